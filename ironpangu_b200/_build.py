@@ -73,12 +73,23 @@ def _run(cmd, cwd=None):
     return r.stdout + r.stderr
 
 
-def build_kernels(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every ``*.cu`` under csrc/kernels for sm_100a into one shared library."""
+def build_kernels(force: bool = False, verbose: bool = False, units=None) -> Path:
+    """Compile every ``*.cu`` under csrc/kernels for sm_100a into one shared library. With ``units`` (file names without the suffix)
+    and no current full library: only these, into a library of their own."""
     cus = sorted(KERNEL_DIR.glob("*.cu"))
     deps = cus + sorted(KERNEL_DIR.glob("*.cuh")) + sorted(KERNEL_DIR.glob("*.h"))
+    target = KERNEL_LIB
     if not force and not _stale(KERNEL_LIB, deps):
         return KERNEL_LIB
+    if units:
+        missing = set(units) - {c.stem for c in cus}
+        if missing:
+            raise ValueError(f"no such kernel sources: {sorted(missing)}")
+        cus = [c for c in cus if c.stem in set(units)]
+        deps = cus + [d for d in deps if d.suffix != ".cu"]
+        target = KERNEL_DIR / f"libifab_kernels_{hashlib.sha256(' '.join(c.stem for c in cus).encode()).hexdigest()[:8]}.so"
+        if not force and not _stale(target, deps):
+            return target
     nvcc = _nvcc()
     objdir = KERNEL_DIR / "build"
     objdir.mkdir(exist_ok=True)
@@ -94,16 +105,16 @@ def build_kernels(force: bool = False, verbose: bool = False) -> Path:
     with ThreadPoolExecutor(max_workers=min(8, len(cus))) as ex:
         results = list(ex.map(one, cus))
     objs = [str(o) for o, _ in results]
-    _run([nvcc, "-shared", "-o", str(KERNEL_LIB), *objs, "-lcudart", "-lcuda"], cwd=KERNEL_DIR)
-    _mark(KERNEL_LIB, deps)
+    _run([nvcc, "-shared", "-o", str(target), *objs, "-lcudart", "-lcuda"], cwd=KERNEL_DIR)
+    _mark(target, deps)
     if verbose:
         for _, out in results:
             print(out)
-    return KERNEL_LIB
+    return target
 
 
-def build_core(force: bool = False) -> Path:
-    """Compile the C++20 host libraries and tools (compiler, planner, runtime services, CLI, server)."""
+def build_core(force: bool = False, tools: bool = True) -> Path:
+    """Compile the C++20 host libraries and, unless ``tools`` is off, the programs (compiler, planner, runtime services, CLI, server)."""
     srcs = sorted(CORE_DIR.glob("*.cpp"))
     deps = srcs + sorted(CORE_DIR.glob("*.h"))
     if srcs and (force or _stale(CORE_LIB, deps)):
@@ -119,7 +130,7 @@ def build_core(force: bool = False) -> Path:
             objs = list(ex.map(one, srcs))
         _run(["g++", "-shared", "-o", str(CORE_LIB), *objs, "-pthread"], cwd=CORE_DIR)
         _mark(CORE_LIB, deps)
-    for bindir, binary in ((CLI_DIR, CLI_BIN), (SERVER_DIR, SERVER_BIN), (TESTS_DIR, TESTS_BIN)):
+    for bindir, binary in () if not tools else ((CLI_DIR, CLI_BIN), (SERVER_DIR, SERVER_BIN), (TESTS_DIR, TESTS_BIN)):
         bsrcs = sorted(bindir.glob("*.cpp"))
         if not bsrcs:
             continue

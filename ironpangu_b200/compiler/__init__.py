@@ -25,10 +25,11 @@ class CompileError(RuntimeError):
 def _load():
     global _lib
     if _lib is None:
-        path = _build.build_core()
+        path = _build.build_core(tools=False)
         lib = C.CDLL(str(path))
         for name, nargs in (("ifab_core_compile", 2), ("ifab_core_write_bundle", 5), ("ifab_core_interpret", 3),
-                            ("ifab_core_read_init_plan", 1), ("ifab_core_read_program", 1), ("ifab_core_validate_bundle", 1)):
+                            ("ifab_core_read_init_plan", 1), ("ifab_core_read_program", 1), ("ifab_core_validate_bundle", 1),
+                            ("ifab_core_pool_create", 2), ("ifab_core_pool_call", 1)):
             fn = getattr(lib, name)
             fn.restype = C.c_void_p
             fn.argtypes = [C.c_char_p] * nargs
@@ -67,6 +68,15 @@ def interpret(source: str, checkpoint_dir: str, tokens: List[int], steps: int = 
     fed token (``watched``: one ``{name: value}`` object per token)."""
     return _call("ifab_core_interpret", source, str(checkpoint_dir),
                  json.dumps({"tokens": tokens, "steps": steps, "logits": logits, "all_logits": all_logits, "watch": watch or []}))
+
+
+def pool_create(manifest: Dict[str, Any], capacities: Dict[str, int]) -> int:
+    """Handle of a new sequence-state pool (``csrc/core/state_pool.h``) with ``capacities`` units per state of a serving manifest."""
+    return int(_call("ifab_core_pool_create", json.dumps(manifest), json.dumps(capacities))["pool"])
+
+
+def pool_call(pool: int, op: str, **request) -> Dict[str, Any]:
+    return _call("ifab_core_pool_call", json.dumps({"pool": pool, "op": op, **request}))
 
 
 def read_init_plan(path: str) -> Dict[str, Any]:

@@ -3,11 +3,14 @@
 // on failure. No exception crosses the boundary.
 #include <cstdlib>
 #include <cstring>
+#include <memory>
+#include <mutex>
 
 #include "contract.h"
 #include "bundle.h"
 #include "interp.h"
 #include "kernel_plugin.h"
+#include "state_pool.h"
 
 using namespace ifab;
 
@@ -47,6 +50,10 @@ program::Options options_from(const Json& j) {
   if (auto v = j.find("bulk_collectives")) o.bulk_collectives = v->as_bool();
   return o;
 }
+// state pools made through the C ABI, by handle
+std::mutex pools_mu;
+std::map<int64_t, std::unique_ptr<runtime::StatePool>> pools;
+int64_t next_pool = 1;
 }  // namespace
 
 extern "C" {
@@ -175,6 +182,72 @@ char* ifab_core_plugin_swiglu(const char* path, const char* target, void* x, voi
     j.set("contract", k.contract());
     j.set("workspace_bytes", k.workspace_bytes());
     return j;
+  });
+}
+
+// Sequence-state pool of a Python engine (one rank): manifest = a serving manifest, capacities = {state: units}.
+char* ifab_core_pool_create(const char* manifest_json, const char* capacities_json) {
+  return guarded([&] {
+    const serving::Manifest m = serving::Manifest::from_json(Json::parse(manifest_json));
+    const Json caps = Json::parse(capacities_json);
+    std::map<runtime::StatePool::Key, uint32_t> cap;
+    for (auto& s : m.states) cap[{s.name, 0}] = (uint32_t)caps.at(s.name).as_int();
+    auto pool = std::make_unique<runtime::StatePool>(m, 1, 1, cap);
+    std::lock_guard<std::mutex> lock(pools_mu);
+    const int64_t id = next_pool++;
+    pools[id] = std::move(pool);
+    Json out = Json::object();
+    out.set("pool", id);
+    return out;
+  });
+}
+// One call on a pool. request: {"pool": id, "op": ...}; reserve {"request", "tokens", "slot"} -> the lease and its bindings; extend
+// {"lease", "generation", "tokens"} and trim {.., "component", "first_live"} -> bindings; retire; usage; close.
+char* ifab_core_pool_call(const char* request_json) {
+  return guarded([&] {
+    const Json q = Json::parse(request_json);
+    std::lock_guard<std::mutex> lock(pools_mu);
+    auto it = pools.find(q.at("pool").as_int());
+    if (it == pools.end()) fail(ErrorKind::Stale, "no such state pool");
+    runtime::StatePool& p = *it->second;
+    const std::string op = q.at("op").as_string();
+    Json out = Json::object();
+    auto show = [&](runtime::Lease l) {
+      Json b = Json::object();
+      for (auto& x : p.bindings(1, l)) {
+        Json u = Json::array();
+        for (uint32_t v : x.units) u.push(v == runtime::kNoUnit ? (int64_t)-1 : (int64_t)v);
+        b.set(x.component, u);
+      }
+      out.set("lease", (int64_t)l.id);
+      out.set("generation", (int64_t)l.generation);
+      out.set("bindings", b);
+    };
+    auto lease = [&] { return runtime::Lease{(uint64_t)q.at("lease").as_int(), (uint64_t)q.at("generation").as_int()}; };
+    if (op == "reserve") {
+      show(p.reserve_at_slot(1, (uint64_t)q.at("request").as_int(), (uint32_t)q.at("tokens").as_int(), (uint32_t)q.at("slot").as_int()));
+    } else if (op == "extend") {
+      p.extend(1, lease(), (uint32_t)q.at("tokens").as_int());
+      show(lease());
+    } else if (op == "trim") {
+      p.trim(1, lease(), q.at("component").as_string(), (uint32_t)q.at("first_live").as_int());
+      show(lease());
+    } else if (op == "retire") {
+      p.retire(1, lease());
+    } else if (op == "usage") {
+      for (auto& u : p.usage()) {
+        Json x = Json::object();
+        x.set("capacity_units", (int64_t)u.capacity_units);
+        x.set("occupied_units", (int64_t)u.occupied_units);
+        x.set("occupied_bytes", (int64_t)u.occupied_bytes);
+        out.set(u.component, x);
+      }
+    } else if (op == "close") {
+      pools.erase(it);
+    } else {
+      invalid("unknown state pool call " + op);
+    }
+    return out;
   });
 }
 

@@ -115,6 +115,66 @@ Lease StatePool::reserve_impl(uint64_t request, uint32_t tokens, int64_t slot) {
   return l;
 }
 
+void StatePool::extend(uint64_t epoch, Lease lease, uint32_t tokens) {
+  guard(epoch);
+  Record& rec = record(lease);
+  if (rec.retired) fail(ErrorKind::Stale, "state pool: lease was retired");
+  if (rec.sealed) invalid("state pool: a sealed lease is read-only");
+  if (tokens <= rec.tokens) return;
+  if (tokens > max_context_) fail(ErrorKind::Capacity, "state pool: reservation exceeds the model context");
+  auto component_of = [&](const Binding& b) -> Component& {
+    for (auto& c : components_)
+      if (c.state.name == b.component) return c;
+    invalid("state pool: no component " + b.component);
+  };
+  auto missing = [&](const Component& c, const Binding& b) -> size_t {
+    if (c.state.storage.kind == Storage::Kind::Slot || b.ring_tokens) return 0;
+    const uint32_t page = c.state.storage.page_tokens;
+    const size_t want = ((size_t)tokens + page - 1) / page;
+    return want > b.units.size() ? want - b.units.size() : 0;
+  };
+  for (auto& b : rec.bindings) {
+    const Component& c = component_of(b);
+    if (c.state.storage.kind == Storage::Kind::Pages && c.state.retention.kind == Retention::Kind::SlidingWindow && !b.ring_tokens &&
+        missing(c, b) > 0)
+      invalid("state pool: " + c.state.name + " was reserved short of its ring and cannot grow");
+    if (c.free_units[b.rank].size() < missing(c, b))
+      fail(ErrorKind::Capacity, "state pool: " + c.state.name + " on rank " + std::to_string(b.rank) + " has " + std::to_string(c.free_units[b.rank].size()) +
+                                    " free units, " + std::to_string(missing(c, b)) + " more needed");
+  }
+  for (auto& b : rec.bindings) {
+    Component& c = component_of(b);
+    for (size_t k = missing(c, b); k > 0; --k) {
+      b.units.push_back(c.free_units[b.rank].back());
+      c.free_units[b.rank].pop_back();
+    }
+  }
+  rec.tokens = tokens;
+}
+
+void StatePool::trim(uint64_t epoch, Lease lease, const std::string& component, uint32_t first_live) {
+  guard(epoch);
+  Record& rec = record(lease);
+  if (rec.retired) fail(ErrorKind::Stale, "state pool: lease was retired");
+  if (rec.sealed || rec.borrowers || rec.in_flight) invalid("state pool: only an idle, unshared lease can be trimmed");
+  for (auto& c : components_) {
+    if (c.state.name != component) continue;
+    if (c.state.storage.kind != Storage::Kind::Pages) invalid("state pool: only paged components can be trimmed");
+    for (auto& b : rec.bindings) {
+      if (b.component != component) continue;
+      if (b.ring_tokens) invalid("state pool: a ring reuses its pages by itself");
+      const size_t dead = std::min<size_t>(first_live / c.state.storage.page_tokens, b.units.size());
+      for (size_t k = 0; k < dead; ++k)
+        if (b.units[k] != kNoUnit) {
+          c.free_units[b.rank].push_back(b.units[k]);
+          b.units[k] = kNoUnit;
+        }
+    }
+    return;
+  }
+  invalid("state pool: no component " + component);
+}
+
 const std::vector<Binding>& StatePool::bindings(uint64_t epoch, Lease lease) const {
   guard(epoch);
   const Record& r = record(lease);
@@ -141,6 +201,7 @@ PageAddress StatePool::page_address(uint64_t epoch, Lease lease, const std::stri
       const uint32_t page = c.state.storage.page_tokens;
       const uint32_t p = b.ring_tokens ? position % b.ring_tokens : position;
       a.unit = b.units.at(p / page);
+      if (a.unit == kNoUnit) fail(ErrorKind::Stale, "state pool: the page of this position was given back");
       a.row = p % page;
       a.byte_offset = (uint64_t)a.unit * c.unit_bytes + (uint64_t)a.row * c.state.storage.row_bytes;
       return a;
@@ -250,7 +311,8 @@ void StatePool::maybe_reclaim(uint64_t id) {
   for (auto& b : r.bindings)
     for (auto& c : components_)
       if (c.state.name == b.component)
-        for (auto u = b.units.rbegin(); u != b.units.rend(); ++u) c.free_units[b.rank].push_back(*u);
+        for (auto u = b.units.rbegin(); u != b.units.rend(); ++u)
+          if (*u != kNoUnit) c.free_units[b.rank].push_back(*u);
   leases_.erase(it);
 }
 
@@ -267,7 +329,7 @@ std::vector<Usage> StatePool::usage() const {
       for (auto& kv : leases_)
         if (kv.second.sealed)
           for (auto& b : kv.second.bindings)
-            if (b.component == c.state.name && b.rank == r) u.sealed_bytes += b.units.size() * c.unit_bytes;
+            if (b.component == c.state.name && b.rank == r) u.sealed_bytes += (uint64_t)(b.units.size() - std::count(b.units.begin(), b.units.end(), kNoUnit)) * c.unit_bytes;
       out.push_back(std::move(u));
     }
   return out;

@@ -17,6 +17,8 @@
 
 namespace ifab::runtime {
 
+constexpr uint32_t kNoUnit = 0xffffffffu;
+
 struct Lease { uint64_t id = 0, generation = 0; };
 struct Borrow { uint64_t id = 0, lease = 0, generation = 0; };
 struct Ticket { uint64_t id = 0; };
@@ -25,7 +27,7 @@ struct SealedLease { uint64_t lease = 0, generation = 0; };
 struct Binding {             // units of one component on one rank
   std::string component;
   uint32_t rank = 0;
-  std::vector<uint32_t> units;   // page ids (Pages) or one slot id (Slot)
+  std::vector<uint32_t> units;   // page ids (Pages; kNoUnit where a page was given back early) or one slot id (Slot)
   uint32_t ring_tokens = 0;      // > 0: positions wrap modulo this many tokens
 };
 struct PageAddress {
@@ -51,6 +53,12 @@ class StatePool {
 
   Lease reserve(uint64_t epoch, uint64_t request, uint32_t tokens);
   Lease reserve_at_slot(uint64_t epoch, uint64_t request, uint32_t tokens, uint32_t slot);   // pin the slot index (resident id)
+  // Grow a lease to cover `tokens` tokens: every position-indexed paged component gets the pages it lacks, all or nothing (a ring
+  // component keeps its ring, which has to cover the growth already). For requests whose length is not known at admission.
+  void extend(uint64_t epoch, Lease lease, uint32_t tokens);
+  // Give back the pages of `component` that hold only positions below `first_live` (a sliding window has passed them for good).
+  // The lease must be idle and neither sealed nor borrowed. Later positions keep their pages.
+  void trim(uint64_t epoch, Lease lease, const std::string& component, uint32_t first_live);
   const std::vector<Binding>& bindings(uint64_t epoch, Lease lease) const;
   PageAddress page_address(uint64_t epoch, Lease lease, const std::string& component, uint32_t rank, uint32_t position) const;
 

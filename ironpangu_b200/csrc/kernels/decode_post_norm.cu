@@ -1,0 +1,194 @@
+// Decode-time linears (1..8 rows per tile) of decoders with an f32 residual stream and norms on sublayer outputs. The weight stream
+// is the one of gemv.cuh (prefetched ahead of the wait on the producer); the prologue finishes the previous sublayer, so a layer
+// needs no row kernels of its own between its linears:
+//
+//   post norm    x_out = x_in + rms(y) * w, operand bf16(x_out). Every CTA computes the rows it needs (a few KB from L2); the CTAs
+//                of the first column write x_out, which must not be x_in (other CTAs still read that)
+//   group norm   operand bf16((o / rms of each group of columns [* gain]) * act(gate)): normalised, gated heads of a recurrent mixer
+//   plain        bf16 rows
+//
+// Epilogue: optional activation, bf16 or f32 result.
+#include "gemv.cuh"
+#include "rope.cuh"
+#include "ifab_kernels.h"
+
+using namespace ifab;
+
+namespace {
+
+enum { PLAIN = 0, POST = 1, GROUP = 2 };
+
+struct Params {
+  const bf16* x; long ldx;                                           // PLAIN
+  const float *y, *norm_w, *x_in; float* x_out; long ldy, ldr;       // POST (ldr: x_in and x_out)
+  const float *o, *gain; const bf16* gate; long ldo, ldg; int groups, gate_act;      // GROUP
+  float eps;
+  const bf16* w;
+  void* z; long ldz; int out_f32, act;
+  int T, N, K;
+};
+
+// stage T rows of the operand; ends with __syncthreads(). `inv`: T * max(groups, 1) floats
+template <int T, int PRO>
+__device__ __forceinline__ void stage_operand(const Params& p, bf16* xs, float* inv, float* red, int t0) {
+  const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, nwarp = nthr >> 5, K = p.K;
+  if (PRO == PLAIN) {
+    for (int t = 0; t < T; ++t) {
+      const bool live = t0 + t < p.T;
+      for (int c = tid * 8; c < K; c += nthr * 8)
+        *reinterpret_cast<uint4*>(xs + t * K + c) = live ? *reinterpret_cast<const uint4*>(p.x + (long)(t0 + t) * p.ldx + c) : make_uint4(0, 0, 0, 0);
+    }
+    __syncthreads();
+    return;
+  }
+  const int groups = PRO == GROUP ? p.groups : 1, n = K / groups;
+  const float* src = PRO == GROUP ? p.o : p.y;
+  const long lds = PRO == GROUP ? p.ldo : p.ldy;
+  if (groups == 1) {
+    for (int t = 0; t < T; ++t) {
+      float ss = 0.f;
+      if (t0 + t < p.T)
+        for (int c = tid * 4; c < K; c += nthr * 4) {
+          const float4 v = *reinterpret_cast<const float4*>(src + (long)(t0 + t) * lds + c);
+          ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+      ss = warp_sum(ss);
+      if (lane == 0) red[t * 8 + warp] = ss;
+    }
+    __syncthreads();
+    if (tid < T) {
+      float s = 0.f;
+      for (int i = 0; i < nwarp; ++i) s += red[tid * 8 + i];
+      inv[tid] = 1.f / sqrtf(s / (float)K + p.eps);
+    }
+  } else {
+    for (int i = warp; i < T * groups; i += nwarp) {
+      const int t = i / groups, g = i - t * groups;
+      float ss = 0.f;
+      if (t0 + t < p.T)
+        for (int c = lane; c < n; c += 32) {
+          const float v = src[(long)(t0 + t) * lds + (long)g * n + c];
+          ss += v * v;
+        }
+      ss = warp_sum(ss);
+      if (lane == 0) inv[i] = 1.f / sqrtf(ss / (float)n + p.eps);
+    }
+  }
+  __syncthreads();
+  for (int t = 0; t < T; ++t) {
+    const long r = t0 + t;
+    const bool live = r < p.T;
+    for (int c = tid * 4; c < K; c += nthr * 4) {
+      float f[4] = {0.f, 0.f, 0.f, 0.f};
+      if (live) {
+        const float4 v = *reinterpret_cast<const float4*>(src + r * lds + c);
+        f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+        if (PRO == POST) {
+          const float iv = inv[t];
+          const float4 w = *reinterpret_cast<const float4*>(p.norm_w + c), x = *reinterpret_cast<const float4*>(p.x_in + r * p.ldr + c);
+          f[0] = x.x + f[0] * iv * w.x;
+          f[1] = x.y + f[1] * iv * w.y;
+          f[2] = x.z + f[2] * iv * w.z;
+          f[3] = x.w + f[3] * iv * w.w;
+          if (blockIdx.x == 0) *reinterpret_cast<float4*>(p.x_out + r * p.ldr + c) = make_float4(f[0], f[1], f[2], f[3]);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            f[i] *= inv[t * groups + (c + i) / n];
+            if (p.gain) f[i] *= p.gain[c + i];
+            f[i] *= activate(__bfloat162float(p.gate[r * p.ldg + c + i]), p.gate_act);
+          }
+        }
+      }
+      __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+      *reinterpret_cast<uint2*>(xs + t * K + c) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+    }
+  }
+  __syncthreads();
+}
+
+template <int T, int R, int PRO>
+__global__ void __launch_bounds__(256) gemv_operand_kernel(Params p) {
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  bf16* xs = reinterpret_cast<bf16*>(smem_raw);
+  float* inv = reinterpret_cast<float*>(xs + (long)T * p.K);
+  __shared__ float red[T * 8];
+  grid_dep_launch();
+  const int t0 = blockIdx.y * T, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n0 = (blockIdx.x * 8 + warp) * R;
+  const bf16* rows[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) rows[r] = (n0 + r < p.N) ? p.w + (long)(n0 + r) * p.K : nullptr;
+  RowBatch<R> pf;
+  prefetch_rows<R>(rows, p.K, pf);
+  grid_dep_wait();
+  stage_operand<T, PRO>(p, xs, inv, red, t0);
+  if (n0 >= p.N) return;
+  float acc[R][T];
+#pragma unroll
+  for (int r = 0; r < R; ++r)
+#pragma unroll
+    for (int t = 0; t < T; ++t) acc[r][t] = 0.f;
+  warp_rows_dot<T, R>(rows, xs, p.K, acc, pf);
+  warp_reduce_acc<T, R>(acc);
+  if (lane == 0) {
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      if (n0 + r >= p.N) continue;
+#pragma unroll
+      for (int t = 0; t < T; ++t) {
+        if (t0 + t >= p.T) continue;
+        const float v = activate(acc[r][t], p.act);
+        if (p.out_f32) reinterpret_cast<float*>(p.z)[(long)(t0 + t) * p.ldz + n0 + r] = v;
+        else reinterpret_cast<bf16*>(p.z)[(long)(t0 + t) * p.ldz + n0 + r] = __float2bfloat16_rn(v);
+      }
+    }
+  }
+}
+
+template <int T, int R, int PRO>
+int launch_one(const Params& p, cudaStream_t s) {
+  const size_t smem = (size_t)T * p.K * sizeof(bf16) + (size_t)T * (PRO == GROUP ? p.groups : 1) * sizeof(float);
+  auto k = gemv_operand_kernel<T, R, PRO>;
+  if (int rc = opt_in_smem(k, smem)) return rc;
+  return launch_chain(k, dim3((p.N + 8 * R - 1) / (8 * R), (p.T + T - 1) / T), dim3(256), smem, s, p);
+}
+template <int T, int PRO>
+int by_rows(const Params& p, cudaStream_t s) {
+  if (p.N >= 148 * 8 * 4 * 2) return launch_one<T, 4, PRO>(p, s);
+  if (p.N >= 148 * 8 * 2 * 2) return launch_one<T, 2, PRO>(p, s);
+  return launch_one<T, 1, PRO>(p, s);
+}
+template <int PRO>
+int dispatch(const Params& p, cudaStream_t s) {
+  if (p.T < 1 || p.N < 1 || p.K < 8 || p.K % 8) return -1;
+  if (p.T <= 1) return by_rows<1, PRO>(p, s);
+  if (p.T <= 2) return by_rows<2, PRO>(p, s);
+  if (p.T <= 4) return by_rows<4, PRO>(p, s);
+  return by_rows<8, PRO>(p, s);
+}
+
+}  // namespace
+
+extern "C" int ifab_gemv_post_norm(const float* y, long ldy, const float* norm_w, float eps, const float* x_in, float* x_out, long ldx, const void* w,
+                                   void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream) {
+  if (ldy % 4 || ldx % 4 || x_in == x_out) return -1;
+  Params p{};
+  p.y = y; p.ldy = ldy; p.norm_w = norm_w; p.eps = eps; p.x_in = x_in; p.x_out = x_out; p.ldr = ldx;
+  p.w = (const bf16*)w; p.z = z; p.ldz = ldz; p.out_f32 = out_f32; p.act = act; p.T = T; p.N = N; p.K = K;
+  return dispatch<POST>(p, (cudaStream_t)stream);
+}
+extern "C" int ifab_gemv_group_norm(const float* o, long ldo, const float* gain, float eps, int groups, const void* gate, long ldg, int gate_act,
+                                    const void* w, void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream) {
+  if (ldo % 4 || groups < 1 || groups > 1024 || K % groups) return -1;
+  Params p{};
+  p.o = o; p.ldo = ldo; p.gain = gain; p.eps = eps; p.groups = groups; p.gate = (const bf16*)gate; p.ldg = ldg; p.gate_act = gate_act;
+  p.w = (const bf16*)w; p.z = z; p.ldz = ldz; p.out_f32 = out_f32; p.act = act; p.T = T; p.N = N; p.K = K;
+  return dispatch<GROUP>(p, (cudaStream_t)stream);
+}
+extern "C" int ifab_gemv_act(const void* x, long ldx, const void* w, void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream) {
+  if (ldx % 8) return -1;
+  Params p{};
+  p.x = (const bf16*)x; p.ldx = ldx;
+  p.w = (const bf16*)w; p.z = z; p.ldz = ldz; p.out_f32 = out_f32; p.act = act; p.T = T; p.N = N; p.K = K;
+  return dispatch<PLAIN>(p, (cudaStream_t)stream);
+}

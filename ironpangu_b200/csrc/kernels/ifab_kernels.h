@@ -73,6 +73,13 @@ int ifab_moe_down_allreduce_decode_fp8(const void* act, const int32_t* ids, cons
 /* ---- tensor-core GEMM (tcgen05 + TMEM + TMA): C[M,N] = A[M,K] * B[N,K]^T (+ residual) ---- */
 int ifab_gemm_bf16(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual,
                    long ldr, int M, int N, int K, uint32_t* status, void* stream);
+/* the same with an activation of the result in the epilogue: 0 none, 1 SiLU, 2 sigmoid, 3 GELU (tanh form) */
+int ifab_gemm_act_bf16(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr, int act,
+                       int M, int N, int K, uint32_t* status, void* stream);
+int ifab_gemm_act_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr, int act,
+                           int persistent, int M, int N, int K, uint32_t* status, void* stream);
+/* C = act(A * B^T) in true f32 */
+int ifab_linear_f32(const float* a, long lda, const float* b, long ldb, float* c, long ldc, int M, int N, int K, int act, void* stream);
 
 /* the same on CTA pairs (tcgen05.mma cta_group::2, 256 x 256 tiles, each CTA loads half of A and half of B); N % 32 == 0 */
 int ifab_gemm_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual,
@@ -252,6 +259,40 @@ int ifab_mhc_post_norm(const void* X, const void* branch, long ldb, const void* 
 /* gated delta rule, one token per row: q, k bf16 [rows, H, dk]; v bf16 [rows, H, dv]; g, beta f32 [rows, H]; state f32 [slots, H, dk, dv] */
 int ifab_delta_rule_decode(const void* q, const void* k, const void* v, const float* g, const float* beta, float* state,
                            const int32_t* slots, void* out, int rows, int H, int dk, int dv, void* stream);
+/* f32 residual stream with the norm on a sublayer's output; `f32`: activations (xa, gate, y) are f32 instead of bf16; gains f32 */
+int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float* x, long ldx, void* xa, long lda, int f32, int T, int D, int vocab,
+                    uint32_t* status, void* stream);
+/* x += rms(y) * w; xa = x, or rms(x) * w2 when w2 is given */
+int ifab_post_norm_add(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, void* xa, long lda, int f32, int T, int D,
+                       void* stream);
+int ifab_rms_rows(const float* x, long ldx, const int32_t* rows, const float* w, float eps, void* y, long ldy, int f32, int T, int D, void* stream);
+int ifab_group_norm_gate(const float* o, long ldo, const float* w, float eps, const void* gate, long ldg, int act, void* y, long ldy, int f32, int T,
+                         int groups, int n, void* stream);
+int ifab_gate_rows(const void* o, long ldo, int head_stride, const void* gate, long ldg, int act, void* y, long ldy, int f32, int T, int H, int n,
+                   void* stream);
+/* decode linears whose prologue finishes the previous sublayer. ..._post_norm: x_out = x_in + rms(y) * w (one CTA column writes it), then
+ * z = act(bf16(x_out) W^T); ..._group_norm: z = act(bf16((o / rms per group [* gain]) * gate_act(gate)) W^T) */
+int ifab_gemv_post_norm(const float* y, long ldy, const float* norm_w, float eps, const float* x_in, float* x_out, long ldx, const void* w, void* z,
+                        long ldz, int out_f32, int act, int T, int N, int K, void* stream);
+int ifab_gemv_group_norm(const float* o, long ldo, const float* gain, float eps, int groups, const void* gate, long ldg, int gate_act, const void* w,
+                         void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream);
+int ifab_gemv_act(const void* x, long ldx, const void* w, void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream);
+/* linear attention with a fixed decay per head over a packed projection row (linear_attn.cu); state f32 [slots, H, d, e], powers f32 [H, 65] */
+int ifab_la_step(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, int H, int d, int e, int rot, int interleaved, const double* freq,
+                 int act, float k_scale, const float* powers, float* state, const int32_t* positions, const int32_t* slots, float* o, long ldo, int T,
+                 void* stream);
+int ifab_la_prepare(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, int H, int d, int e, int rot, int interleaved,
+                    const double* freq, int act, float k_scale, const int32_t* positions, float* q, float* k, float* v, int T, void* stream);
+int ifab_la_chunks(const float* q, const float* k, const float* v, const int32_t* chunks, int n, const int32_t* positions, int H, int d, int e,
+                   const float* powers, float* cstate, uint64_t cstate_bytes, float* state, float* o, long ldo, void* stream);
+/* per-head norm + rotation + cache write, and sliding-window attention with sinks over pages, any head sizes (window_attn.cu) */
+int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, const float* q_gain, const float* k_gain, float eps,
+                            int H, int G, int d, int e, int rot, int interleaved, const double* freq, const int32_t* positions, const int32_t* slots,
+                            const int32_t* page_table, int max_pages, int page_tokens, int num_pages, void* q_out, long ldq, void* k_cache, void* v_cache,
+                            int T, uint32_t* status, void* stream);
+int ifab_window_attn(const void* q, long ldq, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,
+                     const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int H, int G, int d, int e, int window, float scale,
+                     const float* sink, const void* gate, long ldg, int gate_act, void* out, long ldo, int T, uint32_t* status, void* stream);
 /* indexer: q bf16 [T, heads, dim], w f32 [T, heads], keys paged bf16 [pages, page_tokens, dim]; scores = scratch f32 [T, ctx];
  * out int32 [T, topk]: the top-k key positions (<= the query position) in ascending order, -1 padded */
 int ifab_sparse_index(const void* q, const float* w, const void* keys, const int32_t* positions, const int32_t* slots,

@@ -1,0 +1,215 @@
+// Row operators of decoders that keep an f32 residual stream and normalise a sublayer's OUTPUT before adding it:
+//
+//   embed_rows_kernel      x = table[id] (f32) and its copy in the activation type (the operand of the next linears)
+//   post_norm_add_kernel   x += rms(y) * w; copy in the activation type (of rms(x) * w2 when a second gain is given: the norm ahead
+//                          of the output matrix). y is the f32 output of the sublayer's last linear
+//   rms_rows_kernel        rms(x[row]) * w of selected rows, in the activation type (the norm ahead of the output matrix)
+//   group_norm_gate_kernel (o / rms of each group of columns [* w]) * act(gate): the normalised, gated heads of a recurrent
+//                          mixer. group = one head without a gain, or all heads together with one
+//   gate_rows_kernel       o * act(gate), reading heads at a padded stride
+//
+// Every kernel exists for bf16 activations and for f32 ones; norms and the residual are f32 in both.
+#include "rope.cuh"
+#include "ifab_kernels.h"
+
+using namespace ifab;
+
+namespace {
+
+__device__ __forceinline__ void store4(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+__device__ __forceinline__ void store4(bf16* p, const float* f) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+
+template <typename A>
+__global__ void __launch_bounds__(256) embed_rows_kernel(const int32_t* ids, const A* table, long ldt, float* x, long ldx, A* xa, long lda, int D,
+                                                         int vocab, uint32_t* status) {
+  grid_dep_launch();
+  grid_dep_wait();
+  const int t = blockIdx.x;
+  int id = ids[t];
+  if (id < 0 || id >= vocab) {
+    if (threadIdx.x == 0 && status) atomicOr(status, IFAB_STATUS_BAD_INDEX);
+    id = 0;
+  }
+  for (int c = threadIdx.x; c < D; c += blockDim.x) {
+    const A v = table[(long)id * ldt + c];
+    x[(long)t * ldx + c] = to_f32(v);
+    xa[(long)t * lda + c] = v;
+  }
+}
+
+// one CTA per row
+template <typename A>
+__global__ void __launch_bounds__(256) post_norm_add_kernel(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, A* xa,
+                                                            long lda, int D) {
+  __shared__ float red[33];
+  grid_dep_launch();
+  grid_dep_wait();
+  const int t = blockIdx.x;
+  const float* yr = y + (long)t * ldy;
+  float* xr = x + (long)t * ldx;
+  A* ar = xa + (long)t * lda;
+  if (D % 4 == 0 && ldy % 4 == 0 && ldx % 4 == 0 && lda % 4 == 0 && D <= 256 * 16) {     // the row stays in registers between the passes
+    float4 v[4], r[4], g[4];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      r[i] = v[i];
+      g[i] = v[i];
+      if (c < D) {
+        v[i] = *reinterpret_cast<const float4*>(yr + c);
+        r[i] = *reinterpret_cast<const float4*>(xr + c);
+        g[i] = *reinterpret_cast<const float4*>(w + c);
+      }
+      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)D + eps);
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      r[i].x += v[i].x * inv * g[i].x;
+      r[i].y += v[i].y * inv * g[i].y;
+      r[i].z += v[i].z * inv * g[i].z;
+      r[i].w += v[i].w * inv * g[i].w;
+      if (c < D) *reinterpret_cast<float4*>(xr + c) = r[i];
+      ss += r[i].x * r[i].x + r[i].y * r[i].y + r[i].z * r[i].z + r[i].w * r[i].w;
+    }
+    const float inv2 = w2 ? 1.f / sqrtf(block_sum(ss, red) / (float)D + eps) : 1.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      if (c >= D) break;
+      float f[4] = {r[i].x, r[i].y, r[i].z, r[i].w};
+      if (w2) {
+        const float4 h = *reinterpret_cast<const float4*>(w2 + c);
+        f[0] *= inv2 * h.x;
+        f[1] *= inv2 * h.y;
+        f[2] *= inv2 * h.z;
+        f[3] *= inv2 * h.w;
+      }
+      store4(ar + c, f);
+    }
+    return;
+  }
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < D; c += blockDim.x) ss += yr[c] * yr[c];
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)D + eps);
+  ss = 0.f;
+  for (int c = threadIdx.x; c < D; c += blockDim.x) {
+    const float v = xr[c] + yr[c] * inv * w[c];
+    xr[c] = v;
+    ss += v * v;
+    if (!w2) ar[c] = from_f32<A>(v);
+  }
+  if (!w2) return;
+  const float inv2 = 1.f / sqrtf(block_sum(ss, red) / (float)D + eps);
+  for (int c = threadIdx.x; c < D; c += blockDim.x) ar[c] = from_f32<A>(xr[c] * inv2 * w2[c]);
+}
+
+template <typename A>
+__global__ void __launch_bounds__(256) rms_rows_kernel(const float* x, long ldx, const int32_t* rows, const float* w, float eps, A* y, long ldy, int D) {
+  __shared__ float red[33];
+  grid_dep_launch();
+  grid_dep_wait();
+  const int t = blockIdx.x;
+  const float* xr = x + (long)(rows ? rows[t] : t) * ldx;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < D; c += blockDim.x) ss += xr[c] * xr[c];
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)D + eps);
+  for (int c = threadIdx.x; c < D; c += blockDim.x) y[(long)t * ldy + c] = from_f32<A>(xr[c] * inv * w[c]);
+}
+
+// one warp per (row, group) for narrow groups, one CTA per row for a single wide one: grid (ceil(groups / WPB), rows)
+template <typename A, int WARPS_PER_GROUP>
+__global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* o, long ldo, const float* w, float eps, const A* gate, long ldg, int act,
+                                                              A* y, long ldy, int groups, int n) {
+  __shared__ float red[33];
+  grid_dep_launch();
+  grid_dep_wait();
+  const int t = blockIdx.y;
+  constexpr int GPB = 8 / WARPS_PER_GROUP, TPG = 32 * WARPS_PER_GROUP;
+  const int g = blockIdx.x * GPB + threadIdx.x / TPG, i0 = threadIdx.x % TPG;
+  if (WARPS_PER_GROUP == 1 && g >= groups) return;
+  const float* r = o + (long)t * ldo + (long)g * n;
+  float ss = 0.f;
+  for (int c = i0; c < n; c += TPG) ss += r[c] * r[c];
+  ss = WARPS_PER_GROUP == 1 ? warp_sum(ss) : block_sum(ss, red);
+  const float inv = 1.f / sqrtf(ss / (float)n + eps);
+  for (int c = i0; c < n; c += TPG) {
+    float v = r[c] * inv;
+    if (w) v *= w[(long)g * n + c];
+    y[(long)t * ldy + (long)g * n + c] = from_f32<A>(v * activate(to_f32(gate[(long)t * ldg + (long)g * n + c]), act));
+  }
+}
+
+template <typename A>
+__global__ void __launch_bounds__(256) gate_rows_kernel(const A* o, long ldo, int head_stride, const A* gate, long ldg, int act, A* y, long ldy, int H,
+                                                        int n) {
+  grid_dep_launch();
+  grid_dep_wait();
+  const int t = blockIdx.x;
+  for (int c = threadIdx.x; c < H * n; c += blockDim.x) {
+    const int h = c / n, j = c - h * n;
+    y[(long)t * ldy + c] = from_f32<A>(to_f32(o[(long)t * ldo + (long)h * head_stride + j]) * activate(to_f32(gate[(long)t * ldg + c]), act));
+  }
+}
+
+template <typename A>
+int embed(const int32_t* ids, const void* table, long ldt, float* x, long ldx, void* xa, long lda, int T, int D, int vocab, uint32_t* status,
+          cudaStream_t s) {
+  return launch_chain(embed_rows_kernel<A>, dim3(T), dim3(256), 0, s, ids, (const A*)table, ldt, x, ldx, (A*)xa, lda, D, vocab, status);
+}
+template <typename A>
+int group_norm(const float* o, long ldo, const float* w, float eps, const void* gate, long ldg, int act, void* y, long ldy, int T, int groups, int n,
+               cudaStream_t s) {
+  if (n > 512)
+    return launch_chain(group_norm_gate_kernel<A, 8>, dim3(groups, T), dim3(256), 0, s, o, ldo, w, eps, (const A*)gate, ldg, act, (A*)y, ldy, groups, n);
+  return launch_chain(group_norm_gate_kernel<A, 1>, dim3((groups + 7) / 8, T), dim3(256), 0, s, o, ldo, w, eps, (const A*)gate, ldg, act, (A*)y, ldy,
+                      groups, n);
+}
+
+}  // namespace
+
+extern "C" int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float* x, long ldx, void* xa, long lda, int f32, int T, int D,
+                               int vocab, uint32_t* status, void* stream) {
+  if (T < 1 || D < 1 || vocab < 1) return -1;
+  cudaStream_t s = (cudaStream_t)stream;
+  return f32 ? embed<float>(ids, table, ldt, x, ldx, xa, lda, T, D, vocab, status, s) : embed<bf16>(ids, table, ldt, x, ldx, xa, lda, T, D, vocab, status, s);
+}
+
+extern "C" int ifab_post_norm_add(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, void* xa, long lda, int f32, int T, int D,
+                                  void* stream) {
+  if (T < 1 || D < 1) return -1;
+  cudaStream_t s = (cudaStream_t)stream;
+  return f32 ? launch_chain(post_norm_add_kernel<float>, dim3(T), dim3(256), 0, s, y, ldy, w, w2, eps, x, ldx, (float*)xa, lda, D)
+             : launch_chain(post_norm_add_kernel<bf16>, dim3(T), dim3(256), 0, s, y, ldy, w, w2, eps, x, ldx, (bf16*)xa, lda, D);
+}
+
+extern "C" int ifab_rms_rows(const float* x, long ldx, const int32_t* rows, const float* w, float eps, void* y, long ldy, int f32, int T, int D,
+                             void* stream) {
+  if (T < 1 || D < 1) return -1;
+  cudaStream_t s = (cudaStream_t)stream;
+  return f32 ? launch_chain(rms_rows_kernel<float>, dim3(T), dim3(256), 0, s, x, ldx, rows, w, eps, (float*)y, ldy, D)
+             : launch_chain(rms_rows_kernel<bf16>, dim3(T), dim3(256), 0, s, x, ldx, rows, w, eps, (bf16*)y, ldy, D);
+}
+
+extern "C" int ifab_group_norm_gate(const float* o, long ldo, const float* w, float eps, const void* gate, long ldg, int act, void* y, long ldy, int f32,
+                                    int T, int groups, int n, void* stream) {
+  if (T < 1 || groups < 1 || n < 1 || T > 65535) return -1;
+  cudaStream_t s = (cudaStream_t)stream;
+  return f32 ? group_norm<float>(o, ldo, w, eps, gate, ldg, act, y, ldy, T, groups, n, s) : group_norm<bf16>(o, ldo, w, eps, gate, ldg, act, y, ldy, T, groups, n, s);
+}
+
+extern "C" int ifab_gate_rows(const void* o, long ldo, int head_stride, const void* gate, long ldg, int act, void* y, long ldy, int f32, int T, int H, int n,
+                              void* stream) {
+  if (T < 1 || H < 1 || n < 1) return -1;
+  cudaStream_t s = (cudaStream_t)stream;
+  return f32 ? launch_chain(gate_rows_kernel<float>, dim3(T), dim3(256), 0, s, (const float*)o, ldo, head_stride, (const float*)gate, ldg, act, (float*)y, ldy,
+                            H, n)
+             : launch_chain(gate_rows_kernel<bf16>, dim3(T), dim3(256), 0, s, (const bf16*)o, ldo, head_stride, (const bf16*)gate, ldg, act, (bf16*)y, ldy, H, n);
+}

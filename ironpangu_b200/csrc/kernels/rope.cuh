@@ -1,0 +1,55 @@
+// Rotation angles in full precision for any pair layout: the angle position * frequency is formed and reduced in double (the
+// frequencies come as doubles), so cos / sin are exact to float rounding at every position.
+#pragma once
+#include "common.cuh"
+
+namespace ifab {
+
+__device__ __forceinline__ void rope_angle(int pos, double freq, float* c, float* s) {
+  double a = (double)pos * freq;
+  a -= 6.283185307179586 * rint(a * 0.15915494309189535);
+  sincosf((float)a, s, c);
+}
+
+// columns of pair i among the first `rot` columns of a head: (i, i + rot / 2), or (2 i, 2 i + 1) when interleaved
+__device__ __forceinline__ void rope_pair(int i, int rot, int interleaved, int* a, int* b) {
+  *a = interleaved ? 2 * i : i;
+  *b = interleaved ? 2 * i + 1 : i + rot / 2;
+}
+
+// activations and caches exist in bf16 (serving) and f32 (exact mode): loads and stores by type
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(bf16 v) { return __bfloat162float(v); }
+template <typename A>
+__device__ __forceinline__ A from_f32(float v);
+template <>
+__device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float gelu_tanh_f32(float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
+// elementwise activations by number: 0 none, 1 SiLU, 2 sigmoid, 3 GELU (tanh form)
+__device__ __forceinline__ float activate(float z, int act) {
+  switch (act) {
+    case 1: return z * sigmoid_f32(z);
+    case 2: return sigmoid_f32(z);
+    case 3: return gelu_tanh_f32(z);
+    default: return z;
+  }
+}
+
+// sum over the block (blockDim.x a multiple of 32, at most 1024); `red` holds 33 floats; every thread gets the sum
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = blockDim.x >> 5;
+  __syncthreads();
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  float s = 0.f;
+  for (int i = 0; i < n; ++i) s += red[i];
+  return s;
+}
+
+}  // namespace ifab

@@ -13,6 +13,7 @@
 // reference's counterpart is aclnnMatmul on [T<=4096, K] activations (token_executor.h:387-456).
 #include <cstdlib>
 
+#include "rope.cuh"
 #include "tc_gemm_core.cuh"
 #include "ifab_kernels.h"
 
@@ -27,6 +28,7 @@ struct GemmParams {
   int M, N, K;
   uint32_t* status;
   uint32_t spin_limit;
+  int act;               // activation of the result (numbers of activate(); 0: none), after the residual
 };
 
 // store 32 consecutive columns of one row (values already final)
@@ -36,6 +38,10 @@ __device__ __forceinline__ void store_row32(const GemmParams& p, int row, int co
   if (p.residual) {
     const bf16* r = p.residual + (long)row * p.ldr + col;
     for (int i = 0; i < nvalid; ++i) v[i] = bf16_round(v[i]) + __bfloat162float(r[i]);
+  }
+  if (p.act) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) v[i] = activate(v[i], p.act);
   }
   if (p.out_f32) {
     float* out = reinterpret_cast<float*>(p.c) + (long)row * p.ldc + col;
@@ -156,19 +162,24 @@ static bool two_sm_enabled() {
 // C[M,N] = A[M,K] * B[N,K]^T (+ residual). A: row stride lda, B: row stride ldb (elements), K % 8 == 0.
 extern "C" int ifab_gemm_bf16(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32,
                               const void* residual, long ldr, int M, int N, int K, uint32_t* status, void* stream) {
+  return ifab_gemm_act_bf16(a, lda, b, ldb, c, ldc, out_f32, residual, ldr, 0, M, N, K, status, stream);
+}
+
+// The same with an activation of the result in the epilogue (1 SiLU, 2 sigmoid, 3 GELU in the tanh form).
+extern "C" int ifab_gemm_act_bf16(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr,
+                                  int act, int M, int N, int K, uint32_t* status, void* stream) {
   if (M < 1 || N < 1 || K < 8 || K % 8 || lda % 8 || ldb % 8) return -1;
   // from 256 x 256 up: CTA pairs (tcgen05.mma cta_group::2; same accumulation order, same bits) - persistent with two
   // accumulators when there is more than one tile per SM pair, one tile per pair otherwise
   if (M >= 256 && N >= 256 && N % 32 == 0 && two_sm_enabled()) {
     const long tiles = (long)((M + 255) / 256) * ((N + 255) / 256);
-    return tiles > 74 ? ifab_gemm_bf16_2sm_persistent(a, lda, b, ldb, c, ldc, out_f32, residual, ldr, M, N, K, status, stream)
-                      : ifab_gemm_bf16_2sm(a, lda, b, ldb, c, ldc, out_f32, residual, ldr, M, N, K, status, stream);
+    return ifab_gemm_act_bf16_2sm(a, lda, b, ldb, c, ldc, out_f32, residual, ldr, act, tiles > 74, M, N, K, status, stream);
   }
   CUtensorMap ta, tb;
   const int BN = N > 128 ? 256 : 128;
   if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM)) return rc;
   if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)N, (uint64_t)K, (uint64_t)ldb, (uint32_t)BN)) return rc;
-  GemmParams p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u};
+  GemmParams p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, act};
   cudaStream_t s = (cudaStream_t)stream;
   return BN == 256 ? launch<256>(ta, tb, p, s) : launch<128>(ta, tb, p, s);
 }

@@ -16,6 +16,7 @@
 // `ifab_gemm_bf16` uses these kernels from 256 rows and 256 columns up; below that a pair's 256 x 256 tile is mostly padding.
 #include <algorithm>
 
+#include "rope.cuh"
 #include "tc_gemm_core.cuh"
 #include "ifab_kernels.h"
 
@@ -37,6 +38,7 @@ struct Gemm2Params {
   uint32_t* status;
   uint32_t spin_limit;
   int swiglu_f;   // > 0 (persistent kernel only): B = [gate rows 0..F) | up rows F..2F), C[M, F] = silu(A gate^T) * (A up^T)
+  int act;        // activation of the result (numbers of activate(); 0: none), after the residual
 };
 
 __device__ __forceinline__ uint32_t cluster_ctarank() {
@@ -88,6 +90,10 @@ __device__ __forceinline__ void store_row32_2(const Gemm2Params& p, int row, int
     const bf16* r = p.residual + (long)row * p.ldr + col;
 #pragma unroll
     for (int i = 0; i < 32; ++i) v[i] = bf16_round(v[i]) + __bfloat162float(r[i]);
+  }
+  if (p.act) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) v[i] = activate(v[i], p.act);
   }
   if (p.out_f32) {
     float* out = reinterpret_cast<float*>(p.c) + (long)row * p.ldc + col;
@@ -376,34 +382,35 @@ __global__ void __launch_bounds__(192) tc_gemm_2sm_persistent_kernel(const __gri
 
 }  // namespace
 
-// C[M,N] = A[M,K] * B[N,K]^T (+ residual) with CTA pairs on 256 x 256 tiles. N % 32 == 0, K % 8 == 0.
-extern "C" int ifab_gemm_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr,
-                                  int M, int N, int K, uint32_t* status, void* stream) {
+// C[M,N] = act(A[M,K] * B[N,K]^T (+ residual)) with CTA pairs on 256 x 256 tiles. N % 32 == 0, K % 8 == 0. `persistent`: one CTA pair per
+// SM pair walks the tiles with two accumulators in tensor memory, else one pair per tile.
+extern "C" int ifab_gemm_act_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr,
+                                      int act, int persistent, int M, int N, int K, uint32_t* status, void* stream) {
   if (M < 1 || N < 32 || N % 32 || K < 8 || K % 8 || lda % 8 || ldb % 8) return -1;
   CUtensorMap ta, tb;
   if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM)) return rc;
   if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)N, (uint64_t)K, (uint64_t)ldb, HALF_N)) return rc;
-  Gemm2Params p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, 0};
-  if (int rc = opt_in_smem(tc_gemm_2sm_kernel, SMEM2)) return rc;
-  dim3 grid(2 * ((M + 255) / 256), (N + 255) / 256);
-  return launch_chain_cluster(tc_gemm_2sm_kernel, grid, dim3(192), 2, (size_t)SMEM2, (cudaStream_t)stream, ta, tb, p);
-}
-
-// The same with a persistent grid (one CTA pair per SM pair) and two accumulators in tensor memory.
-extern "C" int ifab_gemm_bf16_2sm_persistent(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual,
-                                             long ldr, int M, int N, int K, uint32_t* status, void* stream) {
-  if (M < 1 || N < 32 || N % 32 || K < 8 || K % 8 || lda % 8 || ldb % 8) return -1;
-  CUtensorMap ta, tb;
-  if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM)) return rc;
-  if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)N, (uint64_t)K, (uint64_t)ldb, HALF_N)) return rc;
-  Gemm2Params p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, 0};
+  Gemm2Params p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, 0, act};
+  const int tiles = ((M + 255) / 256) * ((N + 255) / 256);
+  if (!persistent) {
+    if (int rc = opt_in_smem(tc_gemm_2sm_kernel, SMEM2)) return rc;
+    dim3 grid(2 * ((M + 255) / 256), (N + 255) / 256);
+    return launch_chain_cluster(tc_gemm_2sm_kernel, grid, dim3(192), 2, (size_t)SMEM2, (cudaStream_t)stream, ta, tb, p);
+  }
   if (int rc = opt_in_smem(tc_gemm_2sm_persistent_kernel, SMEM2)) return rc;
   int dev = 0, sms = 148;
   cudaGetDevice(&dev);
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-  const int tiles = ((M + 255) / 256) * ((N + 255) / 256);
   const int pairs = std::max(1, std::min(tiles, sms / 2));
   return launch_chain_cluster(tc_gemm_2sm_persistent_kernel, dim3(2 * pairs), dim3(192), 2, (size_t)SMEM2, (cudaStream_t)stream, ta, tb, p);
+}
+extern "C" int ifab_gemm_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr,
+                                  int M, int N, int K, uint32_t* status, void* stream) {
+  return ifab_gemm_act_bf16_2sm(a, lda, b, ldb, c, ldc, out_f32, residual, ldr, 0, 0, M, N, K, status, stream);
+}
+extern "C" int ifab_gemm_bf16_2sm_persistent(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual,
+                                             long ldr, int M, int N, int K, uint32_t* status, void* stream) {
+  return ifab_gemm_act_bf16_2sm(a, lda, b, ldb, c, ldc, out_f32, residual, ldr, 0, 1, M, N, K, status, stream);
 }
 
 // C[M, F] = silu(A gate^T) * (A up^T) with B = [gate rows | up rows] ([2F, K]): the packed gate / up projection of a SwiGLU block in
@@ -414,7 +421,7 @@ extern "C" int ifab_gemm_swiglu_bf16_2sm(const void* a, long lda, const void* b,
   CUtensorMap ta, tb;
   if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM)) return rc;
   if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)2 * F, (uint64_t)K, (uint64_t)ldb, HALF_N)) return rc;
-  Gemm2Params p{c, ldc, 0, nullptr, 0, M, 2 * F, K, status, 4000000u, F};
+  Gemm2Params p{c, ldc, 0, nullptr, 0, M, 2 * F, K, status, 4000000u, F, 0};
   if (int rc = opt_in_smem(tc_gemm_2sm_persistent_kernel, SMEM2)) return rc;
   int dev = 0, sms = 148;
   cudaGetDevice(&dev);

@@ -1,0 +1,211 @@
+// Sliding-window softmax attention with a per-head sink over paged keys / values, for any head sizes (query / key size and value
+// size independent), bf16 or f32 activations and caches.
+//
+//   qk_norm_rope_write_kernel  RMS norm per head of q and k with a shared gain, rotation of the first `rot` columns (either pair
+//                              layout, angles in double), q to its own rows, k and v into the pages of their sequence
+//   window_attn_kernel         one CTA per (row, query head): row at position i sees keys j with 0 <= i - j < window; scores,
+//                              weights and sums in f32; the denominator also holds exp(sink_h). Optional output gate
+//
+// Positions, slots and page tables as in the other paged kernels; pages that fell out of every window may be gone (-1).
+#include "rope.cuh"
+#include "ifab_kernels.h"
+
+using namespace ifab;
+
+namespace {
+
+struct QkParams {
+  const void* proj; long ldp; int q_off, k_off, v_off;
+  const float *q_gain, *k_gain; float eps;           // gains may be null: no norm
+  int H, G, d, e, rot, interleaved;
+  const double* freq;
+  const int32_t *positions, *slots, *page_table;
+  int max_pages, page_tokens, num_pages;
+  void* q_out; long ldq;
+  void *k_cache, *v_cache;
+  int T;
+  uint32_t* status;
+};
+
+// grid (ceil((H + 2 G) / 4), T), 128 threads: one warp per head of a row
+template <typename A>
+__global__ void __launch_bounds__(128) qk_norm_rope_write_kernel(QkParams p) {
+  grid_dep_launch();
+  grid_dep_wait();
+  const int t = blockIdx.y, h = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= p.H + 2 * p.G) return;
+  const int pos = p.positions[t];
+  if (pos < 0) return;
+  const A* row = reinterpret_cast<const A*>(p.proj) + (long)t * p.ldp;
+  long dst_row = -1;
+  if (h >= p.H) {
+    const int lp = pos / p.page_tokens;
+    const int page = lp < p.max_pages ? p.page_table[(long)p.slots[t] * p.max_pages + lp] : -1;
+    if (page < 0 || page >= p.num_pages) {
+      if (lane == 0 && p.status) atomicOr(p.status, IFAB_STATUS_BAD_INDEX);
+      return;
+    }
+    dst_row = (long)page * p.page_tokens + pos % p.page_tokens;
+  }
+  if (h >= p.H + p.G) {
+    const int g = h - p.H - p.G;
+    const A* src = row + p.v_off + (long)g * p.e;
+    A* dst = reinterpret_cast<A*>(p.v_cache) + (dst_row * p.G + g) * p.e;
+    for (int c = lane; c < p.e; c += 32) dst[c] = src[c];
+    return;
+  }
+  const bool is_q = h < p.H;
+  const A* src = is_q ? row + p.q_off + (long)h * p.d : row + p.k_off + (long)(h - p.H) * p.d;
+  A* dst = is_q ? reinterpret_cast<A*>(p.q_out) + (long)t * p.ldq + (long)h * p.d : reinterpret_cast<A*>(p.k_cache) + (dst_row * p.G + h - p.H) * p.d;
+  const float* gain = is_q ? p.q_gain : p.k_gain;
+  float inv = 1.f;
+  if (gain) {
+    float ss = 0.f;
+    for (int c = lane; c < p.d; c += 32) {
+      const float v = to_f32(src[c]);
+      ss += v * v;
+    }
+    inv = 1.f / sqrtf(warp_sum(ss) / (float)p.d + p.eps);
+  }
+  for (int i = lane; i < p.rot / 2; i += 32) {
+    int ia, ib;
+    rope_pair(i, p.rot, p.interleaved, &ia, &ib);
+    float cs, sn;
+    rope_angle(pos, p.freq[i], &cs, &sn);
+    const float a = to_f32(src[ia]) * inv * (gain ? gain[ia] : 1.f), b = to_f32(src[ib]) * inv * (gain ? gain[ib] : 1.f);
+    dst[ia] = from_f32<A>(a * cs - b * sn);
+    dst[ib] = from_f32<A>(b * cs + a * sn);
+  }
+  for (int c = p.rot + lane; c < p.d; c += 32) dst[c] = from_f32<A>(to_f32(src[c]) * inv * (gain ? gain[c] : 1.f));
+}
+
+struct WinParams {
+  const void* q; long ldq;
+  const void *k_cache, *v_cache;
+  const int32_t *positions, *slots, *page_table;
+  int max_pages, page_tokens, num_pages;
+  int H, G, d, e, window;
+  float scale;
+  const float* sink;             // [H] or null
+  const void* gate; long ldg; int gate_act;
+  void* out; long ldo;
+  uint32_t* status;
+};
+
+constexpr int WARPS = 8, KB = 4, EPL = 8;      // lanes own columns lane, lane + 32, ...: up to 256
+
+template <typename A>
+__global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
+  __shared__ float sm_acc[WARPS][256], sm_m[WARPS], sm_l[WARPS];
+  grid_dep_launch();
+  grid_dep_wait();
+  const int h = blockIdx.x, t = blockIdx.y, g = h / (p.H / p.G), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = p.positions[t];
+  if (pos < 0) return;
+  const int32_t* table = p.page_table + (long)p.slots[t] * p.max_pages;
+  const int first = (p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
+  float q[EPL], acc[EPL];
+  const A* qr = reinterpret_cast<const A*>(p.q) + (long)t * p.ldq + (long)h * p.d;
+#pragma unroll
+  for (int u = 0; u < EPL; ++u) {
+    const int c = lane + 32 * u;
+    q[u] = c < p.d ? to_f32(qr[c]) : 0.f;
+    acc[u] = 0.f;
+  }
+  float m = -INFINITY, l = 0.f;
+  for (int k0 = first + warp; k0 <= pos; k0 += WARPS * KB) {
+    float s[KB];
+    long r[KB];
+#pragma unroll
+    for (int b = 0; b < KB; ++b) {
+      const int key = k0 + b * WARPS;
+      r[b] = -1;
+      s[b] = 0.f;
+      if (key <= pos) {
+        const int lp = key / p.page_tokens;
+        const int page = lp < p.max_pages ? table[lp] : -1;
+        if (page < 0 || page >= p.num_pages) {
+          if (lane == 0 && p.status) atomicOr(p.status, IFAB_STATUS_BAD_INDEX);
+        } else {
+          r[b] = ((long)page * p.page_tokens + key % p.page_tokens) * p.G + g;
+          const A* kr = reinterpret_cast<const A*>(p.k_cache) + r[b] * p.d;
+#pragma unroll
+          for (int u = 0; u < EPL; ++u)
+            if (32 * u < p.d && lane + 32 * u < p.d) s[b] = fmaf(q[u], to_f32(kr[lane + 32 * u]), s[b]);
+        }
+      }
+    }
+#pragma unroll
+    for (int b = 0; b < KB; ++b) s[b] = r[b] >= 0 ? warp_sum(s[b]) * p.scale : -INFINITY;
+    float mn = m;
+#pragma unroll
+    for (int b = 0; b < KB; ++b) mn = fmaxf(mn, s[b]);
+    if (mn == -INFINITY) continue;
+    const float corr = expf(m - mn);
+    l *= corr;
+#pragma unroll
+    for (int u = 0; u < EPL; ++u) acc[u] *= corr;
+#pragma unroll
+    for (int b = 0; b < KB; ++b) {
+      if (r[b] < 0) continue;
+      const float w = expf(s[b] - mn);
+      l += w;
+      const A* vr = reinterpret_cast<const A*>(p.v_cache) + r[b] * p.e;
+#pragma unroll
+      for (int u = 0; u < EPL; ++u)
+        if (32 * u < p.e && lane + 32 * u < p.e) acc[u] = fmaf(w, to_f32(vr[lane + 32 * u]), acc[u]);
+    }
+    m = mn;
+  }
+  if (lane == 0) {
+    sm_m[warp] = m;
+    sm_l[warp] = l;
+  }
+#pragma unroll
+  for (int u = 0; u < EPL; ++u) sm_acc[warp][lane + 32 * u] = acc[u];
+  __syncthreads();
+  float M = p.sink ? p.sink[h] : -INFINITY;
+#pragma unroll
+  for (int w = 0; w < WARPS; ++w) M = fmaxf(M, sm_m[w]);
+  float den = p.sink ? expf(p.sink[h] - M) : 0.f, wgt[WARPS];
+#pragma unroll
+  for (int w = 0; w < WARPS; ++w) {
+    wgt[w] = sm_m[w] == -INFINITY ? 0.f : expf(sm_m[w] - M);
+    den += wgt[w] * sm_l[w];
+  }
+  const float inv = den > 0.f ? 1.f / den : 0.f;
+  for (int c = threadIdx.x; c < p.e; c += blockDim.x) {
+    float v = 0.f;
+#pragma unroll
+    for (int w = 0; w < WARPS; ++w) v = fmaf(wgt[w], sm_acc[w][c], v);
+    v *= inv;
+    if (p.gate) v *= activate(to_f32(reinterpret_cast<const A*>(p.gate)[(long)t * p.ldg + (long)h * p.e + c]), p.gate_act);
+    reinterpret_cast<A*>(p.out)[(long)t * p.ldo + (long)h * p.e + c] = from_f32<A>(v);
+  }
+}
+
+}  // namespace
+
+extern "C" int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, const float* q_gain, const float* k_gain,
+                                       float eps, int H, int G, int d, int e, int rot, int interleaved, const double* freq, const int32_t* positions,
+                                       const int32_t* slots, const int32_t* page_table, int max_pages, int page_tokens, int num_pages, void* q_out,
+                                       long ldq, void* k_cache, void* v_cache, int T, uint32_t* status, void* stream) {
+  if (T < 1 || T > 65535 || H < 1 || G < 1 || d < 1 || e < 1 || rot < 0 || rot % 2 || rot > d || (rot && !freq)) return -1;
+  QkParams p{proj, ldp, q_off, k_off, v_off, q_gain, k_gain, eps, H, G, d, e, rot, interleaved, freq, positions, slots, page_table, max_pages, page_tokens,
+             num_pages, q_out, ldq, k_cache, v_cache, T, status};
+  const dim3 grid((H + 2 * G + 3) / 4, T);
+  return f32 ? launch_chain(qk_norm_rope_write_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, p)
+             : launch_chain(qk_norm_rope_write_kernel<bf16>, grid, dim3(128), 0, (cudaStream_t)stream, p);
+}
+
+extern "C" int ifab_window_attn(const void* q, long ldq, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,
+                                const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int H, int G, int d, int e, int window,
+                                float scale, const float* sink, const void* gate, long ldg, int gate_act, void* out, long ldo, int T, uint32_t* status,
+                                void* stream) {
+  if (T < 1 || T > 65535 || H < 1 || G < 1 || H % G || d < 1 || d > 256 || e < 1 || e > 256 || window < 0) return -1;
+  WinParams p{q, ldq, k_cache, v_cache, positions, slots, page_table, max_pages, page_tokens, num_pages, H, G, d, e, window, scale, sink, gate, ldg, gate_act,
+              out, ldo, status};
+  const dim3 grid(H, T);
+  return f32 ? launch_chain(window_attn_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, p)
+             : launch_chain(window_attn_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)stream, p);
+}

@@ -132,6 +132,32 @@ static void test_state_pool() {
   CHECK_THROWS(Capacity, p.reserve_at_slot(7, 6, 16, 1));
   p.poison();
   CHECK_THROWS(Backend, p.reserve(7, 9, 16));
+  // growth on demand and early return of pages that a window has passed
+  StatePool g(m, 3, 2, cap);
+  auto empty = g.usage();
+  Lease gr = g.reserve(3, 1, 10);
+  CHECK(g.bindings(3, gr)[0].units.size() == 1);
+  g.extend(3, gr, 16);
+  CHECK(g.bindings(3, gr)[0].units.size() == 1);
+  g.extend(3, gr, 100);
+  CHECK(g.bindings(3, gr)[0].units.size() == 7 && g.bindings(3, gr)[1].units.size() == 7);
+  CHECK_THROWS(Capacity, g.reserve(3, 2, 32));
+  CHECK_THROWS(Capacity, g.extend(3, gr, 9 * 16));
+  CHECK(g.bindings(3, gr)[0].units.size() == 7);       // a refused growth changes nothing
+  const uint32_t kept = g.bindings(3, gr)[0].units[4];
+  g.trim(3, gr, "kv16", 79);                            // positions 0..63 are dead: four whole pages; 64..79 is not whole
+  CHECK(g.bindings(3, gr)[0].units[3] == kNoUnit && g.bindings(3, gr)[0].units[4] == kept);
+  CHECK_THROWS(Stale, g.page_address(3, gr, "kv16", 0, 63));
+  CHECK(g.page_address(3, gr, "kv16", 0, 64).unit == kept);
+  Lease nb = g.reserve(3, 2, 32);                       // takes returned pages
+  g.extend(3, gr, 130);
+  CHECK(g.bindings(3, gr)[0].units.size() == 9);
+  CHECK_THROWS(Invalid, g.trim(3, gr, "conv", 16));
+  g.retire(3, gr);
+  g.retire(3, nb);
+  CHECK(g.usage() == empty);                            // every page came back exactly once
+  CHECK_THROWS(Stale, g.extend(3, gr, 200));
+
   // sliding window ring
   auto ms = manifest(true);
   std::map<StatePool::Key, uint32_t> cap2;

@@ -1,0 +1,505 @@
+"""Falinex: a decoder whose layers mix by retention, lightning attention or sliding-window attention in any order, with the norm on
+every sublayer's OUTPUT (x += rms(sublayer(x)) * w) over an f32 residual stream, and dense GELU feed-forwards. Layers may share
+another layer's weights (``weights_of``) with a state or cache of their own.
+
+  retention     q, k rotated (half layout), k * dim^-1/2; S = decay S + k v^T, o = S^T q (f32 state); o / rms per head;
+                * silu(W_g x); W_o
+  lightning     q, k, v through SiLU; the same recurrence without rotation or scale; rms over all heads together with a gain;
+                * sigmoid(W_g x); W_o
+  attention     grouped heads; rms of q and k per head with a gain; interleaved rotation; scores * scale over the last ``mask.size``
+                positions; softmax with a learned sink per head in the denominator; * sigmoid(W_g x); W_o
+
+``FalinexDecoder`` runs decode rows (and pieces of prompts up to ``max_tokens`` rows) in one launch chain whose grid depends on the
+row count only, so the engine replays it as a CUDA graph; ``FalinexRows`` runs a packed step - portions of several prompts beside
+decode rows - as matrix-matrix work. Both read the KV pages and recurrent states of ``decoder.state_manager`` (runtime/paged_state.py).
+In bf16 the linears take bf16 operands with f32 accumulation; norms, rotations, scores, recurrences and the residual are f32.
+With ``dtype=torch.float32`` every product is a true f32 FMA.
+
+A checkpoint directory is ``config.json`` (``"architecture": "Falinex"``) + safetensors; see :func:`weight_shapes` for the names."""
+from __future__ import annotations
+
+import json
+from dataclasses import dataclass, field
+from pathlib import Path
+from typing import Dict, List, Optional
+
+import torch
+
+from ..ops import decode as K
+from ..ops import stream_norm as N
+from ..ops import window_attn as WA
+from ..ops.linear_attn import CHUNK, DecayedMixer, chunk_table, rotary_frequencies
+from ..parallel.fabric import Fabric
+from ..runtime.paged_state import PagedState
+
+BF16, F32 = torch.bfloat16, torch.float32
+KERNEL_UNITS = ("misc", "post_norm", "linear_f32", "linear_attn", "window_attn", "decode_post_norm", "decode_moe", "sampling", "tc_gemm", "tc_gemm_2sm")
+
+
+# ---------------------------------------------------------------------------------------------------------------------------
+# configuration
+# ---------------------------------------------------------------------------------------------------------------------------
+@dataclass
+class MixerConfig:
+    kind: str                          # retention | lightning | attention
+    heads: int
+    dim: int
+    vdim: int
+    kv_heads: int = 0                  # attention
+    decay: tuple = ()                  # retention, lightning
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+    window: int = 0                    # attention: 0 = no window
+    scale: float = 1.0                 # attention
+
+    @property
+    def recurrent(self) -> bool:
+        return self.kind != "attention"
+
+    @property
+    def qk_groups(self) -> int:
+        return self.heads if self.recurrent else self.kv_heads
+
+    @property
+    def columns(self) -> List[int]:
+        """Widths of q, k, v and the gate in the packed input projection."""
+        return [self.heads * self.dim, self.qk_groups * self.dim, self.qk_groups * self.vdim, self.heads * self.vdim]
+
+
+@dataclass
+class LayerConfig:
+    mixer: MixerConfig
+    ff: int = 0                        # 0: no feed-forward
+    weights_of: Optional[int] = None
+
+
+@dataclass
+class FalinexConfig:
+    vocab: int
+    width: int
+    eps: float
+    layers: List[LayerConfig] = field(default_factory=list)
+    page_tokens: int = 16
+
+    @staticmethod
+    def from_dict(j: dict) -> "FalinexConfig":
+        if j.get("architecture") != "Falinex":
+            raise ValueError(f"not a Falinex configuration (architecture {j.get('architecture')!r})")
+        layers = []
+        for i, e in enumerate(j["layers"]):
+            m, kind = e["mixer"], e["type"]
+            if kind not in ("retention", "lightning", "attention"):
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            mask = m.get("mask") or {}
+            rot = m.get("rot") or {}
+            mc = MixerConfig(kind, int(m["heads"]), int(m["dim"]), int(m["vdim"]), kv_heads=int(m.get("kv_heads", m["heads"])) if kind == "attention" else 0,
+                             decay=tuple(float(d) for d in m.get("decay", ())), rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)),
+                             window=int(mask.get("size", 0)), scale=float(m.get("scale", 1.0)))
+            mlp = e.get("mlp")
+            if mlp is not None and mlp.get("kind") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+            layers.append(LayerConfig(mc, int(mlp["ff"]) if mlp is not None else 0, e.get("weights_of")))
+        return FalinexConfig(int(j["vocab"]), int(j["width"]), float(j["norm"]["eps"]), layers).validate()
+
+    def to_dict(self) -> dict:
+        out = []
+        for l in self.layers:
+            m = l.mixer
+            d = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim}
+            if m.recurrent:
+                d["decay"] = list(m.decay)
+            else:
+                d.update(kv_heads=m.kv_heads, mask={"size": m.window}, scale=m.scale)
+            if m.rot_dims:
+                d["rot"] = {"base": m.rot_base, "dims": m.rot_dims}
+            e = {"type": m.kind, "mixer": d, "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None}
+            if l.weights_of is not None:
+                e["weights_of"] = l.weights_of
+            out.append(e)
+        return {"architecture": "Falinex", "vocab": self.vocab, "width": self.width, "norm": {"eps": self.eps}, "layers": out}
+
+    def validate(self) -> "FalinexConfig":
+        for i, l in enumerate(self.layers):
+            m = l.mixer
+            if m.rot_dims % 2 or m.rot_dims > m.dim:
+                raise ValueError(f"layer {i}: rotation of {m.rot_dims} columns in heads of {m.dim}")
+            if m.recurrent and len(m.decay) != m.heads:
+                raise ValueError(f"layer {i}: {m.heads} heads but {len(m.decay)} decay factors")
+            if not m.recurrent and (m.kv_heads < 1 or m.heads % m.kv_heads or max(m.dim, m.vdim) > 256):
+                raise ValueError(f"layer {i}: attention heads {m.heads} / {m.kv_heads} of {m.dim} / {m.vdim} columns are not supported")
+            if l.weights_of is not None:
+                j = self.owner(i)
+                if (self.layers[j].mixer, self.layers[j].ff) != (m, l.ff):
+                    raise ValueError(f"layer {i} shares the weights of layer {j} but not its sizes")
+        return self
+
+    def owner(self, i: int) -> int:
+        """The layer whose tensors layer ``i`` uses."""
+        seen = set()
+        while self.layers[i].weights_of is not None:
+            if i in seen or not 0 <= self.layers[i].weights_of < len(self.layers):
+                raise ValueError(f"layer {i}: weights_of does not lead to a layer with weights")
+            seen.add(i)
+            i = self.layers[i].weights_of
+        return i
+
+    @property
+    def window(self) -> int:
+        """The longest window when every attention layer has one, else 0."""
+        w = [l.mixer.window for l in self.layers if not l.mixer.recurrent]
+        return max(w) if w and all(w) else 0
+
+    def param_count(self) -> int:
+        n = 0
+        for shape in weight_shapes(self).values():
+            k = 1
+            for d in shape:
+                k *= d
+            n += k
+        return n
+
+    @staticmethod
+    def tiny() -> "FalinexConfig":
+        """Every mixer, a shared layer, a layer without a feed-forward; odd sizes."""
+        ret = MixerConfig("retention", 3, 24, 40, decay=(0.9, 0.98, 0.995), rot_dims=16, rot_base=1e4)
+        lig = MixerConfig("lightning", 2, 32, 24, decay=(0.8, 0.99))
+        att = MixerConfig("attention", 6, 40, 32, kv_heads=2, rot_dims=24, rot_base=1e5, window=24, scale=0.2)
+        return FalinexConfig(384, 128, 1e-5, [LayerConfig(att, 192), LayerConfig(ret, 0), LayerConfig(lig, 192), LayerConfig(att, 192, 0)]).validate()
+
+    @staticmethod
+    def text2b(layers: int = 24, width: int = 2048, heads: int = 16, kv_heads: int = 4, dim: int = 128, ff: int = 6144, vocab: int = 151936,
+               window: int = 1024) -> "FalinexConfig":
+        """A 2B-class stack: (lightning, retention, retention, attention) repeated."""
+        dec = lambda lo: tuple(1.0 - 2.0 ** -(lo + 6.0 * h / max(1, heads - 1)) for h in range(heads))
+        lig = MixerConfig("lightning", heads, dim, dim, decay=dec(2.0))
+        ret = MixerConfig("retention", heads, dim, dim, decay=dec(5.0), rot_dims=dim, rot_base=1e4)
+        att = MixerConfig("attention", heads, dim, dim, kv_heads=kv_heads, rot_dims=dim, rot_base=1e6, window=window, scale=dim ** -0.5)
+        return FalinexConfig(vocab, width, 1e-5, [LayerConfig((lig, ret, ret, att)[i % 4], ff) for i in range(layers)]).validate()
+
+
+# ---------------------------------------------------------------------------------------------------------------------------
+# weights
+# ---------------------------------------------------------------------------------------------------------------------------
+def weight_shapes(c: FalinexConfig) -> Dict[str, tuple]:
+    """Checkpoint tensor names -> shapes (bf16 in the file)."""
+    s = {"embed": (c.vocab, c.width), "final.norm": (c.width,), "head": (c.vocab, c.width)}
+    for i, l in enumerate(c.layers):
+        if l.weights_of is not None:
+            continue
+        p, m = f"l{i}.", l.mixer
+        q, k, v, g = m.columns
+        s[p + "norm1"] = (c.width,)
+        s.update({p + "mix.q": (q, c.width), p + "mix.k": (k, c.width), p + "mix.v": (v, c.width), p + "mix.g": (g, c.width), p + "mix.o": (c.width, g)})
+        if m.kind == "lightning":
+            s[p + "mix.norm"] = (g,)
+        if m.kind == "attention":
+            s.update({p + "mix.q.norm": (m.dim,), p + "mix.k.norm": (m.dim,), p + "mix.sink": (m.heads,)})
+        if l.ff:
+            s.update({p + "norm2": (c.width,), p + "mlp.up": (l.ff, c.width), p + "mlp.down": (c.width, l.ff)})
+    return s
+
+
+def random_weights(c: FalinexConfig, device, seed: int = 0, std: float = 0.02) -> Dict[str, torch.Tensor]:
+    """Random-init checkpoint tensors: N(0, std) matrices, gains 1 + N(0, std), sinks N(0, 1)."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    out = {}
+    for name, shape in weight_shapes(c).items():
+        t = torch.empty(shape, dtype=BF16, device=device).normal_(0.0, 1.0 if name.endswith("sink") else std, generator=g)
+        out[name] = t + 1.0 if "norm" in name else t
+    return out
+
+
+def save_checkpoint(path, c: FalinexConfig, weights: Dict[str, torch.Tensor]) -> None:
+    """Write ``config.json`` and ``model.safetensors`` (bf16)."""
+    import struct
+
+    d = Path(path)
+    d.mkdir(parents=True, exist_ok=True)
+    (d / "config.json").write_text(json.dumps(c.to_dict(), indent=1))
+    hdr, blobs, at = {}, [], 0
+    for n, t in weights.items():
+        raw = t.detach().to(BF16).cpu().contiguous().view(torch.uint8).numpy().tobytes()
+        hdr[n] = {"dtype": "BF16", "shape": list(t.shape), "data_offsets": [at, at + len(raw)]}
+        blobs.append(raw)
+        at += len(raw)
+    head = json.dumps(hdr).encode()
+    head += b" " * (-len(head) % 8)
+    (d / "model.safetensors").write_bytes(struct.pack("<Q", len(head)) + head + b"".join(blobs))
+
+
+def load_checkpoint(path) -> tuple:
+    """``(config, weights on the host)`` of a checkpoint directory; every expected tensor must be there with its shape."""
+    from ..runtime.plan_engine import SafetensorsDir
+
+    c = FalinexConfig.from_dict(json.loads((Path(path) / "config.json").read_text()))
+    src = SafetensorsDir(str(path))
+    dts = {"BF16": BF16, "F32": F32, "F16": torch.float16}
+    out = {}
+    for name, shape in weight_shapes(c).items():
+        if name not in src.tensors:
+            raise ValueError(f"the checkpoint has no tensor {name}")
+        _, _, _, dt, have = src.tensors[name]
+        if tuple(have) != tuple(shape) or dt not in dts:
+            raise ValueError(f"{name}: {dt} {list(have)} in the checkpoint, {list(shape)} expected")
+        out[name] = torch.from_numpy(src.bytes_of(name).copy()).view(dts[dt]).view(*shape)
+    return c, out
+
+
+def _pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+# ---------------------------------------------------------------------------------------------------------------------------
+# executors
+# ---------------------------------------------------------------------------------------------------------------------------
+class _Rows:
+    """Step buffers for up to ``rows`` rows (leading dimensions padded to 8 elements, padding zero)."""
+
+    def __init__(self, dec: "FalinexDecoder", rows: int, chunked: bool):
+        c, dev, A = dec.cfg, dec.fabric.device, dec.dtype
+        mix = [l.mixer for l in c.layers]
+        z = lambda n, dt=A: torch.zeros(rows, _pad8(n), dtype=dt, device=dev)
+        self.rows = rows
+        self.x, self.x2 = z(c.width, F32), z(c.width, F32)           # residual stream (two: fused prologues write the other one)
+        self.xa, self.y = z(c.width), z(c.width, F32)
+        self.proj = z(max(sum(m.columns) for m in mix))
+        self.o = z(max([m.heads * m.vdim for m in mix if m.recurrent] or [1]), F32)
+        self.q = z(max([m.heads * m.dim for m in mix if not m.recurrent] or [1]))
+        self.mixed = {w: z(w) for w in {m.heads * m.vdim for m in mix}}      # one per width: the padding columns must stay zero
+        self.act = {w: z(w) for w in {l.ff for l in c.layers if l.ff}}
+        self.scratch = None
+        rec = [m for m in mix if m.recurrent]
+        if chunked and rec:
+            f = lambda n: torch.empty(n, dtype=F32, device=dev)
+            nch = rows // CHUNK + dec.num_slots + 1                  # chunks of a step: whole ones and one ragged end per sequence
+            self.scratch = (f(rows * max(m.heads * m.dim for m in rec)), f(rows * max(m.heads * m.dim for m in rec)),
+                            f(rows * max(m.heads * m.vdim for m in rec)), f(nch * max(m.heads * m.dim * m.vdim for m in rec)))
+
+
+class FalinexDecoder:
+    """Decode executor on one GPU: up to ``max_tokens`` (<= 8) rows per step, each with its own position and sequence slot; rows of
+    one sequence inside a step are consecutive and in position order. Greedy next tokens land in ``next_ids``."""
+
+    def __init__(self, cfg: FalinexConfig, weights: Dict[str, torch.Tensor], fabric: Fabric, *, max_tokens: int = 8, max_context: int = 1024, num_slots: int = 1,
+                 pool_tokens: int = 0, keep_logits: bool = False, dtype: torch.dtype = BF16):
+        """``pool_tokens``: tokens the KV page pool holds for all sequences together (0: every slot can reach the full context)."""
+        assert 1 <= max_tokens <= 8 and fabric.world == 1, "the Falinex decoder runs on one GPU"
+        assert dtype in (BF16, F32)
+        c, dev = cfg, fabric.device
+        self.cfg, self.fabric, self.rank, self.world, self.dtype = cfg, fabric, 0, 1, dtype
+        self.T, self.max_context, self.num_slots = max_tokens, max_context, num_slots
+        per_slot = (max_context + c.page_tokens - 1) // c.page_tokens
+        self.num_pages = (pool_tokens + c.page_tokens - 1) // c.page_tokens if pool_tokens else per_slot * num_slots
+        self._load(weights)
+        es = torch.empty((), dtype=dtype).element_size()
+        att = [l.mixer for l in c.layers if not l.mixer.recurrent]
+        rec = [l.mixer for l in c.layers if l.mixer.recurrent]
+        self.state_manager = PagedState(model="falinex", context=max_context, residents=num_slots, page_tokens=c.page_tokens, pool_pages=self.num_pages,
+                                        row_bytes=sum(m.kv_heads * (m.dim + m.vdim) for m in att) * es,
+                                        slot_bytes=sum(m.heads * m.dim * m.vdim for m in rec) * 4, vocab=c.vocab, device=dev, window=c.window)
+        self.page_table = self.state_manager.table
+        for L in self.layers:
+            m = L["m"]
+            if m.recurrent:
+                L["state"] = L["rec"].state(num_slots, dev)
+            else:
+                L["k_cache"] = torch.zeros(self.num_pages, c.page_tokens, m.kv_heads, m.dim, dtype=dtype, device=dev)
+                L["v_cache"] = torch.zeros(self.num_pages, c.page_tokens, m.kv_heads, m.vdim, dtype=dtype, device=dev)
+        T = max_tokens
+        i32 = lambda: torch.zeros(T, dtype=torch.int32, device=dev)
+        self.tokens, self.positions, self.slots, self.next_ids = i32(), i32(), i32(), i32()
+        self.next_vals = torch.zeros(T, dtype=F32, device=dev)
+        self.rows = _Rows(self, T, False)
+        self._logits = torch.empty(T, c.vocab, dtype=F32, device=dev)
+        self.logits = self._logits if keep_logits else None
+        self.partial = torch.empty(((c.vocab + 7) // 8) * 8 * 2, dtype=F32, device=dev)
+        self.sample_scratch = torch.empty(T * ((c.vocab + 4095) // 4096) * 128, dtype=F32, device=dev)
+        self.inv_temp = torch.full((T,), 1e4, dtype=F32, device=dev)
+        # the fused decode chain needs operand widths that are whole 16-byte chunks
+        self.fused = dtype == BF16 and all(n % 8 == 0 for l in c.layers for n in (c.width, l.ff, l.mixer.heads * l.mixer.vdim))
+        self.fused_rows = 2                   # beyond this the CUDA-core products are FMA-bound and the GEMMs take over
+
+    def _load(self, W: Dict[str, torch.Tensor]) -> None:
+        c, dev, A = self.cfg, self.fabric.device, self.dtype
+
+        def mat(*names):
+            """Rows of the named matrices, one after the other; columns padded to 8 elements."""
+            t = torch.cat([W[n].to(dev) for n in names], 0).to(A)
+            return torch.nn.functional.pad(t, (0, _pad8(t.shape[1]) - t.shape[1])).contiguous()
+
+        vec = lambda n: W[n].to(dev).float().contiguous()
+        self.embed, self.head, self.final_norm = mat("embed"), mat("head"), vec("final.norm")
+        built: Dict[int, dict] = {}
+        self.layers: List[dict] = []
+        for i, l in enumerate(c.layers):
+            j = c.owner(i)
+            if j not in built:
+                p, m = f"l{j}.", l.mixer
+                cols = m.columns
+                off = [0, cols[0], cols[0] + cols[1]]
+                S = {"m": m, "norm1": vec(p + "norm1"), "in": mat(*[p + "mix." + n for n in "qkvg"]), "o": mat(p + "mix.o"), "off": off, "gate0": sum(cols[:3]),
+                     "cols": sum(cols), "ff": l.ff}
+                if l.ff:
+                    S.update(norm2=vec(p + "norm2"), up=mat(p + "mlp.up"), down=mat(p + "mlp.down"))
+                if m.recurrent:
+                    ret = m.kind == "retention"
+                    S["rec"] = DecayedMixer(heads=m.heads, dim=m.dim, vdim=m.vdim, decay=m.decay, offsets=off, device=dev, rot_dims=m.rot_dims,
+                                            rot_base=m.rot_base, interleaved=False, act=None if ret else "silu", k_scale=m.dim ** -0.5 if ret else 1.0)
+                    S["gain"] = None if ret else vec(p + "mix.norm")
+                    S["groups"], S["gate_act"] = (m.heads, "silu") if ret else (1, "sigmoid")
+                else:
+                    S.update(q_norm=vec(p + "mix.q.norm"), k_norm=vec(p + "mix.k.norm"), sink=vec(p + "mix.sink"), gate_act="sigmoid",
+                             freq=rotary_frequencies(m.rot_dims, m.rot_base, dev) if m.rot_dims else None)
+                built[j] = S
+            self.layers.append(dict(built[j]))        # shared tensors, own state
+
+    @classmethod
+    def from_checkpoint(cls, path, fabric: Fabric, **kw) -> "FalinexDecoder":
+        c, w = load_checkpoint(path)
+        return cls(c, w, fabric, **kw)
+
+    # -- layers ------------------------------------------------------------------------------------------------------------
+    def _mix(self, B: _Rows, L: dict, m: int, pos, slot, table) -> None:
+        """The mixer of one layer between its input projection (``B.proj``) and the operand of its output projection (``B.mixed``);
+        ``table``: chunk table of a packed step, None for decode rows. Recurrent mixers leave their heads in ``B.o``."""
+        mx, st = L["m"], self.fabric.desc.status
+        proj = B.proj[:m]
+        if mx.recurrent:
+            o = B.o[:m, :mx.heads * mx.vdim]
+            if table is None:
+                L["rec"].step(proj, L["state"], pos, slot, o)
+            else:
+                L["rec"].chunks(proj, L["state"], pos, table, o, B.scratch)
+        else:
+            q = B.q[:m, :mx.heads * mx.dim]
+            WA.qk_norm_rope_write(proj, L["off"], L["q_norm"], L["k_norm"], self.cfg.eps, heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, vdim=mx.vdim,
+                                  rot=mx.rot_dims, interleaved=True, freq=L["freq"], positions=pos, slots=slot, page_table=self.page_table, q_out=q,
+                                  k_cache=L["k_cache"], v_cache=L["v_cache"], status_ptr=st)
+            WA.window_attn(q, L["k_cache"], L["v_cache"], pos, slot, self.page_table, heads=mx.heads, window=mx.window, scale=mx.scale, sink=L["sink"],
+                           gate=proj[:, L["gate0"]:], gate_act=L["gate_act"], out=B.mixed[mx.heads * mx.vdim][:m], status_ptr=st)
+
+    def _layers(self, B: _Rows, m: int, tok, pos, slot, table, final: bool, probe: Optional[list] = None) -> None:
+        """All layers over ``m`` rows as separate row operators and matrix products; the residual ends in ``B.x``, and with ``final`` the
+        normalised rows for the output matrix in ``B.xa``."""
+        c, st, W = self.cfg, self.fabric.desc.status, self.cfg.width
+        x, xa, y = B.x[:m, :W], B.xa[:m], B.y[:m, :W]
+        N.embed_rows(tok, self.embed, x, xa, status_ptr=st)
+        for i, L in enumerate(self.layers):
+            mx = L["m"]
+            hv = mx.heads * mx.vdim
+            last = i + 1 == len(self.layers) and final
+            N.linear(xa, L["in"], B.proj[:m, :L["cols"]], status_ptr=st)
+            self._mix(B, L, m, pos, slot, table)
+            if mx.recurrent:
+                N.group_norm_gate(B.o[:m, :hv], B.proj[:m, L["gate0"]:L["gate0"] + hv], L["gate_act"], c.eps, B.mixed[hv][:m], L["groups"], L["gain"])
+            N.linear(B.mixed[hv][:m], L["o"], y, status_ptr=st)
+            N.post_norm_add(y, L["norm1"], c.eps, x, xa, self.final_norm if last and not L["ff"] else None)
+            if L["ff"]:
+                N.linear(xa, L["up"], B.act[L["ff"]][:m, :L["ff"]], "gelu_tanh", status_ptr=st)
+                N.linear(B.act[L["ff"]][:m], L["down"], y, status_ptr=st)
+                N.post_norm_add(y, L["norm2"], c.eps, x, xa, self.final_norm if last else None)
+            if probe is not None:
+                probe.append(x.clone())
+
+    def _layers_fused(self, B: _Rows, n: int, tok, pos, slot) -> None:
+        """Decode rows: every norm, residual update, gate and activation inside the linear that follows or precedes it. Ends like
+        :meth:`_layers` with ``final``."""
+        c = self.cfg
+        x, x2, xa, y = B.x[:n], B.x2[:n], B.xa[:n], B.y[:n]
+        N.embed_rows(tok, self.embed, x, xa, status_ptr=self.fabric.desc.status)
+        owed = None                            # gain of the sublayer output in y that the residual still lacks
+        for L in self.layers:
+            mx = L["m"]
+            hv, proj = mx.heads * mx.vdim, B.proj[:n]
+            if owed is None:
+                N.gemv_act(xa, L["in"], proj)
+            else:
+                N.gemv_post_norm(y, owed, c.eps, x, x2, L["in"], proj)
+                x, x2 = x2, x
+            self._mix(B, L, n, pos, slot, None)
+            if mx.recurrent:
+                N.gemv_group_norm(B.o[:n, :hv], proj[:, L["gate0"]:], L["gate_act"], c.eps, L["o"], y, L["groups"], L["gain"])
+            else:
+                N.gemv_act(B.mixed[hv][:n], L["o"], y)
+            owed = L["norm1"]
+            if L["ff"]:
+                act = B.act[L["ff"]][:n]
+                N.gemv_post_norm(y, owed, c.eps, x, x2, L["up"], act, "gelu_tanh")
+                x, x2 = x2, x
+                N.gemv_act(act, L["down"], y)
+                owed = L["norm2"]
+        N.post_norm_add(y, owed, c.eps, x, xa, self.final_norm)
+
+    def forward(self, T: Optional[int] = None) -> torch.Tensor:
+        n = self.T if T is None else T
+        B, tok, pos, slot = self.rows, self.tokens[:n], self.positions[:n], self.slots[:n]
+        if self.fused and n <= self.fused_rows:
+            self._layers_fused(B, n, tok, pos, slot)
+        else:
+            self._layers(B, n, tok, pos, slot, None, True)
+        if self.dtype == BF16:
+            K.lm_head_argmax(B.xa[:n], self.head, self.fabric, vocab_offset=0, partial=self.partial, logits=None if self.logits is None else self.logits[:n],
+                             out_ids=self.next_ids[:n], out_vals=self.next_vals[:n])
+        else:
+            N.linear(B.xa[:n], self.head, self._logits[:n])
+            K.sample_topk(self._logits[:n], self.fabric, top_k=1, inv_temperature=self.inv_temp[:n], scratch=self.sample_scratch, out_ids=self.next_ids[:n])
+        return self.next_ids[:n]
+
+    def forward_feedback(self, T: Optional[int] = None) -> torch.Tensor:
+        n = self.T if T is None else T
+        self.forward(n)
+        self.tokens[:n].copy_(self.next_ids[:n])
+        self.positions[:n].add_(1)
+        return self.next_ids[:n]
+
+    def capture(self, T: Optional[int] = None, feedback: bool = False) -> torch.cuda.CUDAGraph:
+        n = self.T if T is None else T
+        self.forward(n)
+        torch.cuda.synchronize()
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):
+            self.forward_feedback(n) if feedback else self.forward(n)
+        return g
+
+
+class FalinexRows:
+    """Packed-step executor: up to ``max_rows`` rows of any sequences (portions of prompts, decode rows), rows of one sequence
+    consecutive and in position order, as one matrix-matrix pass."""
+
+    packed = True              # the engine hands over the rows of a whole step
+    batch_threshold = 8
+
+    def __init__(self, dec: FalinexDecoder, max_rows: int = 512):
+        self.dec, self.M = dec, max_rows
+        self.B = _Rows(dec, max_rows, True)
+        dev = dec.fabric.device
+        self.positions = torch.zeros(max_rows, dtype=torch.int32, device=dev)
+        self.launches = 0
+
+    def plan(self, slots: List[int]) -> torch.Tensor:
+        """Host-side chunk table of a step's rows (int32 ``[n, 4]``); uploaded with the step's control inputs."""
+        return chunk_table(slots)
+
+    def forward_rows(self, tokens: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, select: torch.Tensor, plan: torch.Tensor,
+                     probe: Optional[list] = None) -> torch.Tensor:
+        """f32 logits ``[len(select), vocab]`` of rows ``select``; ``plan`` on the device."""
+        d, c = self.dec, self.dec.cfg
+        m = tokens.numel()
+        assert 1 <= m <= self.M
+        d._layers(self.B, m, tokens, positions, slots, plan, False, probe)
+        xn = torch.zeros(select.numel(), self.B.xa.shape[1], dtype=d.dtype, device=tokens.device)
+        N.rms_rows(self.B.x[:m], d.final_norm, c.eps, xn, select.to(torch.int32))
+        logits = torch.empty(select.numel(), c.vocab, dtype=F32, device=tokens.device)
+        N.linear(xn, d.head, logits, status_ptr=d.fabric.desc.status)
+        return logits
+
+    def forward(self, tokens: torch.Tensor, pos0: int, slot: int = 0) -> torch.Tensor:
+        """A chunk of one sequence; returns the greedy next token (device tensor ``[1]``)."""
+        d, m, dev = self.dec, tokens.numel(), tokens.device
+        pos = torch.arange(pos0, pos0 + m, dtype=torch.int32, device=dev)
+        sl = torch.full((m,), slot, dtype=torch.int32, device=dev)
+        logits = self.forward_rows(tokens, pos, sl, torch.tensor([m - 1], device=dev), self.plan([slot] * m).to(dev))
+        if d.logits is not None:
+            d.logits[:1].copy_(logits)
+        K.sample_topk(logits, d.fabric, top_k=1, inv_temperature=d.inv_temp[:1], scratch=d.sample_scratch, out_ids=d.next_ids[:1])
+        return d.next_ids[:1]

@@ -56,6 +56,23 @@ _SIGS = {
     "ifab_gemv_bf16": [_P, c_long, _P, _P, c_float, c_int, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
     "ifab_gemv_allreduce_bf16": [_P, c_long, _P, _P, c_long, _P, c_long, _P, c_int, c_int, c_int, C.POINTER(IfabFabric), _P],
     "ifab_gemm_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, _P, _P],
+    "ifab_gemm_act_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P, _P],
+    "ifab_linear_f32": [_P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, _P],
+    "ifab_embed_rows": [_P, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, _P, _P],
+    "ifab_post_norm_add": [_P, c_long, _P, _P, c_float, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
+    "ifab_rms_rows": [_P, c_long, _P, _P, c_float, _P, c_long, c_int, c_int, c_int, _P],
+    "ifab_group_norm_gate": [_P, c_long, _P, c_float, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P],
+    "ifab_gate_rows": [_P, c_long, c_int, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P],
+    "ifab_gemv_post_norm": [_P, c_long, _P, c_float, _P, _P, c_long, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
+    "ifab_gemv_group_norm": [_P, c_long, _P, c_float, c_int, _P, c_long, c_int, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
+    "ifab_gemv_act": [_P, c_long, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
+    "ifab_la_step": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_float, _P, _P, _P, _P, _P, c_long, c_int, _P],
+    "ifab_la_prepare": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_float, _P, _P, _P, _P, c_int, _P],
+    "ifab_la_chunks": [_P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, _P, _P, c_u64, _P, _P, c_long, _P],
+    "ifab_qk_norm_rope_write": [_P, c_long, c_int, c_int, c_int, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_int, c_int,
+                                c_int, _P, c_long, _P, _P, c_int, _P, _P],
+    "ifab_window_attn": [_P, c_long, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, c_long, c_int, _P,
+                         c_long, c_int, _P, _P],
     "ifab_gemm_bf16_2sm": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, _P, _P],
     "ifab_gemm_swiglu_bf16_2sm": [_P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, _P, _P],
     "ifab_gemm_bf16_2sm_persistent": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, _P, _P],
@@ -137,8 +154,9 @@ def lib_path() -> Path:
     return _build.KERNEL_LIB
 
 
-def load(build: bool = True):
-    """Return the loaded kernel library, building it first when the sources changed."""
+def load(build: bool = True, units=None):
+    """Return the loaded kernel library, building it first when the sources changed. ``units`` (names of ``.cu`` files without the
+    suffix): a process that runs one model only may ask for a library of just these; it is used when no current full library exists."""
     global _lib
     with _lock:
         if _lib is not None:
@@ -146,7 +164,7 @@ def load(build: bool = True):
         path = _build.KERNEL_LIB
         if build:
             try:
-                path = _build.build_kernels()
+                path = _build.build_kernels(units=units)
             except Exception:
                 if not path.exists():
                     raise

@@ -34,6 +34,9 @@ class DecodeEngine:
         self._graphs = {}
         self._feedback_graphs = {}
         self.transfers = TransferAudit()      # every host <-> device copy of this engine, by role
+        if getattr(decoder, "state_manager", None) is not None:      # pages come from a pool: this engine's one sequence takes its whole context
+            decoder.state_manager.admit(0, decoder.max_context)
+            decoder.state_manager.flush()
         self.h2d_bytes_per_step = 8
         self.d2h_bytes_per_step = 4
 

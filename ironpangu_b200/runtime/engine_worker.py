@@ -88,11 +88,15 @@ class BatchEngine:
     def __init__(self, decoder, model_name: str, context: int, vocab: int, eos: int = -1, greedy_only: bool = False,
                  prefix_slots: int = 0, prefill=None, token_budget: int = 0, use_graphs: bool = True, prefix_namespace: str = ""):
         """``prefill``: optional tensor-core chunk executor (``forward(tokens, pos0, slot)``, attribute ``M`` = rows per call);
-        prompt slices longer than one decode launch group run through it, and the engine advertises ``M`` as its token budget."""
+        prompt slices longer than one decode launch group run through it, and the engine advertises ``M`` as its token budget. An
+        executor with ``packed`` set takes all rows of a step that is wider than a launch group - portions of several prompts
+        beside decode rows - in passes of ``M`` rows. A decoder with a ``state_manager`` has its pages taken and given back here."""
         self.dec, self.name, self.context, self.eos, self.vocab = decoder, model_name, context, eos, vocab
         self.residents = decoder.num_slots
         self.rows = decoder.T
         self.prefill = prefill
+        self.packed = bool(getattr(prefill, "packed", False))
+        self.paged = getattr(decoder, "state_manager", None)
         # one CUDA graph per launch-group width: a decoder step is a few hundred launches, which cost more host time through
         # Python than the kernels take on the device
         self.use_graphs = use_graphs and hasattr(decoder, "capture")
@@ -126,6 +130,8 @@ class BatchEngine:
         self.prefix = (PrefixSnapshots(prefix_slots, self.rows, chunk=self.budget, namespace=prefix_namespace)
                        if prefix_slots > 0 and hasattr(decoder, "caches") else None)
         self.transfers = TransferAudit()
+        self._wanted: Dict[int, List[int]] = {}              # rows of the running step whose logits are asked for (step_logits)
+        self._wanted_logits: Dict[int, torch.Tensor] = {}
         self.trace = None                     # runtime.trace.StepTrace when the runtime option trace_dir is set
         self.allocations_at_ready: Optional[int] = None      # set once the engine has served its first step of every width it will see
         self.audit_counters = {"steps": 0, "launch_groups": 0, "rows": 0, "h2d_bytes": 0, "d2h_bytes": 0, "prefix_rows_copied": 0,
@@ -146,6 +152,8 @@ class BatchEngine:
         a["transfers"] = self.transfers.report()
         a["prepared_execution"] = prepared_execution_report(self)
         a["state_copies"] = state_copy_report(self)
+        if self.paged is not None:
+            a["paged_state"] = self.paged.usage()
         opts = getattr(self, "runtime_options", None)
         if opts is not None:
             a["runtime_options"] = opts.to_dict()
@@ -162,6 +170,8 @@ class BatchEngine:
             raise ValueError("this engine samples greedily only")
         if top_k > self.TOPK_CAP:
             raise ValueError(f"top_k above {self.TOPK_CAP} is not supported")
+        if self.paged is not None:
+            self.paged.admit(resident, reserve)
         self.next_pos[resident] = 0
         self.history[resident] = []
         self.prompt_done[resident] = False
@@ -179,6 +189,8 @@ class BatchEngine:
             self.counts[resident].zero_()
 
     def release(self, resident: int) -> None:
+        if self.paged is not None:
+            self.paged.release(resident)
         self.next_pos[resident] = 0
         self.history[resident] = []
 
@@ -213,11 +225,39 @@ class BatchEngine:
         finally:
             self.trace.end(rec, self.audit_counters)
 
+    def step_logits(self, slices: List[List[int]], tokens: List[int], want: List[List[int]]) -> torch.Tensor:
+        """The step :meth:`step` would run, returning the f32 logits (host ``[rows, vocab]``) of chosen rows: ``want[i]`` lists places
+        among the tokens of slice ``i``. For engines whose every row comes with logits: a packed executor, logits kept by the decoder."""
+        if not (self.packed and self.can_sample):
+            raise ValueError("this engine keeps no logits of arbitrary rows")
+        self._wanted, self._wanted_logits, base = {}, {}, 0
+        for (_, _, count, _), places in zip(slices, want):
+            for w in places:
+                if not 0 <= w < count:
+                    raise ValueError(f"no row {w} in a slice of {count}")
+                self._wanted.setdefault(base + w, []).append(sum(len(v) for v in self._wanted.values()))
+            base += count
+        n = sum(len(v) for v in self._wanted.values())
+        try:
+            self.step(slices, tokens)
+            out = torch.empty(n, self.vocab, dtype=torch.float32)
+            for row, at in self._wanted.items():
+                for i in at:
+                    with self.transfers.scope("request_output"):
+                        self.transfers.d2h(out[i], self._wanted_logits[row], non_blocking=False)
+            return out
+        finally:
+            self._wanted, self._wanted_logits = {}, {}
+
     def _step(self, slices: List[List[int]], tokens: List[int]) -> List[int]:
         d = self.dec
         rows = []                     # (token, position, slot, slice index or -1 when the row does not sample)
         long_slices = []              # prompt slices that go through the matrix-matrix prefill path
         off = 0
+        if self.paged is not None:
+            for resident, position, count, _ in slices:
+                self.paged.ensure(resident, position + count)
+            self.audit_counters["h2d_bytes"] += self.paged.flush()
         for i, (resident, position, count, sample) in enumerate(slices):
             if position != self.next_pos[resident]:
                 raise RuntimeError(f"slice of resident {resident} starts at {position}, expected {self.next_pos[resident]}")
@@ -241,7 +281,7 @@ class BatchEngine:
                         self.counts[resident, local[ok]] += 1
                     continue
                 self.prefix.misses += 1
-            if self.prefill is not None and count > self.rows:
+            if self.prefill is not None and not self.packed and count > self.rows:
                 long_slices.append((i, resident, position, toks, sample))
                 continue
             for k in range(count):
@@ -271,7 +311,7 @@ class BatchEngine:
         if batched:
             # more rows than one decode launch group: all of them as one matrix-matrix pass per `M` rows
             for r0 in range(0, len(rows), self.prefill.M):
-                pending += self._run_rows_batched(rows[r0:r0 + self.prefill.M])
+                pending += self._run_rows_batched(rows[r0:r0 + self.prefill.M], r0)
             rows = []
         for r0 in range(0, len(rows), self.rows):
             part = rows[r0:r0 + self.rows]
@@ -287,10 +327,16 @@ class BatchEngine:
                 tr.h2d(d.slots[:n], hb[2, :n])
             self._run_group(n)
             pending += self._emit(part, n)
+            for j in range(n):
+                if r0 + j in self._wanted:
+                    self._wanted_logits[r0 + j] = d.logits[j].clone()
             self.audit_counters["launch_groups"] += 1
             self.audit_counters["rows"] += n
             self.audit_counters["h2d_bytes"] += 12 * n
         self._collect(pending, out)
+        if self.paged is not None:
+            for resident, position, count, _ in slices:
+                self.paged.advance(resident, position + count)
         # publish the prompt of every sequence that just finished its prefill
         if self.prefix is not None:
             for resident, position, count, sample in slices:
@@ -302,7 +348,7 @@ class BatchEngine:
             raise RuntimeError(f"kernel status word = {d.fabric.status()}")
         return out
 
-    def _run_rows_batched(self, part):
+    def _run_rows_batched(self, part, r0: int = 0):
         """Rows of many sequences (one decode row each, short prompt pieces) through the matrix-matrix path of the prefill
         executor; the sampling rows get their logits from one GEMM and their tokens from the sampling kernel (greedy rows as
         a draw at vanishing temperature). Returns ``[(slice indices, device ids)]`` like :meth:`_emit`."""
@@ -313,8 +359,17 @@ class BatchEngine:
         with self.transfers.scope("control_input"):
             dev = self.transfers.upload(host, d.tokens.device)
         pick = [j for j, r in enumerate(part) if r[3] >= 0]
-        sel = torch.tensor(pick or [n - 1], device=dev.device)
-        logits = self.prefill.forward_rows(dev[0], dev[1], dev[2], sel)
+        asked = [j for j in range(n) if r0 + j in self._wanted]
+        sel = torch.tensor((pick + asked) or [n - 1], device=dev.device)
+        if self.packed:
+            with self.transfers.scope("control_input"):
+                plan = self.transfers.upload(self.prefill.plan([r[2] for r in part]).pin_memory(), d.tokens.device)
+            self.audit_counters["h2d_bytes"] += 4 * plan.numel()
+            logits = self.prefill.forward_rows(dev[0], dev[1], dev[2], sel, plan)
+        else:
+            logits = self.prefill.forward_rows(dev[0], dev[1], dev[2], sel)
+        for i, j in enumerate(asked):
+            self._wanted_logits[r0 + j] = logits[len(pick) + i]
         slots = dev[2].long()
         local = dev[0].long() - self.vocab_offset
         ok = (local >= 0) & (local < self.counts.shape[1])
@@ -485,6 +540,30 @@ def build_engine(args, rank: int, world: int, rec=None) -> BatchEngine:
                                keep_logits=not args.greedy_only)
         mark("state", "K/V pages, delta state, conv history and step workspace")
         eng = BatchEngine(hdec, f"ifab-{args.model}", args.max_model_len, hcfg.vocab, eos=-1, greedy_only=args.greedy_only,
+                          token_budget=args.max_num_batched_tokens, use_graphs=not args.no_graphs)
+        mark("sampling", "per-slot sampling state")
+        return eng
+    if args.model == "checkpoint" or args.model.startswith("falinex"):
+        # families opened from a checkpoint directory (config.json names the architecture), and the presets of Falinex with random weights;
+        # KV pages from one pool, packed steps
+        from ironpangu_b200.models import falinex as F
+        from ironpangu_b200.models import registry
+
+        if world != 1:
+            raise SystemExit("checkpoint models run on one GPU")
+        opts = dict(max_tokens=8, max_context=args.max_model_len, num_slots=args.max_num_seqs, pool_tokens=args.kv_pool_tokens,
+                    keep_logits=True, dtype=torch.float32 if args.dtype == "float32" else torch.bfloat16)
+        rows = max(args.prefill_chunk, 64)
+        if args.model == "checkpoint":
+            if not args.checkpoint:
+                raise SystemExit("--model checkpoint needs --checkpoint DIR")
+            fdec, frows = registry.open_checkpoint(args.checkpoint, fab, max_rows=rows, **opts)
+        else:
+            fcfg = F.FalinexConfig.tiny() if args.model == "falinex-tiny" else F.FalinexConfig.text2b(layers=args.layers or 24)
+            fdec = F.FalinexDecoder(fcfg, F.random_weights(fcfg, dev, seed=args.seed), fab, **opts)
+            frows = F.FalinexRows(fdec, max_rows=rows)
+        mark("weights", "weights, KV page pool, recurrent states and step workspace")
+        eng = BatchEngine(fdec, f"ifab-{args.model}", args.max_model_len, fdec.cfg.vocab, eos=-1, greedy_only=args.greedy_only, prefill=frows,
                           token_budget=args.max_num_batched_tokens, use_graphs=not args.no_graphs)
         mark("sampling", "per-slot sampling state")
         return eng
@@ -716,12 +795,16 @@ def serve(engine, rank: int, world: int, sock_path: str, group=None, agreement="
 
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", default="tiny", choices=["tiny", "flagship", "dense-tiny", "dense2b", "hybrid-tiny", "hybrid2b", "hybrid", "hyper-tiny", "pangu92b", "pangu92b-learned"])
+    ap.add_argument("--model", default="tiny", choices=["tiny", "flagship", "dense-tiny", "dense2b", "hybrid-tiny", "hybrid2b", "hybrid", "hyper-tiny", "pangu92b", "pangu92b-learned",
+                                                         "falinex-tiny", "falinex2b", "checkpoint"],
+                    help="checkpoint: the family that config.json of --checkpoint names (models/registry.py)")
     ap.add_argument("--layers", type=int, default=0)
     ap.add_argument("--seed", type=int, default=0)
     ap.add_argument("--bundle", default="")
     ap.add_argument("--checkpoint", default="")
     ap.add_argument("--definition", default="", help="model document of --model hybrid (contract qwen35_text_v1)")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="float32: true 32-bit products (families that have the mode)")
+    ap.add_argument("--kv-pool-tokens", type=int, default=0, help="tokens of the shared KV page pool (families with one; 0 = every slot can fill its context)")
     ap.add_argument("--max-num-seqs", type=int, default=4)
     ap.add_argument("--max-model-len", type=int, default=256)
     ap.add_argument("--max-num-batched-tokens", type=int, default=0, help="tokens per scheduler step (0 = one launch group of 8 rows)")
