@@ -11,6 +11,7 @@
 // sequences and prefill chunks share one launch). Reference counterparts: attention_qk_prepare /
 // paged_attention_prepare composites (native/src/inferfabric_acl.cpp:1236-1433).
 #include "gemv.cuh"
+#include "rope.cuh"
 #include "ifab_kernels.h"
 
 using namespace ifab;
@@ -79,6 +80,8 @@ struct GqaParams {
   int T, Hq, Hkv, kps, max_splits;
   float* scratch;   // [T][Hq][max_splits][HD + 2]
   uint32_t* status;
+  const float* sink;                              // [Hq]: exp(sink) joins the softmax denominator of the head; or null
+  const bf16* gate; long ldg; int gate_act;       // the result is multiplied by act(gate [T, Hq * HD]); or null
 };
 
 // HD = head_dim (EPL = HD/32 elements per lane), G = query heads per kv head
@@ -212,7 +215,8 @@ __global__ void gqa_merge_kernel(GqaParams p, bf16* out, long ldo) {
   if (threadIdx.x == 0) {
     float M = -INFINITY;
     for (int s = 0; s < ns; ++s) M = fmaxf(M, base[(long)s * (HD + 2) + HD]);
-    float L = 0.f;
+    if (p.sink) M = fmaxf(M, p.sink[h]);
+    float L = p.sink ? __expf(p.sink[h] - M) : 0.f;
     for (int s = 0; s < ns; ++s) {
       const float ms = base[(long)s * (HD + 2) + HD];
       const float w = (ms == -INFINITY) ? 0.f : __expf(ms - M);
@@ -226,7 +230,9 @@ __global__ void gqa_merge_kernel(GqaParams p, bf16* out, long ldo) {
   for (int c = threadIdx.x; c < HD; c += blockDim.x) {
     float v = 0.f;
     for (int s = 0; s < ns; ++s) v += wgt[s] * base[(long)s * (HD + 2) + c];
-    out[(long)t * ldo + (long)h * HD + c] = __float2bfloat16_rn(v * invL);
+    v *= invL;
+    if (p.gate) v *= activate(__bfloat162float(p.gate[(long)t * p.ldg + (long)h * HD + c]), p.gate_act);
+    out[(long)t * ldo + (long)h * HD + c] = __float2bfloat16_rn(v);
   }
 }
 
@@ -268,10 +274,21 @@ extern "C" int ifab_gqa_decode_attention(const void* q, long ldq, const void* k_
                                          int max_pages, int page_tokens, int num_pages, float scale, int T, int Hq, int Hkv,
                                          int head_dim, int keys_per_split, int max_splits, float* scratch,
                                          uint64_t scratch_bytes, void* out, long ldo, uint32_t* status, void* stream) {
-  if (Hkv < 1 || Hq % Hkv || max_splits < 1 || max_splits > 64 || keys_per_split < 8) return -1;
+  return ifab_gqa_window_attention(q, ldq, k_cache, v_cache, positions, slots, page_table, max_pages, page_tokens, num_pages, scale, 0, nullptr, nullptr,
+                                   0, 0, T, Hq, Hkv, head_dim, keys_per_split, max_splits, scratch, scratch_bytes, out, ldo, status, stream);
+}
+
+// The same over the last `window` positions only (0: all), with a sink logit per query head in the denominator and an output gate.
+extern "C" int ifab_gqa_window_attention(const void* q, long ldq, const void* k_cache, const void* v_cache, const int32_t* positions, const int32_t* slots,
+                                         const int32_t* page_table, int max_pages, int page_tokens, int num_pages, float scale, int window,
+                                         const float* sink, const void* gate, long ldg, int gate_act, int T, int Hq, int Hkv, int head_dim,
+                                         int keys_per_split, int max_splits, float* scratch, uint64_t scratch_bytes, void* out, long ldo,
+                                         uint32_t* status, void* stream) {
+  if (Hkv < 1 || Hq % Hkv || max_splits < 1 || max_splits > 64 || keys_per_split < 8 || window < 0) return -1;
   if ((uint64_t)T * Hq * max_splits * (head_dim + 2) * sizeof(float) > scratch_bytes) return -5;
   GqaParams p{(const bf16*)q, ldq, (const bf16*)k_cache, (const bf16*)v_cache, positions, slots, page_table,
-              max_pages, page_tokens, num_pages, scale, 0, T, Hq, Hkv, keys_per_split, max_splits, scratch, status};
+              max_pages, page_tokens, num_pages, scale, window, T, Hq, Hkv, keys_per_split, max_splits, scratch, status, sink, (const bf16*)gate, ldg,
+              gate_act};
   cudaStream_t s = (cudaStream_t)stream;
   switch (head_dim) {
     case 64: return dispatch_g<64>(p, (bf16*)out, ldo, s);

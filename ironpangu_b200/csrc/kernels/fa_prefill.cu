@@ -21,6 +21,7 @@
 // Every wait is bounded; a wait that runs out raises the CTA's abort flag and the status word, the CTA drains its copies,
 // frees its tensor memory and returns. Reference: the fused attention operator of the prompt envelope, up to 4,096 query
 // rows (native/src/token_executor.h:863-909).
+#include "rope.cuh"
 #include "tc_common.cuh"
 #include "ifab_kernels.h"
 
@@ -42,6 +43,9 @@ struct FaParams {
   int m, ctx, kv_group, pos0, window;
   int q_head_stride, k_head_stride, vt_head_stride, vt_row0;
   float scale_log2;                          // softmax scale * log2(e)
+  int e;                                     // value columns per head that are stored, at column h * e (<= 128)
+  const float* sink;                         // [H]: exp(sink) joins the denominator of the head; or null
+  const bf16* gate; long ldg; int gate_act;  // the result is multiplied by act(gate [m, H * e]); or null
   uint32_t* status; uint32_t spin_limit;
 };
 
@@ -51,23 +55,25 @@ struct Bars {
   int abort_flag;
 };
 
-template <int P1, int P2>
+// SPLIT: the weights P enter P V as two bf16 terms (rounded value + remainder), so they keep ~16 bits instead of 8
+template <int P1, int P2, bool SPLIT>
 struct Layout {
   static constexpr int NQ = P1 + P2;                       // 64-column panels of Q and of a K tile
   static constexpr int Q_OFF = 0;
   static constexpr int K_OFF = Q_OFF + NQ * PANEL_BYTES;   // two stages
   static constexpr int V_OFF = K_OFF + 2 * NQ * PANEL_BYTES;
   static constexpr int P_OFF = V_OFF + PV_PANELS * PANEL_BYTES;
-  static constexpr int BAR_OFF = P_OFF + PV_PANELS * PANEL_BYTES;
+  static constexpr int PL_OFF = P_OFF + PV_PANELS * PANEL_BYTES;       // remainder of P
+  static constexpr int BAR_OFF = PL_OFF + (SPLIT ? PV_PANELS * PANEL_BYTES : 0);
   static constexpr int XCH_OFF = BAR_OFF + 256;            // [2 parities][2 column halves][128 rows] tagged 8-byte words: the two threads of a row
   static constexpr int SMEM = XCH_OFF + 2 * PARTS * 128 * 8 + 1024;
 };
 
-template <int P1, int P2>
+template <int P1, int P2, bool SPLIT>
 __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                                                             const __grid_constant__ CUtensorMap tmap_k2, const __grid_constant__ CUtensorMap tmap_vt,
                                                             FaParams p) {
-  using L = Layout<P1, P2>;
+  using L = Layout<P1, P2, SPLIT>;
   constexpr int NQ = L::NQ;
   extern __shared__ unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -173,6 +179,11 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
         const uint64_t da = umma_desc_sw128(pa + pp * PANEL_BYTES), db = umma_desc_sw128(va + pp * PANEL_BYTES);
 #pragma unroll
         for (int k = 0; k < 4; ++k) umma_bf16(tmem + O_COL, da + (uint64_t)(2 * k), db + (uint64_t)(2 * k), idesc, j > 0 || pp > 0 || k > 0);
+        if (SPLIT) {
+          const uint64_t dl = umma_desc_sw128(pa + (L::PL_OFF - L::P_OFF) + pp * PANEL_BYTES);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) umma_bf16(tmem + O_COL, dl + (uint64_t)(2 * k), db + (uint64_t)(2 * k), idesc, true);
+        }
       }
       umma_commit(&B->o_full);
       umma_commit(&B->v_empty);
@@ -244,7 +255,7 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
       const float m_new = moved ? tile_max : m_ref;
       const float corr = (moved && m_ref != -INFINITY) ? exp2f(m_ref - m_new) : 1.f;
       float sum[4] = {0.f, 0.f, 0.f, 0.f};
-      uint4 packed[HK / 8];
+      uint4 packed[HK / 8], rest[SPLIT ? HK / 8 : 1];
 #pragma unroll
       for (int g = 0; g < HK / 8; ++g) {
         float e[8];
@@ -254,6 +265,13 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
           sum[i & 3] += e[i];
         }
         packed[g] = pack8(e);
+        if (SPLIT) {
+          float r8[8];
+          unpack8(packed[g], r8);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) r8[i] = e[i] - r8[i];
+          rest[SPLIT ? g : 0] = pack8(r8);
+        }
       }
       if (j > 0) {
         // P_{j-1} V_{j-1} has completed: the P buffer is free and O is at rest until the next product is issued
@@ -275,6 +293,10 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
       // 8 keys = one 16-byte chunk of this row's 128-byte line; chunk c sits at position c ^ (row % 8)
 #pragma unroll
       for (int g = 0; g < HK / 8; ++g) *reinterpret_cast<uint4*>(prow + (((chunk0 + g) ^ (r & 7)) << 4)) = packed[g];
+      if (SPLIT) {
+#pragma unroll
+        for (int g = 0; g < HK / 8; ++g) *reinterpret_cast<uint4*>(prow + (L::PL_OFF - L::P_OFF) + (((chunk0 + g) ^ (r & 7)) << 4)) = rest[SPLIT ? g : 0];
+      }
       l_run = l_run * corr + ((sum[0] + sum[1]) + (sum[2] + sum[3]));
       m_ref = m_new;
       fence_proxy_async_smem();       // the tensor core reads P through the async proxy
@@ -304,14 +326,31 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
     if (!ok) {
       if (lane == 0) fail();
     } else if (q0 + r < p.m) {
+      if (p.sink) l_run += exp2f(p.sink[h] * 1.4426950408889634f - m_ref);
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      bf16* dst = p.out + (long)(q0 + r) * p.ldo + (long)h * DV + half * HV;
+      const int c0 = half * HV;
+      bf16* dst = p.out + (long)(q0 + r) * p.ldo + (long)h * p.e + c0;
+      const bf16* gr = p.gate ? p.gate + (long)(q0 + r) * p.ldg + (long)h * p.e + c0 : nullptr;
+      const bool wide = ((p.e | (int)(p.ldo & 7) | (p.gate ? (int)(p.ldg & 7) : 0)) & 7) == 0 && (reinterpret_cast<uintptr_t>(p.gate) & 15) == 0;
 #pragma unroll
       for (int c = 0; c < HV; c += 8) {
+        if (c0 + c >= p.e) break;
         float t8[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) t8[i] = o[c + i] * inv;
-        *reinterpret_cast<uint4*>(dst + c) = pack8(t8);
+        if (wide) {
+          if (gr) {
+            float g8[8];
+            unpack8(*reinterpret_cast<const uint4*>(gr + c), g8);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) t8[i] *= activate(g8[i], p.gate_act);
+          }
+          *reinterpret_cast<uint4*>(dst + c) = pack8(t8);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            if (c0 + c + i < p.e) dst[c + i] = __float2bfloat16_rn(gr ? t8[i] * activate(__bfloat162float(gr[c + i]), p.gate_act) : t8[i]);
+        }
       }
     }
   }
@@ -323,12 +362,12 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
   }
 }
 
-template <int P1, int P2>
+template <int P1, int P2, bool SPLIT = false>
 int launch_fa(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tk2, const CUtensorMap& tv, const FaParams& p, int H, cudaStream_t s) {
-  auto k = fa_prefill_kernel<P1, P2>;
-  if (int rc = opt_in_smem(k, Layout<P1, P2>::SMEM)) return rc;
+  auto k = fa_prefill_kernel<P1, P2, SPLIT>;
+  if (int rc = opt_in_smem(k, Layout<P1, P2, SPLIT>::SMEM)) return rc;
   dim3 grid((p.m + BQ - 1) / BQ, H);
-  return launch_chain(k, grid, dim3(THREADS), (size_t)Layout<P1, P2>::SMEM, s, tq, tk, tk2, tv, p);
+  return launch_chain(k, grid, dim3(THREADS), (size_t)Layout<P1, P2, SPLIT>::SMEM, s, tq, tk, tk2, tv, p);
 }
 
 }  // namespace
@@ -356,10 +395,29 @@ extern "C" int ifab_fa_prefill_bf16(const void* q, long ldq, int q_head_stride, 
   }
   if (int rc = make_tmap_bf16_2d(&tv, vt, (uint64_t)vt_rows, (uint64_t)ctx, (uint64_t)ldvt, DV)) return rc;
   FaParams p{(bf16*)out, ldo, m, ctx, kv_group, pos0, window, q_head_stride, k_head_stride, vt_head_stride, vt_row0,
-             scale * 1.4426950408889634f, status, 4000000u};
+             scale * 1.4426950408889634f, DV, nullptr, nullptr, 0, 0, status, 4000000u};
   cudaStream_t s = (cudaStream_t)stream;
   if (d1 == 128 && d2 == 64) return launch_fa<2, 1>(tq, tk, tk2, tv, p, H, s);
   if (d1 == 128 && d2 == 0) return launch_fa<2, 0>(tq, tk, tk2, tv, p, H, s);
   if (d1 == 64 && d2 == 64) return launch_fa<1, 1>(tq, tk, tk2, tv, p, H, s);
   return launch_fa<1, 0>(tq, tk, tk2, tv, p, H, s);
+}
+
+// Windowed grouped-query form with softmax weights of 16 bits instead of 8 in the value product, a sink logit per head, an output gate,
+// and value heads of any width: q [m, H * d] and k [ctx, G * d] with d in {64, 128} columns per head (narrower heads are zero-padded by
+// the caller), vt [G * 128, ldvt >= ctx] (rows past a narrower value head are zero), out and gate [m, H * e], e <= 128.
+extern "C" int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const void* vt, long ldvt, void* out, long ldo, int m, int ctx, int H,
+                                   int kv_group, int d, int e, int pos0, int window, float scale, const float* sink, const void* gate, long ldg, int gate_act,
+                                   uint32_t* status, void* stream) {
+  if (m < 1 || ctx < 1 || H < 1 || kv_group < 1 || H % kv_group || pos0 < 0 || pos0 + m > ctx || window < 0) return -1;
+  if ((d != 64 && d != 128) || e < 1 || e > DV || ldq % 8 || ldk % 8 || ldvt % 8 || ldvt < ctx) return -1;
+  const int G = H / kv_group;
+  CUtensorMap tq, tk, tv;
+  if (int rc = make_tmap_bf16_2d(&tq, q, (uint64_t)m, (uint64_t)H * d, (uint64_t)ldq, BQ)) return rc;
+  if (int rc = make_tmap_bf16_2d(&tk, k, (uint64_t)ctx, (uint64_t)G * d, (uint64_t)ldk, BKEY)) return rc;
+  if (int rc = make_tmap_bf16_2d(&tv, vt, (uint64_t)G * DV, (uint64_t)ctx, (uint64_t)ldvt, DV)) return rc;
+  FaParams p{(bf16*)out, ldo, m, ctx, kv_group, pos0, window, d, d, DV, 0, scale * 1.4426950408889634f, e, sink, (const bf16*)gate, ldg, gate_act, status,
+             4000000u};
+  cudaStream_t s = (cudaStream_t)stream;
+  return d == 128 ? launch_fa<2, 0, true>(tq, tk, tk, tv, p, H, s) : launch_fa<1, 0, true>(tq, tk, tk, tv, p, H, s);
 }

@@ -288,11 +288,21 @@ int ifab_la_chunks(const float* q, const float* k, const float* v, const int32_t
 /* per-head norm + rotation + cache write, and sliding-window attention with sinks over pages, any head sizes (window_attn.cu) */
 int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, const float* q_gain, const float* k_gain, float eps,
                             int H, int G, int d, int e, int rot, int interleaved, const double* freq, const int32_t* positions, const int32_t* slots,
-                            const int32_t* page_table, int max_pages, int page_tokens, int num_pages, void* q_out, long ldq, void* k_cache, void* v_cache,
-                            int T, uint32_t* status, void* stream);
-int ifab_window_attn(const void* q, long ldq, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,
+                            const int32_t* page_table, int max_pages, int page_tokens, int num_pages, void* q_out, long ldq, int q_stride, void* k_cache,
+                            void* v_cache, int T, uint32_t* status, void* stream);
+int ifab_window_attn(const void* q, long ldq, int q_stride, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,
                      const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int H, int G, int d, int e, int window, float scale,
                      const float* sink, const void* gate, long ldg, int gate_act, void* out, long ldo, int T, uint32_t* status, void* stream);
+/* operands of the tensor-core windowed attention: keys / values first .. first + n - 1 of a sequence, heads zero-padded to dp / 128 columns */
+int ifab_ctx_gather_pad(const void* k_cache, const void* v_cache, const int32_t* page_table, int slot, int max_pages, int page_tokens, int num_pages,
+                        int first, int n, int rows, int G, int d, int dp, int e, void* k, void* vt, long ldvt, uint32_t* status, void* stream);
+int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const void* vt, long ldvt, void* out, long ldo, int m, int ctx, int H,
+                        int kv_group, int d, int e, int pos0, int window, float scale, const float* sink, const void* gate, long ldg, int gate_act,
+                        uint32_t* status, void* stream);
+int ifab_gqa_window_attention(const void* q, long ldq, const void* k_cache, const void* v_cache, const int32_t* positions, const int32_t* slots,
+                              const int32_t* page_table, int max_pages, int page_tokens, int num_pages, float scale, int window, const float* sink,
+                              const void* gate, long ldg, int gate_act, int T, int Hq, int Hkv, int head_dim, int keys_per_split, int max_splits,
+                              float* scratch, uint64_t scratch_bytes, void* out, long ldo, uint32_t* status, void* stream);
 /* indexer: q bf16 [T, heads, dim], w f32 [T, heads], keys paged bf16 [pages, page_tokens, dim]; scores = scratch f32 [T, ctx];
  * out int32 [T, topk]: the top-k key positions (<= the query position) in ascending order, -1 padded */
 int ifab_sparse_index(const void* q, const float* w, const void* keys, const int32_t* positions, const int32_t* slots,

@@ -21,7 +21,7 @@ struct QkParams {
   const double* freq;
   const int32_t *positions, *slots, *page_table;
   int max_pages, page_tokens, num_pages;
-  void* q_out; long ldq;
+  void* q_out; long ldq; int q_stride;      // columns from one query head to the next (>= d)
   void *k_cache, *v_cache;
   int T;
   uint32_t* status;
@@ -56,7 +56,7 @@ __global__ void __launch_bounds__(128) qk_norm_rope_write_kernel(QkParams p) {
   }
   const bool is_q = h < p.H;
   const A* src = is_q ? row + p.q_off + (long)h * p.d : row + p.k_off + (long)(h - p.H) * p.d;
-  A* dst = is_q ? reinterpret_cast<A*>(p.q_out) + (long)t * p.ldq + (long)h * p.d : reinterpret_cast<A*>(p.k_cache) + (dst_row * p.G + h - p.H) * p.d;
+  A* dst = is_q ? reinterpret_cast<A*>(p.q_out) + (long)t * p.ldq + (long)h * p.q_stride : reinterpret_cast<A*>(p.k_cache) + (dst_row * p.G + h - p.H) * p.d;
   const float* gain = is_q ? p.q_gain : p.k_gain;
   float inv = 1.f;
   if (gain) {
@@ -89,8 +89,46 @@ struct WinParams {
   const float* sink;             // [H] or null
   const void* gate; long ldg; int gate_act;
   void* out; long ldo;
+  int q_stride;
   uint32_t* status;
 };
+
+// Keys and values first .. first + n - 1 of one sequence out of its pages: k [rows, G * dp] (columns d .. dp - 1 of a head zero) and
+// transposed values vt [G * 128, ld] (rows e .. 127 of a head zero), rows / columns from n on zero - the operands of the tensor-core
+// attention. grid (ceil(rows / 32), G): one CTA per 32 keys of a head, values turned through shared memory.
+__global__ void __launch_bounds__(256) ctx_gather_pad_kernel(const bf16* k_cache, const bf16* v_cache, const int32_t* page_table, int slot, int max_pages,
+                                                             int page_tokens, int num_pages, int first, int n, int G, int d, int dp, int e, bf16* k,
+                                                             bf16* vt, long ldvt, uint32_t* status) {
+  __shared__ bf16 tile[32][128 + 2];
+  __shared__ long src_row[32];
+  grid_dep_launch();
+  grid_dep_wait();
+  const int j0 = blockIdx.x * 32, g = blockIdx.y, t = threadIdx.x;
+  if (t < 32) {
+    long row = -1;
+    if (j0 + t < n) {
+      const int pos = first + j0 + t, lp = pos / page_tokens;
+      const int page = lp < max_pages ? page_table[(long)slot * max_pages + lp] : -1;
+      if (page >= 0 && page < num_pages) row = (long)page * page_tokens + pos % page_tokens;
+      else if (status) atomicOr(status, IFAB_STATUS_BAD_INDEX);
+    }
+    src_row[t] = row;
+  }
+  __syncthreads();
+  const bf16 zero = __float2bfloat16_rn(0.f);
+  for (int i = t; i < 32 * dp; i += 256) {
+    const int kk = i / dp, c = i - kk * dp;
+    const long row = src_row[kk];
+    k[(long)(j0 + kk) * G * dp + (long)g * dp + c] = (row >= 0 && c < d) ? k_cache[(row * G + g) * d + c] : zero;
+  }
+  for (int i = t; i < 32 * 128; i += 256) {
+    const int kk = i >> 7, c = i & 127;
+    const long row = src_row[kk];
+    tile[kk][c] = (row >= 0 && c < e) ? v_cache[(row * G + g) * e + c] : zero;
+  }
+  __syncthreads();
+  for (int c = t >> 5; c < 128; c += 8) vt[((long)g * 128 + c) * ldvt + j0 + (t & 31)] = tile[t & 31][c];
+}
 
 constexpr int WARPS = 8, KB = 4, EPL = 8;      // lanes own columns lane, lane + 32, ...: up to 256
 
@@ -105,7 +143,7 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
   const int32_t* table = p.page_table + (long)p.slots[t] * p.max_pages;
   const int first = (p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
   float q[EPL], acc[EPL];
-  const A* qr = reinterpret_cast<const A*>(p.q) + (long)t * p.ldq + (long)h * p.d;
+  const A* qr = reinterpret_cast<const A*>(p.q) + (long)t * p.ldq + (long)h * p.q_stride;
 #pragma unroll
   for (int u = 0; u < EPL; ++u) {
     const int c = lane + 32 * u;
@@ -189,23 +227,31 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
 extern "C" int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, const float* q_gain, const float* k_gain,
                                        float eps, int H, int G, int d, int e, int rot, int interleaved, const double* freq, const int32_t* positions,
                                        const int32_t* slots, const int32_t* page_table, int max_pages, int page_tokens, int num_pages, void* q_out,
-                                       long ldq, void* k_cache, void* v_cache, int T, uint32_t* status, void* stream) {
-  if (T < 1 || T > 65535 || H < 1 || G < 1 || d < 1 || e < 1 || rot < 0 || rot % 2 || rot > d || (rot && !freq)) return -1;
+                                       long ldq, int q_stride, void* k_cache, void* v_cache, int T, uint32_t* status, void* stream) {
+  if (T < 1 || T > 65535 || H < 1 || G < 1 || d < 1 || e < 1 || rot < 0 || rot % 2 || rot > d || (rot && !freq) || q_stride < d) return -1;
   QkParams p{proj, ldp, q_off, k_off, v_off, q_gain, k_gain, eps, H, G, d, e, rot, interleaved, freq, positions, slots, page_table, max_pages, page_tokens,
-             num_pages, q_out, ldq, k_cache, v_cache, T, status};
+             num_pages, q_out, ldq, q_stride, k_cache, v_cache, T, status};
   const dim3 grid((H + 2 * G + 3) / 4, T);
   return f32 ? launch_chain(qk_norm_rope_write_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, p)
              : launch_chain(qk_norm_rope_write_kernel<bf16>, grid, dim3(128), 0, (cudaStream_t)stream, p);
 }
 
-extern "C" int ifab_window_attn(const void* q, long ldq, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,
+extern "C" int ifab_window_attn(const void* q, long ldq, int q_stride, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,
                                 const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int H, int G, int d, int e, int window,
                                 float scale, const float* sink, const void* gate, long ldg, int gate_act, void* out, long ldo, int T, uint32_t* status,
                                 void* stream) {
   if (T < 1 || T > 65535 || H < 1 || G < 1 || H % G || d < 1 || d > 256 || e < 1 || e > 256 || window < 0) return -1;
   WinParams p{q, ldq, k_cache, v_cache, positions, slots, page_table, max_pages, page_tokens, num_pages, H, G, d, e, window, scale, sink, gate, ldg, gate_act,
-              out, ldo, status};
+              out, ldo, q_stride, status};
   const dim3 grid(H, T);
   return f32 ? launch_chain(window_attn_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, p)
              : launch_chain(window_attn_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)stream, p);
+}
+
+extern "C" int ifab_ctx_gather_pad(const void* k_cache, const void* v_cache, const int32_t* page_table, int slot, int max_pages, int page_tokens,
+                                   int num_pages, int first, int n, int rows, int G, int d, int dp, int e, void* k, void* vt, long ldvt, uint32_t* status,
+                                   void* stream) {
+  if (n < 1 || rows < n || rows % 32 || slot < 0 || first < 0 || G < 1 || d < 1 || dp < d || e < 1 || e > 128 || ldvt < rows) return -1;
+  return launch_chain(ctx_gather_pad_kernel, dim3(rows / 32, G), dim3(256), 0, (cudaStream_t)stream, (const bf16*)k_cache, (const bf16*)v_cache, page_table,
+                      slot, max_pages, page_tokens, num_pages, first, n, G, d, dp, e, (bf16*)k, (bf16*)vt, ldvt, status);
 }

@@ -28,12 +28,14 @@ import torch
 from ..ops import decode as K
 from ..ops import stream_norm as N
 from ..ops import window_attn as WA
-from ..ops.linear_attn import CHUNK, DecayedMixer, chunk_table, rotary_frequencies
+from ..ops.linear_attn import CHUNK, DecayedMixer, DevicePlan, StepPlan, rotary_frequencies
 from ..parallel.fabric import Fabric
 from ..runtime.paged_state import PagedState
 
 BF16, F32 = torch.bfloat16, torch.float32
-KERNEL_UNITS = ("misc", "post_norm", "linear_f32", "linear_attn", "window_attn", "decode_post_norm", "decode_moe", "sampling", "tc_gemm", "tc_gemm_2sm")
+ATTN_ROWS = 64             # rows per launch of the split-KV attention kernels
+KERNEL_UNITS = ("misc", "post_norm", "linear_f32", "linear_attn", "window_attn", "decode_post_norm", "decode_gqa", "fa_prefill", "decode_moe", "sampling",
+                "tc_gemm", "tc_gemm_2sm")
 
 
 # ---------------------------------------------------------------------------------------------------------------------------
@@ -59,6 +61,24 @@ class MixerConfig:
     @property
     def qk_groups(self) -> int:
         return self.heads if self.recurrent else self.kv_heads
+
+    @property
+    def q_shape(self) -> tuple:
+        """(heads, columns from one query head to the next)."""
+        return self.heads, WA.tile_width(self.dim) if self.tiles else self.dim
+
+    @property
+    def tiles(self) -> bool:
+        """Attention whose heads fit the tiles of the tensor-core kernel."""
+        return not self.recurrent and max(self.dim, self.vdim) <= 128
+
+    @property
+    def ctx_shape(self) -> tuple:
+        return self.kv_heads, self.q_shape[1]
+
+    @property
+    def splits(self) -> int:
+        return WA.split_form(self.heads, self.kv_heads, self.dim, self.vdim, self.window) if not self.recurrent and self.q_shape[1] == self.dim else 0
 
     @property
     def columns(self) -> List[int]:
@@ -264,7 +284,20 @@ class _Rows:
         self.xa, self.y = z(c.width), z(c.width, F32)
         self.proj = z(max(sum(m.columns) for m in mix))
         self.o = z(max([m.heads * m.vdim for m in mix if m.recurrent] or [1]), F32)
-        self.q = z(max([m.heads * m.dim for m in mix if not m.recurrent] or [1]))
+        att = [m for m in mix if not m.recurrent]
+        # queries at the stride of the tensor-core tiles where they have one (padding columns stay zero: one buffer per shape)
+        self.q = {m.q_shape: torch.zeros(rows, m.heads * m.q_shape[1], dtype=A, device=dev) for m in att}
+        splits = [m.heads * m.splits * (m.vdim + 2) for m in att if m.splits]
+        self.split_scratch = torch.empty(min(rows, ATTN_ROWS) * max(splits), dtype=F32, device=dev) if splits and A == BF16 else None
+        self.ctx = {}
+        if chunked and A == BF16:
+            for m in att:
+                if m.tiles:
+                    cap = WA.context_rows(rows, m.window) if m.window else (dec.max_context + 31) // 32 * 32
+                    k0, v0 = self.ctx.get(m.ctx_shape, (None, None))
+                    if k0 is None or k0.shape[0] < cap:
+                        self.ctx[m.ctx_shape] = (torch.zeros(cap, m.kv_heads * m.q_shape[1], dtype=A, device=dev),
+                                                 torch.zeros(m.kv_heads * 128, cap, dtype=A, device=dev))
         self.mixed = {w: z(w) for w in {m.heads * m.vdim for m in mix}}      # one per width: the padding columns must stay zero
         self.act = {w: z(w) for w in {l.ff for l in c.layers if l.ff}}
         self.scratch = None
@@ -359,26 +392,41 @@ class FalinexDecoder:
         return cls(c, w, fabric, **kw)
 
     # -- layers ------------------------------------------------------------------------------------------------------------
-    def _mix(self, B: _Rows, L: dict, m: int, pos, slot, table) -> None:
+    def _mix(self, B: _Rows, L: dict, m: int, pos, slot, plan: Optional[DevicePlan]) -> None:
         """The mixer of one layer between its input projection (``B.proj``) and the operand of its output projection (``B.mixed``);
-        ``table``: chunk table of a packed step, None for decode rows. Recurrent mixers leave their heads in ``B.o``."""
+        ``plan``: of a packed step, None for decode rows. Recurrent mixers leave their heads in ``B.o``."""
         mx, st = L["m"], self.fabric.desc.status
         proj = B.proj[:m]
+        hv = mx.heads * mx.vdim
         if mx.recurrent:
-            o = B.o[:m, :mx.heads * mx.vdim]
-            if table is None:
-                L["rec"].step(proj, L["state"], pos, slot, o)
-            else:
-                L["rec"].chunks(proj, L["state"], pos, table, o, B.scratch)
-        else:
-            q = B.q[:m, :mx.heads * mx.dim]
-            WA.qk_norm_rope_write(proj, L["off"], L["q_norm"], L["k_norm"], self.cfg.eps, heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, vdim=mx.vdim,
-                                  rot=mx.rot_dims, interleaved=True, freq=L["freq"], positions=pos, slots=slot, page_table=self.page_table, q_out=q,
-                                  k_cache=L["k_cache"], v_cache=L["v_cache"], status_ptr=st)
-            WA.window_attn(q, L["k_cache"], L["v_cache"], pos, slot, self.page_table, heads=mx.heads, window=mx.window, scale=mx.scale, sink=L["sink"],
-                           gate=proj[:, L["gate0"]:], gate_act=L["gate_act"], out=B.mixed[mx.heads * mx.vdim][:m], status_ptr=st)
+            o = B.o[:m, :hv]
+            if plan is not None and plan.table is not None:
+                L["rec"].chunks(proj, L["state"], pos, plan.table, o, B.scratch)
+            if plan is None or plan.groups:
+                L["rec"].step(proj, L["state"], pos if plan is None else plan.step_positions, slot, o)
+            return
+        q, out = B.q[mx.q_shape][:m], B.mixed[hv][:m]
+        WA.qk_norm_rope_write(proj, L["off"], L["q_norm"], L["k_norm"], self.cfg.eps, heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, vdim=mx.vdim,
+                              rot=mx.rot_dims, interleaved=True, freq=L["freq"], positions=pos, slots=slot, page_table=self.page_table, q_out=q,
+                              k_cache=L["k_cache"], v_cache=L["v_cache"], status_ptr=st)
+        gate = proj[:, L["gate0"]:L["gate0"] + hv]
+        how = dict(heads=mx.heads, window=mx.window, scale=mx.scale, sink=L["sink"], gate_act=L["gate_act"], status_ptr=st)
+        caches = (L["k_cache"], L["v_cache"])
+        tiled = plan is not None and bool(plan.runs) and mx.tiles and self.dtype == BF16
+        if tiled:
+            for r, n, sl, p0 in plan.runs:
+                k, vt = B.ctx[mx.ctx_shape]
+                WA.fa_window(q[r:r + n], *caches, self.page_table, slot=sl, pos0=p0, ctx_k=k, ctx_vt=vt, out=out[r:r + n], gate=gate[r:r + n], **how)
+        groups = [(r, min(m, r + ATTN_ROWS)) for r in range(0, m, ATTN_ROWS)] if not tiled else plan.groups
+        rest = plan.step_positions if tiled else pos
+        if mx.splits and self.dtype == BF16:
+            for lo, hi in groups:
+                WA.gqa_window(q[lo:hi], *caches, rest[lo:hi], slot[lo:hi], self.page_table, splits=mx.splits, scratch=B.split_scratch, out=out[lo:hi],
+                              gate=gate[lo:hi], **how)
+        elif groups:
+            WA.window_attn(q, *caches, rest, slot, self.page_table, out=out, gate=gate, **how)
 
-    def _layers(self, B: _Rows, m: int, tok, pos, slot, table, final: bool, probe: Optional[list] = None) -> None:
+    def _layers(self, B: _Rows, m: int, tok, pos, slot, plan: Optional[DevicePlan], final: bool, probe: Optional[list] = None) -> None:
         """All layers over ``m`` rows as separate row operators and matrix products; the residual ends in ``B.x``, and with ``final`` the
         normalised rows for the output matrix in ``B.xa``."""
         c, st, W = self.cfg, self.fabric.desc.status, self.cfg.width
@@ -389,7 +437,7 @@ class FalinexDecoder:
             hv = mx.heads * mx.vdim
             last = i + 1 == len(self.layers) and final
             N.linear(xa, L["in"], B.proj[:m, :L["cols"]], status_ptr=st)
-            self._mix(B, L, m, pos, slot, table)
+            self._mix(B, L, m, pos, slot, plan)
             if mx.recurrent:
                 N.group_norm_gate(B.o[:m, :hv], B.proj[:m, L["gate0"]:L["gate0"] + hv], L["gate_act"], c.eps, B.mixed[hv][:m], L["groups"], L["gain"])
             N.linear(B.mixed[hv][:m], L["o"], y, status_ptr=st)
@@ -464,7 +512,8 @@ class FalinexDecoder:
 
 class FalinexRows:
     """Packed-step executor: up to ``max_rows`` rows of any sequences (portions of prompts, decode rows), rows of one sequence
-    consecutive and in position order, as one matrix-matrix pass."""
+    consecutive and in position order, as one matrix-matrix pass. Steps without a long run and of at most ``graph_rows_max`` rows
+    (a decode row per running sequence) replay a CUDA graph per row count."""
 
     packed = True              # the engine hands over the rows of a whole step
     batch_threshold = 8
@@ -473,20 +522,40 @@ class FalinexRows:
         self.dec, self.M = dec, max_rows
         self.B = _Rows(dec, max_rows, True)
         dev = dec.fabric.device
-        self.positions = torch.zeros(max_rows, dtype=torch.int32, device=dev)
-        self.launches = 0
+        self.graph_rows_max = min(64, max_rows)
+        self.use_graphs = True
+        self._static = torch.zeros(3, self.graph_rows_max, dtype=torch.int32, device=dev)
+        self._graphs: Dict[int, torch.cuda.CUDAGraph] = {}
 
-    def plan(self, slots: List[int]) -> torch.Tensor:
-        """Host-side chunk table of a step's rows (int32 ``[n, 4]``); uploaded with the step's control inputs."""
-        return chunk_table(slots)
+    def plan(self, slots: List[int], positions: List[int]) -> StepPlan:
+        return StepPlan(slots, positions, group=ATTN_ROWS)
 
-    def forward_rows(self, tokens: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, select: torch.Tensor, plan: torch.Tensor,
+    def _run(self, tokens, positions, slots, plan: StepPlan, control, probe) -> None:
+        d, m = self.dec, tokens.numel()
+        if plan.runs or m > self.graph_rows_max or not self.use_graphs or probe is not None:
+            d._layers(self.B, m, tokens, positions, slots, plan.bind(control, positions), False, probe)
+            return
+        st = self._static[:, :m]
+        st[0].copy_(tokens)
+        st[1].copy_(positions)
+        st[2].copy_(slots)
+        g = self._graphs.get(m)
+        if g is not None:
+            g.replay()
+            return
+        d._layers(self.B, m, *st, None, False)             # the real run of this step (and the warm-up of the capture)
+        torch.cuda.synchronize()
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):                          # records only: no state is touched a second time
+            d._layers(self.B, m, *st, None, False)
+        self._graphs[m] = g
+
+    def forward_rows(self, tokens: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, select: torch.Tensor, plan: StepPlan, control: torch.Tensor,
                      probe: Optional[list] = None) -> torch.Tensor:
-        """f32 logits ``[len(select), vocab]`` of rows ``select``; ``plan`` on the device."""
-        d, c = self.dec, self.dec.cfg
-        m = tokens.numel()
-        assert 1 <= m <= self.M
-        d._layers(self.B, m, tokens, positions, slots, plan, False, probe)
+        """f32 logits ``[len(select), vocab]`` of rows ``select``; ``control``: ``plan.control`` on the device."""
+        d, c, m = self.dec, self.dec.cfg, tokens.numel()
+        assert 1 <= m <= self.M and plan.rows == m
+        self._run(tokens, positions, slots, plan, control, probe)
         xn = torch.zeros(select.numel(), self.B.xa.shape[1], dtype=d.dtype, device=tokens.device)
         N.rms_rows(self.B.x[:m], d.final_norm, c.eps, xn, select.to(torch.int32))
         logits = torch.empty(select.numel(), c.vocab, dtype=F32, device=tokens.device)
@@ -498,7 +567,8 @@ class FalinexRows:
         d, m, dev = self.dec, tokens.numel(), tokens.device
         pos = torch.arange(pos0, pos0 + m, dtype=torch.int32, device=dev)
         sl = torch.full((m,), slot, dtype=torch.int32, device=dev)
-        logits = self.forward_rows(tokens, pos, sl, torch.tensor([m - 1], device=dev), self.plan([slot] * m).to(dev))
+        plan = self.plan([slot] * m, list(range(pos0, pos0 + m)))
+        logits = self.forward_rows(tokens, pos, sl, torch.tensor([m - 1], device=dev), plan, plan.control.to(dev))
         if d.logits is not None:
             d.logits[:1].copy_(logits)
         K.sample_topk(logits, d.fabric, top_k=1, inv_temperature=d.inv_temp[:1], scratch=d.sample_scratch, out_ids=d.next_ids[:1])

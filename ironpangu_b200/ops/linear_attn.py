@@ -2,7 +2,7 @@
 per-sequence f32 states, for any head sizes."""
 from __future__ import annotations
 
-from typing import List, Optional, Sequence
+from typing import Optional, Sequence
 
 import torch
 
@@ -23,19 +23,52 @@ def decay_powers(decay: Sequence[float], device) -> torch.Tensor:
     return torch.tensor([[float(d) ** n for n in range(CHUNK + 1)] for d in decay], dtype=torch.float64).float().to(device)
 
 
-def chunk_table(slots: Sequence[int]) -> torch.Tensor:
-    """Chunks of a packed step: runs of equal consecutive slots (one sequence's rows in position order), cut every CHUNK rows.
-    int32 ``[n, 4]`` on the host: first row, rows, slot, flags (1: first chunk of the run, 2: last)."""
-    out: List[List[int]] = []
-    i, n = 0, len(slots)
-    while i < n:
-        j = i
-        while j < n and slots[j] == slots[i]:
-            j += 1
-        for r in range(i, j, CHUNK):
-            out.append([r, min(CHUNK, j - r), slots[i], (1 if r == i else 0) | (2 if r + CHUNK >= j else 0)])
-        i = j
-    return torch.tensor(out, dtype=torch.int32)
+class StepPlan:
+    """How the rows of a packed step are run: runs of equal consecutive slots (one sequence's rows, in position order) of more than
+    ``short`` rows go by chunks, the others through the decode kernels.
+
+    ``chunks``: ``[first row, rows, slot, flags]`` (1: first chunk of its run, 2: last); ``runs``: ``(first row, rows, slot, first
+    position)`` of the long runs; ``groups``: row ranges ``[lo, hi)`` of at most ``group`` rows that hold every short row. ``control`` is what
+    the device needs of it (int32, host): the chunk table, then - when there are short rows beside long runs - the positions with
+    those of the long runs replaced by -1, so that the decode kernels skip them."""
+
+    def __init__(self, slots: Sequence[int], positions: Sequence[int], short: int = 4, group: int = 64):
+        n = len(slots)
+        self.rows, self.chunks, self.runs, self.groups = n, [], [], []
+        step = list(positions)
+        i = 0
+        while i < n:
+            j = i
+            while j < n and slots[j] == slots[i]:
+                j += 1
+            if j - i > short:
+                self.runs.append((i, j - i, slots[i], positions[i]))
+                for r in range(i, j, CHUNK):
+                    self.chunks.append([r, min(CHUNK, j - r), slots[i], (1 if r == i else 0) | (2 if r + CHUNK >= j else 0)])
+                step[i:j] = [-1] * (j - i)
+            i = j
+        i = 0
+        while i < n:
+            if step[i] < 0:
+                i += 1
+                continue
+            hi = min(n, i + group)
+            last = max(r for r in range(i, hi) if step[r] >= 0)
+            self.groups.append((i, last + 1))
+            i = last + 1
+        flat = [v for c in self.chunks for v in c]
+        self.masked = bool(self.runs) and bool(self.groups)
+        self.control = torch.tensor(flat + (step if self.masked else []) or [0], dtype=torch.int32)
+
+    def bind(self, control: torch.Tensor, positions: torch.Tensor) -> "DevicePlan":
+        """The plan over its control words on the device."""
+        k = 4 * len(self.chunks)
+        return DevicePlan(self, control[:k].view(-1, 4) if k else None, control[k:k + self.rows] if self.masked else positions)
+
+
+class DevicePlan:
+    def __init__(self, plan: StepPlan, table: Optional[torch.Tensor], step_positions: torch.Tensor):
+        self.table, self.step_positions, self.runs, self.groups = table, step_positions, plan.runs, plan.groups
 
 
 class DecayedMixer:
@@ -61,7 +94,7 @@ class DecayedMixer:
                                        slots.data_ptr(), out.data_ptr(), out.stride(0), proj.shape[0], _s()), "la_step")
 
     def chunks(self, proj: torch.Tensor, state: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scratch) -> None:
-        """Prompts: the chunks of ``table`` (see :func:`chunk_table`, on the device). ``scratch``: ``(q, k, v, cstate)`` f32 buffers of at
+        """Prompts: the chunks of ``table`` (``StepPlan.chunks``, on the device). ``scratch``: ``(q, k, v, cstate)`` f32 buffers of at
         least ``rows * H * d``, the same, ``rows * H * e`` and ``chunks * H * d * e`` elements."""
         T = proj.shape[0]
         q, k, v, cs = scratch

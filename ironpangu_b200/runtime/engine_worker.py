@@ -96,6 +96,8 @@ class BatchEngine:
         self.rows = decoder.T
         self.prefill = prefill
         self.packed = bool(getattr(prefill, "packed", False))
+        if self.packed:
+            prefill.use_graphs = use_graphs
         self.paged = getattr(decoder, "state_manager", None)
         # one CUDA graph per launch-group width: a decoder step is a few hundred launches, which cost more host time through
         # Python than the kernels take on the device
@@ -363,9 +365,10 @@ class BatchEngine:
         sel = torch.tensor((pick + asked) or [n - 1], device=dev.device)
         if self.packed:
             with self.transfers.scope("control_input"):
-                plan = self.transfers.upload(self.prefill.plan([r[2] for r in part]).pin_memory(), d.tokens.device)
-            self.audit_counters["h2d_bytes"] += 4 * plan.numel()
-            logits = self.prefill.forward_rows(dev[0], dev[1], dev[2], sel, plan)
+                plan = self.prefill.plan([r[2] for r in part], [r[1] for r in part])
+                control = self.transfers.upload(plan.control.pin_memory(), d.tokens.device)
+            self.audit_counters["h2d_bytes"] += 4 * control.numel()
+            logits = self.prefill.forward_rows(dev[0], dev[1], dev[2], sel, plan, control)
         else:
             logits = self.prefill.forward_rows(dev[0], dev[1], dev[2], sel)
         for i, j in enumerate(asked):
