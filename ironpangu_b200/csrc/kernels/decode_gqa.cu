@@ -212,18 +212,17 @@ __global__ void gqa_merge_kernel(GqaParams p, bf16* out, long ldo) {
   int ns = (n + p.kps - 1) / p.kps;
   if (ns > p.max_splits) ns = p.max_splits;
   const float* base = p.scratch + ((long)t * p.Hq + h) * p.max_splits * (HD + 2);
-  if (threadIdx.x == 0) {
-    float M = -INFINITY;
-    for (int s = 0; s < ns; ++s) M = fmaxf(M, base[(long)s * (HD + 2) + HD]);
+  if (threadIdx.x < 32) {      // up to 64 splits: two per lane
+    const int s0 = threadIdx.x, s1 = threadIdx.x + 32;
+    const float m0 = s0 < ns ? base[(long)s0 * (HD + 2) + HD] : -INFINITY, m1 = s1 < ns ? base[(long)s1 * (HD + 2) + HD] : -INFINITY;
+    const float l0 = s0 < ns ? base[(long)s0 * (HD + 2) + HD + 1] : 0.f, l1 = s1 < ns ? base[(long)s1 * (HD + 2) + HD + 1] : 0.f;
+    float M = warp_max(fmaxf(m0, m1));
     if (p.sink) M = fmaxf(M, p.sink[h]);
-    float L = p.sink ? __expf(p.sink[h] - M) : 0.f;
-    for (int s = 0; s < ns; ++s) {
-      const float ms = base[(long)s * (HD + 2) + HD];
-      const float w = (ms == -INFINITY) ? 0.f : __expf(ms - M);
-      wgt[s] = w;
-      L += w * base[(long)s * (HD + 2) + HD + 1];
-    }
-    Ls = L;
+    const float w0 = m0 == -INFINITY ? 0.f : __expf(m0 - M), w1 = m1 == -INFINITY ? 0.f : __expf(m1 - M);
+    wgt[s0] = w0;
+    wgt[s1] = w1;
+    const float L = warp_sum(w0 * l0 + w1 * l1) + (p.sink ? __expf(p.sink[h] - M) : 0.f);
+    if (threadIdx.x == 0) Ls = L;
   }
   __syncthreads();
   const float invL = Ls > 0.f ? 1.f / Ls : 0.f;
@@ -231,7 +230,7 @@ __global__ void gqa_merge_kernel(GqaParams p, bf16* out, long ldo) {
     float v = 0.f;
     for (int s = 0; s < ns; ++s) v += wgt[s] * base[(long)s * (HD + 2) + c];
     v *= invL;
-    if (p.gate) v *= activate(__bfloat162float(p.gate[(long)t * p.ldg + (long)h * HD + c]), p.gate_act);
+    if (p.gate) v *= activate<true>(__bfloat162float(p.gate[(long)t * p.ldg + (long)h * HD + c]), p.gate_act);
     out[(long)t * ldo + (long)h * HD + c] = __float2bfloat16_rn(v);
   }
 }

@@ -96,7 +96,7 @@ __device__ __forceinline__ void stage_operand(const Params& p, bf16* xs, float* 
           for (int i = 0; i < 4; ++i) {
             f[i] *= inv[t * groups + (c + i) / n];
             if (p.gain) f[i] *= p.gain[c + i];
-            f[i] *= activate(__bfloat162float(p.gate[r * p.ldg + c + i]), p.gate_act);
+            f[i] *= activate<true>(__bfloat162float(p.gate[r * p.ldg + c + i]), p.gate_act);
           }
         }
       }
@@ -137,7 +137,7 @@ __global__ void __launch_bounds__(256) gemv_operand_kernel(Params p) {
 #pragma unroll
       for (int t = 0; t < T; ++t) {
         if (t0 + t >= p.T) continue;
-        const float v = activate(acc[r][t], p.act);
+        const float v = activate<true>(acc[r][t], p.act);
         if (p.out_f32) reinterpret_cast<float*>(p.z)[(long)(t0 + t) * p.ldz + n0 + r] = v;
         else reinterpret_cast<bf16*>(p.z)[(long)(t0 + t) * p.ldz + n0 + r] = __float2bfloat16_rn(v);
       }

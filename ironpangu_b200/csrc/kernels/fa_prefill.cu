@@ -343,13 +343,13 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
             float g8[8];
             unpack8(*reinterpret_cast<const uint4*>(gr + c), g8);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) t8[i] *= activate(g8[i], p.gate_act);
+            for (int i = 0; i < 8; ++i) t8[i] *= activate<true>(g8[i], p.gate_act);
           }
           *reinterpret_cast<uint4*>(dst + c) = pack8(t8);
         } else {
 #pragma unroll
           for (int i = 0; i < 8; ++i)
-            if (c0 + c + i < p.e) dst[c + i] = __float2bfloat16_rn(gr ? t8[i] * activate(__bfloat162float(gr[c + i]), p.gate_act) : t8[i]);
+            if (c0 + c + i < p.e) dst[c + i] = __float2bfloat16_rn(gr ? t8[i] * activate<true>(__bfloat162float(gr[c + i]), p.gate_act) : t8[i]);
         }
       }
     }

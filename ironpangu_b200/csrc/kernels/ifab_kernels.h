@@ -277,17 +277,22 @@ int ifab_gemv_post_norm(const float* y, long ldy, const float* norm_w, float eps
 int ifab_gemv_group_norm(const float* o, long ldo, const float* gain, float eps, int groups, const void* gate, long ldg, int gate_act, const void* w,
                          void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream);
 int ifab_gemv_act(const void* x, long ldx, const void* w, void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream);
-/* linear attention with a fixed decay per head over a packed projection row (linear_attn.cu); state f32 [slots, H, d, e], powers f32 [H, 65] */
-int ifab_la_step(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, int H, int d, int e, int rot, int interleaved, const double* freq,
+/* linear attention with a fixed decay per head over a packed projection row (linear_attn.cu); state f32 [slots, H, e, d], powers f32 [H, 129],
+ * rope float2 [T, rot / 2] of ifab_rope_table */
+int ifab_rope_table(const int32_t* positions, const double* freq, void* cs, int T, int pairs, void* stream);
+int ifab_la_step(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, int H, int d, int e, int rot, int interleaved, const void* rope,
                  int act, float k_scale, const float* powers, float* state, const int32_t* positions, const int32_t* slots, float* o, long ldo, int T,
                  void* stream);
 int ifab_la_prepare(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, int H, int d, int e, int rot, int interleaved,
-                    const double* freq, int act, float k_scale, const int32_t* positions, float* q, float* k, float* v, int T, void* stream);
+                    const void* rope, int act, float k_scale, float* q, float* k, float* v, int T, void* stream);
 int ifab_la_chunks(const float* q, const float* k, const float* v, const int32_t* chunks, int n, const int32_t* positions, int H, int d, int e,
                    const float* powers, float* cstate, uint64_t cstate_bytes, float* state, float* o, long ldo, void* stream);
+int ifab_la_tiles(const void* proj, long ldp, int q_off, int k_off, int v_off, int H, int d, int e, int rot, int interleaved, const void* rope, int act,
+                  float k_scale, const float* powers, const int32_t* chunks, int n, const int32_t* positions, float* cstate, uint64_t cstate_bytes,
+                  float* state, float* o, long ldo, const void* gate, long ldg, int gate_act, void* y, long ldy, float eps, uint32_t* status, void* stream);
 /* per-head norm + rotation + cache write, and sliding-window attention with sinks over pages, any head sizes (window_attn.cu) */
 int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, const float* q_gain, const float* k_gain, float eps,
-                            int H, int G, int d, int e, int rot, int interleaved, const double* freq, const int32_t* positions, const int32_t* slots,
+                            int H, int G, int d, int e, int rot, int interleaved, const void* rope, const int32_t* positions, const int32_t* slots,
                             const int32_t* page_table, int max_pages, int page_tokens, int num_pages, void* q_out, long ldq, int q_stride, void* k_cache,
                             void* v_cache, int T, uint32_t* status, void* stream);
 int ifab_window_attn(const void* q, long ldq, int q_stride, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,

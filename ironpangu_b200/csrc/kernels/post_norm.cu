@@ -143,7 +143,7 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* o, lo
   for (int c = i0; c < n; c += TPG) {
     float v = r[c] * inv;
     if (w) v *= w[(long)g * n + c];
-    y[(long)t * ldy + (long)g * n + c] = from_f32<A>(v * activate(to_f32(gate[(long)t * ldg + (long)g * n + c]), act));
+    y[(long)t * ldy + (long)g * n + c] = from_f32<A>(v * activate<sizeof(A) == 2>(to_f32(gate[(long)t * ldg + (long)g * n + c]), act));
   }
 }
 
@@ -155,7 +155,7 @@ __global__ void __launch_bounds__(256) gate_rows_kernel(const A* o, long ldo, in
   const int t = blockIdx.x;
   for (int c = threadIdx.x; c < H * n; c += blockDim.x) {
     const int h = c / n, j = c - h * n;
-    y[(long)t * ldy + c] = from_f32<A>(to_f32(o[(long)t * ldo + (long)h * head_stride + j]) * activate(to_f32(gate[(long)t * ldg + c]), act));
+    y[(long)t * ldy + c] = from_f32<A>(to_f32(o[(long)t * ldo + (long)h * head_stride + j]) * activate<sizeof(A) == 2>(to_f32(gate[(long)t * ldg + c]), act));
   }
 }
 

@@ -11,6 +11,12 @@ __device__ __forceinline__ void rope_angle(int pos, double freq, float* c, float
   sincosf((float)a, s, c);
 }
 
+// (cos, sin) of pair i for a row of the step: tables float2 [rows, pairs] made once per step (ifab_rope_table)
+struct RopeTable {
+  const float2* cs;      // [rows, rot / 2]
+  int rot, interleaved;  // rotated columns of a head (0: none), pair layout
+};
+
 // columns of pair i among the first `rot` columns of a head: (i, i + rot / 2), or (2 i, 2 i + 1) when interleaved
 __device__ __forceinline__ void rope_pair(int i, int rot, int interleaved, int* a, int* b) {
   *a = interleaved ? 2 * i : i;
@@ -27,15 +33,32 @@ __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <>
 __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
-__device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float gelu_tanh_f32(float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+// rotated value of column c of a head (`head[c']` holds the plain values); columns from rt.rot on pass
+template <typename A>
+__device__ __forceinline__ float rotated(const RopeTable& rt, const float2* row_cs, const A* head, int c) {
+  const int i = rt.interleaved ? c >> 1 : (c < rt.rot / 2 ? c : c - rt.rot / 2);
+  int ia, ib;
+  rope_pair(i, rt.rot, rt.interleaved, &ia, &ib);
+  const float2 t = row_cs[i];
+  const float a = to_f32(head[ia]), b = to_f32(head[ib]);
+  return c == ia ? a * t.x - b * t.y : b * t.x + a * t.y;
+}
+
+// FAST: for results that are rounded to bf16 (the hardware exponential, ~1e-6 relative); GELU's 0.5 (1 + tanh u) is sigmoid(2 u)
+template <bool FAST = false>
+__device__ __forceinline__ float sigmoid_f32(float x) {
+  return FAST ? __fdividef(1.f, 1.f + __expf(-x)) : 1.f / (1.f + expf(-x));      // __fdividef gives 0 for a huge divisor: the limit
+}
+template <bool FAST = false>
+__device__ __forceinline__ float gelu_tanh_f32(float z) { return z * sigmoid_f32<FAST>(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
 
 // elementwise activations by number: 0 none, 1 SiLU, 2 sigmoid, 3 GELU (tanh form)
+template <bool FAST = false>
 __device__ __forceinline__ float activate(float z, int act) {
   switch (act) {
-    case 1: return z * sigmoid_f32(z);
-    case 2: return sigmoid_f32(z);
-    case 3: return gelu_tanh_f32(z);
+    case 1: return z * sigmoid_f32<FAST>(z);
+    case 2: return sigmoid_f32<FAST>(z);
+    case 3: return gelu_tanh_f32<FAST>(z);
     default: return z;
   }
 }

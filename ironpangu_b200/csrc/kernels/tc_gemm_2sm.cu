@@ -93,7 +93,7 @@ __device__ __forceinline__ void store_row32_2(const Gemm2Params& p, int row, int
   }
   if (p.act) {
 #pragma unroll
-    for (int i = 0; i < 32; ++i) v[i] = activate(v[i], p.act);
+    for (int i = 0; i < 32; ++i) v[i] = activate<true>(v[i], p.act);
   }
   if (p.out_f32) {
     float* out = reinterpret_cast<float*>(p.c) + (long)row * p.ldc + col;

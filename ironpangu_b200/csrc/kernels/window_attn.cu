@@ -2,7 +2,7 @@
 // size independent), bf16 or f32 activations and caches.
 //
 //   qk_norm_rope_write_kernel  RMS norm per head of q and k with a shared gain, rotation of the first `rot` columns (either pair
-//                              layout, angles in double), q to its own rows, k and v into the pages of their sequence
+//                              layout), q to its own rows, k and v into the pages of their sequence
 //   window_attn_kernel         one CTA per (row, query head): row at position i sees keys j with 0 <= i - j < window; scores,
 //                              weights and sums in f32; the denominator also holds exp(sink_h). Optional output gate
 //
@@ -14,11 +14,22 @@ using namespace ifab;
 
 namespace {
 
+// cs [T, pairs]: cos and sin of position * freq[i]
+__global__ void __launch_bounds__(128) rope_table_kernel(const int32_t* positions, const double* freq, float2* cs, int T, int pairs) {
+  grid_dep_launch();
+  grid_dep_wait();
+  const long i = (long)blockIdx.x * 128 + threadIdx.x;
+  if (i >= (long)T * pairs) return;
+  float2 v;
+  rope_angle(positions[i / pairs], freq[i % pairs], &v.x, &v.y);
+  cs[i] = v;
+}
+
 struct QkParams {
   const void* proj; long ldp; int q_off, k_off, v_off;
   const float *q_gain, *k_gain; float eps;           // gains may be null: no norm
-  int H, G, d, e, rot, interleaved;
-  const double* freq;
+  int H, G, d, e;
+  RopeTable rope;
   const int32_t *positions, *slots, *page_table;
   int max_pages, page_tokens, num_pages;
   void* q_out; long ldq; int q_stride;      // columns from one query head to the next (>= d)
@@ -67,16 +78,16 @@ __global__ void __launch_bounds__(128) qk_norm_rope_write_kernel(QkParams p) {
     }
     inv = 1.f / sqrtf(warp_sum(ss) / (float)p.d + p.eps);
   }
-  for (int i = lane; i < p.rot / 2; i += 32) {
+  const float2* cs = p.rope.cs + (long)t * (p.rope.rot / 2);
+  for (int i = lane; i < p.rope.rot / 2; i += 32) {
     int ia, ib;
-    rope_pair(i, p.rot, p.interleaved, &ia, &ib);
-    float cs, sn;
-    rope_angle(pos, p.freq[i], &cs, &sn);
+    rope_pair(i, p.rope.rot, p.rope.interleaved, &ia, &ib);
+    const float2 r = cs[i];
     const float a = to_f32(src[ia]) * inv * (gain ? gain[ia] : 1.f), b = to_f32(src[ib]) * inv * (gain ? gain[ib] : 1.f);
-    dst[ia] = from_f32<A>(a * cs - b * sn);
-    dst[ib] = from_f32<A>(b * cs + a * sn);
+    dst[ia] = from_f32<A>(a * r.x - b * r.y);
+    dst[ib] = from_f32<A>(b * r.x + a * r.y);
   }
-  for (int c = p.rot + lane; c < p.d; c += 32) dst[c] = from_f32<A>(to_f32(src[c]) * inv * (gain ? gain[c] : 1.f));
+  for (int c = p.rope.rot + lane; c < p.d; c += 32) dst[c] = from_f32<A>(to_f32(src[c]) * inv * (gain ? gain[c] : 1.f));
 }
 
 struct WinParams {
@@ -217,7 +228,7 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
 #pragma unroll
     for (int w = 0; w < WARPS; ++w) v = fmaf(wgt[w], sm_acc[w][c], v);
     v *= inv;
-    if (p.gate) v *= activate(to_f32(reinterpret_cast<const A*>(p.gate)[(long)t * p.ldg + (long)h * p.e + c]), p.gate_act);
+    if (p.gate) v *= activate<sizeof(A) == 2>(to_f32(reinterpret_cast<const A*>(p.gate)[(long)t * p.ldg + (long)h * p.e + c]), p.gate_act);
     reinterpret_cast<A*>(p.out)[(long)t * p.ldo + (long)h * p.e + c] = from_f32<A>(v);
   }
 }
@@ -225,11 +236,11 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
 }  // namespace
 
 extern "C" int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, const float* q_gain, const float* k_gain,
-                                       float eps, int H, int G, int d, int e, int rot, int interleaved, const double* freq, const int32_t* positions,
+                                       float eps, int H, int G, int d, int e, int rot, int interleaved, const void* rope, const int32_t* positions,
                                        const int32_t* slots, const int32_t* page_table, int max_pages, int page_tokens, int num_pages, void* q_out,
                                        long ldq, int q_stride, void* k_cache, void* v_cache, int T, uint32_t* status, void* stream) {
-  if (T < 1 || T > 65535 || H < 1 || G < 1 || d < 1 || e < 1 || rot < 0 || rot % 2 || rot > d || (rot && !freq) || q_stride < d) return -1;
-  QkParams p{proj, ldp, q_off, k_off, v_off, q_gain, k_gain, eps, H, G, d, e, rot, interleaved, freq, positions, slots, page_table, max_pages, page_tokens,
+  if (T < 1 || T > 65535 || H < 1 || G < 1 || d < 1 || e < 1 || rot < 0 || rot % 2 || rot > d || (rot && !rope) || q_stride < d) return -1;
+  QkParams p{proj, ldp, q_off, k_off, v_off, q_gain, k_gain, eps, H, G, d, e, {(const float2*)rope, rot, interleaved}, positions, slots, page_table, max_pages, page_tokens,
              num_pages, q_out, ldq, q_stride, k_cache, v_cache, T, status};
   const dim3 grid((H + 2 * G + 3) / 4, T);
   return f32 ? launch_chain(qk_norm_rope_write_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, p)
@@ -254,4 +265,10 @@ extern "C" int ifab_ctx_gather_pad(const void* k_cache, const void* v_cache, con
   if (n < 1 || rows < n || rows % 32 || slot < 0 || first < 0 || G < 1 || d < 1 || dp < d || e < 1 || e > 128 || ldvt < rows) return -1;
   return launch_chain(ctx_gather_pad_kernel, dim3(rows / 32, G), dim3(256), 0, (cudaStream_t)stream, (const bf16*)k_cache, (const bf16*)v_cache, page_table,
                       slot, max_pages, page_tokens, num_pages, first, n, G, d, dp, e, (bf16*)k, (bf16*)vt, ldvt, status);
+}
+
+extern "C" int ifab_rope_table(const int32_t* positions, const double* freq, void* cs, int T, int pairs, void* stream) {
+  if (T < 1 || pairs < 1) return -1;
+  return launch_chain(rope_table_kernel, dim3((unsigned)(((long)T * pairs + 127) / 128)), dim3(128), 0, (cudaStream_t)stream, positions, freq, (float2*)cs, T,
+                      pairs);
 }

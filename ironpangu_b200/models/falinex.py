@@ -28,13 +28,13 @@ import torch
 from ..ops import decode as K
 from ..ops import stream_norm as N
 from ..ops import window_attn as WA
-from ..ops.linear_attn import CHUNK, DecayedMixer, DevicePlan, StepPlan, rotary_frequencies
+from ..ops.linear_attn import CHUNK, TILE, DecayedMixer, DevicePlan, RotaryTables, StepPlan
 from ..parallel.fabric import Fabric
 from ..runtime.paged_state import PagedState
 
 BF16, F32 = torch.bfloat16, torch.float32
 ATTN_ROWS = 64             # rows per launch of the split-KV attention kernels
-KERNEL_UNITS = ("misc", "post_norm", "linear_f32", "linear_attn", "window_attn", "decode_post_norm", "decode_gqa", "fa_prefill", "decode_moe", "sampling",
+KERNEL_UNITS = ("misc", "post_norm", "linear_f32", "linear_attn", "linear_attn_tc", "window_attn", "decode_post_norm", "decode_gqa", "fa_prefill", "decode_moe", "sampling",
                 "tc_gemm", "tc_gemm_2sm")
 
 
@@ -300,13 +300,15 @@ class _Rows:
                                                  torch.zeros(m.kv_heads * 128, cap, dtype=A, device=dev))
         self.mixed = {w: z(w) for w in {m.heads * m.vdim for m in mix}}      # one per width: the padding columns must stay zero
         self.act = {w: z(w) for w in {l.ff for l in c.layers if l.ff}}
+        self.rotary = RotaryTables([(m.rot_dims, m.rot_base) for m in mix], rows, dev)
         self.scratch = None
         rec = [m for m in mix if m.recurrent]
         if chunked and rec:
             f = lambda n: torch.empty(n, dtype=F32, device=dev)
-            nch = rows // CHUNK + dec.num_slots + 1                  # chunks of a step: whole ones and one ragged end per sequence
-            self.scratch = (f(rows * max(m.heads * m.dim for m in rec)), f(rows * max(m.heads * m.dim for m in rec)),
-                            f(rows * max(m.heads * m.vdim for m in rec)), f(nch * max(m.heads * m.dim * m.vdim for m in rec)))
+            nch = rows // dec.chunk + dec.num_slots + 1              # chunks of a step: whole ones and one ragged end per sequence
+            wide = 0 if dec.tensor_recurrence else rows              # rows of q, k, v of the f32 form
+            self.scratch = (f(wide * max(m.heads * m.dim for m in rec)), f(wide * max(m.heads * m.dim for m in rec)),
+                            f(wide * max(m.heads * m.vdim for m in rec)), f(nch * max(m.heads * m.dim * m.vdim for m in rec)))
 
 
 class FalinexDecoder:
@@ -324,6 +326,9 @@ class FalinexDecoder:
         per_slot = (max_context + c.page_tokens - 1) // c.page_tokens
         self.num_pages = (pool_tokens + c.page_tokens - 1) // c.page_tokens if pool_tokens else per_slot * num_slots
         self._load(weights)
+        # prompts: recurrences on the tensor cores in bf16 when every head fits a tile, f32 products otherwise
+        self.tensor_recurrence = dtype == BF16 and all(max(l.mixer.dim, l.mixer.vdim) <= 128 for l in c.layers if l.mixer.recurrent)
+        self.chunk = TILE if self.tensor_recurrence else CHUNK
         es = torch.empty((), dtype=dtype).element_size()
         att = [l.mixer for l in c.layers if not l.mixer.recurrent]
         rec = [l.mixer for l in c.layers if l.mixer.recurrent]
@@ -377,12 +382,11 @@ class FalinexDecoder:
                 if m.recurrent:
                     ret = m.kind == "retention"
                     S["rec"] = DecayedMixer(heads=m.heads, dim=m.dim, vdim=m.vdim, decay=m.decay, offsets=off, device=dev, rot_dims=m.rot_dims,
-                                            rot_base=m.rot_base, interleaved=False, act=None if ret else "silu", k_scale=m.dim ** -0.5 if ret else 1.0)
+                                            interleaved=False, act=None if ret else "silu", k_scale=m.dim ** -0.5 if ret else 1.0)
                     S["gain"] = None if ret else vec(p + "mix.norm")
                     S["groups"], S["gate_act"] = (m.heads, "silu") if ret else (1, "sigmoid")
                 else:
-                    S.update(q_norm=vec(p + "mix.q.norm"), k_norm=vec(p + "mix.k.norm"), sink=vec(p + "mix.sink"), gate_act="sigmoid",
-                             freq=rotary_frequencies(m.rot_dims, m.rot_base, dev) if m.rot_dims else None)
+                    S.update(q_norm=vec(p + "mix.q.norm"), k_norm=vec(p + "mix.k.norm"), sink=vec(p + "mix.sink"), gate_act="sigmoid")
                 built[j] = S
             self.layers.append(dict(built[j]))        # shared tensors, own state
 
@@ -392,22 +396,34 @@ class FalinexDecoder:
         return cls(c, w, fabric, **kw)
 
     # -- layers ------------------------------------------------------------------------------------------------------------
-    def _mix(self, B: _Rows, L: dict, m: int, pos, slot, plan: Optional[DevicePlan]) -> None:
+    def _mix(self, B: _Rows, L: dict, m: int, pos, slot, plan: Optional[DevicePlan], norm: bool = True) -> None:
         """The mixer of one layer between its input projection (``B.proj``) and the operand of its output projection (``B.mixed``);
-        ``plan``: of a packed step, None for decode rows. Recurrent mixers leave their heads in ``B.o``."""
+        ``plan``: of a packed step, None for decode rows. Without ``norm`` recurrent mixers leave their heads in ``B.o`` instead (the fused
+        output projection norms and gates them)."""
         mx, st = L["m"], self.fabric.desc.status
         proj = B.proj[:m]
         hv = mx.heads * mx.vdim
+        rope = B.rotary.get(mx.rot_dims, mx.rot_base)
         if mx.recurrent:
-            o = B.o[:m, :hv]
-            if plan is not None and plan.table is not None:
-                L["rec"].chunks(proj, L["state"], pos, plan.table, o, B.scratch)
-            if plan is None or plan.groups:
-                L["rec"].step(proj, L["state"], pos if plan is None else plan.step_positions, slot, o)
+            o, rec, gate = B.o[:m, :hv], L["rec"], proj[:, L["gate0"]:L["gate0"] + hv]
+            long = plan is not None and plan.table is not None
+            alone = long and not plan.groups                       # every row belongs to a long run
+            if long and self.tensor_recurrence:
+                if alone and L["groups"] == mx.heads and L["gain"] is None:
+                    rec.tiles(proj, L["state"], pos, plan.table, rope, B.scratch[3], gated=B.mixed[hv][:m], gate=gate, gate_act=L["gate_act"], eps=self.cfg.eps,
+                              status_ptr=st)
+                    return
+                rec.tiles(proj, L["state"], pos, plan.table, rope, B.scratch[3], out=o, status_ptr=st)
+            elif long:
+                rec.chunks(proj, L["state"], pos, plan.table, rope, o, B.scratch)
+            if not alone:
+                rec.step(proj, L["state"], pos if plan is None else plan.step_positions, slot, rope, o)
+            if norm:
+                N.group_norm_gate(o, gate, L["gate_act"], self.cfg.eps, B.mixed[hv][:m], L["groups"], L["gain"])
             return
         q, out = B.q[mx.q_shape][:m], B.mixed[hv][:m]
         WA.qk_norm_rope_write(proj, L["off"], L["q_norm"], L["k_norm"], self.cfg.eps, heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, vdim=mx.vdim,
-                              rot=mx.rot_dims, interleaved=True, freq=L["freq"], positions=pos, slots=slot, page_table=self.page_table, q_out=q,
+                              rot=mx.rot_dims, interleaved=True, rope=rope, positions=pos, slots=slot, page_table=self.page_table, q_out=q,
                               k_cache=L["k_cache"], v_cache=L["v_cache"], status_ptr=st)
         gate = proj[:, L["gate0"]:L["gate0"] + hv]
         how = dict(heads=mx.heads, window=mx.window, scale=mx.scale, sink=L["sink"], gate_act=L["gate_act"], status_ptr=st)
@@ -432,14 +448,13 @@ class FalinexDecoder:
         c, st, W = self.cfg, self.fabric.desc.status, self.cfg.width
         x, xa, y = B.x[:m, :W], B.xa[:m], B.y[:m, :W]
         N.embed_rows(tok, self.embed, x, xa, status_ptr=st)
+        B.rotary.fill(pos)
         for i, L in enumerate(self.layers):
             mx = L["m"]
             hv = mx.heads * mx.vdim
             last = i + 1 == len(self.layers) and final
             N.linear(xa, L["in"], B.proj[:m, :L["cols"]], status_ptr=st)
             self._mix(B, L, m, pos, slot, plan)
-            if mx.recurrent:
-                N.group_norm_gate(B.o[:m, :hv], B.proj[:m, L["gate0"]:L["gate0"] + hv], L["gate_act"], c.eps, B.mixed[hv][:m], L["groups"], L["gain"])
             N.linear(B.mixed[hv][:m], L["o"], y, status_ptr=st)
             N.post_norm_add(y, L["norm1"], c.eps, x, xa, self.final_norm if last and not L["ff"] else None)
             if L["ff"]:
@@ -455,6 +470,7 @@ class FalinexDecoder:
         c = self.cfg
         x, x2, xa, y = B.x[:n], B.x2[:n], B.xa[:n], B.y[:n]
         N.embed_rows(tok, self.embed, x, xa, status_ptr=self.fabric.desc.status)
+        B.rotary.fill(pos)
         owed = None                            # gain of the sublayer output in y that the residual still lacks
         for L in self.layers:
             mx = L["m"]
@@ -464,7 +480,7 @@ class FalinexDecoder:
             else:
                 N.gemv_post_norm(y, owed, c.eps, x, x2, L["in"], proj)
                 x, x2 = x2, x
-            self._mix(B, L, n, pos, slot, None)
+            self._mix(B, L, n, pos, slot, None, norm=False)
             if mx.recurrent:
                 N.gemv_group_norm(B.o[:n, :hv], proj[:, L["gate0"]:], L["gate_act"], c.eps, L["o"], y, L["groups"], L["gain"])
             else:
@@ -528,7 +544,7 @@ class FalinexRows:
         self._graphs: Dict[int, torch.cuda.CUDAGraph] = {}
 
     def plan(self, slots: List[int], positions: List[int]) -> StepPlan:
-        return StepPlan(slots, positions, group=ATTN_ROWS)
+        return StepPlan(slots, positions, group=ATTN_ROWS, chunk=self.dec.chunk)
 
     def _run(self, tokens, positions, slots, plan: StepPlan, control, probe) -> None:
         d, m = self.dec, tokens.numel()

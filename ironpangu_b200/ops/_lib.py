@@ -67,7 +67,10 @@ _SIGS = {
     "ifab_gemv_group_norm": [_P, c_long, _P, c_float, c_int, _P, c_long, c_int, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
     "ifab_gemv_act": [_P, c_long, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
     "ifab_la_step": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_float, _P, _P, _P, _P, _P, c_long, c_int, _P],
-    "ifab_la_prepare": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_float, _P, _P, _P, _P, c_int, _P],
+    "ifab_la_prepare": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_float, _P, _P, _P, c_int, _P],
+    "ifab_rope_table": [_P, _P, _P, c_int, c_int, _P],
+    "ifab_la_tiles": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_float, _P, _P, c_int, _P, _P, c_u64, _P, _P, c_long,
+                      _P, c_long, c_int, _P, c_long, c_float, _P, _P],
     "ifab_la_chunks": [_P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, _P, _P, c_u64, _P, _P, c_long, _P],
     "ifab_qk_norm_rope_write": [_P, c_long, c_int, c_int, c_int, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_int, c_int,
                                 c_int, _P, c_long, c_int, _P, _P, c_int, _P, _P],

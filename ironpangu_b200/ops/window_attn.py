@@ -11,13 +11,14 @@ from .stream_norm import ACTIVATIONS, _f32, _p, _s
 
 
 def qk_norm_rope_write(proj: torch.Tensor, offsets, q_gain: Optional[torch.Tensor], k_gain: Optional[torch.Tensor], eps: float, *, heads: int, kv_heads: int,
-                       dim: int, vdim: int, rot: int, interleaved: bool, freq: Optional[torch.Tensor], positions: torch.Tensor, slots: torch.Tensor,
+                       dim: int, vdim: int, rot: int, interleaved: bool, rope: Optional[torch.Tensor], positions: torch.Tensor, slots: torch.Tensor,
                        page_table: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, status_ptr=None) -> None:
     """Packed projection rows -> normalised, rotated queries in ``q_out`` (``[T, heads * stride]``, stride >= dim) and normalised, rotated keys / plain values in the pages
-    (``k_cache`` ``[pages, page_tokens, kv_heads, dim]``, ``v_cache`` ``[..., vdim]``)."""
+    (``k_cache`` ``[pages, page_tokens, kv_heads, dim]``, ``v_cache`` ``[..., vdim]``). ``rope``: (cos, sin) of the rows, ``[T, rot / 2, 2]``
+    (``linear_attn.RotaryTables``)."""
     pages, pt = k_cache.shape[:2]
     check(_lib.load().ifab_qk_norm_rope_write(proj.data_ptr(), proj.stride(0), _f32(proj), *offsets, _p(q_gain), _p(k_gain), eps, heads, kv_heads, dim, vdim, rot,
-                                              int(interleaved), _p(freq), positions.data_ptr(), slots.data_ptr(), page_table.data_ptr(), page_table.shape[1],
+                                              int(interleaved), _p(rope), positions.data_ptr(), slots.data_ptr(), page_table.data_ptr(), page_table.shape[1],
                                               pt, pages, q_out.data_ptr(), q_out.stride(0), q_out.shape[1] // heads, k_cache.data_ptr(), v_cache.data_ptr(), proj.shape[0], status_ptr,
                                               _s()), "qk_norm_rope_write")
 

@@ -127,7 +127,7 @@ def falinex_arm(size, prompt: int, chunk: int, batches: List[int], t: Timer, pk)
         pos = torch.full((n,), prompt, dtype=torch.int32, device=dev)
         sl = torch.arange(n, dtype=torch.int32, device=dev)
         state = heads * hd * hd * 4
-        group(f"recurrence step, {n} sequences", rec, lambda L: dec._mix(B, L, n, pos, sl, None), n * (2 * state + 4 * HV * es))
+        group(f"recurrence step, {n} sequences", rec, lambda L: dec._mix(B, L, n, pos, sl, None, norm=False), n * (2 * state + 4 * HV * es))
         keys = min(window, prompt + 1)
         group(f"window attention (norm, rotation, cache write, attention, gate), {n} sequences", att, lambda L: dec._mix(B, L, n, pos, sl, None),
               n * keys * 2 * kv * hd * es + n * (heads + 2 * kv) * hd * es * 2)
@@ -146,9 +146,9 @@ def falinex_arm(size, prompt: int, chunk: int, batches: List[int], t: Timer, pk)
     sl = torch.zeros(m, dtype=torch.int32, device=dev)
     plan = rows.plan([0] * m, list(range(prompt - m, prompt)))
     dp = plan.bind(plan.control.to(dev), pos)
-    C = 64
+    C = dec.chunk
     flops = 2.0 * m * heads * (C * hd + 2 * hd * hd + C * hd)
-    group(f"recurrence chunks, {m} rows", rec, lambda L: dec._mix(B, L, m, pos, sl, dp), m * (3 * HV * es + 4 * HV), flops)
+    group(f"recurrence chunks, head norm, gate, {m} rows", rec, lambda L: dec._mix(B, L, m, pos, sl, dp), m * 5 * HV * es, flops)
     pairs = _visible(m, prompt - m, window)
     group(f"window attention, {m} rows", att, lambda L: dec._mix(B, L, m, pos, sl, dp), m * (2 * heads + 2 * kv) * hd * es, 4.0 * pairs * heads * hd)
     group(f"output norm + residual, {m} rows", rec, lambda L: N.post_norm_add(B.y[:m], L["norm1"], 1e-5, B.x[:m], B.xa[:m]), m * width * (4 + 4 + 4 + 2))
