@@ -48,15 +48,18 @@ class DecodeEngine:
         return None
 
     def _select(self, table, variant, capture):
+        """``(graph, ran)``: the step's graph, and whether the step has just been executed as the warm-up of its capture (a step
+        advances recurrent state, so it must not run a second time)."""
         d = self.dec
-        if variant not in table:
+        ran = variant not in table
+        if ran:
             if variant is not None:
                 d.fuse_override = variant
             capture()
             table[variant] = self._graph if table is self._graphs else self._feedback_graph
             if variant is not None:
                 d.fuse_override = None
-        return table[variant]
+        return table[variant], ran
 
     def _capture(self):
         d = self.dec
@@ -71,18 +74,21 @@ class DecodeEngine:
             d.forward(1)
         self._graph = g
 
-    def _capture_feedback(self):
+    def _feedback_step(self):
         d = self.dec
-        d.forward(1)
+        if hasattr(d, "forward_feedback"):
+            d.forward_feedback(1)
+        else:
+            d.forward(1)
+            d.tokens[:1].copy_(d.next_ids[:1])
+            d.positions[:1].add_(1)
+
+    def _capture_feedback(self):
+        self._feedback_step()
         torch.cuda.synchronize()
         g = torch.cuda.CUDAGraph()
         with torch.cuda.graph(g):
-            if hasattr(d, "forward_feedback"):
-                d.forward_feedback(1)
-            else:
-                d.forward(1)
-                d.tokens[:1].copy_(d.next_ids[:1])
-                d.positions[:1].add_(1)
+            self._feedback_step()
         self._feedback_graph = g
 
     # -- public API --------------------------------------------------------------------------------
@@ -121,8 +127,9 @@ class DecodeEngine:
         with self.transfers.scope("control_input"):
             self.transfers.h2d(self._ctl_dev, self._ctl_host)
         # a capture's warm-up run executes this very step (same token, same position), never a stale one
-        self._graph = self._select(self._graphs, self._variant(self.pos), self._capture)
-        self._graph.replay()
+        self._graph, ran = self._select(self._graphs, self._variant(self.pos), self._capture)
+        if not ran:
+            self._graph.replay()
         with self.transfers.scope("request_output"):
             self.transfers.d2h(self._out_host, self.dec.next_ids[:1])
         torch.cuda.current_stream().synchronize()
@@ -145,8 +152,10 @@ class DecodeEngine:
             d.tokens[:1].fill_(first_token)
             d.positions[:1].fill_(self.pos)
             d.slots[:1].zero_()
-        # warm-up of a capture = the step about to be replayed (same inputs), so it changes no state
-        self._feedback_graph = self._select(self._feedback_graphs, self._variant(self.pos + steps - 1), self._capture_feedback)
-        for _ in range(steps):
+        if steps < 1:
+            return
+        # the warm-up of a capture is the first of these steps
+        self._feedback_graph, ran = self._select(self._feedback_graphs, self._variant(self.pos + steps - 1), self._capture_feedback)
+        for _ in range(steps - 1 if ran else steps):
             self._feedback_graph.replay()
         self.pos += steps
