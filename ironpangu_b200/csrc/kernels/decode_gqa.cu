@@ -197,6 +197,148 @@ __global__ void __launch_bounds__(256) gqa_split_kernel(GqaParams p) {
   }
 }
 
+// The same for groups of up to four query heads: HD / 8 lanes share a key (8 columns, one 16-byte load each), so a warp works on
+// 256 / HD keys at once and a score costs log2(HD / 8) shuffles for all of them; four keys per lane group are in flight, with one update of
+// the running maximum for the four. Every lane group keeps its own maximum, sum and output; they are merged within the warp at the
+// end, then across the warps as above.
+template <int HD, int G>
+__global__ void __launch_bounds__(256, 2) gqa_split_shared_kernel(GqaParams p) {
+  constexpr int C = 8, LP = HD / C, NG = 32 / LP, KB = 4;
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  float* sm_acc = reinterpret_cast<float*>(smem_raw);   // [8][G][HD]
+  float* sm_m = sm_acc + 8 * G * HD;
+  float* sm_l = sm_m + 8 * G;
+  grid_dep_launch();
+  grid_dep_wait();
+  const int split = blockIdx.x, kvh = blockIdx.y, t = blockIdx.z;
+  const int pos = p.positions[t];
+  if (pos < 0) return;
+  int n = pos + 1;
+  if (p.window > 0 && n > p.window) n = p.window;
+  const int first = pos + 1 - n;
+  const int k_begin = split * p.kps;
+  if (k_begin >= n) return;
+  const int k_end = (split == p.max_splits - 1) ? n : min(n, k_begin + p.kps);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = lane / LP, sub = lane % LP;
+  const int slot = p.slots[t];
+  float qf[G][C], acc[G][C], m[G], l[G];
+#pragma unroll
+  for (int g = 0; g < G; ++g) {
+    const bf16* qh = p.q + (long)t * p.ldq + (long)(kvh * G + g) * HD + sub * C;
+#pragma unroll
+    for (int i = 0; i < C; ++i) {
+      qf[g][i] = __bfloat162float(qh[i]) * p.scale;
+      acc[g][i] = 0.f;
+    }
+    m[g] = -INFINITY;
+    l[g] = 0.f;
+  }
+  const long kv_elems = (long)p.Hkv * HD, head = (long)kvh * HD + sub * C;
+  // every lane takes the same number of rounds (the shuffles are warp-wide); a missing key scores -inf
+  for (int k0 = k_begin + warp * NG; k0 < k_end; k0 += 8 * NG * KB) {
+    uint4 kr[KB], vr[KB];
+    bool ok[KB];
+#pragma unroll
+    for (int b = 0; b < KB; ++b) {
+      const int k = k0 + b * 8 * NG + grp;
+      ok[b] = k < k_end;
+      kr[b] = vr[b] = make_uint4(0, 0, 0, 0);
+      if (ok[b]) {
+        const long r = row_of(first + k, slot, p.page_table, p.max_pages, p.page_tokens, p.num_pages);
+        if (r < 0) {
+          if (sub == 0 && p.status) atomicOr(p.status, IFAB_STATUS_BAD_INDEX);
+          ok[b] = false;
+        } else {
+          kr[b] = *reinterpret_cast<const uint4*>(p.k_cache + r * kv_elems + head);
+          vr[b] = *reinterpret_cast<const uint4*>(p.v_cache + r * kv_elems + head);
+        }
+      }
+    }
+    float s[KB][G];
+#pragma unroll
+    for (int b = 0; b < KB; ++b) {
+      float f[8];
+      unpack8(kr[b], f);
+#pragma unroll
+      for (int g = 0; g < G; ++g) {
+        s[b][g] = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s[b][g] = fmaf(qf[g][j], f[j], s[b][g]);
+#pragma unroll
+        for (int o = LP / 2; o > 0; o >>= 1) s[b][g] += __shfl_xor_sync(0xffffffffu, s[b][g], o);
+        if (!ok[b]) s[b][g] = -INFINITY;
+      }
+    }
+#pragma unroll
+    for (int g = 0; g < G; ++g) {
+      const float mn = fmaxf(fmaxf(m[g], fmaxf(s[0][g], s[1][g])), fmaxf(s[2][g], s[3][g]));
+      if (mn > m[g]) {
+        const float corr = __expf(m[g] - mn);
+        l[g] *= corr;
+#pragma unroll
+        for (int i = 0; i < C; ++i) acc[g][i] *= corr;
+        m[g] = mn;
+      }
+#pragma unroll
+      for (int b = 0; b < KB; ++b) {
+        s[b][g] = ok[b] ? __expf(s[b][g] - mn) : 0.f;
+        l[g] += s[b][g];
+      }
+    }
+#pragma unroll
+    for (int b = 0; b < KB; ++b) {
+      float f[8];
+      unpack8(vr[b], f);
+#pragma unroll
+      for (int g = 0; g < G; ++g)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[g][j] = fmaf(s[b][g], f[j], acc[g][j]);
+    }
+  }
+  __syncwarp();
+#pragma unroll
+  for (int g = 0; g < G; ++g) {
+    float M = m[g];
+#pragma unroll
+    for (int o = LP; o < 32; o <<= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+    const float w = m[g] == -INFINITY ? 0.f : __expf(m[g] - M);
+    float L = l[g] * w;
+#pragma unroll
+    for (int o = LP; o < 32; o <<= 1) L += __shfl_xor_sync(0xffffffffu, L, o);
+    if (lane == 0) {
+      sm_m[warp * G + g] = M;
+      sm_l[warp * G + g] = L;
+    }
+#pragma unroll
+    for (int i = 0; i < C; ++i) {
+      float a = acc[g][i] * w;
+#pragma unroll
+      for (int o = LP; o < 32; o <<= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+      if (grp == 0) sm_acc[((long)warp * G + g) * HD + sub * C + i] = a;
+    }
+  }
+  __syncthreads();
+  for (int g = 0; g < G; ++g) {
+    float M = -INFINITY;
+    for (int w = 0; w < 8; ++w) M = fmaxf(M, sm_m[w * G + g]);
+    float wgt[8], L = 0.f;
+    for (int w = 0; w < 8; ++w) {
+      wgt[w] = (sm_m[w * G + g] == -INFINITY) ? 0.f : __expf(sm_m[w * G + g] - M);
+      L += wgt[w] * sm_l[w * G + g];
+    }
+    float* out = p.scratch + (((long)t * p.Hq + kvh * G + g) * p.max_splits + split) * (HD + 2);
+    for (int c = threadIdx.x; c < HD; c += blockDim.x) {
+      float v = 0.f;
+      for (int w = 0; w < 8; ++w) v += wgt[w] * sm_acc[((long)w * G + g) * HD + c];
+      out[c] = v;
+    }
+    if (threadIdx.x == 0) {
+      out[HD] = M;
+      out[HD + 1] = L;
+    }
+  }
+}
+
 // grid (Hq, T), HD threads
 template <int HD>
 __global__ void gqa_merge_kernel(GqaParams p, bf16* out, long ldo) {
@@ -238,7 +380,8 @@ __global__ void gqa_merge_kernel(GqaParams p, bf16* out, long ldo) {
 template <int HD, int G>
 int launch_gqa(const GqaParams& p, bf16* out, long ldo, cudaStream_t s) {
   const size_t smem = (size_t)(8 * G * HD + 16 * G) * sizeof(float);
-  auto k = gqa_split_kernel<HD, G>;
+  constexpr bool shared_keys = HD <= 128 && G <= 4;
+  auto k = shared_keys ? gqa_split_shared_kernel<shared_keys ? HD : 64, shared_keys ? G : 1> : gqa_split_kernel<HD, G>;
   if (int rc = opt_in_smem(k, smem)) return rc;
   dim3 grid(p.max_splits, p.Hkv, p.T);
   if (int rc = launch_chain(k, grid, dim3(256), smem, s, p)) return rc;

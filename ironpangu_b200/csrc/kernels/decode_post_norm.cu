@@ -154,8 +154,9 @@ int launch_one(const Params& p, cudaStream_t s) {
 }
 template <int T, int PRO>
 int by_rows(const Params& p, cudaStream_t s) {
-  if (p.N >= 148 * 8 * 4 * 2) return launch_one<T, 4, PRO>(p, s);
-  if (p.N >= 148 * 8 * 2 * 2) return launch_one<T, 2, PRO>(p, s);
+  // rows per warp: the widest that still gives every SM a CTA (two are resident), so that the grid is one wave
+  if (p.N >= 148 * 8 * 4) return launch_one<T, 4, PRO>(p, s);
+  if (p.N >= 148 * 8 * 2) return launch_one<T, 2, PRO>(p, s);
   return launch_one<T, 1, PRO>(p, s);
 }
 template <int PRO>

@@ -62,11 +62,11 @@ __device__ __forceinline__ void store_row32(const GemmParams& p, int row, int co
   }
 }
 
-template <int BN>
+template <int BN, int ST>
 __global__ void __launch_bounds__(192) tc_gemm_kernel(const __grid_constant__ CUtensorMap tmap_a,
                                                       const __grid_constant__ CUtensorMap tmap_b, GemmParams p) {
   extern __shared__ unsigned char smem_raw[];
-  Pipe<BN> pipe;
+  Pipe<BN, ST> pipe;
   pipe.setup(smem_raw, &tmap_a, &tmap_b);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
@@ -93,12 +93,13 @@ __global__ void __launch_bounds__(192) tc_gemm_kernel(const __grid_constant__ CU
   pipe.teardown();
 }
 
-template <int BN>
+template <int BN, int ST = (BN == 256 ? 4 : BN == 128 ? 6 : BN == 64 ? 8 : 10)>
 int launch(const CUtensorMap& ta, const CUtensorMap& tb, const GemmParams& p, cudaStream_t s) {
-  auto k = tc_gemm_kernel<BN>;
-  if (int rc = opt_in_smem(k, Cfg<BN>::SMEM)) return rc;
+  auto k = tc_gemm_kernel<BN, ST>;
+  constexpr int smem = Cfg<BN, ST>::SMEM;
+  if (int rc = opt_in_smem(k, smem)) return rc;
   dim3 grid((p.N + BN - 1) / BN, (p.M + BM - 1) / BM);
-  return launch_chain(k, grid, dim3(192), (size_t)Cfg<BN>::SMEM, s, ta, tb, p);
+  return launch_chain(k, grid, dim3(192), (size_t)smem, s, ta, tb, p);
 }
 
 }  // namespace
@@ -176,11 +177,19 @@ extern "C" int ifab_gemm_act_bf16(const void* a, long lda, const void* b, long l
     return ifab_gemm_act_bf16_2sm(a, lda, b, ldb, c, ldc, out_f32, residual, ldr, act, tiles > 74, M, N, K, status, stream);
   }
   CUtensorMap ta, tb;
-  const int BN = N > 128 ? 256 : 128;
+  // a single tile row (batched decode) is bound by the stream of B: narrow tiles spread it over the SMs, deep rings keep it in flight
+  int BN = N > 128 ? 256 : 128;
+  if (M <= BM)
+    while (BN > 32 && (N + BN - 1) / BN < 128) BN /= 2;
   if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM)) return rc;
   if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)N, (uint64_t)K, (uint64_t)ldb, (uint32_t)BN)) return rc;
   GemmParams p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, act};
   cudaStream_t s = (cudaStream_t)stream;
-  return BN == 256 ? launch<256>(ta, tb, p, s) : launch<128>(ta, tb, p, s);
+  switch (BN) {
+    case 256: return launch<256>(ta, tb, p, s);
+    case 128: return launch<128>(ta, tb, p, s);
+    case 64: return launch<64>(ta, tb, p, s);
+    default: return launch<32>(ta, tb, p, s);
+  }
 }
 

@@ -35,11 +35,12 @@ def window_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, p
                                        _s()), "window_attn")
 
 
-SPLIT_KEYS = 64            # keys per split of the split-KV decode form
+SPLIT_KEYS = 64            # fewest keys per split of the split-KV decode form
+SPLIT_CTAS = 600           # CTAs the splits of a launch aim at: more rows, longer splits
 
 
 def split_form(heads: int, kv_heads: int, dim: int, vdim: int, window: int) -> int:
-    """Splits of the split-KV decode kernels for this shape, 0 when it needs the general kernel."""
+    """Most splits the split-KV decode kernels take for this shape, 0 when it needs the general kernel."""
     if dim != vdim or dim not in (64, 128, 256) or heads // kv_heads not in (1, 2, 4, 8) or (dim == 256 and heads // kv_heads == 8) or not window:
         return 0
     return max(1, min(64, (window + SPLIT_KEYS - 1) // SPLIT_KEYS))
@@ -48,11 +49,11 @@ def split_form(heads: int, kv_heads: int, dim: int, vdim: int, window: int) -> i
 def gqa_window(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, page_table: torch.Tensor, *,
                heads: int, window: int, scale: float, splits: int, scratch: torch.Tensor, out: torch.Tensor, sink: Optional[torch.Tensor] = None,
                gate: Optional[torch.Tensor] = None, gate_act: Optional[str] = None, status_ptr=None) -> None:
-    """:func:`window_attn` by splits of the window (query heads of a group share the key loads), bf16, shapes of :func:`split_form`."""
+    """:func:`window_attn` by splits of the window (query heads of a group share the key loads), bf16, shapes of :func:`split_form`.
+    ``splits``: the most to use; launches of many rows use fewer, longer ones."""
     pages, pt, G, d = k_cache.shape
-    kps = SPLIT_KEYS
-    while splits * kps < window:
-        kps *= 2
+    splits = max(1, min(splits, SPLIT_CTAS // (q.shape[0] * G)))
+    kps = ((window + splits - 1) // splits + 31) // 32 * 32
     check(_lib.load().ifab_gqa_window_attention(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), positions.data_ptr(), slots.data_ptr(),
                                                 page_table.data_ptr(), page_table.shape[1], pt, pages, scale, window, _p(sink), _p(gate),
                                                 0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], q.shape[0], heads, G, d, kps, splits,
