@@ -28,6 +28,7 @@ struct GemmParams {
   int M, N, K;
   uint32_t* status;
   uint32_t spin_limit;
+  int a_rows;            // rows of A's box
   int act;               // activation of the result (numbers of activate(); 0: none), after the residual
 };
 
@@ -74,7 +75,7 @@ __global__ void __launch_bounds__(192) tc_gemm_kernel(const __grid_constant__ CU
   grid_dep_launch();
   grid_dep_wait();
   if (warp == 0 && lane == 0) {
-    pipe.produce(&tmap_a, &tmap_b, num_kb, m0, n0, -1, p.spin_limit, p.status);
+    pipe.produce(&tmap_a, &tmap_b, num_kb, m0, n0, -1, p.spin_limit, p.status, -1, p.a_rows);
   } else if (warp == 1 && lane == 0) {
     pipe.mma(num_kb, p.spin_limit, p.status);
   } else if (warp >= 2) {
@@ -93,7 +94,7 @@ __global__ void __launch_bounds__(192) tc_gemm_kernel(const __grid_constant__ CU
   pipe.teardown();
 }
 
-template <int BN, int ST = (BN == 256 ? 4 : BN == 128 ? 6 : BN == 64 ? 8 : 10)>
+template <int BN, int ST>
 int launch(const CUtensorMap& ta, const CUtensorMap& tb, const GemmParams& p, cudaStream_t s) {
   auto k = tc_gemm_kernel<BN, ST>;
   constexpr int smem = Cfg<BN, ST>::SMEM;
@@ -177,19 +178,18 @@ extern "C" int ifab_gemm_act_bf16(const void* a, long lda, const void* b, long l
     return ifab_gemm_act_bf16_2sm(a, lda, b, ldb, c, ldc, out_f32, residual, ldr, act, tiles > 74, M, N, K, status, stream);
   }
   CUtensorMap ta, tb;
-  // a single tile row (batched decode) is bound by the stream of B: narrow tiles spread it over the SMs, deep rings keep it in flight
+  // A single tile row (batched decode) is bound by the stream of B: narrow tiles spread it over the SMs, two CTAs on each; the box of A
+  // holds the live rows only.
+  const bool one_row = M <= BM;
   int BN = N > 128 ? 256 : 128;
-  if (M <= BM)
-    while (BN > 32 && (N + BN - 1) / BN < 128) BN /= 2;
-  if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM)) return rc;
+  if (one_row)
+    for (BN = 32; BN < 128 && (N + BN - 1) / BN > 296; BN *= 2) {}
+  const int a_rows = one_row ? (M + 7) / 8 * 8 : BM;
+  if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, (uint32_t)a_rows)) return rc;
   if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)N, (uint64_t)K, (uint64_t)ldb, (uint32_t)BN)) return rc;
-  GemmParams p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, act};
+  GemmParams p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, a_rows, act};
   cudaStream_t s = (cudaStream_t)stream;
-  switch (BN) {
-    case 256: return launch<256>(ta, tb, p, s);
-    case 128: return launch<128>(ta, tb, p, s);
-    case 64: return launch<64>(ta, tb, p, s);
-    default: return launch<32>(ta, tb, p, s);
-  }
+  if (!one_row) return BN == 256 ? launch<256, 4>(ta, tb, p, s) : launch<128, 6>(ta, tb, p, s);
+  return BN == 128 ? launch<128, 3>(ta, tb, p, s) : BN == 64 ? launch<64, 4>(ta, tb, p, s) : launch<32, 5>(ta, tb, p, s);
 }
 

@@ -64,8 +64,8 @@ class MixerConfig:
 
     @property
     def q_shape(self) -> tuple:
-        """(heads, columns from one query head to the next)."""
-        return self.heads, WA.tile_width(self.dim) if self.tiles else self.dim
+        """(heads, columns from one query head to the next, columns of a head)."""
+        return self.heads, WA.tile_width(self.dim) if self.tiles else self.dim, self.dim
 
     @property
     def tiles(self) -> bool:

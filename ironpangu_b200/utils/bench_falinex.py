@@ -175,7 +175,7 @@ def dense_arm(size, params: int, prompt: int, chunk: int, batches: List[int], t:
     from ironpangu_b200.ops import gemm as GM
     from ironpangu_b200.parallel.fabric import Fabric
 
-    width, layers, heads, kv, hd, _, vocab, _ = size
+    width, layers, heads, kv, hd, _, vocab, window = size
     dev = torch.device("cuda", 0)
     cfg = G.DenseConfig(layers=layers, hidden=width, heads=heads, kv_heads=kv, head_dim=hd, ffn=256, vocab=vocab)
     per = (params - cfg.param_count()) / layers / (3 * width)
@@ -213,9 +213,9 @@ def dense_arm(size, params: int, prompt: int, chunk: int, batches: List[int], t:
         ms = t.run(lambda: [fn(l) for l in range(layers)]) / layers
         res["kernels"].append(_line(name, ms, bytes_, flops, pk))
 
-    for n in (1, 64):
+    for n, keys in ((1, prompt + 1), (1, window), (64, prompt + 1), (64, window)):      # also as many keys as the window leaves
         q = torch.zeros(n, (heads + 2 * kv) * hd, dtype=torch.bfloat16, device=dev).normal_()
-        pos = torch.full((n,), prompt, dtype=torch.int32, device=dev)
+        pos = torch.full((n,), keys - 1, dtype=torch.int32, device=dev)
         sl = torch.arange(n, dtype=torch.int32, device=dev)
         out = torch.empty(n, heads * hd, dtype=torch.bfloat16, device=dev)
         scr = torch.empty(n * heads * dec.max_splits * (hd + 2), dtype=torch.float32, device=dev)
@@ -225,7 +225,7 @@ def dense_arm(size, params: int, prompt: int, chunk: int, batches: List[int], t:
             K.gqa_decode_attention(q, dec.k_cache[l], dec.v_cache[l], pos, sl, dec.page_table, heads=heads, kv_heads=kv, head_dim=hd, scale=scale,
                                    keys_per_split=dec.kps, max_splits=dec.max_splits, scratch=scr, out=out, status_ptr=st)
 
-        group(f"attention (rotation, cache write, attention), {n} sequences", attn, n * (prompt + 1) * 2 * kv * hd * es + n * (heads + 2 * kv) * hd * es * 2)
+        group(f"attention (rotation, cache write, attention), {n} sequences, {keys} keys", attn, n * keys * 2 * kv * hd * es + n * (heads + 2 * kv) * hd * es * 2)
     p = lambda l, s: w[f"layers.{l}.{s}"]
     group("qkv projection with norm prologue, 1 row", lambda l: K.gemv(dec.x[:1], p(l, "qkv"), norm_w=p(l, "attn_norm"), eps=cfg.eps, out=dec.qkv[:1]),
           L_bytes(p(0, "qkv")))

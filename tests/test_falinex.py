@@ -455,3 +455,13 @@ def test_trace_replay_program(tmp_path, dtype):
     load = lambda i: torch.from_numpy(np.fromfile(tmp_path / "o" / f"{i}.f32", dtype="<f4")).view(-1, cfg["vocab"])
     assert not (tmp_path / "o" / "1.f32").exists()
     assert logit_error(load(0), wa[[0, 29]]) < lim and logit_error(load(2), torch.stack([wb[11], wa[31], wa[39]])) < lim
+
+
+@pytest.mark.gpu
+def test_worker_preset_and_memory_profile(tmp_path):
+    path = tmp_path / "mem.json"
+    r = subprocess.run([sys.executable, "-m", "ironpangu_b200.runtime.engine_worker", "--model", "falinex-tiny", "--max-num-seqs", "2", "--max-model-len", "128",
+                        "--kv-pool-tokens", "128", "--prefill-chunk", "64", "--memory-profile", str(path), "--profile-only"], capture_output=True, text=True,
+                       timeout=300, cwd=ROOT)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert json.loads(path.read_text())["failed_stage"] is None
