@@ -723,7 +723,7 @@ void DeviceProgram::Impl::dispatch(int T) {
       const int Fs = x.has("shared_weight") ? (int)(dims(x.s("shared_weight") + "|" + x.s("shared_paired_weight"))[0] / 2) : 0;
       const Val& in = V(x.in.at(0));
       kernel(ifab_moe_gate_up_decode(in.ptr, in.ld, norm_w, eps, (const int32_t*)V(x.in[1]).ptr, T, (int)d[2], (int)(d[1] / 2), r.i("topk"), 0, (int)d[0], P(pname),
-                                     shared, Fs, V(k).ptr, st),
+                                     shared, Fs, V(k).ptr, (int)(d[1] / 2), st),
              x.name);
     } else if (x.op == "moe_down_allreduce") {
       const Ins& r = ins[x.in.at(1)];

@@ -110,10 +110,10 @@ struct GateUpParams {
   const bf16* x; long ldx; const bf16* norm_w; float eps;
   const int32_t* ids; int T, D, F, topk, e0, e_local;
   const bf16* w_gu; const bf16* w_sgu; int Fs;
-  bf16* act;
+  bf16* act; int ldact;    // columns from one slot to the next (>= F and Fs)
 };
 
-// grid: (ceil(F/16), T*topk + T). Column y < T*topk is route (t, k); columns after that are the shared
+// grid: (ceil(max(F, Fs)/16), T*topk + T). Column y < T*topk is route (t, k); columns after that are the shared
 // expert of token t. Routes that belong to other ranks exit at once (after the dependency wait).
 __global__ void __launch_bounds__(256) moe_gate_up_kernel(GateUpParams p) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -165,7 +165,7 @@ __global__ void __launch_bounds__(256) moe_gate_up_kernel(GateUpParams p) {
   warp_rows_dot<1, 4>(rows, xs, p.D, acc, pf);
   warp_reduce_acc<1, 4>(acc);
   if (lane == 0) {
-    bf16* out = p.act + ((size_t)t * (p.topk + 1) + slot) * p.F;
+    bf16* out = p.act + ((size_t)t * (p.topk + 1) + slot) * p.ldact;
     out[j0] = __float2bfloat16_rn(silu(bf16_round(acc[0][0])) * bf16_round(acc[2][0]));
     if (j0 + 1 < Fcur) out[j0 + 1] = __float2bfloat16_rn(silu(bf16_round(acc[1][0])) * bf16_round(acc[3][0]));
   }
@@ -176,6 +176,8 @@ struct DownParams {
   const bf16* act; const int32_t* ids; const float* wts;
   int T, D, F, topk, e0, e_local;
   const bf16* w_down; const bf16* w_sdown; int Fs;
+  int ldact; const float* shared_w;               // columns from one slot to the next; weight of the shared expert per row (null: 1)
+  float* y_f32;                                   // [T, D] sums before rounding (one rank), instead of y
   const bf16* residual; long ldr; bf16* y; long ldy;
   FabricView fv; uint64_t* seq; uint32_t* done;
 };
@@ -223,7 +225,7 @@ __global__ void __launch_bounds__(256) moe_down_allreduce_kernel(DownParams p) {
         } else if (slot == p.topk && p.w_sdown != nullptr) {
           local = true;
           w = p.w_sdown;
-          g = 1.f;
+          g = p.shared_w ? p.shared_w[t] : 1.f;
           k = p.Fs;
         }
         const unsigned m = __ballot_sync(0xffffffffu, local);
@@ -256,9 +258,9 @@ __global__ void __launch_bounds__(256) moe_down_allreduce_kernel(DownParams p) {
             const int q = q0 + (int)blockDim.x * j;
             dst[j] = -1;
             if (q < total_c) {
-              const int i = min(q / kch0, n_routes - 1), c = q - s_cbeg[i];
-              v[j] = *reinterpret_cast<const uint4*>(p.act + ((size_t)t * (p.topk + 1) + s_slot[i]) * p.F + c * 8);
-              dst[j] = i * p.F + c * 8;
+              const int i = min(q / kch0, n_routes - 1), c = q - s_cbeg[i];      // only the last route may span more than F
+              v[j] = *reinterpret_cast<const uint4*>(p.act + ((size_t)t * (p.topk + 1) + s_slot[i]) * p.ldact + c * 8);
+              dst[j] = i * p.F + c * 8;                     // the shared expert comes last: it may be wider than F
             }
           }
 #pragma unroll
@@ -271,7 +273,7 @@ __global__ void __launch_bounds__(256) moe_down_allreduce_kernel(DownParams p) {
 #pragma unroll
       for (int r = 0; r < R; ++r) total[r] = 0.f;
       constexpr int MAXC = 6;   // 16-byte chunks per lane and route the per-route form holds in registers (K <= 1536)
-      if ((p.F >> 3) <= 32 * MAXC) {
+      if ((max(p.F, p.Fs) >> 3) <= 32 * MAXC) {
         // One route at a time: weight base, score and activation row are loop invariants, a lane requests its (at most
         // MAXC) chunks of all R rows at once and the chunk loop is straight-line code. The flattened form below spends
         // three times the instructions per chunk on finding out which route a chunk belongs to.
@@ -360,13 +362,20 @@ __global__ void __launch_bounds__(256) moe_down_allreduce_kernel(DownParams p) {
     }
   }
   __syncthreads();
+  if (p.y_f32) {
+    for (int i = threadIdx.x; i < T * RPC; i += blockDim.x) {
+      const int t = i / RPC, c = i % RPC;
+      if (t < p.T && nbase + c < p.D) p.y_f32[(long)t * p.ldy + nbase + c] = slab[i];
+    }
+    return;
+  }
   oneshot_allreduce_slab<T, RPC>(slab, p.fv, p.seq, p.done, nbase, p.T, p.D, p.residual, p.ldr, p.y, p.ldy, nullptr,
                                  &timed_out);
 }
 
 template <int T, int R>
 int launch_down(const DownParams& p, cudaStream_t s) {
-  const size_t smem = (size_t)(p.topk + 1) * p.F * sizeof(bf16);
+  const size_t smem = (size_t)(p.topk * p.F + max(p.F, p.Fs)) * sizeof(bf16);
   auto k = moe_down_allreduce_kernel<T, R>;
   if (int rc = opt_in_smem(k, smem)) return rc;
   dim3 grid((p.D + 8 * R - 1) / (8 * R));
@@ -544,14 +553,36 @@ extern "C" int ifab_router_topk(const void* x, long ldx, const void* norm_w, flo
 
 extern "C" int ifab_moe_gate_up_decode(const void* x, long ldx, const void* norm_w, float eps, const int32_t* ids, int T,
                                        int D, int F, int topk, int e0, int e_local, const void* w_gu,
-                                       const void* w_shared_gu, int Fs, void* act, void* stream) {
-  if (D % 8 != 0 || F % 8 != 0 || Fs % 8 != 0 || Fs > F) return -1;
+                                       const void* w_shared_gu, int Fs, void* act, int ldact, void* stream) {
+  if (D % 8 != 0 || F % 8 != 0 || Fs % 8 != 0 || ldact % 8 != 0 || ldact < F || ldact < Fs) return -1;
   GateUpParams p{(const bf16*)x, ldx, (const bf16*)norm_w, eps, ids, T, D, F, topk, e0, e_local,
-                 (const bf16*)w_gu, (const bf16*)w_shared_gu, Fs, (bf16*)act};
-  dim3 grid((F + 15) / 16, T * topk + T);
+                 (const bf16*)w_gu, (const bf16*)w_shared_gu, Fs, (bf16*)act, ldact};
+  dim3 grid((max(F, w_shared_gu ? Fs : 0) + 15) / 16, T * topk + T);
   const size_t smem = (size_t)D * sizeof(bf16);
   if (int rc = opt_in_smem(moe_gate_up_kernel, smem)) return rc;
   return launch_chain(moe_gate_up_kernel, grid, dim3(256), smem, (cudaStream_t)stream, p);
+}
+
+namespace {
+int run_down(const DownParams& p, cudaStream_t s) {
+  if (p.T <= 1) return dispatch_down<1>(p, s);
+  if (p.T <= 2) return dispatch_down<2>(p, s);
+  if (p.T <= 4) return dispatch_down<4>(p, s);
+  return dispatch_down<8>(p, s);
+}
+}  // namespace
+
+// One rank, f32 result: y [T, ldy] = sum over the chosen experts by weight + shared_w * shared expert. act: slots ldact columns apart (slot topk is the
+// shared expert's)
+extern "C" int ifab_moe_down_f32_decode(const void* act, int ldact, const int32_t* ids, const float* wts, const float* shared_w, int T, int D, int F, int topk,
+                                        int experts, const void* w_down, const void* w_shared_down, int Fs, float* y, long ldy, void* stream) {
+  if (T < 1 || T > 8 || F % 8 != 0 || Fs % 8 != 0 || topk > MAX_TOPK || ldact % 8 != 0 || ldact < F || (w_shared_down && ldact < Fs) || !y) return -1;
+  DownParams p{};
+  p.act = (const bf16*)act; p.ids = ids; p.wts = wts;
+  p.T = T; p.D = D; p.F = F; p.topk = topk; p.e0 = 0; p.e_local = experts;
+  p.w_down = (const bf16*)w_down; p.w_sdown = (const bf16*)w_shared_down; p.Fs = w_shared_down ? Fs : 0;
+  p.ldact = ldact; p.shared_w = shared_w; p.y_f32 = y; p.ldy = ldy;
+  return run_down(p, (cudaStream_t)stream);
 }
 
 extern "C" int ifab_moe_down_allreduce_decode(const void* act, const int32_t* ids, const float* wts, int T, int D, int F,
@@ -559,7 +590,8 @@ extern "C" int ifab_moe_down_allreduce_decode(const void* act, const int32_t* id
                                               const void* w_shared_down, int Fs, const void* residual, long ldr,
                                               void* y, long ldy, const IfabFabric* fab, void* stream) {
   if (T < 1 || T > 8 || F % 8 != 0 || Fs % 8 != 0 || topk > MAX_TOPK || Fs > F) return -1;
-  DownParams p;
+  DownParams p{};
+  p.ldact = F;
   p.act = (const bf16*)act; p.ids = ids; p.wts = wts;
   p.T = T; p.D = D; p.F = F; p.topk = topk; p.e0 = e0; p.e_local = e_local;
   p.w_down = (const bf16*)w_down; p.w_sdown = (const bf16*)w_shared_down; p.Fs = Fs;
@@ -568,11 +600,7 @@ extern "C" int ifab_moe_down_allreduce_decode(const void* act, const int32_t* id
   p.seq = fab->seq; p.done = fab->done;
   if ((size_t)fab->world * T * D * sizeof(uint64_t) > fab->ll_half_bytes) return -3;
   if ((size_t)fab->world * 296 > fab->flag_half_words) return -4;
-  cudaStream_t s = (cudaStream_t)stream;
-  if (T <= 1) return dispatch_down<1>(p, s);
-  if (T <= 2) return dispatch_down<2>(p, s);
-  if (T <= 4) return dispatch_down<4>(p, s);
-  return dispatch_down<8>(p, s);
+  return run_down(p, (cudaStream_t)stream);
 }
 
 extern "C" int ifab_lm_head_argmax(const void* x, long ldx, const void* norm_w, float eps, const void* w, float* logits,

@@ -3,12 +3,15 @@
 // needs no row kernels of its own between its linears:
 //
 //   post norm    x_out = x_in + rms(y) * w, operand bf16(x_out). Every CTA computes the rows it needs (a few KB from L2); the CTAs
-//                of the first column write x_out, which must not be x_in (other CTAs still read that)
+//                of the first column write x_out, which must not be x_in (other CTAs still read that). With a second gain (a norm
+//                ahead of the next sublayer as well) the operand is bf16(rms(x_out) * w2), also stored to xn on request
 //   group norm   operand bf16((o / rms of each group of columns [* gain]) * act(gate)): normalised, gated heads of a recurrent mixer
 //   plain        bf16 rows
 //
-// Epilogue: optional activation, bf16 or f32 result.
+// Epilogue: optional activation, bf16 or f32 result. A router's linear goes on to the selection: the last CTA to finish turns the f32
+// logits into expert ids and weights (moe_select.cuh) and the extra column, when there is one, into the shared expert's weight.
 #include "gemv.cuh"
+#include "moe_select.cuh"
 #include "rope.cuh"
 #include "ifab_kernels.h"
 
@@ -26,11 +29,13 @@ struct Params {
   const bf16* w;
   void* z; long ldz; int out_f32, act;
   int T, N, K;
+  const float* norm2_w; bf16* xn; long ldn;                          // POST: second norm
+  uint32_t* ticket; const float* bias; int E, topk, scoring, renorm; float scale; int32_t* ids; float *wts, *shared_w;      // router: ticket set
 };
 
 // stage T rows of the operand; ends with __syncthreads(). `inv`: T * max(groups, 1) floats
 template <int T, int PRO>
-__device__ __forceinline__ void stage_operand(const Params& p, bf16* xs, float* inv, float* red, int t0) {
+__device__ __forceinline__ void stage_operand(const Params& p, bf16* xs, float* inv, float* red, float* xf, int t0) {
   const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, nwarp = nthr >> 5, K = p.K;
   if (PRO == PLAIN) {
     for (int t = 0; t < T; ++t) {
@@ -75,9 +80,11 @@ __device__ __forceinline__ void stage_operand(const Params& p, bf16* xs, float* 
     }
   }
   __syncthreads();
+  const bool twice = PRO == POST && p.norm2_w;
   for (int t = 0; t < T; ++t) {
     const long r = t0 + t;
     const bool live = r < p.T;
+    float ss = 0.f;
     for (int c = tid * 4; c < K; c += nthr * 4) {
       float f[4] = {0.f, 0.f, 0.f, 0.f};
       if (live) {
@@ -91,6 +98,7 @@ __device__ __forceinline__ void stage_operand(const Params& p, bf16* xs, float* 
           f[2] = x.z + f[2] * iv * w.z;
           f[3] = x.w + f[3] * iv * w.w;
           if (blockIdx.x == 0) *reinterpret_cast<float4*>(p.x_out + r * p.ldr + c) = make_float4(f[0], f[1], f[2], f[3]);
+          ss += f[0] * f[0] + f[1] * f[1] + f[2] * f[2] + f[3] * f[3];
         } else {
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
@@ -100,8 +108,30 @@ __device__ __forceinline__ void stage_operand(const Params& p, bf16* xs, float* 
           }
         }
       }
+      if (twice) {
+        *reinterpret_cast<float4*>(xf + t * K + c) = make_float4(f[0], f[1], f[2], f[3]);
+        continue;
+      }
       __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
       *reinterpret_cast<uint2*>(xs + t * K + c) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+    }
+    if (twice) {
+      ss = warp_sum(ss);
+      if (lane == 0) red[t * 8 + warp] = ss;
+    }
+  }
+  __syncthreads();
+  if (!twice) return;
+  for (int t = 0; t < T; ++t) {
+    float s = 0.f;
+    for (int i = 0; i < nwarp; ++i) s += red[t * 8 + i];
+    const float iv = 1.f / sqrtf(s / (float)K + p.eps);
+    for (int c = tid * 4; c < K; c += nthr * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(xf + t * K + c), w = *reinterpret_cast<const float4*>(p.norm2_w + c);
+      __nv_bfloat162 a = __floats2bfloat162_rn(v.x * iv * w.x, v.y * iv * w.y), b = __floats2bfloat162_rn(v.z * iv * w.z, v.w * iv * w.w);
+      const uint2 u = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+      *reinterpret_cast<uint2*>(xs + t * K + c) = u;
+      if (p.xn && blockIdx.x == 0 && t0 + t < p.T) *reinterpret_cast<uint2*>(p.xn + (long)(t0 + t) * p.ldn + c) = u;
     }
   }
   __syncthreads();
@@ -112,6 +142,7 @@ __global__ void __launch_bounds__(256) gemv_operand_kernel(Params p) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* xs = reinterpret_cast<bf16*>(smem_raw);
   float* inv = reinterpret_cast<float*>(xs + (long)T * p.K);
+  float* xf = inv + 8;                          // POST with a second norm: the updated rows (T <= 8 and K % 8 keep it 16-byte aligned)
   __shared__ float red[T * 8];
   grid_dep_launch();
   const int t0 = blockIdx.y * T, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n0 = (blockIdx.x * 8 + warp) * R;
@@ -121,8 +152,9 @@ __global__ void __launch_bounds__(256) gemv_operand_kernel(Params p) {
   RowBatch<R> pf;
   prefetch_rows<R>(rows, p.K, pf);
   grid_dep_wait();
-  stage_operand<T, PRO>(p, xs, inv, red, t0);
-  if (n0 >= p.N) return;
+  stage_operand<T, PRO>(p, xs, inv, red, xf, t0);
+  const bool router = PRO == POST && p.ticket;
+  if (n0 >= p.N && !router) return;
   float acc[R][T];
 #pragma unroll
   for (int r = 0; r < R; ++r)
@@ -143,11 +175,26 @@ __global__ void __launch_bounds__(256) gemv_operand_kernel(Params p) {
       }
     }
   }
+  if (!router) return;
+  __shared__ int is_last;
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    is_last = atomicAdd(p.ticket, 1u) == gridDim.x - 1;
+    if (is_last) *p.ticket = 0;
+  }
+  __syncthreads();
+  if (!is_last || warp >= p.T) return;          // one row tile: warp t selects for row t
+  __threadfence();
+  const float* logits = reinterpret_cast<const float*>(p.z) + (long)warp * p.ldz;
+  select_topk_row(logits, p.bias, p.E, p.topk, p.scoring, p.renorm, p.scale, p.ids + (long)warp * p.topk, p.wts + (long)warp * p.topk);
+  if (p.shared_w && lane == 0) p.shared_w[warp] = sigmoid_f32(__ldcg(logits + p.E));
 }
 
 template <int T, int R, int PRO>
 int launch_one(const Params& p, cudaStream_t s) {
-  const size_t smem = (size_t)T * p.K * sizeof(bf16) + (size_t)T * (PRO == GROUP ? p.groups : 1) * sizeof(float);
+  const size_t smem = (size_t)T * p.K * sizeof(bf16) + (PRO == GROUP ? (size_t)T * p.groups : 8) * sizeof(float) +
+                      (PRO == POST && p.norm2_w ? (size_t)T * p.K * sizeof(float) : 0);
   auto k = gemv_operand_kernel<T, R, PRO>;
   if (int rc = opt_in_smem(k, smem)) return rc;
   return launch_chain(k, dim3((p.N + 8 * R - 1) / (8 * R), (p.T + T - 1) / T), dim3(256), smem, s, p);
@@ -170,12 +217,28 @@ int dispatch(const Params& p, cudaStream_t s) {
 
 }  // namespace
 
-extern "C" int ifab_gemv_post_norm(const float* y, long ldy, const float* norm_w, float eps, const float* x_in, float* x_out, long ldx, const void* w,
-                                   void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream) {
+extern "C" int ifab_gemv_post_norm(const float* y, long ldy, const float* norm_w, const float* norm2_w, float eps, const float* x_in, float* x_out, long ldx,
+                                   const void* w, void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream) {
   if (ldy % 4 || ldx % 4 || x_in == x_out) return -1;
   Params p{};
+  p.norm2_w = norm2_w;
   p.y = y; p.ldy = ldy; p.norm_w = norm_w; p.eps = eps; p.x_in = x_in; p.x_out = x_out; p.ldr = ldx;
   p.w = (const bf16*)w; p.z = z; p.ldz = ldz; p.out_f32 = out_f32; p.act = act; p.T = T; p.N = N; p.K = K;
+  return dispatch<POST>(p, (cudaStream_t)stream);
+}
+// The router of a sublayer pair: x_out as above, xn = bf16(rms(x_out) * norm2_w), f32 logits [T, N] = xn w^T (T <= 8), then ids / wts of the chosen
+// of the first E columns and, when N = E + 1, shared_w = sigmoid(logits[:, E]). ticket: one zeroed word (left zero again)
+extern "C" int ifab_router_post_norm(const float* y, long ldy, const float* norm_w, const float* norm2_w, float eps, const float* x_in, float* x_out, long ldx,
+                                     void* xn, long ldn, const void* w, float* logits, long ldz, const float* bias, int E, int topk, int scoring, int renorm,
+                                     float scale, int32_t* ids, float* wts, float* shared_w, uint32_t* ticket, int T, int N, int K, void* stream) {
+  if (ldy % 4 || ldx % 4 || ldn % 4 || x_in == x_out || T > 8 || !ticket || !norm2_w || E < 1 || E > 32 * SELECT_PER_LANE || topk < 1 || topk > MAX_TOPK ||
+      topk > E || N < E || N > E + 1 || (shared_w && N != E + 1) || scoring < 0 || scoring > 2)
+    return -1;
+  Params p{};
+  p.y = y; p.ldy = ldy; p.norm_w = norm_w; p.norm2_w = norm2_w; p.eps = eps; p.x_in = x_in; p.x_out = x_out; p.ldr = ldx;
+  p.xn = (bf16*)xn; p.ldn = ldn; p.ticket = ticket; p.bias = bias; p.E = E; p.topk = topk; p.scoring = scoring; p.renorm = renorm; p.scale = scale;
+  p.ids = ids; p.wts = wts; p.shared_w = shared_w;
+  p.w = (const bf16*)w; p.z = logits; p.ldz = ldz; p.out_f32 = 1; p.act = 0; p.T = T; p.N = N; p.K = K;
   return dispatch<POST>(p, (cudaStream_t)stream);
 }
 extern "C" int ifab_gemv_group_norm(const float* o, long ldo, const float* gain, float eps, int groups, const void* gate, long ldg, int gate_act,

@@ -1,7 +1,7 @@
 // Prompt (prefill) attention on the 5th-generation tensor cores: softmax(Q K^T) V for a chunk of consecutive tokens of one
 // sequence against that sequence's whole context, causal, optional sliding window. One CTA = 128 query rows of one head.
 //
-//   warp 0      TMA producer: the Q tile once, then per 128-key tile the K panels (two shared-memory stages) and the V^T
+//   warp 0      TMA producer: the Q tile once, then per 128-key tile the K panels (two shared-memory stages; one where they would not fit) and the V^T
 //               panels (one stage), all 128-byte-swizzled [128 rows x 64 columns] boxes, never multicast
 //   warp 1      allocates tensor memory; one lane issues tcgen05.mma: S_j = Q K_j^T into one of two TMEM score buffers (so
 //               S_{j+1} is computed while the softmax warps work on S_j), then O_j = P_j V_j once P_j is in shared memory
@@ -46,6 +46,7 @@ struct FaParams {
   int e;                                     // value columns per head that are stored, at column h * e (<= 128)
   const float* sink;                         // [H]: exp(sink) joins the denominator of the head; or null
   const bf16* gate; long ldg; int gate_act;  // the result is multiplied by act(gate [m, H * e]); or null
+  int gate_head;                             // the gate has one value per head instead: [m, H]
   uint32_t* status; uint32_t spin_limit;
 };
 
@@ -59,9 +60,10 @@ struct Bars {
 template <int P1, int P2, bool SPLIT>
 struct Layout {
   static constexpr int NQ = P1 + P2;                       // 64-column panels of Q and of a K tile
+  static constexpr int KST = SPLIT && NQ > 2 ? 1 : 2;      // stages of K tiles
   static constexpr int Q_OFF = 0;
-  static constexpr int K_OFF = Q_OFF + NQ * PANEL_BYTES;   // two stages
-  static constexpr int V_OFF = K_OFF + 2 * NQ * PANEL_BYTES;
+  static constexpr int K_OFF = Q_OFF + NQ * PANEL_BYTES;
+  static constexpr int V_OFF = K_OFF + KST * NQ * PANEL_BYTES;
   static constexpr int P_OFF = V_OFF + PV_PANELS * PANEL_BYTES;
   static constexpr int PL_OFF = P_OFF + PV_PANELS * PANEL_BYTES;       // remainder of P
   static constexpr int BAR_OFF = PL_OFF + (SPLIT ? PV_PANELS * PANEL_BYTES : 0);
@@ -74,7 +76,7 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
                                                             const __grid_constant__ CUtensorMap tmap_k2, const __grid_constant__ CUtensorMap tmap_vt,
                                                             FaParams p) {
   using L = Layout<P1, P2, SPLIT>;
-  constexpr int NQ = L::NQ;
+  constexpr int NQ = L::NQ, KST = L::KST;
   extern __shared__ unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   unsigned char* Qs = smem + L::Q_OFF;
@@ -130,7 +132,7 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
     for (int pp = 0; pp < NQ; ++pp) tma_load_2d(Qs + pp * PANEL_BYTES, &tmap_q, &B->q_full, h * p.q_head_stride + pp * 64, q0);
     int armed_k = 0, armed_v = 0;
     for (int j = 0; j < n_tiles && !*abort_flag; ++j) {
-      const int key0 = (t_begin + j) * BKEY, s = j & 1, round = j >> 1;
+      const int key0 = (t_begin + j) * BKEY, s = j % KST, round = j / KST;
       if (round > 0 && !mbar_wait(&B->k_empty[s], (round - 1) & 1, p.spin_limit)) { fail(); break; }
       unsigned char* kd = Ks + s * NQ * PANEL_BYTES;
       mbar_expect_tx(&B->k_full[s], NQ * PANEL_BYTES);
@@ -145,7 +147,7 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
     if (*abort_flag) {
       // every copy this thread issued must land before the CTA may exit
       mbar_wait(&B->q_full, 0, p.spin_limit);
-      for (int j = max(0, armed_k - 2); j < armed_k; ++j) mbar_wait(&B->k_full[j & 1], (j >> 1) & 1, p.spin_limit);
+      for (int j = max(0, armed_k - KST); j < armed_k; ++j) mbar_wait(&B->k_full[j % KST], (j / KST) & 1, p.spin_limit);
       if (armed_v > 0) mbar_wait(&B->v_full, (armed_v - 1) & 1, p.spin_limit);
     }
   } else if (warp == 1 && lane == 0) {
@@ -153,10 +155,10 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
     constexpr uint32_t idesc = umma_idesc_bf16(BQ, 128);
     bool ok = mbar_wait(&B->q_full, 0, p.spin_limit);
     auto issue_scores = [&](int j) {
-      const int s = j & 1;
-      if (!mbar_wait(&B->k_full[s], (j >> 1) & 1, p.spin_limit) || *abort_flag) return false;
+      const int s = j & 1, ks = j % KST;
+      if (!mbar_wait(&B->k_full[ks], (j / KST) & 1, p.spin_limit) || *abort_flag) return false;
       tc_fence_after();
-      const uint32_t qa = smem_u32(Qs), ka = smem_u32(Ks + s * NQ * PANEL_BYTES);
+      const uint32_t qa = smem_u32(Qs), ka = smem_u32(Ks + ks * NQ * PANEL_BYTES);
 #pragma unroll
       for (int pp = 0; pp < NQ; ++pp) {
         const uint64_t da = umma_desc_sw128(qa + pp * PANEL_BYTES), db = umma_desc_sw128(ka + pp * PANEL_BYTES);
@@ -164,7 +166,7 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
         for (int k = 0; k < 4; ++k) umma_bf16(tmem + S_COL + (uint32_t)s * 128u, da + (uint64_t)(2 * k), db + (uint64_t)(2 * k), idesc, pp > 0 || k > 0);
       }
       umma_commit(&B->s_full[s]);
-      umma_commit(&B->k_empty[s]);
+      umma_commit(&B->k_empty[ks]);
       return true;
     };
     if (ok && n_tiles > 0) ok = issue_scores(0);
@@ -327,11 +329,12 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
       if (lane == 0) fail();
     } else if (q0 + r < p.m) {
       if (p.sink) l_run += exp2f(p.sink[h] * 1.4426950408889634f - m_ref);
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if (p.gate && p.gate_head) inv *= activate<true>(__bfloat162float(p.gate[(long)(q0 + r) * p.ldg + h]), p.gate_act);
       const int c0 = half * HV;
       bf16* dst = p.out + (long)(q0 + r) * p.ldo + (long)h * p.e + c0;
-      const bf16* gr = p.gate ? p.gate + (long)(q0 + r) * p.ldg + (long)h * p.e + c0 : nullptr;
-      const bool wide = ((p.e | (int)(p.ldo & 7) | (p.gate ? (int)(p.ldg & 7) : 0)) & 7) == 0 && (reinterpret_cast<uintptr_t>(p.gate) & 15) == 0;
+      const bf16* gr = p.gate && !p.gate_head ? p.gate + (long)(q0 + r) * p.ldg + (long)h * p.e + c0 : nullptr;
+      const bool wide = ((p.e | (int)(p.ldo & 7) | (gr ? (int)(p.ldg & 7) : 0)) & 7) == 0 && (!gr || (reinterpret_cast<uintptr_t>(p.gate) & 15) == 0);
 #pragma unroll
       for (int c = 0; c < HV; c += 8) {
         if (c0 + c >= p.e) break;
@@ -395,7 +398,7 @@ extern "C" int ifab_fa_prefill_bf16(const void* q, long ldq, int q_head_stride, 
   }
   if (int rc = make_tmap_bf16_2d(&tv, vt, (uint64_t)vt_rows, (uint64_t)ctx, (uint64_t)ldvt, DV)) return rc;
   FaParams p{(bf16*)out, ldo, m, ctx, kv_group, pos0, window, q_head_stride, k_head_stride, vt_head_stride, vt_row0,
-             scale * 1.4426950408889634f, DV, nullptr, nullptr, 0, 0, status, 4000000u};
+             scale * 1.4426950408889634f, DV, nullptr, nullptr, 0, 0, 0, status, 4000000u};
   cudaStream_t s = (cudaStream_t)stream;
   if (d1 == 128 && d2 == 64) return launch_fa<2, 1>(tq, tk, tk2, tv, p, H, s);
   if (d1 == 128 && d2 == 0) return launch_fa<2, 0>(tq, tk, tk2, tv, p, H, s);
@@ -403,21 +406,26 @@ extern "C" int ifab_fa_prefill_bf16(const void* q, long ldq, int q_head_stride, 
   return launch_fa<1, 0>(tq, tk, tk2, tv, p, H, s);
 }
 
-// Windowed grouped-query form with softmax weights of 16 bits instead of 8 in the value product, a sink logit per head, an output gate,
-// and value heads of any width: q [m, H * d] and k [ctx, G * d] with d in {64, 128} columns per head (narrower heads are zero-padded by
-// the caller), vt [G * 128, ldvt >= ctx] (rows past a narrower value head are zero), out and gate [m, H * e], e <= 128.
-extern "C" int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const void* vt, long ldvt, void* out, long ldo, int m, int ctx, int H,
-                                   int kv_group, int d, int e, int pos0, int window, float scale, const float* sink, const void* gate, long ldg, int gate_act,
-                                   uint32_t* status, void* stream) {
+// Windowed form with softmax weights of 16 bits instead of 8 in the value product, a sink logit per head, an output gate, and value heads
+// of any width: q [m, H * (d + d2)] and k [ctx, G * d] with d in {64, 128} columns per head (narrower heads are zero-padded by the caller),
+// k2 [ctx, d2] key columns shared by all heads (d2 0 or 64), vt [G * 128, ldvt >= ctx] (rows past a narrower value head are zero), out
+// [m, H * e], e <= 128; gate [m, H * e], or [m, H] with gate_per_head.
+extern "C" int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const void* k2, long ldk2, int d2, const void* vt, long ldvt, void* out, long ldo,
+                                   int m, int ctx, int H, int kv_group, int d, int e, int pos0, int window, float scale, const float* sink, const void* gate,
+                                   long ldg, int gate_act, int gate_per_head, uint32_t* status, void* stream) {
   if (m < 1 || ctx < 1 || H < 1 || kv_group < 1 || H % kv_group || pos0 < 0 || pos0 + m > ctx || window < 0) return -1;
-  if ((d != 64 && d != 128) || e < 1 || e > DV || ldq % 8 || ldk % 8 || ldvt % 8 || ldvt < ctx) return -1;
+  if ((d != 64 && d != 128) || (d2 != 0 && d2 != 64) || (d2 && (!k2 || ldk2 % 8)) || e < 1 || e > DV || ldq % 8 || ldk % 8 || ldvt % 8 || ldvt < ctx) return -1;
   const int G = H / kv_group;
-  CUtensorMap tq, tk, tv;
-  if (int rc = make_tmap_bf16_2d(&tq, q, (uint64_t)m, (uint64_t)H * d, (uint64_t)ldq, BQ)) return rc;
+  CUtensorMap tq, tk, tk2, tv;
+  if (int rc = make_tmap_bf16_2d(&tq, q, (uint64_t)m, (uint64_t)H * (d + d2), (uint64_t)ldq, BQ)) return rc;
   if (int rc = make_tmap_bf16_2d(&tk, k, (uint64_t)ctx, (uint64_t)G * d, (uint64_t)ldk, BKEY)) return rc;
+  tk2 = tk;
+  if (d2)
+    if (int rc = make_tmap_bf16_2d(&tk2, k2, (uint64_t)ctx, (uint64_t)d2, (uint64_t)ldk2, BKEY)) return rc;
   if (int rc = make_tmap_bf16_2d(&tv, vt, (uint64_t)G * DV, (uint64_t)ctx, (uint64_t)ldvt, DV)) return rc;
-  FaParams p{(bf16*)out, ldo, m, ctx, kv_group, pos0, window, d, d, DV, 0, scale * 1.4426950408889634f, e, sink, (const bf16*)gate, ldg, gate_act, status,
-             4000000u};
+  FaParams p{(bf16*)out, ldo, m, ctx, kv_group, pos0, window, d + d2, d, DV, 0, scale * 1.4426950408889634f, e, sink, (const bf16*)gate, ldg, gate_act,
+             gate_per_head, status, 4000000u};
   cudaStream_t s = (cudaStream_t)stream;
-  return d == 128 ? launch_fa<2, 0, true>(tq, tk, tk, tv, p, H, s) : launch_fa<1, 0, true>(tq, tk, tk, tv, p, H, s);
+  if (d2) return d == 128 ? launch_fa<2, 1, true>(tq, tk, tk2, tv, p, H, s) : launch_fa<1, 1, true>(tq, tk, tk2, tv, p, H, s);
+  return d == 128 ? launch_fa<2, 0, true>(tq, tk, tk2, tv, p, H, s) : launch_fa<1, 0, true>(tq, tk, tk2, tv, p, H, s);
 }

@@ -80,6 +80,15 @@ int ifab_gemm_act_bf16_2sm(const void* a, long lda, const void* b, long ldb, voi
                            int persistent, int M, int N, int K, uint32_t* status, void* stream);
 /* C = act(A * B^T) in true f32 */
 int ifab_linear_f32(const float* a, long lda, const float* b, long ldb, float* c, long ldc, int M, int N, int K, int act, void* stream);
+/* n products at strides sa, sb, sc; and products grouped by the tile table of ifab_moe_dispatch (rows of A through `index` when given; pair: A is
+ * [gate | up], taken as silu(gate) * up) */
+int ifab_linear_f32_batched(const float* a, long lda, long sa, const float* b, long ldb, long sb, float* c, long ldc, long sc, int n, int M, int N, int K,
+                            void* stream);
+int ifab_grouped_linear_f32(const float* a, long lda, const int32_t* index, int pair, const float* b, int N, int K, const int32_t* tiles,
+                            const int32_t* num_tiles, int max_tiles, int rows, float* c, long ldc, void* stream);
+/* one product per head, heads side by side in the rows of A and C: C[t, h * c_stride + n] = sum_k A[t, h * a_stride + k] B[h, n, k] (tcgen05) */
+int ifab_gemm_heads_bf16(const void* a, long lda, int a_stride, const void* b, long ldb, void* c, long ldc, int c_stride, int out_f32, int heads, int M, int N,
+                         int K, uint32_t* status, void* stream);
 
 /* the same on CTA pairs (tcgen05.mma cta_group::2, 256 x 256 tiles, each CTA loads half of A and half of B); N % 32 == 0 */
 int ifab_gemm_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual,
@@ -167,7 +176,18 @@ int ifab_router_topk(const void* x, long ldx, const void* norm_w, float eps, con
                      float scale, uint32_t* ticket, void* xn, long ldxn, void* stream);
 int ifab_moe_gate_up_decode(const void* x, long ldx, const void* norm_w, float eps, const int32_t* ids, int T, int D,
                             int F, int topk, int e0, int e_local, const void* w_gu, const void* w_shared_gu, int Fs,
-                            void* act, void* stream);
+                            void* act, int ldact, void* stream);
+/* one rank: y f32 [T, ldy] = the same sum before rounding, the shared expert's row weighted by shared_w [T] (null: 1). In both, `act` slots are
+ * ldact columns apart (slot topk is the shared expert's, which may be wider or narrower than F) */
+int ifab_moe_down_f32_decode(const void* act, int ldact, const int32_t* ids, const float* wts, const float* shared_w, int T, int D, int F, int topk,
+                             int experts, const void* w_down, const void* w_shared_down, int Fs, float* y, long ldy, void* stream);
+/* routed experts of decoders with an f32 residual (moe_rows.cu): logits f32 [M, ld] (column E: the shared expert's gate, used when shared_w is given) ->
+ * ids, wts [M, topk]; scoring 0 softmax, 1 sigmoid, 2 logit + bias selected, softmax over the chosen. combine_norm: y = weighted sum of the permuted
+ * rows (+ shared_w * shared), x += rms(y) * w, xa = rms(x) * w2 (x without w2) */
+int ifab_moe_route(const float* logits, long ld, const float* bias, int M, int E, int topk, int scoring, int renorm, float scale, int32_t* ids, float* wts,
+                   float* shared_w, void* stream);
+int ifab_moe_combine_norm(const void* y, long ldy, const int32_t* route_row, const float* wts, int topk, const void* shared, long lds, const float* shared_w,
+                          const float* w, const float* w2, float eps, float* x, long ldx, void* xa, long lda, int f32, int M, int D, void* stream);
 int ifab_moe_down_allreduce_decode(const void* act, const int32_t* ids, const float* wts, int T, int D, int F, int topk,
                                    int e0, int e_local, const void* w_down, const void* w_shared_down, int Fs,
                                    const void* residual, long ldr, void* y, long ldy, const IfabFabric* fab,
@@ -260,8 +280,9 @@ int ifab_mhc_post_norm(const void* X, const void* branch, long ldb, const void* 
 int ifab_delta_rule_decode(const void* q, const void* k, const void* v, const float* g, const float* beta, float* state,
                            const int32_t* slots, void* out, int rows, int H, int dk, int dv, void* stream);
 /* f32 residual stream with the norm on a sublayer's output; `f32`: activations (xa, gate, y) are f32 instead of bf16; gains f32 */
-int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float* x, long ldx, void* xa, long lda, int f32, int T, int D, int vocab,
-                    uint32_t* status, void* stream);
+/* x = table[id] * scale; xa = x, or rms(x) * w when w is given */
+int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float scale, const float* w, float eps, float* x, long ldx, void* xa, long lda, int f32,
+                    int T, int D, int vocab, uint32_t* status, void* stream);
 /* x += rms(y) * w; xa = x, or rms(x) * w2 when w2 is given */
 int ifab_post_norm_add(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, void* xa, long lda, int f32, int T, int D,
                        void* stream);
@@ -271,9 +292,13 @@ int ifab_group_norm_gate(const float* o, long ldo, const float* w, float eps, co
 int ifab_gate_rows(const void* o, long ldo, int head_stride, const void* gate, long ldg, int act, void* y, long ldy, int f32, int T, int H, int n,
                    void* stream);
 /* decode linears whose prologue finishes the previous sublayer. ..._post_norm: x_out = x_in + rms(y) * w (one CTA column writes it), then
- * z = act(bf16(x_out) W^T); ..._group_norm: z = act(bf16((o / rms per group [* gain]) * gate_act(gate)) W^T) */
-int ifab_gemv_post_norm(const float* y, long ldy, const float* norm_w, float eps, const float* x_in, float* x_out, long ldx, const void* w, void* z,
-                        long ldz, int out_f32, int act, int T, int N, int K, void* stream);
+ * z = act(bf16(x_out) W^T), or of bf16(rms(x_out) * norm2_w) when norm2_w is given; ..._group_norm: z = act(bf16((o / rms per group [* gain]) * gate_act(gate)) W^T) */
+int ifab_gemv_post_norm(const float* y, long ldy, const float* norm_w, const float* norm2_w, float eps, const float* x_in, float* x_out, long ldx,
+                        const void* w, void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream);
+/* the same with both norms as a router: xn = the operand, f32 logits, then ids / wts (and shared_w = sigmoid(logits[:, E]) when N = E + 1), T <= 8 */
+int ifab_router_post_norm(const float* y, long ldy, const float* norm_w, const float* norm2_w, float eps, const float* x_in, float* x_out, long ldx, void* xn,
+                          long ldn, const void* w, float* logits, long ldz, const float* bias, int E, int topk, int scoring, int renorm, float scale,
+                          int32_t* ids, float* wts, float* shared_w, uint32_t* ticket, int T, int N, int K, void* stream);
 int ifab_gemv_group_norm(const float* o, long ldo, const float* gain, float eps, int groups, const void* gate, long ldg, int gate_act, const void* w,
                          void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream);
 int ifab_gemv_act(const void* x, long ldx, const void* w, void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream);
@@ -301,9 +326,26 @@ int ifab_window_attn(const void* q, long ldq, int q_stride, const void* k_cache,
 /* operands of the tensor-core windowed attention: keys / values first .. first + n - 1 of a sequence, heads zero-padded to dp / 128 columns */
 int ifab_ctx_gather_pad(const void* k_cache, const void* v_cache, const int32_t* page_table, int slot, int max_pages, int page_tokens, int num_pages,
                         int first, int n, int rows, int G, int d, int dp, int e, void* k, void* vt, long ldvt, uint32_t* status, void* stream);
-int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const void* vt, long ldvt, void* out, long ldo, int m, int ctx, int H,
-                        int kv_group, int d, int e, int pos0, int window, float scale, const float* sink, const void* gate, long ldg, int gate_act,
-                        uint32_t* status, void* stream);
+int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const void* k2, long ldk2, int d2, const void* vt, long ldvt, void* out, long ldo,
+                        int m, int ctx, int H, int kv_group, int d, int e, int pos0, int window, float scale, const float* sink, const void* gate, long ldg,
+                        int gate_act, int gate_per_head, uint32_t* status, void* stream);
+/* latent attention over paged rows [latent padded to Lp | rotated key part padded to Rp], any sizes, bf16 or f32 (latent_attn.cu). splits <= 64, the last
+ * takes what is left of the keys a row sees; scratch f32 [T, H, splits, Lp + 2] */
+int ifab_latent_prepare(const void* proj, long ldp, int f32, int q_off, int q_rank, int kv_off, int kv_rank, int rot_dim, const float* q_gain,
+                        const float* kv_gain, float eps, const void* rope, int rot, const int32_t* positions, const int32_t* slots, const int32_t* page_table,
+                        int max_pages, int page_tokens, int num_pages, void* cq, long ldc, void* cache, int Lp, int Rp, int T, uint32_t* status, void* stream);
+int ifab_rotate_heads(void* q, long ldq, int f32, int head_stride, int off, int H, int rot, const void* rope, int T, void* stream);
+int ifab_latent_absorb(void* q, long ldq, int head_stride, int rot_off, const void* w_uk, const void* rope, int rot, float* q_lat, int T, int H, int d, int Lp,
+                       void* stream);
+int ifab_latent_split(const float* q_lat, const void* q_rot, long ldq, int head_stride, const void* cache, int f32, int Lp, int Rp, const int32_t* positions,
+                      const int32_t* slots, const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int window, float scale, int T, int H,
+                      int kps, int splits, float* scratch, uint64_t scratch_bytes, uint32_t* status, void* stream);
+int ifab_latent_merge(const float* scratch, const int32_t* positions, int window, int kps, int splits, const void* gate, long ldg, int f32, int T, int H, int Lp,
+                      void* o_lat, long ldo, void* stream);
+int ifab_latent_merge_vup(const float* scratch, const int32_t* positions, int window, int kps, int splits, const void* gate, long ldg, int T, int H, int Lp,
+                          const void* w_uv, int vdim, void* out, long ldo, void* stream);
+int ifab_latent_gather(const void* cache, const int32_t* page_table, int slot, int max_pages, int page_tokens, int num_pages, int first, int n, int rows, int Lp,
+                       int Rp, int tile, void* lat, void* rot, uint32_t* status, void* stream);
 int ifab_gqa_window_attention(const void* q, long ldq, const void* k_cache, const void* v_cache, const int32_t* positions, const int32_t* slots,
                               const int32_t* page_table, int max_pages, int page_tokens, int num_pages, float scale, int window, const float* sink,
                               const void* gate, long ldg, int gate_act, int T, int Hq, int Hkv, int head_dim, int keys_per_split, int max_splits,

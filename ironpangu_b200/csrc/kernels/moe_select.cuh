@@ -2,6 +2,7 @@
 //
 // Softmax scoring (0): probabilities over all experts, the k largest, optionally renormalised to sum 1.
 // Sigmoid scoring (1): sigmoid scores, selection on score + bias, weights = score / sum of the selected scores.
+// Biased-logit scoring (2): selection on logit + bias, weights = softmax over the selected ones only.
 // Ties go to the lower expert index, so the result does not depend on lane order. Supports up to 256 experts.
 #pragma once
 #include "common.cuh"
@@ -31,6 +32,9 @@ __device__ __forceinline__ void select_topk_scores(float (&score)[SELECT_PER_LAN
         score[i] = __expf(score[i] - mx);
         denom += score[i];
         sel[i] = score[i];
+      } else if (scoring == 2) {
+        if (bias) score[i] += bias[ei];
+        sel[i] = score[i];
       } else {
         score[i] = 1.f / (1.f + __expf(-score[i]));
         sel[i] = score[i] + (bias ? bias[ei] : 0.f);
@@ -43,7 +47,7 @@ __device__ __forceinline__ void select_topk_scores(float (&score)[SELECT_PER_LAN
   denom = warp_sum(denom);
   float picked_w[MAX_TOPK];
   int picked_e[MAX_TOPK];
-  float wsum = 0.f;
+  float wsum = 0.f, top = 0.f;
   for (int k = 0; k < topk; ++k) {
     float bv = -INFINITY;
     int bi = 0x7fffffff;
@@ -66,13 +70,15 @@ __device__ __forceinline__ void select_topk_scores(float (&score)[SELECT_PER_LAN
     }
     raw = warp_sum(raw);
     picked_e[k] = bi;
-    picked_w[k] = (scoring == 0) ? raw / denom : raw;
+    picked_w[k] = (scoring == 0) ? raw / denom : scoring == 2 ? expf(raw - (k ? top : raw)) : raw;
+    if (k == 0) top = raw;
     wsum += picked_w[k];
   }
   if (lane == 0) {
     for (int k = 0; k < topk; ++k) {
       float w = picked_w[k];
       if (scoring == 0) { if (renorm) w = w / wsum; }
+      else if (scoring == 2) w = w / wsum;
       else w = w / (wsum + 1e-20f);
       ids[k] = picked_e[k];
       wts[k] = w * scale;

@@ -1,6 +1,7 @@
 // Row operators of decoders that keep an f32 residual stream and normalise a sublayer's OUTPUT before adding it:
 //
-//   embed_rows_kernel      x = table[id] (f32) and its copy in the activation type (the operand of the next linears)
+//   embed_rows_kernel      x = table[id] * scale (f32) and its copy in the activation type (the operand of the next linears), of rms(x) * w
+//                          when a gain is given (the norm ahead of the first sublayer)
 //   post_norm_add_kernel   x += rms(y) * w; copy in the activation type (of rms(x) * w2 when a second gain is given: the norm ahead
 //                          of the output matrix). y is the f32 output of the sublayer's last linear
 //   rms_rows_kernel        rms(x[row]) * w of selected rows, in the activation type (the norm ahead of the output matrix)
@@ -23,8 +24,9 @@ __device__ __forceinline__ void store4(bf16* p, const float* f) {
 }
 
 template <typename A>
-__global__ void __launch_bounds__(256) embed_rows_kernel(const int32_t* ids, const A* table, long ldt, float* x, long ldx, A* xa, long lda, int D,
-                                                         int vocab, uint32_t* status) {
+__global__ void __launch_bounds__(256) embed_rows_kernel(const int32_t* ids, const A* table, long ldt, float scale, const float* w, float eps, float* x, long ldx,
+                                                         A* xa, long lda, int D, int vocab, uint32_t* status) {
+  __shared__ float red[33];
   grid_dep_launch();
   grid_dep_wait();
   const int t = blockIdx.x;
@@ -33,11 +35,16 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(const int32_t* ids, con
     if (threadIdx.x == 0 && status) atomicOr(status, IFAB_STATUS_BAD_INDEX);
     id = 0;
   }
+  float ss = 0.f;
   for (int c = threadIdx.x; c < D; c += blockDim.x) {
-    const A v = table[(long)id * ldt + c];
-    x[(long)t * ldx + c] = to_f32(v);
-    xa[(long)t * lda + c] = v;
+    const float v = to_f32(table[(long)id * ldt + c]) * scale;
+    x[(long)t * ldx + c] = v;
+    if (!w) xa[(long)t * lda + c] = from_f32<A>(v);
+    ss += v * v;
   }
+  if (!w) return;
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)D + eps);
+  for (int c = threadIdx.x; c < D; c += blockDim.x) xa[(long)t * lda + c] = from_f32<A>(to_f32(table[(long)id * ldt + c]) * scale * inv * w[c]);
 }
 
 // one CTA per row
@@ -160,9 +167,9 @@ __global__ void __launch_bounds__(256) gate_rows_kernel(const A* o, long ldo, in
 }
 
 template <typename A>
-int embed(const int32_t* ids, const void* table, long ldt, float* x, long ldx, void* xa, long lda, int T, int D, int vocab, uint32_t* status,
-          cudaStream_t s) {
-  return launch_chain(embed_rows_kernel<A>, dim3(T), dim3(256), 0, s, ids, (const A*)table, ldt, x, ldx, (A*)xa, lda, D, vocab, status);
+int embed(const int32_t* ids, const void* table, long ldt, float scale, const float* w, float eps, float* x, long ldx, void* xa, long lda, int T, int D, int vocab,
+          uint32_t* status, cudaStream_t s) {
+  return launch_chain(embed_rows_kernel<A>, dim3(T), dim3(256), 0, s, ids, (const A*)table, ldt, scale, w, eps, x, ldx, (A*)xa, lda, D, vocab, status);
 }
 template <typename A>
 int group_norm(const float* o, long ldo, const float* w, float eps, const void* gate, long ldg, int act, void* y, long ldy, int T, int groups, int n,
@@ -175,11 +182,12 @@ int group_norm(const float* o, long ldo, const float* w, float eps, const void* 
 
 }  // namespace
 
-extern "C" int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float* x, long ldx, void* xa, long lda, int f32, int T, int D,
-                               int vocab, uint32_t* status, void* stream) {
+extern "C" int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float scale, const float* w, float eps, float* x, long ldx, void* xa, long lda,
+                               int f32, int T, int D, int vocab, uint32_t* status, void* stream) {
   if (T < 1 || D < 1 || vocab < 1) return -1;
   cudaStream_t s = (cudaStream_t)stream;
-  return f32 ? embed<float>(ids, table, ldt, x, ldx, xa, lda, T, D, vocab, status, s) : embed<bf16>(ids, table, ldt, x, ldx, xa, lda, T, D, vocab, status, s);
+  return f32 ? embed<float>(ids, table, ldt, scale, w, eps, x, ldx, xa, lda, T, D, vocab, status, s)
+             : embed<bf16>(ids, table, ldt, scale, w, eps, x, ldx, xa, lda, T, D, vocab, status, s);
 }
 
 extern "C" int ifab_post_norm_add(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, void* xa, long lda, int f32, int T, int D,

@@ -9,31 +9,26 @@ another layer's weights (``weights_of``) with a state or cache of their own.
   attention     grouped heads; rms of q and k per head with a gain; interleaved rotation; scores * scale over the last ``mask.size``
                 positions; softmax with a learned sink per head in the denominator; * sigmoid(W_g x); W_o
 
-``FalinexDecoder`` runs decode rows (and pieces of prompts up to ``max_tokens`` rows) in one launch chain whose grid depends on the
-row count only, so the engine replays it as a CUDA graph; ``FalinexRows`` runs a packed step - portions of several prompts beside
-decode rows - as matrix-matrix work. Both read the KV pages and recurrent states of ``decoder.state_manager`` (runtime/paged_state.py).
+``FalinexDecoder`` and ``FalinexRows`` are the decode and packed-step executors (``stream_decoder.py``).
 In bf16 the linears take bf16 operands with f32 accumulation; norms, rotations, scores, recurrences and the residual are f32.
 With ``dtype=torch.float32`` every product is a true f32 FMA.
 
 A checkpoint directory is ``config.json`` (``"architecture": "Falinex"``) + safetensors; see :func:`weight_shapes` for the names."""
 from __future__ import annotations
 
-import json
 from dataclasses import dataclass, field
-from pathlib import Path
 from typing import Dict, List, Optional
 
 import torch
 
-from ..ops import decode as K
 from ..ops import stream_norm as N
 from ..ops import window_attn as WA
-from ..ops.linear_attn import CHUNK, TILE, DecayedMixer, DevicePlan, RotaryTables, StepPlan
+from ..ops.linear_attn import CHUNK, TILE, DecayedMixer, DevicePlan, RotaryTables
 from ..parallel.fabric import Fabric
-from ..runtime.paged_state import PagedState
+from . import checkpoint
+from .checkpoint import pad8
+from .stream_decoder import ATTN_ROWS, BF16, F32, StreamDecoder, StreamRows
 
-BF16, F32 = torch.bfloat16, torch.float32
-ATTN_ROWS = 64             # rows per launch of the split-KV attention kernels
 KERNEL_UNITS = ("misc", "post_norm", "linear_f32", "linear_attn", "linear_attn_tc", "window_attn", "decode_post_norm", "decode_gqa", "fa_prefill", "decode_moe", "sampling",
                 "tc_gemm", "tc_gemm_2sm")
 
@@ -170,13 +165,7 @@ class FalinexConfig:
         return max(w) if w and all(w) else 0
 
     def param_count(self) -> int:
-        n = 0
-        for shape in weight_shapes(self).values():
-            k = 1
-            for d in shape:
-                k *= d
-            n += k
-        return n
+        return checkpoint.param_count(weight_shapes(self))
 
     @staticmethod
     def tiny() -> "FalinexConfig":
@@ -195,6 +184,9 @@ class FalinexConfig:
         ret = MixerConfig("retention", heads, dim, dim, decay=dec(5.0), rot_dims=dim, rot_base=1e4)
         att = MixerConfig("attention", heads, dim, dim, kv_heads=kv_heads, rot_dims=dim, rot_base=1e6, window=window, scale=dim ** -0.5)
         return FalinexConfig(vocab, width, 1e-5, [LayerConfig((lig, ret, ret, att)[i % 4], ff) for i in range(layers)]).validate()
+
+
+PRESETS = {"falinex-tiny": FalinexConfig.tiny, "falinex2b": FalinexConfig.text2b}
 
 
 # ---------------------------------------------------------------------------------------------------------------------------
@@ -231,42 +223,12 @@ def random_weights(c: FalinexConfig, device, seed: int = 0, std: float = 0.02) -
 
 def save_checkpoint(path, c: FalinexConfig, weights: Dict[str, torch.Tensor]) -> None:
     """Write ``config.json`` and ``model.safetensors`` (bf16)."""
-    import struct
-
-    d = Path(path)
-    d.mkdir(parents=True, exist_ok=True)
-    (d / "config.json").write_text(json.dumps(c.to_dict(), indent=1))
-    hdr, blobs, at = {}, [], 0
-    for n, t in weights.items():
-        raw = t.detach().to(BF16).cpu().contiguous().view(torch.uint8).numpy().tobytes()
-        hdr[n] = {"dtype": "BF16", "shape": list(t.shape), "data_offsets": [at, at + len(raw)]}
-        blobs.append(raw)
-        at += len(raw)
-    head = json.dumps(hdr).encode()
-    head += b" " * (-len(head) % 8)
-    (d / "model.safetensors").write_bytes(struct.pack("<Q", len(head)) + head + b"".join(blobs))
+    checkpoint.save(path, c, weights)
 
 
 def load_checkpoint(path) -> tuple:
     """``(config, weights on the host)`` of a checkpoint directory; every expected tensor must be there with its shape."""
-    from ..runtime.plan_engine import SafetensorsDir
-
-    c = FalinexConfig.from_dict(json.loads((Path(path) / "config.json").read_text()))
-    src = SafetensorsDir(str(path))
-    dts = {"BF16": BF16, "F32": F32, "F16": torch.float16}
-    out = {}
-    for name, shape in weight_shapes(c).items():
-        if name not in src.tensors:
-            raise ValueError(f"the checkpoint has no tensor {name}")
-        _, _, _, dt, have = src.tensors[name]
-        if tuple(have) != tuple(shape) or dt not in dts:
-            raise ValueError(f"{name}: {dt} {list(have)} in the checkpoint, {list(shape)} expected")
-        out[name] = torch.from_numpy(src.bytes_of(name).copy()).view(dts[dt]).view(*shape)
-    return c, out
-
-
-def _pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
+    return checkpoint.load(path, FalinexConfig.from_dict, weight_shapes)
 
 
 # ---------------------------------------------------------------------------------------------------------------------------
@@ -278,7 +240,7 @@ class _Rows:
     def __init__(self, dec: "FalinexDecoder", rows: int, chunked: bool):
         c, dev, A = dec.cfg, dec.fabric.device, dec.dtype
         mix = [l.mixer for l in c.layers]
-        z = lambda n, dt=A: torch.zeros(rows, _pad8(n), dtype=dt, device=dev)
+        z = lambda n, dt=A: torch.zeros(rows, pad8(n), dtype=dt, device=dev)
         self.rows = rows
         self.x, self.x2 = z(c.width, F32), z(c.width, F32)           # residual stream (two: fused prologues write the other one)
         self.xa, self.y = z(c.width), z(c.width, F32)
@@ -311,61 +273,17 @@ class _Rows:
                             f(wide * max(m.heads * m.vdim for m in rec)), f(nch * max(m.heads * m.dim * m.vdim for m in rec)))
 
 
-class FalinexDecoder:
-    """Decode executor on one GPU: up to ``max_tokens`` (<= 8) rows per step, each with its own position and sequence slot; rows of
-    one sequence inside a step are consecutive and in position order. Greedy next tokens land in ``next_ids``."""
+class FalinexDecoder(StreamDecoder):
+    """Decode executor: see :class:`StreamDecoder`."""
 
-    def __init__(self, cfg: FalinexConfig, weights: Dict[str, torch.Tensor], fabric: Fabric, *, max_tokens: int = 8, max_context: int = 1024, num_slots: int = 1,
-                 pool_tokens: int = 0, keep_logits: bool = False, dtype: torch.dtype = BF16):
-        """``pool_tokens``: tokens the KV page pool holds for all sequences together (0: every slot can reach the full context)."""
-        assert 1 <= max_tokens <= 8 and fabric.world == 1, "the Falinex decoder runs on one GPU"
-        assert dtype in (BF16, F32)
-        c, dev = cfg, fabric.device
-        self.cfg, self.fabric, self.rank, self.world, self.dtype = cfg, fabric, 0, 1, dtype
-        self.T, self.max_context, self.num_slots = max_tokens, max_context, num_slots
-        per_slot = (max_context + c.page_tokens - 1) // c.page_tokens
-        self.num_pages = (pool_tokens + c.page_tokens - 1) // c.page_tokens if pool_tokens else per_slot * num_slots
-        self._load(weights)
-        # prompts: recurrences on the tensor cores in bf16 when every head fits a tile, f32 products otherwise
-        self.tensor_recurrence = dtype == BF16 and all(max(l.mixer.dim, l.mixer.vdim) <= 128 for l in c.layers if l.mixer.recurrent)
-        self.chunk = TILE if self.tensor_recurrence else CHUNK
-        es = torch.empty((), dtype=dtype).element_size()
-        att = [l.mixer for l in c.layers if not l.mixer.recurrent]
-        rec = [l.mixer for l in c.layers if l.mixer.recurrent]
-        self.state_manager = PagedState(model="falinex", context=max_context, residents=num_slots, page_tokens=c.page_tokens, pool_pages=self.num_pages,
-                                        row_bytes=sum(m.kv_heads * (m.dim + m.vdim) for m in att) * es,
-                                        slot_bytes=sum(m.heads * m.dim * m.vdim for m in rec) * 4, vocab=c.vocab, device=dev, window=c.window)
-        self.page_table = self.state_manager.table
-        for L in self.layers:
-            m = L["m"]
-            if m.recurrent:
-                L["state"] = L["rec"].state(num_slots, dev)
-            else:
-                L["k_cache"] = torch.zeros(self.num_pages, c.page_tokens, m.kv_heads, m.dim, dtype=dtype, device=dev)
-                L["v_cache"] = torch.zeros(self.num_pages, c.page_tokens, m.kv_heads, m.vdim, dtype=dtype, device=dev)
-        T = max_tokens
-        i32 = lambda: torch.zeros(T, dtype=torch.int32, device=dev)
-        self.tokens, self.positions, self.slots, self.next_ids = i32(), i32(), i32(), i32()
-        self.next_vals = torch.zeros(T, dtype=F32, device=dev)
-        self.rows = _Rows(self, T, False)
-        self._logits = torch.empty(T, c.vocab, dtype=F32, device=dev)
-        self.logits = self._logits if keep_logits else None
-        self.partial = torch.empty(((c.vocab + 7) // 8) * 8 * 2, dtype=F32, device=dev)
-        self.sample_scratch = torch.empty(T * ((c.vocab + 4095) // 4096) * 128, dtype=F32, device=dev)
-        self.inv_temp = torch.full((T,), 1e4, dtype=F32, device=dev)
-        # the fused decode chain needs operand widths that are whole 16-byte chunks
-        self.fused = dtype == BF16 and all(n % 8 == 0 for l in c.layers for n in (c.width, l.ff, l.mixer.heads * l.mixer.vdim))
-        self.fused_rows = 2                   # beyond this the CUDA-core products are FMA-bound and the GEMMs take over
+    name = "falinex"
+
+    def make_rows(self, rows: int, chunked: bool) -> _Rows:
+        return _Rows(self, rows, chunked)
 
     def _load(self, W: Dict[str, torch.Tensor]) -> None:
-        c, dev, A = self.cfg, self.fabric.device, self.dtype
-
-        def mat(*names):
-            """Rows of the named matrices, one after the other; columns padded to 8 elements."""
-            t = torch.cat([W[n].to(dev) for n in names], 0).to(A)
-            return torch.nn.functional.pad(t, (0, _pad8(t.shape[1]) - t.shape[1])).contiguous()
-
-        vec = lambda n: W[n].to(dev).float().contiguous()
+        c, dev = self.cfg, self.fabric.device
+        mat, vec = (lambda *n: self._mat(W, *n)), (lambda n: self._vec(W, n))
         self.embed, self.head, self.final_norm = mat("embed"), mat("head"), vec("final.norm")
         built: Dict[int, dict] = {}
         self.layers: List[dict] = []
@@ -389,6 +307,28 @@ class FalinexDecoder:
                     S.update(q_norm=vec(p + "mix.q.norm"), k_norm=vec(p + "mix.k.norm"), sink=vec(p + "mix.sink"), gate_act="sigmoid")
                 built[j] = S
             self.layers.append(dict(built[j]))        # shared tensors, own state
+
+        # prompts: recurrences on the tensor cores in bf16 when every head fits a tile, f32 products otherwise
+        self.tensor_recurrence = self.dtype == BF16 and all(max(l.mixer.dim, l.mixer.vdim) <= 128 for l in c.layers if l.mixer.recurrent)
+        self.chunk = TILE if self.tensor_recurrence else CHUNK
+        # the fused decode chain needs operand widths that are whole 16-byte chunks
+        self.fused = self.dtype == BF16 and all(n % 8 == 0 for l in c.layers for n in (c.width, l.ff, l.mixer.heads * l.mixer.vdim))
+
+    def _state_bytes(self) -> tuple:
+        es = torch.empty((), dtype=self.dtype).element_size()
+        att = [l.mixer for l in self.cfg.layers if not l.mixer.recurrent]
+        rec = [l.mixer for l in self.cfg.layers if l.mixer.recurrent]
+        return sum(m.kv_heads * (m.dim + m.vdim) for m in att) * es, sum(m.heads * m.dim * m.vdim for m in rec) * 4
+
+    def _make_states(self) -> None:
+        c, dev = self.cfg, self.fabric.device
+        for L in self.layers:
+            m = L["m"]
+            if m.recurrent:
+                L["state"] = L["rec"].state(self.num_slots, dev)
+            else:
+                L["k_cache"] = torch.zeros(self.num_pages, c.page_tokens, m.kv_heads, m.dim, dtype=self.dtype, device=dev)
+                L["v_cache"] = torch.zeros(self.num_pages, c.page_tokens, m.kv_heads, m.vdim, dtype=self.dtype, device=dev)
 
     @classmethod
     def from_checkpoint(cls, path, fabric: Fabric, **kw) -> "FalinexDecoder":
@@ -494,98 +434,6 @@ class FalinexDecoder:
                 owed = L["norm2"]
         N.post_norm_add(y, owed, c.eps, x, xa, self.final_norm)
 
-    def forward(self, T: Optional[int] = None) -> torch.Tensor:
-        n = self.T if T is None else T
-        B, tok, pos, slot = self.rows, self.tokens[:n], self.positions[:n], self.slots[:n]
-        if self.fused and n <= self.fused_rows:
-            self._layers_fused(B, n, tok, pos, slot)
-        else:
-            self._layers(B, n, tok, pos, slot, None, True)
-        if self.dtype == BF16:
-            K.lm_head_argmax(B.xa[:n], self.head, self.fabric, vocab_offset=0, partial=self.partial, logits=None if self.logits is None else self.logits[:n],
-                             out_ids=self.next_ids[:n], out_vals=self.next_vals[:n])
-        else:
-            N.linear(B.xa[:n], self.head, self._logits[:n])
-            K.sample_topk(self._logits[:n], self.fabric, top_k=1, inv_temperature=self.inv_temp[:n], scratch=self.sample_scratch, out_ids=self.next_ids[:n])
-        return self.next_ids[:n]
 
-    def forward_feedback(self, T: Optional[int] = None) -> torch.Tensor:
-        n = self.T if T is None else T
-        self.forward(n)
-        self.tokens[:n].copy_(self.next_ids[:n])
-        self.positions[:n].add_(1)
-        return self.next_ids[:n]
-
-    def capture(self, T: Optional[int] = None, feedback: bool = False) -> torch.cuda.CUDAGraph:
-        n = self.T if T is None else T
-        self.forward(n)
-        torch.cuda.synchronize()
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
-            self.forward_feedback(n) if feedback else self.forward(n)
-        return g
-
-
-class FalinexRows:
-    """Packed-step executor: up to ``max_rows`` rows of any sequences (portions of prompts, decode rows), rows of one sequence
-    consecutive and in position order, as one matrix-matrix pass. Steps without a long run and of at most ``graph_rows_max`` rows
-    (a decode row per running sequence) replay a CUDA graph per row count."""
-
-    packed = True              # the engine hands over the rows of a whole step
-    batch_threshold = 8
-
-    def __init__(self, dec: FalinexDecoder, max_rows: int = 512):
-        self.dec, self.M = dec, max_rows
-        self.B = _Rows(dec, max_rows, True)
-        dev = dec.fabric.device
-        self.graph_rows_max = min(64, max_rows)
-        self.use_graphs = True
-        self._static = torch.zeros(3, self.graph_rows_max, dtype=torch.int32, device=dev)
-        self._graphs: Dict[int, torch.cuda.CUDAGraph] = {}
-
-    def plan(self, slots: List[int], positions: List[int]) -> StepPlan:
-        return StepPlan(slots, positions, group=ATTN_ROWS, chunk=self.dec.chunk)
-
-    def _run(self, tokens, positions, slots, plan: StepPlan, control, probe) -> None:
-        d, m = self.dec, tokens.numel()
-        if plan.runs or m > self.graph_rows_max or not self.use_graphs or probe is not None:
-            d._layers(self.B, m, tokens, positions, slots, plan.bind(control, positions), False, probe)
-            return
-        st = self._static[:, :m]
-        st[0].copy_(tokens)
-        st[1].copy_(positions)
-        st[2].copy_(slots)
-        g = self._graphs.get(m)
-        if g is not None:
-            g.replay()
-            return
-        d._layers(self.B, m, *st, None, False)             # the real run of this step (and the warm-up of the capture)
-        torch.cuda.synchronize()
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):                          # records only: no state is touched a second time
-            d._layers(self.B, m, *st, None, False)
-        self._graphs[m] = g
-
-    def forward_rows(self, tokens: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, select: torch.Tensor, plan: StepPlan, control: torch.Tensor,
-                     probe: Optional[list] = None) -> torch.Tensor:
-        """f32 logits ``[len(select), vocab]`` of rows ``select``; ``control``: ``plan.control`` on the device."""
-        d, c, m = self.dec, self.dec.cfg, tokens.numel()
-        assert 1 <= m <= self.M and plan.rows == m
-        self._run(tokens, positions, slots, plan, control, probe)
-        xn = torch.zeros(select.numel(), self.B.xa.shape[1], dtype=d.dtype, device=tokens.device)
-        N.rms_rows(self.B.x[:m], d.final_norm, c.eps, xn, select.to(torch.int32))
-        logits = torch.empty(select.numel(), c.vocab, dtype=F32, device=tokens.device)
-        N.linear(xn, d.head, logits, status_ptr=d.fabric.desc.status)
-        return logits
-
-    def forward(self, tokens: torch.Tensor, pos0: int, slot: int = 0) -> torch.Tensor:
-        """A chunk of one sequence; returns the greedy next token (device tensor ``[1]``)."""
-        d, m, dev = self.dec, tokens.numel(), tokens.device
-        pos = torch.arange(pos0, pos0 + m, dtype=torch.int32, device=dev)
-        sl = torch.full((m,), slot, dtype=torch.int32, device=dev)
-        plan = self.plan([slot] * m, list(range(pos0, pos0 + m)))
-        logits = self.forward_rows(tokens, pos, sl, torch.tensor([m - 1], device=dev), plan, plan.control.to(dev))
-        if d.logits is not None:
-            d.logits[:1].copy_(logits)
-        K.sample_topk(logits, d.fabric, top_k=1, inv_temperature=d.inv_temp[:1], scratch=d.sample_scratch, out_ids=d.next_ids[:1])
-        return d.next_ids[:1]
+class FalinexRows(StreamRows):
+    """Packed-step executor: see :class:`StreamRows`."""

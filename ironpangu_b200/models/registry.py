@@ -17,12 +17,14 @@ class Family:
     decoder: str               # class with from_checkpoint(path, fabric, ...)
     rows: str                  # packed-step executor over that decoder
     exact: bool                # has a true 32-bit mode
+    presets: Tuple[str, ...] = ()      # names of PRESETS of the module: configurations served with random weights
 
     def load(self):
         return importlib.import_module(f"ironpangu_b200.models.{self.module}")
 
 
-FAMILIES: Tuple[Family, ...] = (Family("Falinex", "falinex", "FalinexDecoder", "FalinexRows", True),)
+FAMILIES: Tuple[Family, ...] = (Family("Falinex", "falinex", "FalinexDecoder", "FalinexRows", True, ("falinex-tiny", "falinex2b")),
+                                Family("Ponenex", "ponenex", "PonenexDecoder", "PonenexRows", True, ("ponenex-tiny", "ponenex-text")))
 
 
 def family_of(checkpoint_dir) -> Family:
@@ -33,6 +35,23 @@ def family_of(checkpoint_dir) -> Family:
         if f.architecture == name:
             return f
     raise ValueError(f"no model family for architecture {name!r} (known: {', '.join(f.architecture for f in FAMILIES)})")
+
+
+def preset_names() -> Tuple[str, ...]:
+    return tuple(n for f in FAMILIES for n in f.presets)
+
+
+def open_preset(name: str, fabric, *, layers: int = 0, seed: int = 0, max_rows: int = 512, **decoder_options):
+    """``(decoder, packed-step executor)`` of a preset configuration with random weights; ``layers`` keeps the first so many."""
+    f = next((f for f in FAMILIES if name in f.presets), None)
+    if f is None:
+        raise ValueError(f"no preset {name!r} (known: {', '.join(preset_names())})")
+    mod = f.load()
+    cfg = mod.PRESETS[name]()
+    if layers:
+        cfg.layers = cfg.layers[:layers]
+    dec = getattr(mod, f.decoder)(cfg, mod.random_weights(cfg, fabric.device, seed=seed), fabric, **decoder_options)
+    return dec, getattr(mod, f.rows)(dec, max_rows=max_rows)
 
 
 def open_checkpoint(checkpoint_dir, fabric, *, max_rows: int = 512, **decoder_options):

@@ -58,12 +58,12 @@ _SIGS = {
     "ifab_gemm_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, _P, _P],
     "ifab_gemm_act_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P, _P],
     "ifab_linear_f32": [_P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, _P],
-    "ifab_embed_rows": [_P, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, _P, _P],
+    "ifab_embed_rows": [_P, _P, c_long, c_float, _P, c_float, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, _P, _P],
     "ifab_post_norm_add": [_P, c_long, _P, _P, c_float, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
     "ifab_rms_rows": [_P, c_long, _P, _P, c_float, _P, c_long, c_int, c_int, c_int, _P],
     "ifab_group_norm_gate": [_P, c_long, _P, c_float, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P],
     "ifab_gate_rows": [_P, c_long, c_int, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P],
-    "ifab_gemv_post_norm": [_P, c_long, _P, c_float, _P, _P, c_long, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
+    "ifab_gemv_post_norm": [_P, c_long, _P, _P, c_float, _P, _P, c_long, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
     "ifab_gemv_group_norm": [_P, c_long, _P, c_float, c_int, _P, c_long, c_int, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
     "ifab_gemv_act": [_P, c_long, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
     "ifab_la_step": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_float, _P, _P, _P, _P, _P, c_long, c_int, _P],
@@ -75,19 +75,36 @@ _SIGS = {
     "ifab_qk_norm_rope_write": [_P, c_long, c_int, c_int, c_int, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_int, c_int,
                                 c_int, _P, c_long, c_int, _P, _P, c_int, _P, _P],
     "ifab_ctx_gather_pad": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_long, _P, _P],
-    "ifab_fa_window_bf16": [_P, c_long, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, c_long,
-                            c_int, _P, _P],
+    "ifab_fa_window_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                            c_float, _P, _P, c_long, c_int, c_int, _P, _P],
     "ifab_gqa_window_attention": [_P, c_long, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int,
                                   c_int, _P, c_u64, _P, c_long, _P, _P],
     "ifab_window_attn": [_P, c_long, c_int, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, c_long, c_int, _P,
                          c_long, c_int, _P, _P],
+    "ifab_moe_down_f32_decode": [_P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, c_long, _P],
+    "ifab_moe_route": [_P, c_long, _P, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, _P, _P],
+    "ifab_moe_combine_norm": [_P, c_long, _P, _P, c_int, _P, c_long, _P, _P, _P, c_float, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
+    "ifab_linear_f32_batched": [_P, c_long, c_long, _P, c_long, c_long, _P, c_long, c_long, c_int, c_int, c_int, c_int, _P],
+    "ifab_grouped_linear_f32": [_P, c_long, _P, c_int, _P, c_int, c_int, _P, _P, c_int, c_int, _P, c_long, _P],
+    "ifab_gemm_heads_bf16": [_P, c_long, c_int, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P],
+    "ifab_router_post_norm": [_P, c_long, _P, _P, c_float, _P, _P, c_long, _P, c_long, _P, _P, c_long, _P, c_int, c_int, c_int, c_int, c_float, _P, _P, _P,
+                              _P, c_int, c_int, c_int, _P],
+    "ifab_latent_prepare": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, c_int, _P, _P, _P, c_int, c_int, c_int, _P, c_long,
+                            _P, c_int, c_int, c_int, _P, _P],
+    "ifab_rotate_heads": [_P, c_long, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P],
+    "ifab_latent_absorb": [_P, c_long, c_int, c_int, _P, _P, c_int, _P, c_int, c_int, c_int, c_int, _P],
+    "ifab_latent_split": [_P, _P, c_long, c_int, _P, c_int, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, _P,
+                          c_u64, _P, _P],
+    "ifab_latent_merge": [_P, _P, c_int, c_int, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P, c_long, _P],
+    "ifab_latent_merge_vup": [_P, _P, c_int, c_int, c_int, _P, c_long, c_int, c_int, c_int, _P, c_int, _P, c_long, _P],
+    "ifab_latent_gather": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P],
     "ifab_gemm_bf16_2sm": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, _P, _P],
     "ifab_gemm_swiglu_bf16_2sm": [_P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, _P, _P],
     "ifab_gemm_bf16_2sm_persistent": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, _P, _P],
     "ifab_gemm_allreduce_bf16": [_P, c_long, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, C.POINTER(IfabFabric), _P],
     "ifab_gemm_reduce_scatter_bf16": [_P, c_long, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, C.POINTER(IfabFabric), _P],
     "ifab_router_topk": [_P, c_long, _P, c_float, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, c_long, _P],
-    "ifab_moe_gate_up_decode": [_P, c_long, _P, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, _P],
+    "ifab_moe_gate_up_decode": [_P, c_long, _P, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, c_int, _P],
     "ifab_moe_down_allreduce_decode": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, c_long, _P,
                                        c_long, C.POINTER(IfabFabric), _P],
     "ifab_moe_block_decode": [_P, c_long, _P, c_float, _P, _P, c_int, c_int, c_int, c_int, c_float, _P, _P, _P, _P, c_int, c_int,

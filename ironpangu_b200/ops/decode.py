@@ -120,7 +120,7 @@ def moe_gate_up(x: torch.Tensor, ids: torch.Tensor, w_gu: torch.Tensor, e0: int,
                 act: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Gate/up projections + SwiGLU of the routes owned by this rank (and of the shared-expert shard).
 
-    ``w_gu``: ``[E_local, 2F, D]``; ``act``: ``[T, topk+1, F]`` (slot ``topk`` is the shared expert)."""
+    ``w_gu``: ``[E_local, 2F, D]``; ``act``: ``[T, topk+1, >= F]`` (slot ``topk`` is the shared expert, which may be wider than F)."""
     T, D = x.shape
     topk = ids.shape[1]
     e_local, twoF, _ = w_gu.shape
@@ -129,7 +129,7 @@ def moe_gate_up(x: torch.Tensor, ids: torch.Tensor, w_gu: torch.Tensor, e0: int,
     if act is None:
         act = torch.zeros(T, topk + 1, F, dtype=BF16, device=x.device)
     check(_lib.load().ifab_moe_gate_up_decode(x.data_ptr(), _rows(x), _ptr(norm_w), eps, ids.data_ptr(), T, D, F, topk,
-                                              e0, e_local, w_gu.data_ptr(), _ptr(w_shared_gu), Fs, act.data_ptr(),
+                                              e0, e_local, w_gu.data_ptr(), _ptr(w_shared_gu), Fs, act.data_ptr(), act.shape[2],
                                               _stream()), "moe_gate_up")
     return act
 

@@ -27,12 +27,13 @@ def _f32(t: torch.Tensor) -> int:
     return int(t.dtype == torch.float32)
 
 
-def embed_rows(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, xa: torch.Tensor, status_ptr: Optional[int] = None) -> None:
-    """``x`` (f32 residual) and ``xa`` (activation copy) = rows ``ids`` of ``table``."""
+def embed_rows(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, xa: torch.Tensor, *, scale: float = 1.0, gain: Optional[torch.Tensor] = None,
+               eps: float = 0.0, status_ptr: Optional[int] = None) -> None:
+    """``x`` (f32 residual) = rows ``ids`` of ``table`` times ``scale``; ``xa`` (activation type) = x, or ``rms(x) * gain``."""
     T, D = x.shape
     assert ids.dtype == torch.int32 and x.dtype == torch.float32 and table.dtype == xa.dtype
-    check(_lib.load().ifab_embed_rows(ids.data_ptr(), table.data_ptr(), table.stride(0), x.data_ptr(), x.stride(0), xa.data_ptr(), xa.stride(0), _f32(xa),
-                                      T, D, table.shape[0], status_ptr, _s()), "embed_rows")
+    check(_lib.load().ifab_embed_rows(ids.data_ptr(), table.data_ptr(), table.stride(0), scale, _p(gain), eps, x.data_ptr(), x.stride(0), xa.data_ptr(),
+                                      xa.stride(0), _f32(xa), T, D, table.shape[0], status_ptr, _s()), "embed_rows")
 
 
 def post_norm_add(y: torch.Tensor, w: torch.Tensor, eps: float, x: torch.Tensor, xa: torch.Tensor, final: Optional[torch.Tensor] = None) -> None:
@@ -66,12 +67,13 @@ def gate_rows(o: torch.Tensor, head_stride: int, gate: torch.Tensor, act: str, o
 
 
 def gemv_post_norm(y: torch.Tensor, norm_w: torch.Tensor, eps: float, x_in: torch.Tensor, x_out: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
-                   act: Optional[str] = None) -> None:
-    """``x_out = x_in + rms(y) * norm_w``; ``out = act(bf16(x_out) @ w.T)`` in one launch (decode rows)."""
+                   act: Optional[str] = None, next_norm: Optional[torch.Tensor] = None) -> None:
+    """``x_out = x_in + rms(y) * norm_w``; ``out = act(bf16(x_out) @ w.T)``, or of ``bf16(rms(x_out) * next_norm)``, in one launch (decode
+    rows)."""
     T, K = y.shape
     N = w.shape[0]
     assert w.shape[1] == K and w.is_contiguous() and x_in.stride(0) == x_out.stride(0)
-    check(_lib.load().ifab_gemv_post_norm(y.data_ptr(), y.stride(0), norm_w.data_ptr(), eps, x_in.data_ptr(), x_out.data_ptr(), x_in.stride(0), w.data_ptr(),
+    check(_lib.load().ifab_gemv_post_norm(y.data_ptr(), y.stride(0), norm_w.data_ptr(), _p(next_norm), eps, x_in.data_ptr(), x_out.data_ptr(), x_in.stride(0), w.data_ptr(),
                                           out.data_ptr(), out.stride(0), _f32(out), ACTIVATIONS[act], T, N, K, _s()), "gemv_post_norm")
 
 

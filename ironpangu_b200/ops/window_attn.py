@@ -86,6 +86,6 @@ def fa_window(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, pag
     lib = _lib.load()
     check(lib.ifab_ctx_gather_pad(k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr(), slot, page_table.shape[1], pt, pages, first, n, rows, G, d,
                                   dp, e, ctx_k.data_ptr(), ctx_vt.data_ptr(), ctx_vt.stride(0), status_ptr, _s()), "ctx_gather_pad")
-    check(lib.ifab_fa_window_bf16(q.data_ptr(), q.stride(0), ctx_k.data_ptr(), ctx_k.stride(0), ctx_vt.data_ptr(), ctx_vt.stride(0), out.data_ptr(),
+    check(lib.ifab_fa_window_bf16(q.data_ptr(), q.stride(0), ctx_k.data_ptr(), ctx_k.stride(0), None, 0, 0, ctx_vt.data_ptr(), ctx_vt.stride(0), out.data_ptr(),
                                   out.stride(0), m, n, heads, heads // G, dp, e, pos0 - first, window, scale, _p(sink), _p(gate),
-                                  0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], status_ptr, _s()), "fa_window")
+                                  0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], 0, status_ptr, _s()), "fa_window")

@@ -546,25 +546,21 @@ def build_engine(args, rank: int, world: int, rec=None) -> BatchEngine:
                           token_budget=args.max_num_batched_tokens, use_graphs=not args.no_graphs)
         mark("sampling", "per-slot sampling state")
         return eng
-    if args.model == "checkpoint" or args.model.startswith("falinex"):
-        # families opened from a checkpoint directory (config.json names the architecture), and the presets of Falinex with random weights;
-        # KV pages from one pool, packed steps
-        from ironpangu_b200.models import falinex as F
-        from ironpangu_b200.models import registry
+    from ironpangu_b200.models import registry
 
+    if args.model == "checkpoint" or args.model in registry.preset_names():
+        # families opened from a checkpoint directory (config.json names the architecture), and their presets with random weights; KV pages
+        # from one pool, packed steps
         if world != 1:
             raise SystemExit("checkpoint models run on one GPU")
         opts = dict(max_tokens=8, max_context=args.max_model_len, num_slots=args.max_num_seqs, pool_tokens=args.kv_pool_tokens,
-                    keep_logits=True, dtype=torch.float32 if args.dtype == "float32" else torch.bfloat16)
-        rows = max(args.prefill_chunk, 64)
+                    keep_logits=True, dtype=torch.float32 if args.dtype == "float32" else torch.bfloat16, max_rows=max(args.prefill_chunk, 64))
         if args.model == "checkpoint":
             if not args.checkpoint:
                 raise SystemExit("--model checkpoint needs --checkpoint DIR")
-            fdec, frows = registry.open_checkpoint(args.checkpoint, fab, max_rows=rows, **opts)
+            fdec, frows = registry.open_checkpoint(args.checkpoint, fab, **opts)
         else:
-            fcfg = F.FalinexConfig.tiny() if args.model == "falinex-tiny" else F.FalinexConfig.text2b(layers=args.layers or 24)
-            fdec = F.FalinexDecoder(fcfg, F.random_weights(fcfg, dev, seed=args.seed), fab, **opts)
-            frows = F.FalinexRows(fdec, max_rows=rows)
+            fdec, frows = registry.open_preset(args.model, fab, layers=args.layers, seed=args.seed, **opts)
         mark("weights", "weights, KV page pool, recurrent states and step workspace")
         eng = BatchEngine(fdec, f"ifab-{args.model}", args.max_model_len, fdec.cfg.vocab, eos=-1, greedy_only=args.greedy_only, prefill=frows,
                           token_budget=args.max_num_batched_tokens, use_graphs=not args.no_graphs)
@@ -797,9 +793,11 @@ def serve(engine, rank: int, world: int, sock_path: str, group=None, agreement="
 
 
 def main() -> None:
+    from ironpangu_b200.models import registry
+
     ap = argparse.ArgumentParser()
     ap.add_argument("--model", default="tiny", choices=["tiny", "flagship", "dense-tiny", "dense2b", "hybrid-tiny", "hybrid2b", "hybrid", "hyper-tiny", "pangu92b", "pangu92b-learned",
-                                                         "falinex-tiny", "falinex2b", "checkpoint"],
+                                                         *registry.preset_names(), "checkpoint"],
                     help="checkpoint: the family that config.json of --checkpoint names (models/registry.py)")
     ap.add_argument("--layers", type=int, default=0)
     ap.add_argument("--seed", type=int, default=0)
