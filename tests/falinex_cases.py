@@ -60,9 +60,3 @@ def weights(cfg, seed=0):
 def tokens(cfg, n, seed=0):
     return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(1000 + seed)).tolist()
 
-
-def logit_error(got, want):
-    """Largest rms difference of a row of logits, mean taken off, over the spread of the wanted logits."""
-    d = got.double() - want
-    d = d - d.mean(-1, keepdim=True)
-    return float((d.pow(2).mean(-1).sqrt() / want.std()).max())

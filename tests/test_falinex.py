@@ -12,7 +12,9 @@ import pytest
 import torch
 
 import falinex_oracle as O
-from falinex_cases import CASES, attention, config, lightning, logit_error, retention, tokens, weights
+from falinex_cases import CASES, attention, config, lightning, retention, tokens, weights
+from stream_rig import Rig as StreamRig
+from stream_rig import cut, logit_error, random_batches
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 BF16, F32 = torch.bfloat16, torch.float32
@@ -182,54 +184,8 @@ def test_replay_admits_batches_and_releases():
 # ---------------------------------------------------------------------------------------------------------------------------
 # GPU: the model through the engine
 # ---------------------------------------------------------------------------------------------------------------------------
-class Rig:
-    """The serving engine over one configuration; ``run`` feeds (request, count) steps and returns each request's logits of every row."""
-
-    def __init__(self, cfg, dtype, *, context=320, pool=0, residents=4, rows=256, seed=0, graphs=True):
-        from ironpangu_b200.models import falinex as F
-        from ironpangu_b200.parallel.fabric import Fabric
-        from ironpangu_b200.runtime.engine_worker import BatchEngine
-
-        self.cfg, self.fab, self.w = cfg, Fabric(0, 1), weights(cfg, seed)
-        self.dec = F.FalinexDecoder(F.FalinexConfig.from_dict(cfg), self.w, self.fab, max_context=context, num_slots=residents, pool_tokens=pool,
-                                    keep_logits=True, dtype=dtype)
-        self.eng = BatchEngine(self.dec, "t", context, cfg["vocab"], prefill=F.FalinexRows(self.dec, max_rows=rows), use_graphs=graphs)
-
-    def run(self, requests, steps):
-        """requests: id -> tokens; steps: lists of (id, count). A request ends with its last token; ids with '#' run the tokens of the
-        part before it once more."""
-        from ironpangu_b200.runtime.replay import Replay
-
-        r, at, out = Replay(self.eng), {}, {}
-        for n, step in enumerate(steps):
-            entries, end, got = [], [], []
-            for name, count in step:
-                toks = requests[name.split("#")[0]]
-                lo = at.get(name, 0)
-                part = toks[lo:lo + count]
-                entries.append({"id": name, "tokens": part, "want": list(range(len(part)))})
-                got += [name] * len(part)
-                at[name] = lo + len(part)
-                if at[name] == len(toks):
-                    end.append(name)
-            logits = r.step({"step": n, "entries": entries, "end": end})
-            for i, name in enumerate(got):
-                out.setdefault(name, []).append(logits[i])
-        assert self.fab.status() == 0
-        return {k: torch.stack(v) for k, v in out.items()}
-
-    def close(self):
-        self.dec.state_manager.close()
-        self.fab.close()
-
-
-def _cut(rnd, n, sizes):
-    out = []
-    while n:
-        c = min(n, rnd.choice(sizes))
-        out.append(c)
-        n -= c
-    return out
+def Rig(cfg, dtype, *, seed=0, **kw):
+    return StreamRig(cfg, weights(cfg, seed), dtype, **kw)
 
 
 @pytest.mark.gpu
@@ -242,7 +198,7 @@ def test_whole_prompts_portions_and_decoding(name, dtype):
     toks = tokens(cfg, n)
     want = O.forward(cfg, rig.w, toks)
     rnd = random.Random(name)
-    schedules = {"whole": [n], "token by token": [1] * 40, "prompt, then decoding": [n - 70] + [1] * 70, "portions": _cut(rnd, n, [2, 3, 5, 9, 17, 33, 64, 65]),
+    schedules = {"whole": [n], "token by token": [1] * 40, "prompt, then decoding": [n - 70] + [1] * 70, "portions": cut(rnd, n, [2, 3, 5, 9, 17, 33, 64, 65]),
                  "pairs": [2] * 30, "first tokens": [1, 2, 3, 1, 5, 16, 15, 2]}
     for what, cuts in schedules.items():
         got = rig.run({"a": toks[:sum(cuts)]}, [[("a", c)] for c in cuts])["a"]
@@ -263,22 +219,7 @@ def test_unequal_requests_in_one_batch_with_reused_pages_and_slots(name, dtype):
     lens = {"a": 150, "b": 23, "c": 97, "d": 5, "e": 64, "f": 33, "g": 121}
     reqs = {k: tokens(cfg, n, i) for i, (k, n) in enumerate(lens.items())}
     want = {k: O.forward(cfg, rig.w, t) for k, t in reqs.items()}
-    waiting, live, steps = list(reqs) + ["a#2", "d#2"], {}, []
-    while waiting or live:
-        while waiting and len(live) < 4 and sum((v + 63) // 64 * 64 for v in (len(reqs[k.split("#")[0]]) for k in list(live) + waiting[:1])) <= 448:
-            k = waiting.pop(0)
-            live[k] = len(reqs[k.split("#")[0]])
-        step = []
-        for k in list(live):
-            if rnd.random() < 0.2:
-                continue
-            c = min(live[k], rnd.choice([1, 1, 1, 2, 3, 16, 29, 64]))
-            step.append((k, c))
-            live[k] -= c
-            if not live[k]:
-                del live[k]
-        if step:
-            steps.append(step)
+    steps = random_batches(rnd, lens, list(reqs) + ["a#2", "d#2"], 4, 448, [1, 1, 1, 2, 3, 16, 29, 64])
     got = rig.run(reqs, steps)
     for k, g in got.items():
         e = logit_error(g, want[k.split("#")[0]])
