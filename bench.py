@@ -34,10 +34,11 @@ def parse():
     ap.add_argument("--impl", default="native", choices=["native", "reference", "nccl_cublas"])
     ap.add_argument("--model", default="flagship", choices=["flagship", "tiny", "dense2b"],
                     help="flagship: the 92B-class MLA+MoE model of the headline metric; dense2b: the Qwen-style 2B dense GQA decoder")
-    ap.add_argument("--design", default="", choices=["", "falinex"],
-                    help="falinex: instead of the headline run, prefill and decode throughput of the Falinex design beside the dense model at equal "
-                         "size, one JSON line per size (ironpangu_b200/utils/bench_falinex.py; one GPU)")
-    ap.add_argument("--design-sizes", default="small,2b,8b", help="sizes of --design falinex")
+    ap.add_argument("--design", default="", choices=["", "falinex", "ponenex"],
+                    help="instead of the headline run, prefill and decode throughput of a design beside its closest other model at equal size, one JSON "
+                         "line per size (one GPU): falinex beside the dense model (ironpangu_b200/utils/bench_falinex.py), ponenex beside the MLA + MoE "
+                         "model (bench_ponenex.py)")
+    ap.add_argument("--design-sizes", default="", help="sizes of --design, comma separated (default: all)")
     ap.add_argument("--context", type=int, default=512)
     ap.add_argument("--prefill", default="gemm", choices=["gemm", "decode"],
                     help="gemm: tensor-core prefill path (native impl only); decode: prompt through the decode kernels, 8 rows a time")
@@ -175,13 +176,14 @@ def main():
                           "no Rust toolchain in this image (pip install of the reference tree fails: no setup.py/pyproject)"}))
         return 0
 
-    if args.design == "falinex":
-        from ironpangu_b200.utils import bench_falinex
+    if args.design:
+        import importlib
 
+        arm = importlib.import_module(f"ironpangu_b200.utils.bench_{args.design}")
         sampler = ClockSampler(0)
         sampler.start()
         try:
-            return bench_falinex.main(["--sizes", args.design_sizes])
+            return arm.main(["--sizes", args.design_sizes] if args.design_sizes else [])
         finally:
             print(json.dumps({"bench": args.design, "clocks": sampler.stop()}))
 

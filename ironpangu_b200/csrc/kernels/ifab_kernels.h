@@ -334,13 +334,21 @@ int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const 
 int ifab_latent_prepare(const void* proj, long ldp, int f32, int q_off, int q_rank, int kv_off, int kv_rank, int rot_dim, const float* q_gain,
                         const float* kv_gain, float eps, const void* rope, int rot, const int32_t* positions, const int32_t* slots, const int32_t* page_table,
                         int max_pages, int page_tokens, int num_pages, void* cq, long ldc, void* cache, int Lp, int Rp, int T, uint32_t* status, void* stream);
+int ifab_latent_query(const void* proj, long ldp, int q_off, int q_rank, int kv_off, int kv_rank, int rot_dim, const void* q_gain, const float* kv_gain,
+                      float eps, const void* rope, int rot, const int32_t* positions, const int32_t* slots, const int32_t* page_table, int max_pages,
+                      int page_tokens, int num_pages, void* cache, int Lp, int Rp, const void* w_uq, int N, void* q, long ldq, int T, uint32_t* status,
+                      void* stream);
 int ifab_rotate_heads(void* q, long ldq, int f32, int head_stride, int off, int H, int rot, const void* rope, int T, void* stream);
 int ifab_latent_absorb(void* q, long ldq, int head_stride, int rot_off, const void* w_uk, const void* rope, int rot, float* q_lat, int T, int H, int d, int Lp,
                        void* stream);
 int ifab_latent_split(const float* q_lat, const void* q_rot, long ldq, int head_stride, const void* cache, int f32, int Lp, int Rp, const int32_t* positions,
                       const int32_t* slots, const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int window, float scale, int T, int H,
                       int kps, int splits, float* scratch, uint64_t scratch_bytes, uint32_t* status, void* stream);
-int ifab_latent_merge(const float* scratch, const int32_t* positions, int window, int kps, int splits, const void* gate, long ldg, int f32, int T, int H, int Lp,
+/* for many rows: splits * sub partials (sub warps of a CTA share four heads; 1 from 17 heads on) */
+int ifab_latent_batch(const float* q_lat, const void* q_rot, long ldq, int head_stride, const void* cache, int Lp, int Rp, const int32_t* positions,
+                      const int32_t* slots, const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int window, float scale, int T, int H,
+                      int kps, int splits, int sub, float* scratch, uint64_t scratch_bytes, uint32_t* status, void* stream);
+int ifab_latent_merge(const float* scratch, const int32_t* positions, int window, int kps, int splits, int sub, const void* gate, long ldg, int f32, int T, int H, int Lp,
                       void* o_lat, long ldo, void* stream);
 int ifab_latent_merge_vup(const float* scratch, const int32_t* positions, int window, int kps, int splits, const void* gate, long ldg, int T, int H, int Lp,
                           const void* w_uv, int vdim, void* out, long ldo, void* stream);

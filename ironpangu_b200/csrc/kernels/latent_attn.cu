@@ -4,11 +4,15 @@
 //
 //   latent_prepare_kernel   one packed projection row -> normed query latent (operand of the query up-projection), and into the page of
 //                           the row's sequence: normed latent, rotated key part
+//   latent_query_kernel     the same for a few rows (decode) in one launch with the query up-projection: the first CTAs stream W_uq and norm the
+//                           query latent while they stage it, the last T write the pages
 //   rotate_heads_kernel     rotation of the rotated columns of every query head, in place (half layout)
 //   latent_absorb_kernel    q_lat[h] = q_unrotated[h] W_uk[h] for a few rows (decode), rotation of the rest included
 //   latent_split_kernel     split-KV attention over the pages with an optional sliding window: every warp scores four keys for HG heads
 //                           at once; the HG x 4 sums are reduced through a transposing butterfly, so each lane ends with ONE
 //                           (key, head) score, takes one exponential and the weights are broadcast back
+//   latent_batch_kernel     the same for many rows: the warps of a CTA split the HEADS first (four each) and the keys only with what is left of them; the
+//                           keys of a split pass through a ring of shared-memory stages (cp.async) once for all heads
 //   latent_merge_kernel     log-sum-exp merge of the splits, head gate -> o_lat rows (operand of the value up-projection)
 //   latent_merge_vup_kernel merge, gate and value up-projection for a few rows (decode)
 //   latent_gather_kernel    the rows a run of queries can see, out of the pages into dense operands of the tensor-core form
@@ -133,6 +137,57 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(PrepareParams p) {
   grid_dep_launch();
   grid_dep_wait();
   prepare_row<A>(p, blockIdx.x, red);
+}
+
+template <int T, int R>
+__global__ void __launch_bounds__(256) latent_query_kernel(PrepareParams p, const bf16* w_uq, const bf16* q_gain, int N, int ctas, bf16* q, long ldq, int rows) {
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  bf16* xs = reinterpret_cast<bf16*>(smem_raw);
+  __shared__ float red[T * 33];
+  grid_dep_launch();
+  if ((int)blockIdx.x >= ctas) {
+    grid_dep_wait();
+    prepare_row<bf16>(p, blockIdx.x - ctas, red);
+    return;
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n0 = (blockIdx.x * 8 + warp) * R;
+  const bf16* w[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) w[r] = n0 + r < N ? w_uq + (long)(n0 + r) * p.q_rank : nullptr;
+  RowBatch<R> pf;
+  prefetch_rows<R>(w, p.q_rank, pf);
+  grid_dep_wait();
+  stage_x<T>(xs, reinterpret_cast<const bf16*>(p.proj) + p.q_off, p.ldp, 0, rows, p.q_rank, q_gain, p.eps, false, red);
+  if (n0 >= N) return;
+  float acc[R][T];
+#pragma unroll
+  for (int r = 0; r < R; ++r)
+#pragma unroll
+    for (int t = 0; t < T; ++t) acc[r][t] = 0.f;
+  warp_rows_dot<T, R>(w, xs, p.q_rank, acc, pf);
+  warp_reduce_acc<T, R>(acc);
+  if (lane == 0) {
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+#pragma unroll
+      for (int t = 0; t < T; ++t)
+        if (n0 + r < N && t < rows) q[(long)t * ldq + n0 + r] = __float2bfloat16_rn(acc[r][t]);
+  }
+}
+
+template <int T, int R>
+int launch_query(const PrepareParams& p, const bf16* w_uq, const bf16* q_gain, int N, bf16* q, long ldq, int rows, cudaStream_t s) {
+  const size_t smem = (size_t)T * p.q_rank * sizeof(bf16);
+  auto k = latent_query_kernel<T, R>;
+  if (int rc = opt_in_smem(k, smem)) return rc;
+  const int ctas = (N + 8 * R - 1) / (8 * R);
+  return launch_chain(k, dim3(ctas + rows), dim3(256), smem, s, p, w_uq, q_gain, N, ctas, q, ldq, rows);
+}
+template <int T>
+int query_rows(const PrepareParams& p, const bf16* w_uq, const bf16* q_gain, int N, bf16* q, long ldq, int rows, cudaStream_t s) {
+  if (N >= 148 * 8 * 4) return launch_query<T, 4>(p, w_uq, q_gain, N, q, ldq, rows, s);
+  if (N >= 148 * 8 * 2) return launch_query<T, 2>(p, w_uq, q_gain, N, q, ldq, rows, s);
+  return launch_query<T, 1>(p, w_uq, q_gain, N, q, ldq, rows, s);
 }
 
 template <typename A>
@@ -411,9 +466,171 @@ __global__ void __launch_bounds__(256) latent_split_kernel(SplitParams p) {
 }
 
 // ------------------------------------------------------------------------------------------------
+constexpr int TILE_KEYS = 32, STAGES = 3;
+
+__device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool live) {
+  const uint32_t dst = (uint32_t)__cvta_generic_to_shared(smem);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(gmem), "r"(live ? 16 : 0) : "memory");      // 0 bytes read: zero fill
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// bf16; grid (splits, ceil(H / 32), T). `sub` of the eight warps share four heads, each takes every sub-th batch of keys and writes partials of its
+// own: split s leaves partials s * sub .. s * sub + sub - 1
+template <int NL>
+__global__ void __launch_bounds__(256) latent_batch_kernel(SplitParams p, int sub) {
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  bf16* ring = reinterpret_cast<bf16*>(smem_raw);                // [STAGES][TILE_KEYS][Lp + Rp]
+  constexpr int HG = 4, V = KB * HG, GRP = 32 / V;
+  grid_dep_launch();
+  grid_dep_wait();
+  const int split = blockIdx.x, t = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int groups = WARPS / sub, part = warp / groups, h0 = (blockIdx.y * WARPS + warp % groups) * HG;
+  const int pos = p.pg.positions[t];
+  if (pos < 0) return;
+  int first, count;
+  visible(pos, p.window, &first, &count);
+  const int k_begin = split * p.kps;
+  if (k_begin >= count) return;
+  const int k_end = split == p.splits - 1 ? count : min(count, k_begin + p.kps);
+  const int slot = p.pg.slots[t], row = p.Lp + p.Rp, chunks = row / 8, tiles = (k_end - k_begin + TILE_KEYS - 1) / TILE_KEYS;
+  // copies: eight threads per key, each finds its key's page one tile ahead of the copy
+  const int my_row = threadIdx.x >> 3, lane8 = threadIdx.x & 7;
+  auto find = [&](int tile) -> long {
+    const int k = k_begin + tile * TILE_KEYS + my_row;
+    if (k >= k_end) return -1;
+    const long r = page_row(p.pg, slot, first + k);
+    if (r < 0 && lane8 == 0 && p.pg.status) atomicOr(p.pg.status, IFAB_STATUS_BAD_INDEX);
+    return r;
+  };
+  auto copy = [&](int tile, long r) {
+    bf16* dst = ring + ((long)(tile % STAGES) * TILE_KEYS + my_row) * row;
+    const bf16* src = reinterpret_cast<const bf16*>(p.cache) + (r < 0 ? 0 : r) * row;
+    for (int c = lane8; c < chunks; c += 8) cp_async16(dst + c * 8, src + c * 8, r >= 0);
+  };
+  long next = find(0);
+#pragma unroll
+  for (int i = 0; i < STAGES - 1; ++i) {
+    if (i < tiles) copy(i, next);
+    cp_async_commit();
+    next = find(i + 1);
+  }
+  float ql[HG][NL * 8], qr[HG][2], acc[HG][NL * 8];
+#pragma unroll
+  for (int g = 0; g < HG; ++g) {
+    const bool live = h0 + g < p.H;
+    const float* a = p.q_lat + ((long)t * p.H + h0 + g) * p.Lp;
+    const bf16* b = reinterpret_cast<const bf16*>(p.q_rot) + (long)t * p.ldq + (long)(h0 + g) * p.head_stride;
+#pragma unroll
+    for (int i = 0; i < NL; ++i) {
+      const int c = i * 256 + lane * 8;
+      float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (live && c < p.Lp) load8(a + c, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        ql[g][i * 8 + j] = f[j] * p.scale;
+        acc[g][i * 8 + j] = 0.f;
+      }
+    }
+    const int c = lane * 2;
+    qr[g][0] = live && c < p.Rp ? __bfloat162float(b[c]) * p.scale : 0.f;
+    qr[g][1] = live && c < p.Rp ? __bfloat162float(b[c + 1]) * p.scale : 0.f;
+  }
+  const int my_key = (lane / GRP) / HG;
+  float m = -INFINITY, l = 0.f;
+  for (int tile = 0; tile < tiles; ++tile) {
+    cp_async_wait<STAGES - 2>();
+    __syncthreads();                             // the tile has landed for every thread, and nobody still reads the stage refilled below
+    if (tile + STAGES - 1 < tiles) copy(tile + STAGES - 1, next);
+    cp_async_commit();
+    next = find(tile + STAGES);
+    const bf16* keys = ring + (long)(tile % STAGES) * TILE_KEYS * row;
+    const int live_keys = min(TILE_KEYS, k_end - k_begin - tile * TILE_KEYS);
+    for (int k0 = part * KB; k0 < live_keys; k0 += KB * sub) {
+      Raw8<bf16> rl[KB][NL];
+      float s[V];
+#pragma unroll
+      for (int j = 0; j < KB; ++j) {
+        const bf16* kr = keys + (long)(k0 + j) * row;
+        float2 x = make_float2(0.f, 0.f);
+        if (lane * 2 < p.Rp) x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(kr + p.Lp + lane * 2));
+        float kf[NL * 8];
+#pragma unroll
+        for (int i = 0; i < NL; ++i) {
+          if (i * 256 + lane * 8 < p.Lp) rl[j][i].load(kr + i * 256 + lane * 8);
+          else rl[j][i].zero();
+          rl[j][i].get(kf + i * 8);
+        }
+#pragma unroll
+        for (int g = 0; g < HG; ++g) {
+          float v0 = qr[g][0] * x.x, v1 = qr[g][1] * x.y;
+#pragma unroll
+          for (int i = 0; i < NL * 8; i += 2) {
+            v0 = fmaf(ql[g][i], kf[i], v0);
+            v1 = fmaf(ql[g][i + 1], kf[i + 1], v1);
+          }
+          s[j * HG + g] = v0 + v1;
+        }
+      }
+      float sc = transpose_sum<V>(s);
+      if (k0 + my_key >= live_keys) sc = -INFINITY;
+      float mx = fmaxf(sc, __shfl_xor_sync(0xffffffffu, sc, 16));
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
+      const bool moved = mx > m;
+      const float mn = moved ? mx : m;
+      const float w = sc == -INFINITY ? 0.f : __expf(sc - mn), corr = moved ? (m == -INFINITY ? 0.f : __expf(m - mn)) : 1.f;
+      m = mn;
+      l = l * corr + w;
+      if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+        for (int g = 0; g < HG; ++g) {
+          const float cg = __shfl_sync(0xffffffffu, corr, g * GRP);
+#pragma unroll
+          for (int i = 0; i < NL * 8; ++i) acc[g][i] *= cg;
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < KB; ++j) {
+        float kf[NL * 8];
+#pragma unroll
+        for (int i = 0; i < NL; ++i) rl[j][i].get(kf + i * 8);
+#pragma unroll
+        for (int g = 0; g < HG; ++g) {
+          const float wj = __shfl_sync(0xffffffffu, w, (j * HG + g) * GRP);
+#pragma unroll
+          for (int i = 0; i < NL * 8; ++i) acc[g][i] = fmaf(wj, kf[i], acc[g][i]);
+        }
+      }
+    }
+  }
+  cp_async_wait<0>();
+  l += __shfl_xor_sync(0xffffffffu, l, 16);
+  l += __shfl_xor_sync(0xffffffffu, l, 8);
+#pragma unroll
+  for (int g = 0; g < HG; ++g) {
+    const float mg = __shfl_sync(0xffffffffu, m, g * GRP), lg = __shfl_sync(0xffffffffu, l, g * GRP);
+    if (h0 + g >= p.H) continue;
+    float* out = p.scratch + ((((long)t * p.H + h0 + g) * p.splits + split) * sub + part) * (p.Lp + 2);
+#pragma unroll
+    for (int i = 0; i < NL; ++i) {
+      const int c = i * 256 + lane * 8;
+      if (c < p.Lp) {
+#pragma unroll
+        for (int j = 0; j < 8; j += 2) *reinterpret_cast<float2*>(out + c + j) = make_float2(acc[g][i * 8 + j], acc[g][i * 8 + j + 1]);      // rows of Lp + 2 floats
+      }
+    }
+    if (lane == 0) {
+      out[p.Lp] = mg;
+      out[p.Lp + 1] = lg;
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
 struct MergeParams {
   const float* scratch; const int32_t* positions;
-  int window, kps, splits, H, Lp;
+  int window, kps, splits, sub, H, Lp;       // sub: partials per split
   const void* gate; long ldg;                // [T, H]: head h of row t is multiplied by sigmoid(gate); or null
 };
 
@@ -422,9 +639,9 @@ template <bool FAST>
 __device__ __forceinline__ int merge_weights(const MergeParams& p, int t, int h, int pos, float gate, float* wgt, const float** base) {
   int first, count;
   visible(pos, p.window, &first, &count);
-  const int n = min(p.splits, (count + p.kps - 1) / p.kps);
-  *base = p.scratch + ((long)t * p.H + h) * p.splits * (p.Lp + 2);
-  if (threadIdx.x < 32) {                    // splits <= 64: two per lane
+  const int n = min(p.splits, (count + p.kps - 1) / p.kps) * p.sub;
+  *base = p.scratch + ((long)t * p.H + h) * p.splits * p.sub * (p.Lp + 2);
+  if (threadIdx.x < 32) {                    // at most 64 partials: two per lane
     const int s0 = threadIdx.x, s1 = threadIdx.x + 32;
     const float m0 = s0 < n ? (*base)[(long)s0 * (p.Lp + 2) + p.Lp] : -INFINITY, m1 = s1 < n ? (*base)[(long)s1 * (p.Lp + 2) + p.Lp] : -INFINITY;
     const float l0 = s0 < n ? (*base)[(long)s0 * (p.Lp + 2) + p.Lp + 1] : 0.f, l1 = s1 < n ? (*base)[(long)s1 * (p.Lp + 2) + p.Lp + 1] : 0.f;
@@ -544,6 +761,14 @@ int split_sizes(const SplitParams& p, cudaStream_t s) {
   return wide ? split_heads<A, 4, 4>(p, s) : split_heads<A, 4, 1>(p, s);
 }
 
+template <int NL>
+int launch_batch(const SplitParams& p, int sub, cudaStream_t s) {
+  const size_t smem = (size_t)STAGES * TILE_KEYS * (p.Lp + p.Rp) * sizeof(bf16);
+  auto k = latent_batch_kernel<NL>;
+  if (int rc = opt_in_smem(k, smem)) return rc;
+  return launch_chain(k, dim3(p.splits, (p.H + 31) / 32, p.T), dim3(256), smem, s, p, sub);
+}
+
 bool bad_geometry(int Lp, int Rp) { return Lp < 8 || Lp > 1024 || Lp % 8 || Rp < 0 || Rp > 256 || Rp % 8; }
 
 }  // namespace
@@ -559,6 +784,24 @@ extern "C" int ifab_latent_prepare(const void* proj, long ldp, int f32, int q_of
                   {positions, slots, page_table, max_pages, page_tokens, num_pages, status}, cq, ldc, cache, Lp, Rp};
   return f32 ? launch_chain(latent_prepare_kernel<float>, dim3(T), dim3(256), 0, (cudaStream_t)stream, p)
              : launch_chain(latent_prepare_kernel<bf16>, dim3(T), dim3(256), 0, (cudaStream_t)stream, p);
+}
+
+// decode rows (T <= 8), bf16: q [T, N] = rms(query latent) w_uq^T and the pages of the rows; w_uq [N, q_rank], q_rank % 8 == 0, bf16 gain
+extern "C" int ifab_latent_query(const void* proj, long ldp, int q_off, int q_rank, int kv_off, int kv_rank, int rot_dim, const void* q_gain, const float* kv_gain,
+                                 float eps, const void* rope, int rot, const int32_t* positions, const int32_t* slots, const int32_t* page_table, int max_pages,
+                                 int page_tokens, int num_pages, void* cache, int Lp, int Rp, const void* w_uq, int N, void* q, long ldq, int T, uint32_t* status,
+                                 void* stream) {
+  if (T < 1 || T > 8 || N < 1 || q_rank < 8 || q_rank % 8 || q_off % 8 || ldp % 8 || kv_rank < 1 || kv_rank > Lp || rot_dim < 0 || rot_dim > Rp || rot < 0 ||
+      rot % 2 || rot > rot_dim || (rot && !rope) || bad_geometry(Lp, Rp))
+    return -1;
+  PrepareParams p{proj, ldp, q_off, q_rank, kv_off, kv_rank, rot_dim, nullptr, kv_gain, eps, (const float2*)rope, rot,
+                  {positions, slots, page_table, max_pages, page_tokens, num_pages, status}, nullptr, 0, cache, Lp, Rp};
+  cudaStream_t s = (cudaStream_t)stream;
+  const bf16 *w = (const bf16*)w_uq, *g = (const bf16*)q_gain;
+  if (T <= 1) return query_rows<1>(p, w, g, N, (bf16*)q, ldq, T, s);
+  if (T <= 2) return query_rows<2>(p, w, g, N, (bf16*)q, ldq, T, s);
+  if (T <= 4) return query_rows<4>(p, w, g, N, (bf16*)q, ldq, T, s);
+  return query_rows<8>(p, w, g, N, (bf16*)q, ldq, T, s);
 }
 
 extern "C" int ifab_rotate_heads(void* q, long ldq, int f32, int head_stride, int off, int H, int rot, const void* rope, int T, void* stream) {
@@ -585,10 +828,23 @@ extern "C" int ifab_latent_split(const float* q_lat, const void* q_rot, long ldq
   return f32 ? split_sizes<float>(p, (cudaStream_t)stream) : split_sizes<bf16>(p, (cudaStream_t)stream);
 }
 
-extern "C" int ifab_latent_merge(const float* scratch, const int32_t* positions, int window, int kps, int splits, const void* gate, long ldg, int f32, int T,
+// the same with bf16 pages, Lp <= 512, Rp <= 64, for launches of many rows: `sub` (1, 2, 4 or 8, 32 heads / sub or fewer in all when above 1) warps per
+// four heads, splits * sub partials
+extern "C" int ifab_latent_batch(const float* q_lat, const void* q_rot, long ldq, int head_stride, const void* cache, int Lp, int Rp, const int32_t* positions,
+                                 const int32_t* slots, const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int window, float scale, int T,
+                                 int H, int kps, int splits, int sub, float* scratch, uint64_t scratch_bytes, uint32_t* status, void* stream) {
+  if (T < 1 || T > 65535 || H < 1 || window < 0 || kps < 1 || splits < 1 || bad_geometry(Lp, Rp) || Lp > 512 || Rp > 64) return -1;
+  if ((sub != 1 && sub != 2 && sub != 4 && sub != 8) || (sub > 1 && H * sub > 32) || splits * sub > 64) return -1;
+  if ((uint64_t)T * H * splits * sub * (Lp + 2) * sizeof(float) > scratch_bytes) return -5;
+  SplitParams p{q_lat, q_rot, ldq, head_stride, cache, Lp, Rp, {positions, slots, page_table, max_pages, page_tokens, num_pages, status}, window, scale, T, H,
+                kps, splits, scratch};
+  return Lp <= 256 ? launch_batch<1>(p, sub, (cudaStream_t)stream) : launch_batch<2>(p, sub, (cudaStream_t)stream);
+}
+
+extern "C" int ifab_latent_merge(const float* scratch, const int32_t* positions, int window, int kps, int splits, int sub, const void* gate, long ldg, int f32, int T,
                                  int H, int Lp, void* o_lat, long ldo, void* stream) {
-  if (T < 1 || T > 65535 || H < 1 || window < 0 || kps < 1 || splits < 1 || splits > 64 || bad_geometry(Lp, 0)) return -1;
-  MergeParams p{scratch, positions, window, kps, splits, H, Lp, gate, ldg};
+  if (T < 1 || T > 65535 || H < 1 || window < 0 || kps < 1 || splits < 1 || sub < 1 || splits * sub > 64 || bad_geometry(Lp, 0)) return -1;
+  MergeParams p{scratch, positions, window, kps, splits, sub, H, Lp, gate, ldg};
   return f32 ? launch_chain(latent_merge_kernel<float>, dim3(H, T), dim3(128), 0, (cudaStream_t)stream, p, (float*)o_lat, ldo)
              : launch_chain(latent_merge_kernel<bf16>, dim3(H, T), dim3(128), 0, (cudaStream_t)stream, p, (bf16*)o_lat, ldo);
 }
@@ -596,7 +852,7 @@ extern "C" int ifab_latent_merge(const float* scratch, const int32_t* positions,
 extern "C" int ifab_latent_merge_vup(const float* scratch, const int32_t* positions, int window, int kps, int splits, const void* gate, long ldg, int T, int H,
                                      int Lp, const void* w_uv, int vdim, void* out, long ldo, void* stream) {
   if (T < 1 || T > 65535 || H < 1 || window < 0 || kps < 1 || splits < 1 || splits > 64 || vdim < 1 || bad_geometry(Lp, 0)) return -1;
-  MergeParams p{scratch, positions, window, kps, splits, H, Lp, gate, ldg};
+  MergeParams p{scratch, positions, window, kps, splits, 1, H, Lp, gate, ldg};
   return launch_chain(latent_merge_vup_kernel, dim3(H, T, (vdim + 63) / 64), dim3(256), (size_t)Lp * sizeof(bf16), (cudaStream_t)stream, p, (const bf16*)w_uv, vdim,
                       (bf16*)out, ldo);
 }

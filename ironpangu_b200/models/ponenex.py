@@ -29,7 +29,7 @@ from . import checkpoint
 from .checkpoint import pad8
 from .stream_decoder import ATTN_ROWS, BF16, F32, StreamDecoder, StreamRows
 
-KERNEL_UNITS = ("misc", "post_norm", "linear_f32", "latent_attn", "tc_heads", "moe_rows", "moe_prefill", "tc_grouped", "decode_post_norm", "decode_linear", "window_attn",
+KERNEL_UNITS = ("misc", "post_norm", "linear_f32", "latent_attn", "tc_heads", "moe_rows", "moe_prefill", "tc_grouped", "decode_post_norm", "window_attn",
                 "fa_prefill", "decode_moe", "sampling", "tc_gemm", "tc_gemm_2sm")
 
 

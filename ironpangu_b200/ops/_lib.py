@@ -91,11 +91,15 @@ _SIGS = {
                               _P, c_int, c_int, c_int, _P],
     "ifab_latent_prepare": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, c_int, _P, _P, _P, c_int, c_int, c_int, _P, c_long,
                             _P, c_int, c_int, c_int, _P, _P],
+    "ifab_latent_query": [_P, c_long, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, c_int, _P, _P, _P, c_int, c_int, c_int, _P, c_int, c_int, _P,
+                          c_int, _P, c_long, c_int, _P, _P],
     "ifab_rotate_heads": [_P, c_long, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P],
     "ifab_latent_absorb": [_P, c_long, c_int, c_int, _P, _P, c_int, _P, c_int, c_int, c_int, c_int, _P],
     "ifab_latent_split": [_P, _P, c_long, c_int, _P, c_int, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, _P,
                           c_u64, _P, _P],
-    "ifab_latent_merge": [_P, _P, c_int, c_int, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P, c_long, _P],
+    "ifab_latent_batch": [_P, _P, c_long, c_int, _P, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int, _P, c_u64,
+                          _P, _P],
+    "ifab_latent_merge": [_P, _P, c_int, c_int, c_int, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P, c_long, _P],
     "ifab_latent_merge_vup": [_P, _P, c_int, c_int, c_int, _P, c_long, c_int, c_int, c_int, _P, c_int, _P, c_long, _P],
     "ifab_latent_gather": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P],
     "ifab_gemm_bf16_2sm": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, _P, _P],
@@ -190,8 +194,10 @@ def load(build: bool = True, units=None):
         if build:
             try:
                 path = _build.build_kernels(units=units)
-            except Exception:
-                if not path.exists():
+            except Exception as e:
+                # no compiler here: a library built elsewhere may do. Sources that do not compile are an error: an older library would
+                # be called with the wrong arguments
+                if not path.exists() or str(e).startswith("build failed"):
                     raise
         if not path.exists():
             raise RuntimeError(f"{path} is missing: run `python -m ironpangu_b200._build`")

@@ -17,7 +17,6 @@ import torch
 
 from . import _lib
 from ._lib import check
-from . import decode as K
 from . import stream_norm as N
 from .stream_norm import ACTIVATIONS, _f32, _p, _s
 from .window_attn import context_rows, tile_width
@@ -26,6 +25,8 @@ BF16, F32 = torch.bfloat16, torch.float32
 SPLIT_KEYS = 32            # fewest keys of a split (one batch of every warp)
 SPLIT_CTAS = 600           # CTAs the splits of a launch aim at: more rows, longer splits
 MAX_SPLITS = 64
+BATCH_ROWS = 8             # rows from which the warps of a CTA split the heads instead of the keys
+BATCH_CTAS = 148
 V_TILE = 128               # value columns per head of the tensor-core prompt kernel
 
 
@@ -76,6 +77,20 @@ class LatentShape:
         """Columns of the unrotated and of the rotated part of a query head as the kernels take it."""
         return (tile_width(self.dim), 64) if self.tiles and dtype == BF16 else (_pad(self.dim), self.rot_cols)
 
+    def batched(self, rows: int) -> bool:
+        """A launch of ``rows`` rows takes the kernel whose warps split the heads."""
+        return rows >= BATCH_ROWS and self.heads >= 4 and self.latent_cols <= 512 and self.rot_cols <= 64
+
+    def batch_splitting(self, rows: int, max_context: int) -> tuple:
+        """(splits, keys per split, partials per split) of that kernel: about one CTA per SM."""
+        keys = min(self.window, max_context) if self.window else max_context
+        sub = 8
+        while sub > 1 and self.heads * sub > 32:
+            sub //= 2
+        n = max(1, min(MAX_SPLITS // sub, (keys + 63) // 64, BATCH_CTAS // (rows * ((self.heads + 31) // 32))))
+        kps = ((keys + n - 1) // n + 31) // 32 * 32
+        return (keys + kps - 1) // kps, kps, sub
+
     @property
     def in_cols(self) -> int:
         """Columns of the packed input projection: query latent, key / value latent, rotated key part, head gates; the key part starts at a
@@ -106,8 +121,8 @@ class LatentBuffers:
         self.q_lat = z(self.group * max(s.heads * s.latent_cols for s in shapes), dt=F32)
         self.o_lat = z(self.group * max(s.heads * s.latent_cols for s in shapes))
         self.mixed = {s.heads * s.vdim: z(rows, _pad(s.heads * s.vdim)) for s in shapes}
-        self.scratch = torch.empty(max(most_splits(s, n, max_context) * n * s.heads * (s.latent_cols + 2) for s in shapes for n in range(1, self.group + 1)),
-                                   dtype=F32, device=device)
+        partials = lambda s, n: max(most_splits(s, n, max_context), s.batch_splitting(n, max_context)[0] * s.batch_splitting(n, max_context)[2])
+        self.scratch = torch.empty(max(partials(s, n) * n * s.heads * (s.latent_cols + 2) for s in shapes for n in range(1, self.group + 1)), dtype=F32, device=device)
         self.lat, self.k, self.vt, self.rot, self.cap = {}, None, None, None, 0
         tiled = [s for s in shapes if s.tiles]
         if chunked and dtype == BF16 and tiled:
@@ -167,13 +182,13 @@ class LatentMixer:
     def _q(self, B: LatentBuffers) -> torch.Tensor:
         return B.q[self.shape.heads, self.q_parts[0], self.q_parts[1]]
 
-    def prepare(self, B: LatentBuffers, m: int, rope, pos, slot, table, eps: float, status_ptr, norm_query: bool = True) -> None:
-        """Projection rows -> normed query latent in ``B.cq`` (unless the query up-projection norms it itself), pages of the rows written."""
+    def prepare(self, B: LatentBuffers, m: int, rope, pos, slot, table, eps: float, status_ptr) -> None:
+        """Projection rows -> normed query latent in ``B.cq``, pages of the rows written."""
         s = self.shape
-        cq = B.cq[s.q_rank] if norm_query else None
+        cq = B.cq[s.q_rank]
         check(_lib.load().ifab_latent_prepare(B.proj.data_ptr(), B.proj.stride(0), _f32(B.proj), 0, s.q_rank, s.kv_off, s.kv_rank, s.rot_dim, self.q_gain.data_ptr(),
-                                              self.kv_gain.data_ptr(), eps, _p(rope), s.rot_dims, *self._paging(pos, slot, table), _p(cq),
-                                              0 if cq is None else cq.stride(0), self.cache.data_ptr(), s.latent_cols, s.rot_cols, m, status_ptr, _s()),
+                                              self.kv_gain.data_ptr(), eps, _p(rope), s.rot_dims, *self._paging(pos, slot, table), cq.data_ptr(),
+                                              cq.stride(0), self.cache.data_ptr(), s.latent_cols, s.rot_cols, m, status_ptr, _s()),
               "latent_prepare")
 
     def rotate(self, q: torch.Tensor, rope) -> None:
@@ -196,11 +211,12 @@ class LatentMixer:
                                             B.scratch.data_ptr(), B.scratch.numel() * 4, status_ptr, _s()), "latent_split")
 
     def decode(self, B: LatentBuffers, m: int, rope, pos, slot, table, eps: float, status_ptr) -> None:
-        """A few bf16 rows from ``B.proj`` to ``B.mixed``: six launches."""
+        """A few bf16 rows (at most 8) from ``B.proj`` to ``B.mixed``: query projection (pages written beside it), absorb, split, merge + values."""
         s, (n1, n2) = self.shape, self.q_parts
         q, lib, H, Lp = self._q(B)[:m], _lib.load(), s.heads, s.latent_cols
-        self.prepare(B, m, rope, pos, slot, table, eps, status_ptr, norm_query=False)
-        K.gemv(B.proj[:m, :s.q_rank], self.w_uq, norm_w=self.q_gain_act, eps=eps, out=q)
+        check(lib.ifab_latent_query(B.proj.data_ptr(), B.proj.stride(0), 0, s.q_rank, s.kv_off, s.kv_rank, s.rot_dim, self.q_gain_act.data_ptr(),
+                                    self.kv_gain.data_ptr(), eps, _p(rope), s.rot_dims, *self._paging(pos, slot, table), self.cache.data_ptr(), Lp, s.rot_cols,
+                                    self.w_uq.data_ptr(), q.shape[1], q.data_ptr(), q.stride(0), m, status_ptr, _s()), "latent_query")
         check(lib.ifab_latent_absorb(q.data_ptr(), q.stride(0), n1 + n2, n1, self.w_uk.data_ptr(), _p(rope), s.rot_dims, B.q_lat.data_ptr(), m, H, s.dim, Lp, _s()),
               "latent_absorb")
         how = self.splitting(m)
@@ -216,11 +232,17 @@ class LatentMixer:
         out = B.mixed[H * s.vdim][lo:hi]
         q_lat, o_lat = B.q_lat[:n * H * Lp].view(n, H * Lp), B.o_lat[:n * H * Lp].view(n, H * Lp)
         heads_product(q, n1 + n2, self.w_uk_t, q_lat, Lp, H, s.dim, status_ptr)
-        how = self.splitting(n)
-        pos, slot = pos[lo:hi], slot[lo:hi]
-        self._split(B, q, q_lat, pos, slot, table, how, status_ptr)
+        pos, slot, sub = pos[lo:hi], slot[lo:hi], 1
+        if self.dtype == BF16 and s.batched(n):
+            splits, kps, sub = s.batch_splitting(n, self.max_context)
+            check(lib.ifab_latent_batch(q_lat.data_ptr(), q[:, n1:].data_ptr(), q.stride(0), n1 + n2, self.cache.data_ptr(), Lp, s.rot_cols,
+                                        *self._paging(pos, slot, table), s.window, s.scale, n, H, kps, splits, sub, B.scratch.data_ptr(), B.scratch.numel() * 4,
+                                        status_ptr, _s()), "latent_batch")
+        else:
+            splits, kps = self.splitting(n)
+            self._split(B, q, q_lat, pos, slot, table, (splits, kps), status_ptr)
         gate = B.proj[lo:hi, s.gate_off:]
-        check(lib.ifab_latent_merge(B.scratch.data_ptr(), pos.data_ptr(), s.window, how[1], how[0], gate.data_ptr(), gate.stride(0), _f32(o_lat), n, H, Lp,
+        check(lib.ifab_latent_merge(B.scratch.data_ptr(), pos.data_ptr(), s.window, kps, splits, sub, gate.data_ptr(), gate.stride(0), _f32(o_lat), n, H, Lp,
                                     o_lat.data_ptr(), o_lat.stride(0), _s()), "latent_merge")
         heads_product(o_lat, Lp, self.w_uv, out, s.vdim, H, Lp, status_ptr)
 
