@@ -13,7 +13,7 @@ import torch
 
 from ..ops import decode as K
 from ..ops import stream_norm as N
-from ..ops.linear_attn import DevicePlan, StepPlan
+from ..ops.linear_attn import StepPlan
 from ..parallel.fabric import Fabric
 from ..runtime.paged_state import PagedState
 from .checkpoint import pad8
@@ -169,6 +169,3 @@ class StreamRows:
             d.logits[:1].copy_(logits)
         K.sample_topk(logits, d.fabric, top_k=1, inv_temperature=d.inv_temp[:1], scratch=d.sample_scratch, out_ids=d.next_ids[:1])
         return d.next_ids[:1]
-
-
-__all__ = ["StreamDecoder", "StreamRows", "DevicePlan", "StepPlan", "ATTN_ROWS", "BF16", "F32"]

@@ -14,7 +14,7 @@ from typing import Dict, List
 
 import torch
 
-from .bench_falinex import L_bytes, Timer, _line, _visible, peaks
+from .bench_falinex import Timer, _line, _visible, peaks
 
 BF16, F32 = torch.bfloat16, torch.float32
 SIZES = {          # layers, width, heads, query rank, experts, top, expert ff, vocabulary, window (heads 128 + 64 / 128, latent 512, one shared expert)
@@ -53,7 +53,7 @@ class Costs:
         return hit * self.unit + self.unit + 2.0 * self.experts * self.width, rows * (self.top + 1) * self.unit
 
 
-def _result(params, fab) -> Dict:
+def _result(params) -> Dict:
     return {"params_m": round(params / 1e6), "prefill": {}, "decode": {}, "kernels": []}
 
 
@@ -85,7 +85,7 @@ def ponenex_arm(size, prompt: int, chunk: int, batches: List[int], t: Timer, pk)
         dec.state_manager.admit(r, ctx)
     dec.state_manager.flush()
     toks = torch.randint(0, C.vocab, (prompt,), dtype=torch.int32, device=dev)
-    res = _result(cfg.param_count(), fab)
+    res = _result(cfg.param_count())
 
     def prefill():
         for p0 in range(0, prompt, chunk):
@@ -174,7 +174,7 @@ def mla_arm(size, prompt: int, chunk: int, batches: List[int], t: Timer, pk) -> 
     pre = MlaMoePrefill(dec, max_rows=chunk)
     pre.use_graphs = False                          # chunks of the timed prompt are launched like the other arm's
     toks = torch.randint(0, C.vocab, (prompt,), dtype=torch.int32, device=dev)
-    res = _result(cfg.param_count(), fab)
+    res = _result(cfg.param_count())
 
     def prefill():
         for p0 in range(0, prompt, chunk):
