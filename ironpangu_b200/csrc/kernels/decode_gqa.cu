@@ -10,6 +10,7 @@
 // Query rows carry their own position and sequence slot (continuous batching: rows of different
 // sequences and prefill chunks share one launch). Reference counterparts: attention_qk_prepare /
 // paged_attention_prepare composites (native/src/inferfabric_acl.cpp:1236-1433).
+#include "attn_rule.cuh"
 #include "gemv.cuh"
 #include "rope.cuh"
 #include "ifab_kernels.h"
@@ -82,6 +83,8 @@ struct GqaParams {
   uint32_t* status;
   const float* sink;                              // [Hq]: exp(sink) joins the softmax denominator of the head; or null
   const bf16* gate; long ldg; int gate_act;       // the result is multiplied by act(gate [T, Hq * HD]); or null
+  int gate_head;                                  // the gate has one value per head instead: [T, Hq]
+  ScoreRule rule;
 };
 
 // HD = head_dim (EPL = HD/32 elements per lane), G = query heads per kv head
@@ -97,9 +100,7 @@ __global__ void __launch_bounds__(256) gqa_split_kernel(GqaParams p) {
   const int split = blockIdx.x, kvh = blockIdx.y, t = blockIdx.z;
   const int pos = p.positions[t];
   if (pos < 0) return;
-  int n = pos + 1;
-  if (p.window > 0 && n > p.window) n = p.window;
-  const int first = pos + 1 - n;
+  const int first = first_key(pos, p.window, p.rule.chunked), n = pos + 1 - first;
   const int k_begin = split * p.kps;
   if (k_begin >= n) return;
   // the last split also takes every key beyond max_splits * keys_per_split, so a long context is slower, never clipped
@@ -157,6 +158,7 @@ __global__ void __launch_bounds__(256) gqa_split_kernel(GqaParams p) {
 #pragma unroll
         for (int i = 0; i < EPL; ++i) s = fmaf(qf[g][i], kf[j][i], s);
         s = warp_sum(s) * p.scale;
+        if (!p.rule.plain()) s = ruled_score<true>(s, p.rule, p.rule.slopes ? p.rule.slopes[kvh * G + g] : 0.f, n - 1 - (kb + 8 * j));
         const float mn = fmaxf(m[g], s);
         const float corr = __expf(m[g] - mn), pe = __expf(s - mn);
         l[g] = l[g] * corr + pe;
@@ -213,15 +215,14 @@ __global__ void __launch_bounds__(256, 2) gqa_split_shared_kernel(GqaParams p) {
   const int split = blockIdx.x, kvh = blockIdx.y, t = blockIdx.z;
   const int pos = p.positions[t];
   if (pos < 0) return;
-  int n = pos + 1;
-  if (p.window > 0 && n > p.window) n = p.window;
-  const int first = pos + 1 - n;
+  const int first = first_key(pos, p.window, p.rule.chunked), n = pos + 1 - first;
   const int k_begin = split * p.kps;
   if (k_begin >= n) return;
   const int k_end = (split == p.max_splits - 1) ? n : min(n, k_begin + p.kps);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = lane / LP, sub = lane % LP;
   const int slot = p.slots[t];
-  float qf[G][C], acc[G][C], m[G], l[G];
+  float qf[G][C], acc[G][C], m[G], l[G], slope[G];
+  const bool ruled = !p.rule.plain();
 #pragma unroll
   for (int g = 0; g < G; ++g) {
     const bf16* qh = p.q + (long)t * p.ldq + (long)(kvh * G + g) * HD + sub * C;
@@ -232,6 +233,7 @@ __global__ void __launch_bounds__(256, 2) gqa_split_shared_kernel(GqaParams p) {
     }
     m[g] = -INFINITY;
     l[g] = 0.f;
+    slope[g] = p.rule.slopes ? p.rule.slopes[kvh * G + g] : 0.f;
   }
   const long kv_elems = (long)p.Hkv * HD, head = (long)kvh * HD + sub * C;
   // every lane takes the same number of rounds (the shuffles are warp-wide); a missing key scores -inf
@@ -266,6 +268,7 @@ __global__ void __launch_bounds__(256, 2) gqa_split_shared_kernel(GqaParams p) {
         for (int j = 0; j < 8; ++j) s[b][g] = fmaf(qf[g][j], f[j], s[b][g]);
 #pragma unroll
         for (int o = LP / 2; o > 0; o >>= 1) s[b][g] += __shfl_xor_sync(0xffffffffu, s[b][g], o);
+        if (ruled) s[b][g] = ruled_score<true>(s[b][g], p.rule, slope[g], n - 1 - (k0 + b * 8 * NG + grp));
         if (!ok[b]) s[b][g] = -INFINITY;
       }
     }
@@ -349,8 +352,7 @@ __global__ void gqa_merge_kernel(GqaParams p, bf16* out, long ldo) {
   const int h = blockIdx.x, t = blockIdx.y;
   const int pos = p.positions[t];
   if (pos < 0) return;
-  int n = pos + 1;
-  if (p.window > 0 && n > p.window) n = p.window;
+  const int n = pos + 1 - first_key(pos, p.window, p.rule.chunked);
   int ns = (n + p.kps - 1) / p.kps;
   if (ns > p.max_splits) ns = p.max_splits;
   const float* base = p.scratch + ((long)t * p.Hq + h) * p.max_splits * (HD + 2);
@@ -372,7 +374,7 @@ __global__ void gqa_merge_kernel(GqaParams p, bf16* out, long ldo) {
     float v = 0.f;
     for (int s = 0; s < ns; ++s) v += wgt[s] * base[(long)s * (HD + 2) + c];
     v *= invL;
-    if (p.gate) v *= activate<true>(__bfloat162float(p.gate[(long)t * p.ldg + (long)h * HD + c]), p.gate_act);
+    if (p.gate) v *= activate<true>(__bfloat162float(p.gate[(long)t * p.ldg + (p.gate_head ? h : (long)h * HD + c)]), p.gate_act);
     out[(long)t * ldo + (long)h * HD + c] = __float2bfloat16_rn(v);
   }
 }
@@ -416,21 +418,22 @@ extern "C" int ifab_gqa_decode_attention(const void* q, long ldq, const void* k_
                                          int max_pages, int page_tokens, int num_pages, float scale, int T, int Hq, int Hkv,
                                          int head_dim, int keys_per_split, int max_splits, float* scratch,
                                          uint64_t scratch_bytes, void* out, long ldo, uint32_t* status, void* stream) {
-  return ifab_gqa_window_attention(q, ldq, k_cache, v_cache, positions, slots, page_table, max_pages, page_tokens, num_pages, scale, 0, nullptr, nullptr,
-                                   0, 0, T, Hq, Hkv, head_dim, keys_per_split, max_splits, scratch, scratch_bytes, out, ldo, status, stream);
+  return ifab_gqa_window_attention(q, ldq, k_cache, v_cache, positions, slots, page_table, max_pages, page_tokens, num_pages, scale, 0, 0.f, nullptr, 0, nullptr, nullptr,
+                                   0, 0, 0, T, Hq, Hkv, head_dim, keys_per_split, max_splits, scratch, scratch_bytes, out, ldo, status, stream);
 }
 
-// The same over the last `window` positions only (0: all), with a sink logit per query head in the denominator and an output gate.
+// The same over the last `window` positions (0: all) or, `chunked`, the query's own stretch of as many; with a cap of the scores (0: none), slopes [Hq]
+// of the distance bias, a sink logit per query head in the denominator and an output gate, [T, Hq * HD] or [T, Hq].
 extern "C" int ifab_gqa_window_attention(const void* q, long ldq, const void* k_cache, const void* v_cache, const int32_t* positions, const int32_t* slots,
-                                         const int32_t* page_table, int max_pages, int page_tokens, int num_pages, float scale, int window,
-                                         const float* sink, const void* gate, long ldg, int gate_act, int T, int Hq, int Hkv, int head_dim,
+                                         const int32_t* page_table, int max_pages, int page_tokens, int num_pages, float scale, int window, float cap,
+                                         const float* slopes, int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, int T, int Hq, int Hkv, int head_dim,
                                          int keys_per_split, int max_splits, float* scratch, uint64_t scratch_bytes, void* out, long ldo,
                                          uint32_t* status, void* stream) {
-  if (Hkv < 1 || Hq % Hkv || max_splits < 1 || max_splits > 64 || keys_per_split < 8 || window < 0) return -1;
+  if (Hkv < 1 || Hq % Hkv || max_splits < 1 || max_splits > 64 || keys_per_split < 8 || window < 0 || cap < 0.f) return -1;
   if ((uint64_t)T * Hq * max_splits * (head_dim + 2) * sizeof(float) > scratch_bytes) return -5;
   GqaParams p{(const bf16*)q, ldq, (const bf16*)k_cache, (const bf16*)v_cache, positions, slots, page_table,
               max_pages, page_tokens, num_pages, scale, window, T, Hq, Hkv, keys_per_split, max_splits, scratch, status, sink, (const bf16*)gate, ldg,
-              gate_act};
+              gate_act, gate_per_head, {cap, slopes, chunked}};
   cudaStream_t s = (cudaStream_t)stream;
   switch (head_dim) {
     case 64: return dispatch_g<64>(p, (bf16*)out, ldo, s);

@@ -5,7 +5,7 @@
 //   router_topk_kernel        f32 router projection, one CTA per expert (+RMSNorm prologue); the
 //                             last CTA to finish turns the logits into top-k ids and weights
 //                             (softmax top-k or sigmoid+bias)
-//   moe_gate_up_kernel        one CTA column per route: gate/up rows of the routed expert, SwiGLU
+//   moe_gate_up_kernel        one CTA column per route: gate/up rows of the routed expert, gated unit
 //   moe_down_allreduce_kernel score-weighted sum of the local experts' down projections (+ the
 //                             tensor-parallel shard of the shared expert) + one-shot all-reduce
 //   lm_head_argmax_kernel     vocabulary-sharded logits + greedy selection; the last CTA exchanges
@@ -13,9 +13,11 @@
 //
 // Reference counterparts: router_projection/router_select, route_quantize, expert_gmm,
 // expert_reduce and allreduce (native/src/token_executor.h:957-1205) and emit (:1206-1274).
+#include "attn_rule.cuh"
 #include "gemv.cuh"
 #include "oneshot_ar.cuh"
 #include "moe_select.cuh"
+#include "rope.cuh"
 #include "ifab_kernels.h"
 
 using namespace ifab;
@@ -111,6 +113,7 @@ struct GateUpParams {
   const int32_t* ids; int T, D, F, topk, e0, e_local;
   const bf16* w_gu; const bf16* w_sgu; int Fs;
   bf16* act; int ldact;    // columns from one slot to the next (>= F and Fs)
+  GatedUnit unit;
 };
 
 // grid: (ceil(max(F, Fs)/16), T*topk + T). Column y < T*topk is route (t, k); columns after that are the shared
@@ -166,8 +169,8 @@ __global__ void __launch_bounds__(256) moe_gate_up_kernel(GateUpParams p) {
   warp_reduce_acc<1, 4>(acc);
   if (lane == 0) {
     bf16* out = p.act + ((size_t)t * (p.topk + 1) + slot) * p.ldact;
-    out[j0] = __float2bfloat16_rn(silu(bf16_round(acc[0][0])) * bf16_round(acc[2][0]));
-    if (j0 + 1 < Fcur) out[j0 + 1] = __float2bfloat16_rn(silu(bf16_round(acc[1][0])) * bf16_round(acc[3][0]));
+    out[j0] = __float2bfloat16_rn(gated_bf16(acc[0][0], acc[2][0], p.unit));
+    if (j0 + 1 < Fcur) out[j0 + 1] = __float2bfloat16_rn(gated_bf16(acc[1][0], acc[3][0], p.unit));
   }
 }
 
@@ -397,6 +400,7 @@ struct HeadParams {
   float2* partial;     // [grid][T] (value, index-as-int-bits)
   int32_t* out_ids; float* out_vals;
   FabricView fv; uint64_t* seq; uint32_t* done;
+  float cap;           // > 0: logits are cap tanh(logit / cap)
 };
 
 template <int T, int R>
@@ -433,6 +437,7 @@ __global__ void __launch_bounds__(256) lm_head_argmax_kernel(HeadParams p) {
 #pragma unroll
         for (int r = 0; r < R; ++r) {
           if (n0 + r >= p.V) continue;
+          if (p.cap > 0.f) acc[r][t] = soft_limit<true>(acc[r][t], p.cap);
           if (p.logits && t < p.T) p.logits[(size_t)t * p.V + n0 + r] = acc[r][t];
           if (acc[r][t] > bv) { bv = acc[r][t]; bi = p.vocab_offset + n0 + r; }
         }
@@ -554,9 +559,17 @@ extern "C" int ifab_router_topk(const void* x, long ldx, const void* norm_w, flo
 extern "C" int ifab_moe_gate_up_decode(const void* x, long ldx, const void* norm_w, float eps, const int32_t* ids, int T,
                                        int D, int F, int topk, int e0, int e_local, const void* w_gu,
                                        const void* w_shared_gu, int Fs, void* act, int ldact, void* stream) {
+  return ifab_moe_gate_up_unit_decode(x, ldx, norm_w, eps, ids, T, D, F, topk, e0, e_local, w_gu, w_shared_gu, Fs, act, ldact, 0, 0.f, 0.f, stream);
+}
+// The same with the gated unit by number (rope.cuh).
+extern "C" int ifab_moe_gate_up_unit_decode(const void* x, long ldx, const void* norm_w, float eps, const int32_t* ids, int T, int D, int F, int topk, int e0,
+                                            int e_local, const void* w_gu, const void* w_shared_gu, int Fs, void* act, int ldact, int unit, float limit,
+                                            float alpha, void* stream) {
+  const GatedUnit gu{unit, limit, alpha};
+  if (!gated_ok(gu)) return -1;
   if (D % 8 != 0 || F % 8 != 0 || Fs % 8 != 0 || ldact % 8 != 0 || ldact < F || ldact < Fs) return -1;
   GateUpParams p{(const bf16*)x, ldx, (const bf16*)norm_w, eps, ids, T, D, F, topk, e0, e_local,
-                 (const bf16*)w_gu, (const bf16*)w_shared_gu, Fs, (bf16*)act, ldact};
+                 (const bf16*)w_gu, (const bf16*)w_shared_gu, Fs, (bf16*)act, ldact, gu};
   dim3 grid((max(F, w_shared_gu ? Fs : 0) + 15) / 16, T * topk + T);
   const size_t smem = (size_t)D * sizeof(bf16);
   if (int rc = opt_in_smem(moe_gate_up_kernel, smem)) return rc;
@@ -606,8 +619,15 @@ extern "C" int ifab_moe_down_allreduce_decode(const void* act, const int32_t* id
 extern "C" int ifab_lm_head_argmax(const void* x, long ldx, const void* norm_w, float eps, const void* w, float* logits,
                                    int T, int V_local, int K, int vocab_offset, void* partial, uint64_t partial_bytes,
                                    int32_t* out_ids, float* out_vals, const IfabFabric* fab, void* stream) {
-  if (T < 1 || T > 8 || K % 8 != 0) return -1;
+  return ifab_lm_head_capped_argmax(x, ldx, norm_w, eps, w, logits, 0.f, T, V_local, K, vocab_offset, partial, partial_bytes, out_ids, out_vals, fab, stream);
+}
+// The same for logits cap tanh(logit / cap) (cap 0: none).
+extern "C" int ifab_lm_head_capped_argmax(const void* x, long ldx, const void* norm_w, float eps, const void* w, float* logits, float cap, int T, int V_local, int K,
+                                          int vocab_offset, void* partial, uint64_t partial_bytes, int32_t* out_ids, float* out_vals, const IfabFabric* fab,
+                                          void* stream) {
+  if (T < 1 || T > 8 || K % 8 != 0 || cap < 0.f) return -1;
   HeadParams p;
+  p.cap = cap;
   p.x = (const bf16*)x; p.ldx = ldx; p.norm_w = (const bf16*)norm_w; p.eps = eps;
   p.w = (const bf16*)w; p.logits = logits; p.T = T; p.V = V_local; p.K = K; p.vocab_offset = vocab_offset;
   p.partial = (float2*)partial; p.out_ids = out_ids; p.out_vals = out_vals;

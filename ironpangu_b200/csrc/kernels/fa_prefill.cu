@@ -21,6 +21,7 @@
 // Every wait is bounded; a wait that runs out raises the CTA's abort flag and the status word, the CTA drains its copies,
 // frees its tensor memory and returns. Reference: the fused attention operator of the prompt envelope, up to 4,096 query
 // rows (native/src/token_executor.h:863-909).
+#include "attn_rule.cuh"
 #include "rope.cuh"
 #include "tc_common.cuh"
 #include "ifab_kernels.h"
@@ -48,6 +49,9 @@ struct FaParams {
   const bf16* gate; long ldg; int gate_act;  // the result is multiplied by act(gate [m, H * e]); or null
   int gate_head;                             // the gate has one value per head instead: [m, H]
   uint32_t* status; uint32_t spin_limit;
+  int chunked;                               // `window` is the size of the stretches that queries stay in (attn_rule.cuh)
+  float cap_log2, cap_exp;                   // RULED: cap * log2(e) (0: no cap) and 2 * scale * log2(e) / cap
+  const float* slopes;                       // RULED: distance bias [H], or null
 };
 
 struct Bars {
@@ -71,7 +75,7 @@ struct Layout {
   static constexpr int SMEM = XCH_OFF + 2 * PARTS * 128 * 8 + 1024;
 };
 
-template <int P1, int P2, bool SPLIT>
+template <int P1, int P2, bool SPLIT, bool RULED>
 __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                                                             const __grid_constant__ CUtensorMap tmap_k2, const __grid_constant__ CUtensorMap tmap_vt,
                                                             FaParams p) {
@@ -91,7 +95,7 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
   // key tiles this query tile can see: up to the position of its last live row, from the window's start
   const int last_row = min(q0 + BQ, p.m) - 1;
   const int t_end = min((p.ctx + BKEY - 1) / BKEY, (p.pos0 + last_row) / BKEY + 1);
-  const int t_begin = p.window > 0 ? max(0, p.pos0 + q0 - p.window + 1) / BKEY : 0;
+  const int t_begin = first_key(p.pos0 + q0, p.window, p.chunked) / BKEY;
   const int n_tiles = t_end - t_begin;
 
   if (threadIdx.x == 0) {
@@ -197,7 +201,8 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
     const int quarter = warp & 3, half = (warp - 4) >> 2, r = quarter * 32 + lane;     // `half`: which of the PARTS column ranges
     const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
     const int q_pos = p.pos0 + q0 + r;
-    const int lo = p.window > 0 ? q_pos - p.window + 1 : 0;     // first visible key
+    const int lo = first_key(q_pos, p.window, p.chunked);       // first visible key
+    const float slope = RULED && p.slopes ? p.slopes[h] * 1.4426950408889634f : 0.f;
     constexpr int HK = BKEY / PARTS, HV = DV / PARTS;
     float m_ref = -INFINITY, l_run = 0.f;     // reference maximum (base-2 domain, may lag the true maximum by up to 8); sum over this thread's columns
     bool ok = true;
@@ -247,7 +252,13 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
 #pragma unroll
       for (int i = 0; i < HK; ++i) {
         const int key = key0 + i;
-        sv[i] = (key <= q_pos && key >= lo) ? sv[i] * p.scale_log2 : -INFINITY;
+        float z = sv[i] * p.scale_log2;
+        if (RULED) {
+          // cap tanh(s / cap) = cap - 2 cap / (1 + exp(2 s / cap))
+          if (p.cap_log2 > 0.f) z = p.cap_log2 - __fdividef(2.f * p.cap_log2, 1.f + exp2f(sv[i] * p.cap_exp));
+          z -= slope * (float)(q_pos - key);
+        }
+        sv[i] = (key <= q_pos && key >= lo) ? z : -INFINITY;
         mx[i & 3] = fmaxf(mx[i & 3], sv[i]);
       }
       const float my_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
@@ -365,9 +376,9 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
   }
 }
 
-template <int P1, int P2, bool SPLIT = false>
+template <int P1, int P2, bool SPLIT = false, bool RULED = false>
 int launch_fa(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tk2, const CUtensorMap& tv, const FaParams& p, int H, cudaStream_t s) {
-  auto k = fa_prefill_kernel<P1, P2, SPLIT>;
+  auto k = fa_prefill_kernel<P1, P2, SPLIT, RULED>;
   if (int rc = opt_in_smem(k, Layout<P1, P2, SPLIT>::SMEM)) return rc;
   dim3 grid((p.m + BQ - 1) / BQ, H);
   return launch_chain(k, grid, dim3(THREADS), (size_t)Layout<P1, P2, SPLIT>::SMEM, s, tq, tk, tk2, tv, p);
@@ -398,7 +409,7 @@ extern "C" int ifab_fa_prefill_bf16(const void* q, long ldq, int q_head_stride, 
   }
   if (int rc = make_tmap_bf16_2d(&tv, vt, (uint64_t)vt_rows, (uint64_t)ctx, (uint64_t)ldvt, DV)) return rc;
   FaParams p{(bf16*)out, ldo, m, ctx, kv_group, pos0, window, q_head_stride, k_head_stride, vt_head_stride, vt_row0,
-             scale * 1.4426950408889634f, DV, nullptr, nullptr, 0, 0, 0, status, 4000000u};
+             scale * 1.4426950408889634f, DV, nullptr, nullptr, 0, 0, 0, status, 4000000u, 0, 0.f, 0.f, nullptr};
   cudaStream_t s = (cudaStream_t)stream;
   if (d1 == 128 && d2 == 64) return launch_fa<2, 1>(tq, tk, tk2, tv, p, H, s);
   if (d1 == 128 && d2 == 0) return launch_fa<2, 0>(tq, tk, tk2, tv, p, H, s);
@@ -409,10 +420,11 @@ extern "C" int ifab_fa_prefill_bf16(const void* q, long ldq, int q_head_stride, 
 // Windowed form with softmax weights of 16 bits instead of 8 in the value product, a sink logit per head, an output gate, and value heads
 // of any width: q [m, H * (d + d2)] and k [ctx, G * d] with d in {64, 128} columns per head (narrower heads are zero-padded by the caller),
 // k2 [ctx, d2] key columns shared by all heads (d2 0 or 64), vt [G * 128, ldvt >= ctx] (rows past a narrower value head are zero), out
-// [m, H * e], e <= 128; gate [m, H * e], or [m, H] with gate_per_head.
+// [m, H * e], e <= 128; gate [m, H * e], or [m, H] with gate_per_head. `chunked`: `window` is the size of the stretches queries stay in (position 0 of
+// the operands starts one); cap (0: none) and slopes [H] (or null) act on the scores (attn_rule.cuh), without k2.
 extern "C" int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const void* k2, long ldk2, int d2, const void* vt, long ldvt, void* out, long ldo,
-                                   int m, int ctx, int H, int kv_group, int d, int e, int pos0, int window, float scale, const float* sink, const void* gate,
-                                   long ldg, int gate_act, int gate_per_head, uint32_t* status, void* stream) {
+                                   int m, int ctx, int H, int kv_group, int d, int e, int pos0, int window, float scale, float cap, const float* slopes,
+                                   int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, uint32_t* status, void* stream) {
   if (m < 1 || ctx < 1 || H < 1 || kv_group < 1 || H % kv_group || pos0 < 0 || pos0 + m > ctx || window < 0) return -1;
   if ((d != 64 && d != 128) || (d2 != 0 && d2 != 64) || (d2 && (!k2 || ldk2 % 8)) || e < 1 || e > DV || ldq % 8 || ldk % 8 || ldvt % 8 || ldvt < ctx) return -1;
   const int G = H / kv_group;
@@ -424,8 +436,10 @@ extern "C" int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long 
     if (int rc = make_tmap_bf16_2d(&tk2, k2, (uint64_t)ctx, (uint64_t)d2, (uint64_t)ldk2, BKEY)) return rc;
   if (int rc = make_tmap_bf16_2d(&tv, vt, (uint64_t)G * DV, (uint64_t)ctx, (uint64_t)ldvt, DV)) return rc;
   FaParams p{(bf16*)out, ldo, m, ctx, kv_group, pos0, window, d + d2, d, DV, 0, scale * 1.4426950408889634f, e, sink, (const bf16*)gate, ldg, gate_act,
-             gate_per_head, status, 4000000u};
+             gate_per_head, status, 4000000u, chunked, cap * 1.4426950408889634f, cap > 0.f ? 2.f * scale * 1.4426950408889634f / cap : 0.f, slopes};
   cudaStream_t s = (cudaStream_t)stream;
+  if (cap > 0.f || slopes)
+    return d2 ? -1 : d == 128 ? launch_fa<2, 0, true, true>(tq, tk, tk2, tv, p, H, s) : launch_fa<1, 0, true, true>(tq, tk, tk2, tv, p, H, s);
   if (d2) return d == 128 ? launch_fa<2, 1, true>(tq, tk, tk2, tv, p, H, s) : launch_fa<1, 1, true>(tq, tk, tk2, tv, p, H, s);
   return d == 128 ? launch_fa<2, 0, true>(tq, tk, tk2, tv, p, H, s) : launch_fa<1, 0, true>(tq, tk, tk2, tv, p, H, s);
 }

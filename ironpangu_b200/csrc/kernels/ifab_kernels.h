@@ -78,14 +78,25 @@ int ifab_gemm_act_bf16(const void* a, long lda, const void* b, long ldb, void* c
                        int M, int N, int K, uint32_t* status, void* stream);
 int ifab_gemm_act_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr, int act,
                            int persistent, int M, int N, int K, uint32_t* status, void* stream);
-/* C = act(A * B^T) in true f32 */
-int ifab_linear_f32(const float* a, long lda, const float* b, long ldb, float* c, long ldc, int M, int N, int K, int act, void* stream);
+/* the same with a bias [N] (f32, or null) and, for cap > 0, a soft limit cap tanh(result / cap) after the activation */
+int ifab_gemm_epilogue_bf16(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr, const float* bias,
+                            int act, float cap, int M, int N, int K, uint32_t* status, void* stream);
+int ifab_gemm_epilogue_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr,
+                                const float* bias, int act, float cap, int persistent, int M, int N, int K, uint32_t* status, void* stream);
+/* first half of a gated feed-forward, any number of rows: b = [gate rows | up rows] ([2F, K]), c[M, F] = unit(a gate^T, a up^T). Units: 0 silu(g) u,
+ * 1 relu(g) u, 2 g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = u within [-limit, limit] */
+int ifab_gemm_gated_bf16(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int unit, float limit, float alpha, int M, int F, int K,
+                         uint32_t* status, void* stream);
+int ifab_gemm_gated_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int unit, float limit, float alpha, int M, int F, int K,
+                             uint32_t* status, void* stream);
+/* C = act(A * B^T + bias) in true f32, softly limited for cap > 0 */
+int ifab_linear_f32(const float* a, long lda, const float* b, long ldb, float* c, long ldc, const float* bias, float cap, int M, int N, int K, int act, void* stream);
 /* n products at strides sa, sb, sc; and products grouped by the tile table of ifab_moe_dispatch (rows of A through `index` when given; pair: A is
- * [gate | up], taken as silu(gate) * up) */
+ * [gate | up], taken as the gated unit of that number) */
 int ifab_linear_f32_batched(const float* a, long lda, long sa, const float* b, long ldb, long sb, float* c, long ldc, long sc, int n, int M, int N, int K,
                             void* stream);
-int ifab_grouped_linear_f32(const float* a, long lda, const int32_t* index, int pair, const float* b, int N, int K, const int32_t* tiles,
-                            const int32_t* num_tiles, int max_tiles, int rows, float* c, long ldc, void* stream);
+int ifab_grouped_linear_f32(const float* a, long lda, const int32_t* index, int pair, int unit, float limit, float alpha, const float* b, int N,
+                            int K, const int32_t* tiles, const int32_t* num_tiles, int max_tiles, int rows, float* c, long ldc, void* stream);
 /* one product per head, heads side by side in the rows of A and C: C[t, h * c_stride + n] = sum_k A[t, h * a_stride + k] B[h, n, k] (tcgen05) */
 int ifab_gemm_heads_bf16(const void* a, long lda, int a_stride, const void* b, long ldb, void* c, long ldc, int c_stride, int out_f32, int heads, int M, int N,
                          int K, uint32_t* status, void* stream);
@@ -119,6 +130,8 @@ int ifab_allgather_gemm_bf16(void* const* a_peers, long lda, const void* b, long
 int ifab_grouped_gemm_bf16(const void* a, long lda, int rows_max, const void* b, int experts, int N, int K,
                            const int32_t* tiles, const int32_t* num_tiles, int max_tiles, void* c, long ldc, int mode,
                            uint32_t* status, void* stream);
+int ifab_grouped_gemm_gated_bf16(const void* a, long lda, int rows_max, const void* b, int experts, int N, int K, const int32_t* tiles, const int32_t* num_tiles,
+                                 int max_tiles, void* c, long ldc, int mode, int unit, float limit, float alpha, uint32_t* status, void* stream);
 /* router for any number of rows (blocks of 8 per CTA); xn (optional) receives the RMS-normalised rows */
 int ifab_router_block(const void* x, long ldx, const void* norm_w, float eps, const float* w_router, const float* bias,
                       float* logits, int32_t* ids, float* wts, void* xn, long ldxn, int M, int D, int E, int topk,
@@ -177,17 +190,21 @@ int ifab_router_topk(const void* x, long ldx, const void* norm_w, float eps, con
 int ifab_moe_gate_up_decode(const void* x, long ldx, const void* norm_w, float eps, const int32_t* ids, int T, int D,
                             int F, int topk, int e0, int e_local, const void* w_gu, const void* w_shared_gu, int Fs,
                             void* act, int ldact, void* stream);
+int ifab_moe_gate_up_unit_decode(const void* x, long ldx, const void* norm_w, float eps, const int32_t* ids, int T, int D, int F, int topk, int e0, int e_local,
+                                 const void* w_gu, const void* w_shared_gu, int Fs, void* act, int ldact, int unit, float limit, float alpha, void* stream);
 /* one rank: y f32 [T, ldy] = the same sum before rounding, the shared expert's row weighted by shared_w [T] (null: 1). In both, `act` slots are
  * ldact columns apart (slot topk is the shared expert's, which may be wider or narrower than F) */
 int ifab_moe_down_f32_decode(const void* act, int ldact, const int32_t* ids, const float* wts, const float* shared_w, int T, int D, int F, int topk,
                              int experts, const void* w_down, const void* w_shared_down, int Fs, float* y, long ldy, void* stream);
 /* routed experts of decoders with an f32 residual (moe_rows.cu): logits f32 [M, ld] (column E: the shared expert's gate, used when shared_w is given) ->
- * ids, wts [M, topk]; scoring 0 softmax, 1 sigmoid, 2 logit + bias selected, softmax over the chosen. combine_norm: y = weighted sum of the permuted
- * rows (+ shared_w * shared), x += rms(y) * w, xa = rms(x) * w2 (x without w2) */
-int ifab_moe_route(const float* logits, long ld, const float* bias, int M, int E, int topk, int scoring, int renorm, float scale, int32_t* ids, float* wts,
-                   float* shared_w, void* stream);
+ * ids, wts [M, topk]; scoring 0 softmax, 1 sigmoid, 2 logit + bias selected, softmax over the chosen, 3 sigmoid + bias selected, sigmoid (over the sum with
+ * renorm); of `groups` groups of neighbours only the `keep` best are open (moe_select.cuh). combine_norm: y = weighted sum of the permuted rows
+ * (+ shared_w * shared), x += rms(y) * w (without w: y + base) (+ extra), xa = rms(x) * w2 (x without w2) */
+int ifab_moe_route(const float* logits, long ld, const float* bias, int M, int E, int topk, int scoring, int renorm, float scale, int groups, int keep, int32_t* ids,
+                   float* wts, float* shared_w, void* stream);
 int ifab_moe_combine_norm(const void* y, long ldy, const int32_t* route_row, const float* wts, int topk, const void* shared, long lds, const float* shared_w,
-                          const float* w, const float* w2, float eps, float* x, long ldx, void* xa, long lda, int f32, int M, int D, void* stream);
+                          const float* w, const float* w2, float eps, const float* base, long ldb, const float* extra, long lde, float* x, long ldx, void* xa,
+                          long lda, int f32, int M, int D, void* stream);
 int ifab_moe_down_allreduce_decode(const void* act, const int32_t* ids, const float* wts, int T, int D, int F, int topk,
                                    int e0, int e_local, const void* w_down, const void* w_shared_down, int Fs,
                                    const void* residual, long ldr, void* y, long ldy, const IfabFabric* fab,
@@ -210,6 +227,9 @@ int ifab_lm_head_argmax(const void* x, long ldx, const void* norm_w, float eps, 
                         int T, int V_local, int K, int vocab_offset, void* partial /* >= grid*T*8 bytes */,
                         uint64_t partial_bytes, int32_t* out_ids, float* out_vals, const IfabFabric* fab,
                         void* stream);
+/* the same for logits cap tanh(logit / cap) (0: none) */
+int ifab_lm_head_capped_argmax(const void* x, long ldx, const void* norm_w, float eps, const void* w, float* logits, float cap, int T, int V_local, int K,
+                               int vocab_offset, void* partial, uint64_t partial_bytes, int32_t* out_ids, float* out_vals, const IfabFabric* fab, void* stream);
 
 /* ---- sampling on vocabulary-sharded logits: temperature, penalties, top-k <= 64, min-p, top-p, counter-based draw ---- */
 int ifab_sample_topk(const float* logits, long ld, int T, int V_local, int vocab_offset, int top_k,
@@ -280,12 +300,14 @@ int ifab_mhc_post_norm(const void* X, const void* branch, long ldb, const void* 
 int ifab_delta_rule_decode(const void* q, const void* k, const void* v, const float* g, const float* beta, float* state,
                            const int32_t* slots, void* out, int rows, int H, int dk, int dv, void* stream);
 /* f32 residual stream with the norm on a sublayer's output; `f32`: activations (xa, gate, y) are f32 instead of bf16; gains f32 */
-/* x = table[id] * scale; xa = x, or rms(x) * w when w is given */
-int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float scale, const float* w, float eps, float* x, long ldx, void* xa, long lda, int f32,
-                    int T, int D, int vocab, uint32_t* status, void* stream);
-/* x += rms(y) * w; xa = x, or rms(x) * w2 when w2 is given */
-int ifab_post_norm_add(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, void* xa, long lda, int f32, int T, int D,
-                       void* stream);
+/* x = table[id] * scale (and once more to copy, when given); xa = x, or rms(x) * w when w is given */
+int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float scale, const float* w, float eps, float* x, long ldx, float* copy, void* xa, long lda,
+                    int f32, int T, int D, int vocab, uint32_t* status, void* stream);
+/* x += rms(y) * w (y without w, nothing without y) (+ extra); xa = x, or rms(x) * w2 when w2 is given */
+int ifab_post_norm_add(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, const float* extra, long lde, void* xa, long lda,
+                       int f32, int T, int D, void* stream);
+/* y [T, F] = gated unit of gu[:, c] and gu[:, up + c] */
+int ifab_gated_rows(const void* gu, long ld, int up, int unit, float limit, float alpha, void* y, long ldy, int f32, int T, int F, void* stream);
 int ifab_rms_rows(const float* x, long ldx, const int32_t* rows, const float* w, float eps, void* y, long ldy, int f32, int T, int D, void* stream);
 int ifab_group_norm_gate(const float* o, long ldo, const float* w, float eps, const void* gate, long ldg, int act, void* y, long ldy, int f32, int T,
                          int groups, int n, void* stream);
@@ -301,7 +323,15 @@ int ifab_router_post_norm(const float* y, long ldy, const float* norm_w, const f
                           int32_t* ids, float* wts, float* shared_w, uint32_t* ticket, int T, int N, int K, void* stream);
 int ifab_gemv_group_norm(const float* o, long ldo, const float* gain, float eps, int groups, const void* gate, long ldg, int gate_act, const void* w,
                          void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream);
-int ifab_gemv_act(const void* x, long ldx, const void* w, void* z, long ldz, int out_f32, int act, int T, int N, int K, void* stream);
+/* z = act(x W^T + bias + addend), bias and addend (f32 rows, may be z) or null */
+int ifab_gemv_act(const void* x, long ldx, const void* w, const float* bias, const float* addend, long ldadd, void* z, long ldz, int out_f32, int act, int T, int N,
+                  int K, void* stream);
+/* front of a layer with parallel sublayers, T <= 2: x_out = x_in (+ y) (+ extra), h = rms(x_out) * norm_w -> projection z = h W^T + bias, gated unit of
+ * [gate | up] rows, router logits and selection */
+int ifab_parallel_in_decode(const float* y, long ldy, const float* extra, long lde, const float* norm_w, float eps, const float* x_in, float* x_out, long ldx,
+                            void* xn, long ldn, const void* w, const float* bias, void* z, long ldz, int N, const void* w_gu, int F, int unit, float limit,
+                            float alpha, void* unit_out, long ldu, const void* w_router, float* logits, long ldl, const float* correction, int E, int topk,
+                            int scoring, int renorm, float scale, int groups, int keep, int32_t* ids, float* wts, uint32_t* ticket, int T, int K, void* stream);
 /* linear attention with a fixed decay per head over a packed projection row (linear_attn.cu); state f32 [slots, H, e, d], powers f32 [H, 129],
  * rope float2 [T, rot / 2] of ifab_rope_table */
 int ifab_rope_table(const int32_t* positions, const double* freq, void* cs, int T, int pairs, void* stream);
@@ -315,20 +345,22 @@ int ifab_la_chunks(const float* q, const float* k, const float* v, const int32_t
 int ifab_la_tiles(const void* proj, long ldp, int q_off, int k_off, int v_off, int H, int d, int e, int rot, int interleaved, const void* rope, int act,
                   float k_scale, const float* powers, const int32_t* chunks, int n, const int32_t* positions, float* cstate, uint64_t cstate_bytes,
                   float* state, float* o, long ldo, const void* gate, long ldg, int gate_act, void* y, long ldy, float eps, uint32_t* status, void* stream);
-/* per-head norm + rotation + cache write, and sliding-window attention with sinks over pages, any head sizes (window_attn.cu) */
+/* norm per head (or, `whole`, over all heads of q and of k with a gain per column) + rotation + cache write, and attention over a window or a chunk of the
+ * pages with score caps, distance biases, sinks and gates (attn_rule.cuh), any head sizes (window_attn.cu) */
 int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, const float* q_gain, const float* k_gain, float eps,
                             int H, int G, int d, int e, int rot, int interleaved, const void* rope, const int32_t* positions, const int32_t* slots,
                             const int32_t* page_table, int max_pages, int page_tokens, int num_pages, void* q_out, long ldq, int q_stride, void* k_cache,
-                            void* v_cache, int T, uint32_t* status, void* stream);
+                            void* v_cache, int whole, int T, uint32_t* status, void* stream);
 int ifab_window_attn(const void* q, long ldq, int q_stride, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,
-                     const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int H, int G, int d, int e, int window, float scale,
-                     const float* sink, const void* gate, long ldg, int gate_act, void* out, long ldo, int T, uint32_t* status, void* stream);
+                     const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int H, int G, int d, int e, int window, float scale, float cap,
+                     const float* slopes, int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, void* out, long ldo, int T,
+                     uint32_t* status, void* stream);
 /* operands of the tensor-core windowed attention: keys / values first .. first + n - 1 of a sequence, heads zero-padded to dp / 128 columns */
 int ifab_ctx_gather_pad(const void* k_cache, const void* v_cache, const int32_t* page_table, int slot, int max_pages, int page_tokens, int num_pages,
                         int first, int n, int rows, int G, int d, int dp, int e, void* k, void* vt, long ldvt, uint32_t* status, void* stream);
 int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const void* k2, long ldk2, int d2, const void* vt, long ldvt, void* out, long ldo,
-                        int m, int ctx, int H, int kv_group, int d, int e, int pos0, int window, float scale, const float* sink, const void* gate, long ldg,
-                        int gate_act, int gate_per_head, uint32_t* status, void* stream);
+                        int m, int ctx, int H, int kv_group, int d, int e, int pos0, int window, float scale, float cap, const float* slopes, int chunked,
+                        const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, uint32_t* status, void* stream);
 /* latent attention over paged rows [latent padded to Lp | rotated key part padded to Rp], any sizes, bf16 or f32 (latent_attn.cu). splits <= 64, the last
  * takes what is left of the keys a row sees; scratch f32 [T, H, splits, Lp + 2] */
 int ifab_latent_prepare(const void* proj, long ldp, int f32, int q_off, int q_rank, int kv_off, int kv_rank, int rot_dim, const float* q_gain,
@@ -355,8 +387,8 @@ int ifab_latent_merge_vup(const float* scratch, const int32_t* positions, int wi
 int ifab_latent_gather(const void* cache, const int32_t* page_table, int slot, int max_pages, int page_tokens, int num_pages, int first, int n, int rows, int Lp,
                        int Rp, int tile, void* lat, void* rot, uint32_t* status, void* stream);
 int ifab_gqa_window_attention(const void* q, long ldq, const void* k_cache, const void* v_cache, const int32_t* positions, const int32_t* slots,
-                              const int32_t* page_table, int max_pages, int page_tokens, int num_pages, float scale, int window, const float* sink,
-                              const void* gate, long ldg, int gate_act, int T, int Hq, int Hkv, int head_dim, int keys_per_split, int max_splits,
+                              const int32_t* page_table, int max_pages, int page_tokens, int num_pages, float scale, int window, float cap, const float* slopes,
+                              int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, int T, int Hq, int Hkv, int head_dim, int keys_per_split, int max_splits,
                               float* scratch, uint64_t scratch_bytes, void* out, long ldo, uint32_t* status, void* stream);
 /* indexer: q bf16 [T, heads, dim], w f32 [T, heads], keys paged bf16 [pages, page_tokens, dim]; scores = scratch f32 [T, ctx];
  * out int32 [T, topk]: the top-k key positions (<= the query position) in ascending order, -1 padded */

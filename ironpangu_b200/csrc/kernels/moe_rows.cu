@@ -4,7 +4,8 @@
 //   moe_route_kernel         f32 router logits (+ bias) -> ids and weights of the chosen experts (moe_select.cuh), and the shared
 //                            expert's weight sigmoid(logits[:, E]) when the logits carry that column
 //   moe_combine_norm_kernel  y = sum of the chosen experts' rows by weight + shared weight * shared row (f32, slot order); then the
-//                            residual update x += rms(y) * w and the next operand xa = rms(x) * w2 (or x)
+//                            residual update x += rms(y) * w and the next operand xa = rms(x) * w2 (or x). Without w, y is added
+//                            as it is, together with f32 rows `base` (what ran beside the experts) and `extra`
 #include "moe_select.cuh"
 #include "rope.cuh"
 #include "ifab_kernels.h"
@@ -17,6 +18,7 @@ struct RouteParams {
   const float* logits; long ld; const float* bias;
   int M, E, topk, scoring, renorm; float scale;
   int32_t* ids; float* wts; float* shared_w;
+  int groups, keep;
 };
 
 // one warp per row
@@ -26,7 +28,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(RouteParams p) {
   const int m = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (m >= p.M) return;
   const float* z = p.logits + (long)m * p.ld;
-  select_topk_row(z, p.bias, p.E, p.topk, p.scoring, p.renorm, p.scale, p.ids + (long)m * p.topk, p.wts + (long)m * p.topk);
+  select_topk_row(z, p.bias, p.E, p.topk, p.scoring, p.renorm, p.scale, p.ids + (long)m * p.topk, p.wts + (long)m * p.topk, p.groups, p.keep);
   if (p.shared_w && lane == 0) p.shared_w[m] = sigmoid_f32(z[p.E]);
 }
 
@@ -51,6 +53,7 @@ struct CombineNormParams {
   const void* shared; long lds; const float* shared_w;      // shared expert's rows (or null) and their weights (null: 1)
   const float *w, *w2; float eps;
   float* x; long ldx; void* xa; long lda;
+  const float *base, *extra; long ldb, lde;      // rows of the residual update (without w), or null
   int D, Dp;                             // Dp: D padded to 4 columns; the padding of every operand is zero
 };
 
@@ -96,7 +99,7 @@ __global__ void __launch_bounds__(256) moe_combine_norm_kernel(CombineNormParams
       for (int j = 0; j < 4; ++j) ss += v[i][j] * v[i][j];
     }
   }
-  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)p.D + p.eps);
+  const float inv = p.w ? 1.f / sqrtf(block_sum(ss, red) / (float)p.D + p.eps) : 1.f;
   float* xr = p.x + (long)m * p.ldx;
   A* ar = reinterpret_cast<A*>(p.xa) + (long)m * p.lda;
   ss = 0.f;
@@ -106,9 +109,21 @@ __global__ void __launch_bounds__(256) moe_combine_norm_kernel(CombineNormParams
     if (c < p.Dp) {
       float r[4];
       load4(xr + c, r);
+      if (p.base) {
+        float f[4];
+        load4(p.base + (long)m * p.ldb + c, f);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[i][j] += f[j];
+      }
+      if (p.extra) {
+        float f[4];
+        load4(p.extra + (long)m * p.lde + c, f);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) r[j] += f[j];
+      }
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        v[i][j] = c + j < p.D ? r[j] + v[i][j] * inv * p.w[c + j] : 0.f;
+        v[i][j] = c + j < p.D ? r[j] + (p.w ? v[i][j] * inv * p.w[c + j] : v[i][j]) : 0.f;
         ss += v[i][j] * v[i][j];
       }
       store4(xr + c, v[i]);
@@ -138,19 +153,20 @@ int combine(const CombineNormParams& p, int M, cudaStream_t s) {
 
 }  // namespace
 
-extern "C" int ifab_moe_route(const float* logits, long ld, const float* bias, int M, int E, int topk, int scoring, int renorm, float scale, int32_t* ids,
-                              float* wts, float* shared_w, void* stream) {
-  if (M < 1 || E < 1 || E > 32 * SELECT_PER_LANE || topk < 1 || topk > MAX_TOPK || topk > E || scoring < 0 || scoring > 2) return -1;
-  RouteParams p{logits, ld, bias, M, E, topk, scoring, renorm, scale, ids, wts, shared_w};
+extern "C" int ifab_moe_route(const float* logits, long ld, const float* bias, int M, int E, int topk, int scoring, int renorm, float scale, int groups, int keep,
+                              int32_t* ids, float* wts, float* shared_w, void* stream) {
+  if (M < 1 || !select_ok(E, topk, scoring, groups, keep)) return -1;
+  RouteParams p{logits, ld, bias, M, E, topk, scoring, renorm, scale, ids, wts, shared_w, groups, keep};
   return launch_chain(moe_route_kernel, dim3((M + 3) / 4), dim3(128), 0, (cudaStream_t)stream, p);
 }
 
 extern "C" int ifab_moe_combine_norm(const void* y, long ldy, const int32_t* route_row, const float* wts, int topk, const void* shared, long lds,
-                                     const float* shared_w, const float* w, const float* w2, float eps, float* x, long ldx, void* xa, long lda, int f32, int M,
-                                     int D, void* stream) {
+                                     const float* shared_w, const float* w, const float* w2, float eps, const float* base, long ldb, const float* extra, long lde,
+                                     float* x, long ldx, void* xa, long lda, int f32, int M, int D, void* stream) {
   const int Dp = (D + 3) / 4 * 4;
   if (M < 1 || D < 1 || topk < 1 || topk > MAX_TOPK || ldy % 4 || ldx % 4 || lda % 4 || (shared && lds % 4) || ldy < Dp || ldx < Dp || lda < Dp || (shared && lds < Dp))
     return -1;
-  CombineNormParams p{y, ldy, route_row, wts, topk, shared, lds, shared_w, w, w2, eps, x, ldx, xa, lda, D, Dp};
+  if ((w && base) || (base && (ldb % 4 || ldb < Dp)) || (extra && (lde % 4 || lde < Dp))) return -1;
+  CombineNormParams p{y, ldy, route_row, wts, topk, shared, lds, shared_w, w, w2, eps, x, ldx, xa, lda, base, extra, ldb, lde, D, Dp};
   return f32 ? combine<float>(p, M, (cudaStream_t)stream) : combine<bf16>(p, M, (cudaStream_t)stream);
 }

@@ -1,13 +1,15 @@
 // Row operators of decoders that keep an f32 residual stream and normalise a sublayer's OUTPUT before adding it:
 //
 //   embed_rows_kernel      x = table[id] * scale (f32) and its copy in the activation type (the operand of the next linears), of rms(x) * w
-//                          when a gain is given (the norm ahead of the first sublayer)
+//                          when a gain is given (the norm ahead of the first sublayer); a second f32 copy on request
 //   post_norm_add_kernel   x += rms(y) * w; copy in the activation type (of rms(x) * w2 when a second gain is given: the norm ahead
-//                          of the output matrix). y is the f32 output of the sublayer's last linear
+//                          of the output matrix). y is the f32 output of the sublayer's last linear; without w
+//                          it is added as it is, without y nothing is; rows of `extra` join the update
 //   rms_rows_kernel        rms(x[row]) * w of selected rows, in the activation type (the norm ahead of the output matrix)
 //   group_norm_gate_kernel (o / rms of each group of columns [* w]) * act(gate): the normalised, gated heads of a recurrent
 //                          mixer. group = one head without a gain, or all heads together with one
 //   gate_rows_kernel       o * act(gate), reading heads at a padded stride
+//   gated_rows_kernel      [gate | up] rows -> the gated unit's value (rope.cuh)
 //
 // Every kernel exists for bf16 activations and for f32 ones; norms and the residual are f32 in both.
 #include "rope.cuh"
@@ -25,7 +27,7 @@ __device__ __forceinline__ void store4(bf16* p, const float* f) {
 
 template <typename A>
 __global__ void __launch_bounds__(256) embed_rows_kernel(const int32_t* ids, const A* table, long ldt, float scale, const float* w, float eps, float* x, long ldx,
-                                                         A* xa, long lda, int D, int vocab, uint32_t* status) {
+                                                         float* copy, A* xa, long lda, int D, int vocab, uint32_t* status) {
   __shared__ float red[33];
   grid_dep_launch();
   grid_dep_wait();
@@ -39,6 +41,7 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(const int32_t* ids, con
   for (int c = threadIdx.x; c < D; c += blockDim.x) {
     const float v = to_f32(table[(long)id * ldt + c]) * scale;
     x[(long)t * ldx + c] = v;
+    if (copy) copy[(long)t * ldx + c] = v;
     if (!w) xa[(long)t * lda + c] = from_f32<A>(v);
     ss += v * v;
   }
@@ -49,16 +52,17 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(const int32_t* ids, con
 
 // one CTA per row
 template <typename A>
-__global__ void __launch_bounds__(256) post_norm_add_kernel(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, A* xa,
-                                                            long lda, int D) {
+__global__ void __launch_bounds__(256) post_norm_add_kernel(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx,
+                                                            const float* extra, long lde, A* xa, long lda, int D) {
   __shared__ float red[33];
   grid_dep_launch();
   grid_dep_wait();
   const int t = blockIdx.x;
-  const float* yr = y + (long)t * ldy;
+  const float* yr = y ? y + (long)t * ldy : nullptr;
+  const float* er = extra ? extra + (long)t * lde : nullptr;
   float* xr = x + (long)t * ldx;
   A* ar = xa + (long)t * lda;
-  if (D % 4 == 0 && ldy % 4 == 0 && ldx % 4 == 0 && lda % 4 == 0 && D <= 256 * 16) {     // the row stays in registers between the passes
+  if (D % 4 == 0 && ldy % 4 == 0 && ldx % 4 == 0 && lda % 4 == 0 && lde % 4 == 0 && D <= 256 * 16) {     // the row stays in registers between the passes
     float4 v[4], r[4], g[4];
     float ss = 0.f;
 #pragma unroll
@@ -66,15 +70,22 @@ __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* y, long
       const int c = (threadIdx.x + i * 256) * 4;
       v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
       r[i] = v[i];
-      g[i] = v[i];
+      g[i] = make_float4(1.f, 1.f, 1.f, 1.f);
       if (c < D) {
-        v[i] = *reinterpret_cast<const float4*>(yr + c);
+        if (yr) v[i] = *reinterpret_cast<const float4*>(yr + c);
         r[i] = *reinterpret_cast<const float4*>(xr + c);
-        g[i] = *reinterpret_cast<const float4*>(w + c);
+        if (w) g[i] = *reinterpret_cast<const float4*>(w + c);
+        if (er) {
+          const float4 e = *reinterpret_cast<const float4*>(er + c);
+          r[i].x += e.x;
+          r[i].y += e.y;
+          r[i].z += e.z;
+          r[i].w += e.w;
+        }
       }
       ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
     }
-    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)D + eps);
+    const float inv = w ? 1.f / sqrtf(block_sum(ss, red) / (float)D + eps) : 1.f;
     ss = 0.f;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
@@ -104,11 +115,13 @@ __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* y, long
     return;
   }
   float ss = 0.f;
-  for (int c = threadIdx.x; c < D; c += blockDim.x) ss += yr[c] * yr[c];
-  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)D + eps);
+  if (yr && w)
+    for (int c = threadIdx.x; c < D; c += blockDim.x) ss += yr[c] * yr[c];
+  const float inv = yr && w ? 1.f / sqrtf(block_sum(ss, red) / (float)D + eps) : 1.f;
   ss = 0.f;
   for (int c = threadIdx.x; c < D; c += blockDim.x) {
-    const float v = xr[c] + yr[c] * inv * w[c];
+    float v = xr[c] + (er ? er[c] : 0.f);
+    if (yr) v += yr[c] * inv * (w ? w[c] : 1.f);
     xr[c] = v;
     ss += v * v;
     if (!w2) ar[c] = from_f32<A>(v);
@@ -167,9 +180,17 @@ __global__ void __launch_bounds__(256) gate_rows_kernel(const A* o, long ldo, in
 }
 
 template <typename A>
-int embed(const int32_t* ids, const void* table, long ldt, float scale, const float* w, float eps, float* x, long ldx, void* xa, long lda, int T, int D, int vocab,
-          uint32_t* status, cudaStream_t s) {
-  return launch_chain(embed_rows_kernel<A>, dim3(T), dim3(256), 0, s, ids, (const A*)table, ldt, scale, w, eps, x, ldx, (A*)xa, lda, D, vocab, status);
+__global__ void __launch_bounds__(256) gated_rows_kernel(const A* gu, long ld, int up, GatedUnit unit, A* y, long ldy, int F) {
+  grid_dep_launch();
+  grid_dep_wait();
+  const A* r = gu + (long)blockIdx.x * ld;
+  for (int c = threadIdx.x; c < F; c += blockDim.x) y[(long)blockIdx.x * ldy + c] = from_f32<A>(gated_value<sizeof(A) == 2>(to_f32(r[c]), to_f32(r[up + c]), unit));
+}
+
+template <typename A>
+int embed(const int32_t* ids, const void* table, long ldt, float scale, const float* w, float eps, float* x, long ldx, float* copy, void* xa, long lda, int T, int D,
+          int vocab, uint32_t* status, cudaStream_t s) {
+  return launch_chain(embed_rows_kernel<A>, dim3(T), dim3(256), 0, s, ids, (const A*)table, ldt, scale, w, eps, x, ldx, copy, (A*)xa, lda, D, vocab, status);
 }
 template <typename A>
 int group_norm(const float* o, long ldo, const float* w, float eps, const void* gate, long ldg, int act, void* y, long ldy, int T, int groups, int n,
@@ -182,20 +203,30 @@ int group_norm(const float* o, long ldo, const float* w, float eps, const void* 
 
 }  // namespace
 
-extern "C" int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float scale, const float* w, float eps, float* x, long ldx, void* xa, long lda,
-                               int f32, int T, int D, int vocab, uint32_t* status, void* stream) {
+// copy: a second f32 copy of x (row stride ldx), or null
+extern "C" int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float scale, const float* w, float eps, float* x, long ldx, float* copy, void* xa,
+                               long lda, int f32, int T, int D, int vocab, uint32_t* status, void* stream) {
   if (T < 1 || D < 1 || vocab < 1) return -1;
   cudaStream_t s = (cudaStream_t)stream;
-  return f32 ? embed<float>(ids, table, ldt, scale, w, eps, x, ldx, xa, lda, T, D, vocab, status, s)
-             : embed<bf16>(ids, table, ldt, scale, w, eps, x, ldx, xa, lda, T, D, vocab, status, s);
+  return f32 ? embed<float>(ids, table, ldt, scale, w, eps, x, ldx, copy, xa, lda, T, D, vocab, status, s)
+             : embed<bf16>(ids, table, ldt, scale, w, eps, x, ldx, copy, xa, lda, T, D, vocab, status, s);
 }
 
-extern "C" int ifab_post_norm_add(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, void* xa, long lda, int f32, int T, int D,
-                                  void* stream) {
+extern "C" int ifab_post_norm_add(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, const float* extra, long lde, void* xa,
+                                  long lda, int f32, int T, int D, void* stream) {
   if (T < 1 || D < 1) return -1;
   cudaStream_t s = (cudaStream_t)stream;
-  return f32 ? launch_chain(post_norm_add_kernel<float>, dim3(T), dim3(256), 0, s, y, ldy, w, w2, eps, x, ldx, (float*)xa, lda, D)
-             : launch_chain(post_norm_add_kernel<bf16>, dim3(T), dim3(256), 0, s, y, ldy, w, w2, eps, x, ldx, (bf16*)xa, lda, D);
+  return f32 ? launch_chain(post_norm_add_kernel<float>, dim3(T), dim3(256), 0, s, y, ldy, w, w2, eps, x, ldx, extra, lde, (float*)xa, lda, D)
+             : launch_chain(post_norm_add_kernel<bf16>, dim3(T), dim3(256), 0, s, y, ldy, w, w2, eps, x, ldx, extra, lde, (bf16*)xa, lda, D);
+}
+
+// y [T, F] = unit(gu[:, c], gu[:, up + c])
+extern "C" int ifab_gated_rows(const void* gu, long ld, int up, int unit, float limit, float alpha, void* y, long ldy, int f32, int T, int F, void* stream) {
+  const GatedUnit u{unit, limit, alpha};
+  if (T < 1 || F < 1 || up < F || !gated_ok(u)) return -1;
+  cudaStream_t s = (cudaStream_t)stream;
+  return f32 ? launch_chain(gated_rows_kernel<float>, dim3(T), dim3(256), 0, s, (const float*)gu, ld, up, u, (float*)y, ldy, F)
+             : launch_chain(gated_rows_kernel<bf16>, dim3(T), dim3(256), 0, s, (const bf16*)gu, ld, up, u, (bf16*)y, ldy, F);
 }
 
 extern "C" int ifab_rms_rows(const float* x, long ldx, const int32_t* rows, const float* w, float eps, void* y, long ldy, int f32, int T, int D,

@@ -63,6 +63,29 @@ __device__ __forceinline__ float activate(float z, int act) {
   }
 }
 
+// What a gated feed-forward makes of its two projections: 0 silu(g) u, 1 relu(g) u, 2 g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit) and
+// u' = u within [-limit, limit]
+struct GatedUnit {
+  int kind;
+  float limit, alpha;
+};
+template <bool FAST = false>
+__device__ __forceinline__ float gated_value(float g, float u, const GatedUnit& unit) {
+  if (unit.kind == 1) return fmaxf(g, 0.f) * u;
+  if (unit.kind == 2) {
+    g = fminf(g, unit.limit);
+    return g * sigmoid_f32<FAST>(unit.alpha * g) * (fminf(fmaxf(u, -unit.limit), unit.limit) + 1.f);
+  }
+  return g * sigmoid_f32<FAST>(g) * u;
+}
+// the same of projections that count as bf16 rows for SiLU units (the form of the kernels that store them)
+__device__ __forceinline__ float gated_bf16(float g, float u, const GatedUnit& unit) {
+  if (unit.kind) return gated_value<true>(g, u, unit);
+  g = bf16_round(g);
+  return g / (1.f + __expf(-g)) * bf16_round(u);
+}
+__host__ __forceinline__ bool gated_ok(const GatedUnit& u) { return u.kind >= 0 && u.kind <= 2 && (u.kind != 2 || u.limit > 0.f); }
+
 // sum over the block (blockDim.x a multiple of 32, at most 1024); `red` holds 33 floats; every thread gets the sum
 __device__ __forceinline__ float block_sum(float v, float* red) {
   v = warp_sum(v);

@@ -16,6 +16,7 @@
 // `ifab_gemm_bf16` uses these kernels from 256 rows and 256 columns up; below that a pair's 256 x 256 tile is mostly padding.
 #include <algorithm>
 
+#include "attn_rule.cuh"
 #include "rope.cuh"
 #include "tc_gemm_core.cuh"
 #include "ifab_kernels.h"
@@ -37,8 +38,10 @@ struct Gemm2Params {
   int M, N, K;
   uint32_t* status;
   uint32_t spin_limit;
-  int swiglu_f;   // > 0 (persistent kernel only): B = [gate rows 0..F) | up rows F..2F), C[M, F] = silu(A gate^T) * (A up^T)
-  int act;        // activation of the result (numbers of activate(); 0: none), after the residual
+  int swiglu_f;   // > 0 (persistent kernel only): B = [gate rows 0..F) | up rows F..2F), C[M, F] = unit(A gate^T, A up^T)
+  int act;        // activation of the result (numbers of activate(); 0: none), after bias and residual
+  const float* bias; float cap;      // [N] or null; > 0: cap tanh(result / cap)
+  GatedUnit unit;
 };
 
 __device__ __forceinline__ uint32_t cluster_ctarank() {
@@ -86,6 +89,10 @@ __device__ __forceinline__ void umma_commit_pair(uint64_t* bar) {
 
 __device__ __forceinline__ void store_row32_2(const Gemm2Params& p, int row, int col, float* v) {
   if (row >= p.M || col >= (p.swiglu_f > 0 ? p.swiglu_f : p.N)) return;
+  if (p.bias) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) v[i] += p.bias[col + i];
+  }
   if (p.residual) {
     const bf16* r = p.residual + (long)row * p.ldr + col;
 #pragma unroll
@@ -94,6 +101,10 @@ __device__ __forceinline__ void store_row32_2(const Gemm2Params& p, int row, int
   if (p.act) {
 #pragma unroll
     for (int i = 0; i < 32; ++i) v[i] = activate<true>(v[i], p.act);
+  }
+  if (p.cap > 0.f) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) v[i] = soft_limit<true>(v[i], p.cap);
   }
   if (p.out_f32) {
     float* out = reinterpret_cast<float*>(p.c) + (long)row * p.ldc + col;
@@ -351,10 +362,7 @@ __global__ void __launch_bounds__(192) tc_gemm_2sm_persistent_kernel(const __gri
           tmem_ld_32x32(tm_row + (uint32_t)(HALF_N + c0), u);
           tmem_ld_wait();
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const float g = bf16_round(v[i]);
-            v[i] = g / (1.f + __expf(-g)) * bf16_round(u[i]);
-          }
+          for (int i = 0; i < 32; ++i) v[i] = gated_bf16(v[i], u[i], p.unit);
           store_row32_2(p, row, n0 + c0, v);
         }
       } else {
@@ -386,11 +394,15 @@ __global__ void __launch_bounds__(192) tc_gemm_2sm_persistent_kernel(const __gri
 // SM pair walks the tiles with two accumulators in tensor memory, else one pair per tile.
 extern "C" int ifab_gemm_act_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr,
                                       int act, int persistent, int M, int N, int K, uint32_t* status, void* stream) {
+  return ifab_gemm_epilogue_bf16_2sm(a, lda, b, ldb, c, ldc, out_f32, residual, ldr, nullptr, act, 0.f, persistent, M, N, K, status, stream);
+}
+extern "C" int ifab_gemm_epilogue_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr,
+                                           const float* bias, int act, float cap, int persistent, int M, int N, int K, uint32_t* status, void* stream) {
   if (M < 1 || N < 32 || N % 32 || K < 8 || K % 8 || lda % 8 || ldb % 8) return -1;
   CUtensorMap ta, tb;
   if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM)) return rc;
   if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)N, (uint64_t)K, (uint64_t)ldb, HALF_N)) return rc;
-  Gemm2Params p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, 0, act};
+  Gemm2Params p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, 0, act, bias, cap, {}};
   const int tiles = ((M + 255) / 256) * ((N + 255) / 256);
   if (!persistent) {
     if (int rc = opt_in_smem(tc_gemm_2sm_kernel, SMEM2)) return rc;
@@ -413,15 +425,20 @@ extern "C" int ifab_gemm_bf16_2sm_persistent(const void* a, long lda, const void
   return ifab_gemm_act_bf16_2sm(a, lda, b, ldb, c, ldc, out_f32, residual, ldr, 0, 1, M, N, K, status, stream);
 }
 
-// C[M, F] = silu(A gate^T) * (A up^T) with B = [gate rows | up rows] ([2F, K]): the packed gate / up projection of a SwiGLU block in
-// one persistent CTA-pair launch (gate and up of the same 128 output columns share an accumulator). F % 32 == 0, K % 8 == 0.
 extern "C" int ifab_gemm_swiglu_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int M, int F, int K, uint32_t* status,
                                          void* stream) {
-  if (M < 1 || F < 32 || F % 32 || K < 8 || K % 8 || lda % 8 || ldb % 8) return -1;
+  return ifab_gemm_gated_bf16_2sm(a, lda, b, ldb, c, ldc, 0, 0.f, 0.f, M, F, K, status, stream);
+}
+// C[M, F] = unit(A gate^T, A up^T) with B = [gate rows | up rows] ([2F, K]): the packed gate / up projection of a gated feed-forward in
+// one persistent CTA-pair launch (gate and up of the same 128 output columns share an accumulator). F % 32 == 0, K % 8 == 0.
+extern "C" int ifab_gemm_gated_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int unit, float limit, float alpha, int M, int F,
+                                        int K, uint32_t* status, void* stream) {
+  const GatedUnit gu{unit, limit, alpha};
+  if (!gated_ok(gu) || M < 1 || F < 32 || F % 32 || K < 8 || K % 8 || lda % 8 || ldb % 8) return -1;
   CUtensorMap ta, tb;
   if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM)) return rc;
   if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)2 * F, (uint64_t)K, (uint64_t)ldb, HALF_N)) return rc;
-  Gemm2Params p{c, ldc, 0, nullptr, 0, M, 2 * F, K, status, 4000000u, F, 0};
+  Gemm2Params p{c, ldc, 0, nullptr, 0, M, 2 * F, K, status, 4000000u, F, 0, nullptr, 0.f, gu};
   if (int rc = opt_in_smem(tc_gemm_2sm_persistent_kernel, SMEM2)) return rc;
   int dev = 0, sms = 148;
   cudaGetDevice(&dev);

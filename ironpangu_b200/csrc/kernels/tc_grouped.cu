@@ -8,10 +8,12 @@
 //                           covers the worst case and CTAs beyond num_tiles leave at once - no host round trip.
 // Modes:
 //   plain    C[row, n] = A[row, :] . B[e][n, :]                                    (down projection)
-//   swiglu   B holds gate rows [0, F) and up rows [F, 2F); one accumulator of 256 columns receives 128 gate and the
-//            128 matching up columns (two TMA boxes per stage), the epilogue stores silu(gate) * up -> C[row, F]
+//   gated    B holds gate rows [0, F) and up rows [F, 2F); one accumulator of 256 columns receives 128 gate and the
+//            128 matching up columns (two TMA boxes per stage), the epilogue stores the unit's value (silu(gate) * up or
+//            another of rope.cuh) -> C[row, F]
 // Rows of a tile that belong to the next expert (the tile is only partly valid) are computed and thrown away.
 // Reference counterparts: expert_gmm + expert_act_quantize (native/src/token_executor.h:1054-1167).
+#include "rope.cuh"
 #include "tc_gemm_core.cuh"
 #include "ifab_kernels.h"
 
@@ -27,6 +29,7 @@ struct GroupedParams {
   int N, K, F;          // F: columns of the swiglu output (N = 2F); unused in plain mode
   uint32_t* status;
   uint32_t spin_limit;
+  GatedUnit unit;
 };
 
 template <int BN, bool SWIGLU>
@@ -65,10 +68,7 @@ __global__ void __launch_bounds__(192) tc_grouped_kernel(const __grid_constant__
           tmem_ld_32x32(tm + (uint32_t)(NOUT + c0), u);
           tmem_ld_wait();
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const float g = bf16_round(v[i]);
-            v[i] = g / (1.f + __expf(-g)) * bf16_round(u[i]);
-          }
+          for (int i = 0; i < 32; ++i) v[i] = gated_bf16(v[i], u[i], p.unit);
         } else {
           tmem_ld_wait();
         }
@@ -105,11 +105,19 @@ int launch_grouped(const CUtensorMap& ta, const CUtensorMap& tb, const GroupedPa
 extern "C" int ifab_grouped_gemm_bf16(const void* a, long lda, int rows_max, const void* b, int experts, int N, int K,
                                       const int32_t* tiles, const int32_t* num_tiles, int max_tiles, void* c, long ldc, int mode,
                                       uint32_t* status, void* stream) {
+  return ifab_grouped_gemm_gated_bf16(a, lda, rows_max, b, experts, N, K, tiles, num_tiles, max_tiles, c, ldc, mode, 0, 0.f, 0.f, status, stream);
+}
+// The same with the gated unit of mode 1 by number (0 SiLU, 1 ReLU, 2 limited).
+extern "C" int ifab_grouped_gemm_gated_bf16(const void* a, long lda, int rows_max, const void* b, int experts, int N, int K, const int32_t* tiles,
+                                            const int32_t* num_tiles, int max_tiles, void* c, long ldc, int mode, int unit, float limit, float alpha,
+                                            uint32_t* status, void* stream) {
+  const GatedUnit gu{unit, limit, alpha};
+  if (!gated_ok(gu)) return -1;
   if (rows_max < 1 || experts < 1 || N < 8 || K < 8 || K % 8 || lda % 8 || ldc % 8 || max_tiles < 1 || max_tiles > 65535) return -1;
   if (mode == 1 && (N % 16)) return -1;
   CUtensorMap ta, tb;
   if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)rows_max, (uint64_t)K, (uint64_t)lda, BM)) return rc;
-  GroupedParams p{reinterpret_cast<const int4*>(tiles), num_tiles, (bf16*)c, ldc, N, K, N / 2, status, 4000000u};
+  GroupedParams p{reinterpret_cast<const int4*>(tiles), num_tiles, (bf16*)c, ldc, N, K, N / 2, status, 4000000u, gu};
   cudaStream_t s = (cudaStream_t)stream;
   if (mode == 1) {
     if (int rc = make_tmap_bf16_3d(&tb, b, (uint64_t)experts, (uint64_t)N, (uint64_t)K, (uint64_t)K, (uint64_t)N * K, 128)) return rc;

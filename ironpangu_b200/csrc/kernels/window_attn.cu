@@ -1,12 +1,16 @@
-// Sliding-window softmax attention with a per-head sink over paged keys / values, for any head sizes (query / key size and value
-// size independent), bf16 or f32 activations and caches.
+// Softmax attention over a window or a chunk of paged keys / values with sinks, score caps, distance biases and output gates
+// (attn_rule.cuh), for any head sizes (query / key size and value size independent), bf16 or f32 activations and caches.
 //
 //   qk_norm_rope_write_kernel  RMS norm per head of q and k with a shared gain, rotation of the first `rot` columns (either pair
 //                              layout), q to its own rows, k and v into the pages of their sequence
-//   window_attn_kernel         one CTA per (row, query head): row at position i sees keys j with 0 <= i - j < window; scores,
-//                              weights and sums in f32; the denominator also holds exp(sink_h). Optional output gate
+//   qk_rows_norm_write_kernel  the same with the norm over all heads of q (and all of k) together, a gain per column
+//   window_attn_kernel         one CTA per (row, query head): scores, weights and sums in f32; the denominator also holds
+//                              exp(sink_h). Optional output gate, a value per column or per head
+//
+// v may be the columns of k (v_off == k_off): the values are then the keys as projected.
 //
 // Positions, slots and page tables as in the other paged kernels; pages that fell out of every window may be gone (-1).
+#include "attn_rule.cuh"
 #include "rope.cuh"
 #include "ifab_kernels.h"
 
@@ -90,6 +94,75 @@ __global__ void __launch_bounds__(128) qk_norm_rope_write_kernel(QkParams p) {
   for (int c = p.rope.rot + lane; c < p.d; c += 32) dst[c] = from_f32<A>(to_f32(src[c]) * inv * (gain ? gain[c] : 1.f));
 }
 
+// grid T, 256 threads: the two row sums first, then pairs of neighbouring columns
+template <typename A>
+__global__ void __launch_bounds__(256) qk_rows_norm_write_kernel(QkParams p) {
+  __shared__ float red[2][8];
+  grid_dep_launch();
+  grid_dep_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = p.positions[t];
+  if (pos < 0) return;
+  const A* row = reinterpret_cast<const A*>(p.proj) + (long)t * p.ldp;
+  const int lp = pos / p.page_tokens;
+  const int page = lp < p.max_pages ? p.page_table[(long)p.slots[t] * p.max_pages + lp] : -1;
+  if (page < 0 || page >= p.num_pages) {
+    if (threadIdx.x == 0 && p.status) atomicOr(p.status, IFAB_STATUS_BAD_INDEX);
+    return;
+  }
+  const long dst_row = (long)page * p.page_tokens + pos % p.page_tokens;
+  const int nq = p.H * p.d, nk = p.G * p.d, nv = p.G * p.e;
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x; c < nq; c += 256) {
+    const float v = to_f32(row[p.q_off + c]);
+    sq += v * v;
+  }
+  for (int c = threadIdx.x; c < nk; c += 256) {
+    const float v = to_f32(row[p.k_off + c]);
+    sk += v * v;
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) {
+    red[0][warp] = sq;
+    red[1][warp] = sk;
+  }
+  A* vd = reinterpret_cast<A*>(p.v_cache) + dst_row * nv;
+  for (int c = threadIdx.x; c < nv; c += 256) vd[c] = row[p.v_off + c];
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    sq += red[0][i];
+    sk += red[1][i];
+  }
+  const float iq = 1.f / sqrtf(sq / (float)nq + p.eps), ik = 1.f / sqrtf(sk / (float)nk + p.eps);
+  const float2* cs = p.rope.cs + (long)t * (p.rope.rot / 2);
+  const int half = p.rope.rot / 2, units = half + p.d - p.rope.rot;      // of a head: pairs, then single columns
+  A* qd = reinterpret_cast<A*>(p.q_out) + (long)t * p.ldq;
+  A* kd = reinterpret_cast<A*>(p.k_cache) + dst_row * nk;
+  for (int i = threadIdx.x; i < (p.H + p.G) * units; i += 256) {
+    const int h = i / units, u = i - h * units;
+    const bool is_q = h < p.H;
+    const int c0 = (is_q ? h : h - p.H) * p.d;                           // of the head among its projection's columns
+    const A* src = row + (is_q ? p.q_off : p.k_off) + c0;
+    const float* gain = (is_q ? p.q_gain : p.k_gain) + c0;
+    A* dst = is_q ? qd + (long)h * p.q_stride : kd + c0;
+    const float inv = is_q ? iq : ik;
+    if (u < half) {
+      int ia, ib;
+      rope_pair(u, p.rope.rot, p.rope.interleaved, &ia, &ib);
+      const float2 r = cs[u];
+      const float a = to_f32(src[ia]) * inv * gain[ia], b = to_f32(src[ib]) * inv * gain[ib];
+      dst[ia] = from_f32<A>(a * r.x - b * r.y);
+      dst[ib] = from_f32<A>(b * r.x + a * r.y);
+    } else {
+      const int c = p.rope.rot + u - half;
+      dst[c] = from_f32<A>(to_f32(src[c]) * inv * gain[c]);
+    }
+  }
+}
+
 struct WinParams {
   const void* q; long ldq;
   const void *k_cache, *v_cache;
@@ -102,6 +175,8 @@ struct WinParams {
   void* out; long ldo;
   int q_stride;
   uint32_t* status;
+  ScoreRule rule;
+  int gate_head;                 // the gate has one value per head: [T, H]
 };
 
 // Keys and values first .. first + n - 1 of one sequence out of its pages: k [rows, G * dp] (columns d .. dp - 1 of a head zero) and
@@ -152,7 +227,8 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
   const int pos = p.positions[t];
   if (pos < 0) return;
   const int32_t* table = p.page_table + (long)p.slots[t] * p.max_pages;
-  const int first = (p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
+  const int first = first_key(pos, p.window, p.rule.chunked);
+  const float slope = p.rule.slopes ? p.rule.slopes[h] : 0.f;
   float q[EPL], acc[EPL];
   const A* qr = reinterpret_cast<const A*>(p.q) + (long)t * p.ldq + (long)h * p.q_stride;
 #pragma unroll
@@ -186,6 +262,11 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
     }
 #pragma unroll
     for (int b = 0; b < KB; ++b) s[b] = r[b] >= 0 ? warp_sum(s[b]) * p.scale : -INFINITY;
+    if (!p.rule.plain()) {
+#pragma unroll
+      for (int b = 0; b < KB; ++b)
+        if (r[b] >= 0) s[b] = ruled_score<sizeof(A) == 2>(s[b], p.rule, slope, pos - k0 - b * WARPS);
+    }
     float mn = m;
 #pragma unroll
     for (int b = 0; b < KB; ++b) mn = fmaxf(mn, s[b]);
@@ -228,7 +309,7 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
 #pragma unroll
     for (int w = 0; w < WARPS; ++w) v = fmaf(wgt[w], sm_acc[w][c], v);
     v *= inv;
-    if (p.gate) v *= activate<sizeof(A) == 2>(to_f32(reinterpret_cast<const A*>(p.gate)[(long)t * p.ldg + (long)h * p.e + c]), p.gate_act);
+    if (p.gate) v *= activate<sizeof(A) == 2>(to_f32(reinterpret_cast<const A*>(p.gate)[(long)t * p.ldg + (p.gate_head ? h : (long)h * p.e + c)]), p.gate_act);
     reinterpret_cast<A*>(p.out)[(long)t * p.ldo + (long)h * p.e + c] = from_f32<A>(v);
   }
 }
@@ -238,10 +319,15 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
 extern "C" int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, const float* q_gain, const float* k_gain,
                                        float eps, int H, int G, int d, int e, int rot, int interleaved, const void* rope, const int32_t* positions,
                                        const int32_t* slots, const int32_t* page_table, int max_pages, int page_tokens, int num_pages, void* q_out,
-                                       long ldq, int q_stride, void* k_cache, void* v_cache, int T, uint32_t* status, void* stream) {
+                                       long ldq, int q_stride, void* k_cache, void* v_cache, int whole, int T, uint32_t* status, void* stream) {
   if (T < 1 || T > 65535 || H < 1 || G < 1 || d < 1 || e < 1 || rot < 0 || rot % 2 || rot > d || (rot && !rope) || q_stride < d) return -1;
   QkParams p{proj, ldp, q_off, k_off, v_off, q_gain, k_gain, eps, H, G, d, e, {(const float2*)rope, rot, interleaved}, positions, slots, page_table, max_pages, page_tokens,
              num_pages, q_out, ldq, q_stride, k_cache, v_cache, T, status};
+  if (whole) {
+    if (!q_gain || !k_gain) return -1;
+    return f32 ? launch_chain(qk_rows_norm_write_kernel<float>, dim3(T), dim3(256), 0, (cudaStream_t)stream, p)
+               : launch_chain(qk_rows_norm_write_kernel<bf16>, dim3(T), dim3(256), 0, (cudaStream_t)stream, p);
+  }
   const dim3 grid((H + 2 * G + 3) / 4, T);
   return f32 ? launch_chain(qk_norm_rope_write_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, p)
              : launch_chain(qk_norm_rope_write_kernel<bf16>, grid, dim3(128), 0, (cudaStream_t)stream, p);
@@ -249,11 +335,11 @@ extern "C" int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int 
 
 extern "C" int ifab_window_attn(const void* q, long ldq, int q_stride, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,
                                 const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int H, int G, int d, int e, int window,
-                                float scale, const float* sink, const void* gate, long ldg, int gate_act, void* out, long ldo, int T, uint32_t* status,
-                                void* stream) {
-  if (T < 1 || T > 65535 || H < 1 || G < 1 || H % G || d < 1 || d > 256 || e < 1 || e > 256 || window < 0) return -1;
+                                float scale, float cap, const float* slopes, int chunked, const float* sink, const void* gate, long ldg, int gate_act,
+                                int gate_per_head, void* out, long ldo, int T, uint32_t* status, void* stream) {
+  if (cap < 0.f || T < 1 || T > 65535 || H < 1 || G < 1 || H % G || d < 1 || d > 256 || e < 1 || e > 256 || window < 0) return -1;
   WinParams p{q, ldq, k_cache, v_cache, positions, slots, page_table, max_pages, page_tokens, num_pages, H, G, d, e, window, scale, sink, gate, ldg, gate_act,
-              out, ldo, q_stride, status};
+              out, ldo, q_stride, status, {cap, slopes, chunked}, gate_per_head};
   const dim3 grid(H, T);
   return f32 ? launch_chain(window_attn_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, p)
              : launch_chain(window_attn_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)stream, p);

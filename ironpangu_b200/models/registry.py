@@ -24,7 +24,8 @@ class Family:
 
 
 FAMILIES: Tuple[Family, ...] = (Family("Falinex", "falinex", "FalinexDecoder", "FalinexRows", True, ("falinex-tiny", "falinex2b")),
-                                Family("Ponenex", "ponenex", "PonenexDecoder", "PonenexRows", True, ("ponenex-tiny", "ponenex-text")))
+                                Family("Ponenex", "ponenex", "PonenexDecoder", "PonenexRows", True, ("ponenex-tiny", "ponenex-text")),
+                                Family("Mikutar", "mikutar", "MikutarDecoder", "MikutarRows", True, ("mikutar-tiny", "mikutar-text")))
 
 
 def family_of(checkpoint_dir) -> Family:

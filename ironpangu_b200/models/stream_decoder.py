@@ -34,6 +34,7 @@ class StreamDecoder:
     name = "stream"
     chunk = 128            # rows per chunk of a packed step's long runs
     short_rows = 4         # runs of at most this many rows take the decode kernels inside a packed step
+    logit_cap = 0.0        # > 0: logits are cap * tanh(logit / cap)
     fused_rows = 2         # beyond this the CUDA-core products are FMA-bound and the GEMMs take over
 
     def __init__(self, cfg, weights: Dict[str, torch.Tensor], fabric: Fabric, *, max_tokens: int = 8, max_context: int = 1024, num_slots: int = 1,
@@ -82,9 +83,9 @@ class StreamDecoder:
             self._layers(B, n, tok, pos, slot, None, True)
         if self.dtype == BF16:
             K.lm_head_argmax(B.xa[:n], self.head, self.fabric, vocab_offset=0, partial=self.partial, logits=None if self.logits is None else self.logits[:n],
-                             out_ids=self.next_ids[:n], out_vals=self.next_vals[:n])
+                             out_ids=self.next_ids[:n], out_vals=self.next_vals[:n], cap=self.logit_cap)
         else:
-            N.linear(B.xa[:n], self.head, self._logits[:n])
+            N.linear(B.xa[:n], self.head, self._logits[:n], cap=self.logit_cap)
             K.sample_topk(self._logits[:n], self.fabric, top_k=1, inv_temperature=self.inv_temp[:n], scratch=self.sample_scratch, out_ids=self.next_ids[:n])
         return self.next_ids[:n]
 
@@ -155,7 +156,7 @@ class StreamRows:
         xn = torch.zeros(select.numel(), self.B.xa.shape[1], dtype=d.dtype, device=tokens.device)
         N.rms_rows(self.B.x[:m], d.final_norm, c.eps, xn, select.to(torch.int32))
         logits = torch.empty(select.numel(), c.vocab, dtype=F32, device=tokens.device)
-        N.linear(xn, d.head, logits, status_ptr=d.fabric.desc.status)
+        N.linear(xn, d.head, logits, status_ptr=d.fabric.desc.status, cap=d.logit_cap)
         return logits
 
     def forward(self, tokens: torch.Tensor, pos0: int, slot: int = 0) -> torch.Tensor:

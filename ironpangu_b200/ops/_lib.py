@@ -57,15 +57,20 @@ _SIGS = {
     "ifab_gemv_allreduce_bf16": [_P, c_long, _P, _P, c_long, _P, c_long, _P, c_int, c_int, c_int, C.POINTER(IfabFabric), _P],
     "ifab_gemm_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, _P, _P],
     "ifab_gemm_act_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P, _P],
-    "ifab_linear_f32": [_P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, _P],
-    "ifab_embed_rows": [_P, _P, c_long, c_float, _P, c_float, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, _P, _P],
-    "ifab_post_norm_add": [_P, c_long, _P, _P, c_float, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
+    "ifab_gemm_epilogue_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, _P, c_int, c_float, c_int, c_int, c_int, _P, _P],
+    "ifab_gemm_gated_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, c_float, c_float, c_int, c_int, c_int, _P, _P],
+    "ifab_linear_f32": [_P, c_long, _P, c_long, _P, c_long, _P, c_float, c_int, c_int, c_int, c_int, _P],
+    "ifab_embed_rows": [_P, _P, c_long, c_float, _P, c_float, _P, c_long, _P, _P, c_long, c_int, c_int, c_int, c_int, _P, _P],
+    "ifab_post_norm_add": [_P, c_long, _P, _P, c_float, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
+    "ifab_gated_rows": [_P, c_long, c_int, c_int, c_float, c_float, _P, c_long, c_int, c_int, c_int, _P],
+    "ifab_parallel_in_decode": [_P, c_long, _P, c_long, _P, c_float, _P, _P, c_long, _P, c_long, _P, _P, _P, c_long, c_int, _P, c_int, c_int, c_float, c_float, _P, c_long,
+                                _P, _P, c_long, _P, c_int, c_int, c_int, c_int, c_float, c_int, c_int, _P, _P, _P, c_int, c_int, _P],
     "ifab_rms_rows": [_P, c_long, _P, _P, c_float, _P, c_long, c_int, c_int, c_int, _P],
     "ifab_group_norm_gate": [_P, c_long, _P, c_float, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P],
     "ifab_gate_rows": [_P, c_long, c_int, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P],
     "ifab_gemv_post_norm": [_P, c_long, _P, _P, c_float, _P, _P, c_long, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
     "ifab_gemv_group_norm": [_P, c_long, _P, c_float, c_int, _P, c_long, c_int, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
-    "ifab_gemv_act": [_P, c_long, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
+    "ifab_gemv_act": [_P, c_long, _P, _P, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, c_int, _P],
     "ifab_la_step": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_float, _P, _P, _P, _P, _P, c_long, c_int, _P],
     "ifab_la_prepare": [_P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_float, _P, _P, _P, c_int, _P],
     "ifab_rope_table": [_P, _P, _P, c_int, c_int, _P],
@@ -73,19 +78,19 @@ _SIGS = {
                       _P, c_long, c_int, _P, c_long, c_float, _P, _P],
     "ifab_la_chunks": [_P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, _P, _P, c_u64, _P, _P, c_long, _P],
     "ifab_qk_norm_rope_write": [_P, c_long, c_int, c_int, c_int, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_int, c_int,
-                                c_int, _P, c_long, c_int, _P, _P, c_int, _P, _P],
+                                c_int, _P, c_long, c_int, _P, _P, c_int, c_int, _P, _P],
     "ifab_ctx_gather_pad": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_long, _P, _P],
     "ifab_fa_window_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                            c_float, _P, _P, c_long, c_int, c_int, _P, _P],
-    "ifab_gqa_window_attention": [_P, c_long, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int,
-                                  c_int, _P, c_u64, _P, c_long, _P, _P],
-    "ifab_window_attn": [_P, c_long, c_int, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, c_long, c_int, _P,
-                         c_long, c_int, _P, _P],
+                            c_float, c_float, _P, c_int, _P, _P, c_long, c_int, c_int, _P, _P],
+    "ifab_gqa_window_attention": [_P, c_long, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, c_float, _P, c_int, _P, _P, c_long, c_int, c_int, c_int, c_int,
+                                  c_int, c_int, c_int, c_int, _P, c_u64, _P, c_long, _P, _P],
+    "ifab_window_attn": [_P, c_long, c_int, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, _P, c_int, _P, _P,
+                         c_long, c_int, c_int, _P, c_long, c_int, _P, _P],
     "ifab_moe_down_f32_decode": [_P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, c_long, _P],
-    "ifab_moe_route": [_P, c_long, _P, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, _P, _P],
-    "ifab_moe_combine_norm": [_P, c_long, _P, _P, c_int, _P, c_long, _P, _P, _P, c_float, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
+    "ifab_moe_route": [_P, c_long, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, _P, _P, _P, _P],
+    "ifab_moe_combine_norm": [_P, c_long, _P, _P, c_int, _P, c_long, _P, _P, _P, c_float, _P, c_long, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
     "ifab_linear_f32_batched": [_P, c_long, c_long, _P, c_long, c_long, _P, c_long, c_long, c_int, c_int, c_int, c_int, _P],
-    "ifab_grouped_linear_f32": [_P, c_long, _P, c_int, _P, c_int, c_int, _P, _P, c_int, c_int, _P, c_long, _P],
+    "ifab_grouped_linear_f32": [_P, c_long, _P, c_int, c_int, c_float, c_float, _P, c_int, c_int, _P, _P, c_int, c_int, _P, c_long, _P],
     "ifab_gemm_heads_bf16": [_P, c_long, c_int, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P],
     "ifab_router_post_norm": [_P, c_long, _P, _P, c_float, _P, _P, c_long, _P, c_long, _P, _P, c_long, _P, c_int, c_int, c_int, c_int, c_float, _P, _P, _P,
                               _P, c_int, c_int, c_int, _P],
@@ -109,6 +114,7 @@ _SIGS = {
     "ifab_gemm_reduce_scatter_bf16": [_P, c_long, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, C.POINTER(IfabFabric), _P],
     "ifab_router_topk": [_P, c_long, _P, c_float, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, c_long, _P],
     "ifab_moe_gate_up_decode": [_P, c_long, _P, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, c_int, _P],
+    "ifab_moe_gate_up_unit_decode": [_P, c_long, _P, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, c_int, c_int, c_float, c_float, _P],
     "ifab_moe_down_allreduce_decode": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, c_long, _P,
                                        c_long, C.POINTER(IfabFabric), _P],
     "ifab_moe_block_decode": [_P, c_long, _P, c_float, _P, _P, c_int, c_int, c_int, c_int, c_float, _P, _P, _P, _P, c_int, c_int,
@@ -124,6 +130,8 @@ _SIGS = {
                                            c_long, C.POINTER(IfabFabric), _P],
     "ifab_lm_head_argmax": [_P, c_long, _P, c_float, _P, _P, c_int, c_int, c_int, c_int, _P, c_u64, _P, _P,
                             C.POINTER(IfabFabric), _P],
+    "ifab_lm_head_capped_argmax": [_P, c_long, _P, c_float, _P, _P, c_float, c_int, c_int, c_int, c_int, _P, c_u64, _P, _P,
+                                   C.POINTER(IfabFabric), _P],
     "ifab_sample_topk": [_P, c_long, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P, c_long, _P, _P, _P, _P, c_u64, _P, _P,
                          C.POINTER(IfabFabric), _P],
     "ifab_mla_kv_write": [_P, c_long, _P, c_float, c_float, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, _P, _P],
@@ -160,6 +168,7 @@ _SIGS = {
     "ifab_kv_dequantize_q8": [_P, _P, c_long, _P],
     "ifab_quantize_int8": [_P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
     "ifab_grouped_gemm_bf16": [_P, c_long, c_int, _P, c_int, c_int, c_int, _P, _P, c_int, _P, c_long, c_int, _P, _P],
+    "ifab_grouped_gemm_gated_bf16": [_P, c_long, c_int, _P, c_int, c_int, c_int, _P, _P, c_int, _P, c_long, c_int, c_int, c_float, c_float, _P, _P],
     "ifab_router_block": [_P, c_long, _P, c_float, _P, _P, _P, _P, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int,
                           c_float, _P],
     "ifab_moe_dispatch": [_P, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P, c_int, _P],

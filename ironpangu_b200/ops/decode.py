@@ -117,8 +117,8 @@ def router_topk(x: torch.Tensor, w_router: torch.Tensor, topk: int, *, norm_w: O
 
 def moe_gate_up(x: torch.Tensor, ids: torch.Tensor, w_gu: torch.Tensor, e0: int, *,
                 norm_w: Optional[torch.Tensor] = None, eps: float = 1e-5, w_shared_gu: Optional[torch.Tensor] = None,
-                act: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Gate/up projections + SwiGLU of the routes owned by this rank (and of the shared-expert shard).
+                act: Optional[torch.Tensor] = None, unit=None) -> torch.Tensor:
+    """Gate/up projections + SwiGLU (or ``unit``, a ``stream_norm.GatedUnit``) of the routes owned by this rank (and of the shared-expert shard).
 
     ``w_gu``: ``[E_local, 2F, D]``; ``act``: ``[T, topk+1, >= F]`` (slot ``topk`` is the shared expert, which may be wider than F)."""
     T, D = x.shape
@@ -128,9 +128,9 @@ def moe_gate_up(x: torch.Tensor, ids: torch.Tensor, w_gu: torch.Tensor, e0: int,
     Fs = 0 if w_shared_gu is None else w_shared_gu.shape[0] // 2
     if act is None:
         act = torch.zeros(T, topk + 1, F, dtype=BF16, device=x.device)
-    check(_lib.load().ifab_moe_gate_up_decode(x.data_ptr(), _rows(x), _ptr(norm_w), eps, ids.data_ptr(), T, D, F, topk,
-                                              e0, e_local, w_gu.data_ptr(), _ptr(w_shared_gu), Fs, act.data_ptr(), act.shape[2],
-                                              _stream()), "moe_gate_up")
+    check(_lib.load().ifab_moe_gate_up_unit_decode(x.data_ptr(), _rows(x), _ptr(norm_w), eps, ids.data_ptr(), T, D, F, topk,
+                                                   e0, e_local, w_gu.data_ptr(), _ptr(w_shared_gu), Fs, act.data_ptr(), act.shape[2],
+                                                   *(unit.args if unit is not None else (0, 0.0, 0.0)), _stream()), "moe_gate_up")
     return act
 
 
@@ -276,8 +276,9 @@ def moe_down_allreduce_fp8(act: torch.Tensor, ids: torch.Tensor, wts: torch.Tens
 def lm_head_argmax(x: torch.Tensor, w: torch.Tensor, fabric, *, norm_w: Optional[torch.Tensor] = None,
                    eps: float = 1e-5, vocab_offset: int = 0, partial: Optional[torch.Tensor] = None,
                    logits: Optional[torch.Tensor] = None, out_ids: Optional[torch.Tensor] = None,
-                   out_vals: Optional[torch.Tensor] = None):
-    """Vocabulary-sharded lm_head + greedy token selection (cross-rank exchange inside the kernel)."""
+                   out_vals: Optional[torch.Tensor] = None, cap: float = 0.0):
+    """Vocabulary-sharded lm_head + greedy token selection (cross-rank exchange inside the kernel). ``cap`` > 0: logits are
+    ``cap * tanh(logit / cap)``."""
     T, K = x.shape
     V = w.shape[0]
     dev = x.device
@@ -285,9 +286,9 @@ def lm_head_argmax(x: torch.Tensor, w: torch.Tensor, fabric, *, norm_w: Optional
         partial = torch.empty(((V + 7) // 8) * 8 * 2, dtype=torch.float32, device=dev)
     if out_ids is None:
         out_ids = torch.empty(T, dtype=torch.int32, device=dev)
-    check(_lib.load().ifab_lm_head_argmax(x.data_ptr(), _rows(x), _ptr(norm_w), eps, w.data_ptr(), _ptr(logits), T, V, K,
-                                          vocab_offset, partial.data_ptr(), partial.numel() * partial.element_size(),
-                                          out_ids.data_ptr(), _ptr(out_vals), C.byref(fabric.desc), _stream()),
+    check(_lib.load().ifab_lm_head_capped_argmax(x.data_ptr(), _rows(x), _ptr(norm_w), eps, w.data_ptr(), _ptr(logits), cap, T, V, K,
+                                                 vocab_offset, partial.data_ptr(), partial.numel() * partial.element_size(),
+                                                 out_ids.data_ptr(), _ptr(out_vals), C.byref(fabric.desc), _stream()),
           "lm_head_argmax")
     return out_ids
 

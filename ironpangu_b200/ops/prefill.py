@@ -23,15 +23,16 @@ def _p(t: Optional[torch.Tensor]) -> Optional[int]:
 
 
 def grouped_gemm(a: torch.Tensor, b: torch.Tensor, tiles: torch.Tensor, num_tiles: torch.Tensor, out: torch.Tensor, *,
-                 swiglu: bool = False, status_ptr: Optional[int] = None) -> torch.Tensor:
+                 swiglu: bool = False, unit=None, status_ptr: Optional[int] = None) -> torch.Tensor:
     """``out[r] = a[r] @ b[expert(r)].T`` over the 128-row tiles listed in ``tiles`` (int32 ``[max_tiles, 4]``:
-    expert, first row, valid rows, 0); with ``swiglu`` ``b`` is ``[E, 2F, K]`` and ``out`` is ``[rows, F]``."""
+    expert, first row, valid rows, 0); with ``swiglu`` ``b`` is ``[E, 2F, K]`` and ``out`` is ``[rows, F]``, with ``unit``
+    (``stream_norm.GatedUnit``) the same for another gated unit."""
     rows, K = a.shape
     E, N, Kb = b.shape
     assert Kb == K and a.stride(1) == 1 and b.is_contiguous() and out.stride(1) == 1 and tiles.dtype == torch.int32
-    check(_lib.load().ifab_grouped_gemm_bf16(a.data_ptr(), a.stride(0), rows, b.data_ptr(), E, N, K, tiles.data_ptr(),
-                                             num_tiles.data_ptr(), tiles.shape[0], out.data_ptr(), out.stride(0), int(swiglu),
-                                             status_ptr, _s()), "grouped_gemm")
+    check(_lib.load().ifab_grouped_gemm_gated_bf16(a.data_ptr(), a.stride(0), rows, b.data_ptr(), E, N, K, tiles.data_ptr(),
+                                                   num_tiles.data_ptr(), tiles.shape[0], out.data_ptr(), out.stride(0), int(swiglu or unit is not None),
+                                                   *(unit.args if unit is not None else (0, 0.0, 0.0)), status_ptr, _s()), "grouped_gemm")
     return out
 
 

@@ -3,6 +3,7 @@
 kernel. Thin wrappers: current stream, no allocation when outputs are given, no fallback."""
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -12,6 +13,30 @@ from ._lib import check
 
 BF16 = torch.bfloat16
 ACTIVATIONS = {None: 0, "silu": 1, "sigmoid": 2, "gelu_tanh": 3}
+
+
+UNITS = {"silu": 0, "relu": 1, "limited": 2}
+
+
+@dataclass(frozen=True)
+class GatedUnit:
+    """What a gated feed-forward makes of its two projections g and u: ``silu`` silu(g) u; ``relu`` relu(g) u; ``limited`` g' sigmoid(alpha g')
+    (u' + 1) with g' = min(g, limit) and u' = u within [-limit, limit]."""
+
+    kind: str = "silu"
+    limit: float = 0.0
+    alpha: float = 1.0
+
+    def check(self) -> None:
+        if self.kind not in UNITS or (self.kind == "limited" and self.limit <= 0):
+            raise ValueError(f"gated unit {self} is not supported")
+
+    @property
+    def args(self) -> tuple:
+        return UNITS[self.kind], self.limit, self.alpha
+
+
+SILU = GatedUnit()
 
 
 def _s() -> int:
@@ -28,20 +53,31 @@ def _f32(t: torch.Tensor) -> int:
 
 
 def embed_rows(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, xa: torch.Tensor, *, scale: float = 1.0, gain: Optional[torch.Tensor] = None,
-               eps: float = 0.0, status_ptr: Optional[int] = None) -> None:
-    """``x`` (f32 residual) = rows ``ids`` of ``table`` times ``scale``; ``xa`` (activation type) = x, or ``rms(x) * gain``."""
+               eps: float = 0.0, copy: Optional[torch.Tensor] = None, status_ptr: Optional[int] = None) -> None:
+    """``x`` (f32 residual) = rows ``ids`` of ``table`` times ``scale``; ``xa`` (activation type) = x, or ``rms(x) * gain``. ``copy``: a second
+    place for x."""
     T, D = x.shape
+    assert copy is None or copy.stride(0) == x.stride(0)
     assert ids.dtype == torch.int32 and x.dtype == torch.float32 and table.dtype == xa.dtype
-    check(_lib.load().ifab_embed_rows(ids.data_ptr(), table.data_ptr(), table.stride(0), scale, _p(gain), eps, x.data_ptr(), x.stride(0), xa.data_ptr(),
+    check(_lib.load().ifab_embed_rows(ids.data_ptr(), table.data_ptr(), table.stride(0), scale, _p(gain), eps, x.data_ptr(), x.stride(0), _p(copy), xa.data_ptr(),
                                       xa.stride(0), _f32(xa), T, D, table.shape[0], status_ptr, _s()), "embed_rows")
 
 
-def post_norm_add(y: torch.Tensor, w: torch.Tensor, eps: float, x: torch.Tensor, xa: torch.Tensor, final: Optional[torch.Tensor] = None) -> None:
-    """``x += rms(y) * w`` in f32; ``xa`` = x, or ``rms(x) * final`` (the norm ahead of the output matrix)."""
+def post_norm_add(y: Optional[torch.Tensor], w: Optional[torch.Tensor], eps: float, x: torch.Tensor, xa: torch.Tensor, final: Optional[torch.Tensor] = None,
+                  extra: Optional[torch.Tensor] = None) -> None:
+    """``x += rms(y) * w [+ extra]`` in f32 (``y`` as it is without ``w``, nothing without ``y``); ``xa`` = x, or ``rms(x) * final`` (the norm
+    ahead of the next linears)."""
     T, D = x.shape
-    assert y.dtype == x.dtype == w.dtype == torch.float32
-    check(_lib.load().ifab_post_norm_add(y.data_ptr(), y.stride(0), w.data_ptr(), _p(final), eps, x.data_ptr(), x.stride(0), xa.data_ptr(), xa.stride(0),
-                                         _f32(xa), T, D, _s()), "post_norm_add")
+    assert all(t is None or t.dtype == torch.float32 for t in (y, w, x, extra))
+    check(_lib.load().ifab_post_norm_add(_p(y), 0 if y is None else y.stride(0), _p(w), _p(final), eps, x.data_ptr(), x.stride(0), _p(extra),
+                                         0 if extra is None else extra.stride(0), xa.data_ptr(), xa.stride(0), _f32(xa), T, D, _s()), "post_norm_add")
+
+
+def gated_rows(gu: torch.Tensor, unit: GatedUnit, out: torch.Tensor) -> None:
+    """``out`` ``[T, F]`` = the gated unit of the halves of ``gu`` ``[T, 2 * n]`` (their first F columns)."""
+    T, F = out.shape
+    assert gu.dtype == out.dtype
+    check(_lib.load().ifab_gated_rows(gu.data_ptr(), gu.stride(0), gu.shape[1] // 2, *unit.args, out.data_ptr(), out.stride(0), _f32(out), T, F, _s()), "gated_rows")
 
 
 def rms_rows(x: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
@@ -87,22 +123,40 @@ def gemv_group_norm(o: torch.Tensor, gate: torch.Tensor, gate_act: str, eps: flo
                                            w.data_ptr(), out.data_ptr(), out.stride(0), _f32(out), 0, T, N, K, _s()), "gemv_group_norm")
 
 
-def gemv_act(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: Optional[str] = None) -> None:
-    """``out = act(x @ w.T)`` for decode rows."""
+def gemv_act(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: Optional[str] = None, bias: Optional[torch.Tensor] = None,
+             addend: Optional[torch.Tensor] = None) -> None:
+    """``out = act(x @ w.T + bias + addend)`` for decode rows; ``bias`` f32 ``[N]``, ``addend`` f32 rows (may be ``out``)."""
     T, K = x.shape
     assert w.shape[1] == K and w.is_contiguous() and x.dtype == BF16
-    check(_lib.load().ifab_gemv_act(x.data_ptr(), x.stride(0), w.data_ptr(), out.data_ptr(), out.stride(0), _f32(out), ACTIVATIONS[act], T, w.shape[0], K,
-                                    _s()), "gemv_act")
+    check(_lib.load().ifab_gemv_act(x.data_ptr(), x.stride(0), w.data_ptr(), _p(bias), _p(addend), 0 if addend is None else addend.stride(0), out.data_ptr(),
+                                    out.stride(0), _f32(out), ACTIVATIONS[act], T, w.shape[0], K, _s()), "gemv_act")
 
 
-def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: Optional[str] = None, status_ptr: Optional[int] = None) -> None:
-    """``out = act(x @ w.T)`` for any number of rows: the tensor-core GEMM for bf16 operands (bf16 or f32 result), true f32 otherwise."""
+def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: Optional[str] = None, status_ptr: Optional[int] = None,
+           bias: Optional[torch.Tensor] = None, cap: float = 0.0) -> None:
+    """``out = act(x @ w.T + bias)`` for any number of rows: the tensor-core GEMM for bf16 operands (bf16 or f32 result), true f32 otherwise.
+    ``bias``: f32 ``[N]``; ``cap`` > 0: ``cap * tanh(out / cap)`` at the end."""
     T, K = x.shape
     N = w.shape[0]
     assert w.shape[1] == K and x.dtype == w.dtype and x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() >= N)
     if x.dtype == torch.float32:
-        check(_lib.load().ifab_linear_f32(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), T, N, K, ACTIVATIONS[act], _s()),
-              "linear_f32")
+        check(_lib.load().ifab_linear_f32(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), _p(bias), cap, T, N, K,
+                                          ACTIVATIONS[act], _s()), "linear_f32")
     else:
-        check(_lib.load().ifab_gemm_act_bf16(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), _f32(out), None, 0,
-                                             ACTIVATIONS[act], T, N, K, status_ptr, _s()), "gemm_act")
+        check(_lib.load().ifab_gemm_epilogue_bf16(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), _f32(out), None, 0,
+                                                  _p(bias), ACTIVATIONS[act], cap, T, N, K, status_ptr, _s()), "gemm_epilogue")
+
+
+def gated_linear(x: torch.Tensor, w: torch.Tensor, unit: GatedUnit, out: torch.Tensor, pair: Optional[torch.Tensor] = None, status_ptr: Optional[int] = None) -> None:
+    """``out`` ``[T, F]`` = the gated unit of ``x @ gate.T`` and ``x @ up.T`` with ``w`` = [gate | up] ``[2 F, K]``: one launch for bf16; in f32 the
+    two projections go through ``pair`` ``[T, 2 F]``."""
+    T, K = x.shape
+    F = w.shape[0] // 2
+    assert w.shape == (2 * F, K) and out.shape == (T, F) and x.dtype == w.dtype == out.dtype and out.stride(1) == 1 and x.stride(1) == 1
+    if x.dtype == torch.float32:
+        linear(x, w, pair)
+        gated_rows(pair, unit, out)
+    else:
+        check(_lib.load().ifab_gemm_gated_bf16(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), *unit.args, T, F, K, status_ptr,
+                                               _s()), "gemm_gated")

@@ -1,37 +1,45 @@
-"""Sliding-window softmax attention with sinks over paged keys / values (``csrc/kernels/window_attn.cu``)."""
+"""Softmax attention over a window or a chunk of paged keys / values, with sinks, score caps, distance biases and output gates
+(``csrc/kernels/window_attn.cu``, ``decode_gqa.cu``, ``fa_prefill.cu``), and a grouped-query attention layer over them.
+
+The mask: the last ``window`` positions (0: all), or with ``chunked`` the positions of the query's own stretch of ``window``, counted from
+position 0 of the sequence. A score is ``q k scale``, with ``cap`` > 0 ``cap * tanh(score / cap)``, and with ``slopes`` (f32 ``[heads]``) less
+``slope * (distance of the key)``. A gate has a value per column of the result, or one per head (``gate_head``)."""
 from __future__ import annotations
 
-from typing import Optional
+from dataclasses import dataclass
+from typing import Dict, Optional
 
 import torch
 
 from . import _lib
+from . import stream_norm as N
 from ._lib import check
 from .stream_norm import ACTIVATIONS, _f32, _p, _s
 
 
 def qk_norm_rope_write(proj: torch.Tensor, offsets, q_gain: Optional[torch.Tensor], k_gain: Optional[torch.Tensor], eps: float, *, heads: int, kv_heads: int,
                        dim: int, vdim: int, rot: int, interleaved: bool, rope: Optional[torch.Tensor], positions: torch.Tensor, slots: torch.Tensor,
-                       page_table: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, status_ptr=None) -> None:
+                       page_table: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, whole: bool = False, status_ptr=None) -> None:
     """Packed projection rows -> normalised, rotated queries in ``q_out`` (``[T, heads * stride]``, stride >= dim) and normalised, rotated keys / plain values in the pages
     (``k_cache`` ``[pages, page_tokens, kv_heads, dim]``, ``v_cache`` ``[..., vdim]``). ``rope``: (cos, sin) of the rows, ``[T, rot / 2, 2]``
-    (``linear_attn.RotaryTables``)."""
+    (``linear_attn.RotaryTables``). The norm is per head with one gain of ``dim`` columns, or with ``whole`` over all columns of q and all of k,
+    with a gain for each. ``offsets``: where q, k and v start in a row (v may be k)."""
     pages, pt = k_cache.shape[:2]
     check(_lib.load().ifab_qk_norm_rope_write(proj.data_ptr(), proj.stride(0), _f32(proj), *offsets, _p(q_gain), _p(k_gain), eps, heads, kv_heads, dim, vdim, rot,
                                               int(interleaved), _p(rope), positions.data_ptr(), slots.data_ptr(), page_table.data_ptr(), page_table.shape[1],
-                                              pt, pages, q_out.data_ptr(), q_out.stride(0), q_out.shape[1] // heads, k_cache.data_ptr(), v_cache.data_ptr(), proj.shape[0], status_ptr,
+                                              pt, pages, q_out.data_ptr(), q_out.stride(0), q_out.shape[1] // heads, k_cache.data_ptr(), v_cache.data_ptr(), int(whole), proj.shape[0], status_ptr,
                                               _s()), "qk_norm_rope_write")
 
 
 def window_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, page_table: torch.Tensor, *,
                 heads: int, window: int, scale: float, out: torch.Tensor, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                gate_act: Optional[str] = None, status_ptr=None) -> None:
-    """Rows of any sequences: row at position i attends keys j with 0 <= i - j < window (0: all), exp(sink) joins the denominator,
-    the result is multiplied by ``gate_act(gate)``."""
+                gate_act: Optional[str] = None, gate_head: bool = False, chunked: bool = False, cap: float = 0.0, slopes: Optional[torch.Tensor] = None,
+                status_ptr=None) -> None:
+    """Rows of any sequences, any head sizes: exp(sink) joins the denominator, the result is multiplied by ``gate_act(gate)``."""
     pages, pt, G, d = k_cache.shape
     check(_lib.load().ifab_window_attn(q.data_ptr(), q.stride(0), q.shape[1] // heads, k_cache.data_ptr(), v_cache.data_ptr(), _f32(q), positions.data_ptr(), slots.data_ptr(),
-                                       page_table.data_ptr(), page_table.shape[1], pt, pages, heads, G, d, v_cache.shape[3], window, scale, _p(sink), _p(gate),
-                                       0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], out.data_ptr(), out.stride(0), q.shape[0], status_ptr,
+                                       page_table.data_ptr(), page_table.shape[1], pt, pages, heads, G, d, v_cache.shape[3], window, scale, cap, _p(slopes), int(chunked), _p(sink), _p(gate),
+                                       0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], int(gate_head), out.data_ptr(), out.stride(0), q.shape[0], status_ptr,
                                        _s()), "window_attn")
 
 
@@ -48,15 +56,16 @@ def split_form(heads: int, kv_heads: int, dim: int, vdim: int, window: int) -> i
 
 def gqa_window(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, page_table: torch.Tensor, *,
                heads: int, window: int, scale: float, splits: int, scratch: torch.Tensor, out: torch.Tensor, sink: Optional[torch.Tensor] = None,
-               gate: Optional[torch.Tensor] = None, gate_act: Optional[str] = None, status_ptr=None) -> None:
+               gate: Optional[torch.Tensor] = None, gate_act: Optional[str] = None, gate_head: bool = False, chunked: bool = False, cap: float = 0.0,
+               slopes: Optional[torch.Tensor] = None, status_ptr=None) -> None:
     """:func:`window_attn` by splits of the window (query heads of a group share the key loads), bf16, shapes of :func:`split_form`.
     ``splits``: the most to use; launches of many rows use fewer, longer ones."""
     pages, pt, G, d = k_cache.shape
     splits = max(1, min(splits, SPLIT_CTAS // (q.shape[0] * G)))
     kps = ((window + splits - 1) // splits + 31) // 32 * 32
     check(_lib.load().ifab_gqa_window_attention(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), positions.data_ptr(), slots.data_ptr(),
-                                                page_table.data_ptr(), page_table.shape[1], pt, pages, scale, window, _p(sink), _p(gate),
-                                                0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], q.shape[0], heads, G, d, kps, splits,
+                                                page_table.data_ptr(), page_table.shape[1], pt, pages, scale, window, cap, _p(slopes), int(chunked), _p(sink), _p(gate),
+                                                0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], int(gate_head), q.shape[0], heads, G, d, kps, splits,
                                                 scratch.data_ptr(), scratch.numel() * 4, out.data_ptr(), out.stride(0), status_ptr, _s()), "gqa_window")
 
 
@@ -72,14 +81,15 @@ def context_rows(count: int, window: int) -> int:
 
 def fa_window(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor, *, slot: int, pos0: int, heads: int, window: int,
               scale: float, ctx_k: torch.Tensor, ctx_vt: torch.Tensor, out: torch.Tensor, sink: Optional[torch.Tensor] = None,
-              gate: Optional[torch.Tensor] = None, gate_act: Optional[str] = None, status_ptr=None) -> None:
+              gate: Optional[torch.Tensor] = None, gate_act: Optional[str] = None, gate_head: bool = False, chunked: bool = False, cap: float = 0.0,
+              slopes: Optional[torch.Tensor] = None, status_ptr=None) -> None:
     """Prompt attention of consecutive positions ``pos0 ..`` of one sequence (keys already in its pages) on the tensor cores: the keys
     and values the rows can see are gathered out of the pages into ``ctx_k`` ``[rows, kv_heads * tile]`` / ``ctx_vt`` ``[kv_heads * 128,
     rows]``. ``q``: ``[m, heads * tile]``, columns past the head width zero; ``window`` 0: the whole context."""
     pages, pt, G, d = k_cache.shape
     m, e = q.shape[0], v_cache.shape[3]
     dp = q.shape[1] // heads
-    first = max(0, pos0 - window + 1) if window else 0
+    first = 0 if not window else pos0 // window * window if chunked else max(0, pos0 - window + 1)
     n = pos0 + m - first
     rows = (n + 31) // 32 * 32
     assert dp == tile_width(d) and e <= 128 and ctx_k.shape[0] >= rows and ctx_vt.shape[1] >= rows and ctx_k.shape[1] == G * dp
@@ -87,5 +97,141 @@ def fa_window(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, pag
     check(lib.ifab_ctx_gather_pad(k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr(), slot, page_table.shape[1], pt, pages, first, n, rows, G, d,
                                   dp, e, ctx_k.data_ptr(), ctx_vt.data_ptr(), ctx_vt.stride(0), status_ptr, _s()), "ctx_gather_pad")
     check(lib.ifab_fa_window_bf16(q.data_ptr(), q.stride(0), ctx_k.data_ptr(), ctx_k.stride(0), None, 0, 0, ctx_vt.data_ptr(), ctx_vt.stride(0), out.data_ptr(),
-                                  out.stride(0), m, n, heads, heads // G, dp, e, pos0 - first, window, scale, _p(sink), _p(gate),
-                                  0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], 0, status_ptr, _s()), "fa_window")
+                                  out.stride(0), m, n, heads, heads // G, dp, e, pos0 - first, window, scale, cap, _p(slopes), int(chunked), _p(sink), _p(gate),
+                                  0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], int(gate_head), status_ptr, _s()), "fa_window")
+
+
+# ---------------------------------------------------------------------------------------------------------------------------
+# a grouped-query attention layer
+# ---------------------------------------------------------------------------------------------------------------------------
+@dataclass(frozen=True)
+class GroupedShape:
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int = 0                # 0: no mask but the causal one
+    chunked: bool = False
+    cap: float = 0.0               # soft limit of the scores
+    biased: bool = False           # distance bias with slope 2^(-8 (h + 1) / heads)
+    rot_dims: int = 0              # rotated columns of a head, interleaved pairs
+    rot_base: float = 10000.0
+    norm: bool = False             # rms of all of q and of all of k before the rotation
+    keys_are_values: bool = False  # values = keys as projected
+    bias: bool = False             # of the q, k and output projections
+
+    def check(self) -> None:
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
+            raise ValueError(f"attention: {self.heads} heads over {self.kv_heads} key / value heads are not supported")
+        if max(self.dim, self.vdim) > 256 or (self.keys_are_values and self.dim != self.vdim):
+            raise ValueError(f"attention: heads of {self.dim} / {self.vdim} columns are not supported")
+        if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.dim:
+            raise ValueError(f"attention: rotation of {self.rot_dims} columns in heads of {self.dim}")
+        if self.window < 0 or self.cap < 0:
+            raise ValueError("attention: window and cap must not be negative")
+
+    @property
+    def offsets(self) -> tuple:
+        """Where q, k, v and the head gates start in a projection row, and where it ends."""
+        q, k = self.heads * self.dim, self.kv_heads * self.dim
+        v = 0 if self.keys_are_values else self.kv_heads * self.vdim
+        return 0, q, q if self.keys_are_values else q + k, q + k + v, q + k + v + self.heads
+
+    @property
+    def in_cols(self) -> int:
+        """Columns of the packed projection, filled up to whole stores of the GEMMs."""
+        return (self.offsets[4] + 31) // 32 * 32
+
+    @property
+    def tiles(self) -> bool:
+        return max(self.dim, self.vdim) <= 128
+
+    @property
+    def q_stride(self) -> int:
+        return tile_width(self.dim) if self.tiles else self.dim
+
+    @property
+    def splits(self) -> int:
+        return split_form(self.heads, self.kv_heads, self.dim, self.vdim, self.window) if self.q_stride == self.dim else 0
+
+    @property
+    def row(self) -> int:
+        """Elements a token holds in the pages."""
+        return self.kv_heads * (self.dim + self.vdim)
+
+
+class GroupedBuffers:
+    """Work buffers of the grouped attention layers of a model for up to ``rows`` rows; ``chunked``: for packed steps."""
+
+    def __init__(self, shapes, rows: int, dtype: torch.dtype, device, *, chunked: bool, max_context: int, group: int):
+        self.group = group
+        z = lambda *s: torch.zeros(*s, dtype=dtype, device=device)
+        self.proj = z(rows, max(s.in_cols for s in shapes))
+        # queries at the stride of the tensor-core tiles where they have one (padding columns stay zero: one buffer per shape)
+        self.q = {(s.heads, s.q_stride, s.dim): z(rows, s.heads * s.q_stride) for s in shapes}
+        need = [s.heads * s.splits * (s.vdim + 2) for s in shapes if s.splits]
+        self.scratch = torch.empty(min(rows, group) * max(need), dtype=torch.float32, device=device) if need and dtype == torch.bfloat16 else None
+        self.ctx = {}
+        if chunked and dtype == torch.bfloat16:
+            for s in shapes:
+                cap = (max_context + 31) // 32 * 32
+                if s.window:
+                    cap = min(cap, context_rows(rows, s.window))
+                key = (s.kv_heads, s.q_stride)
+                if s.tiles and (key not in self.ctx or self.ctx[key][0].shape[0] < cap):
+                    self.ctx[key] = z(cap, s.kv_heads * s.q_stride), z(s.kv_heads * 128, cap)
+
+
+class GroupedAttention:
+    """One grouped-query attention layer with a gate per head: its weights in the layouts the kernels take, and the launches between the
+    packed input projection and the operand of the output projection. The output matrix (``W[p + "o"]``) is the caller's."""
+
+    def __init__(self, shape: GroupedShape, W: Dict[str, torch.Tensor], p: str, device, dtype: torch.dtype):
+        """``W[p + name]`` for q, k, v (unless the keys are the values), g, with biases q.b, k.b and with norms q.norm, k.norm."""
+        s = shape
+        self.shape = s
+        get = lambda n: W[p + n].to(device)
+        mats = [get(n).to(dtype) for n in ("q", "k") + (() if s.keys_are_values else ("v",)) + ("g",)]
+        width = mats[0].shape[1]
+        self.w_in = torch.zeros(s.in_cols, (width + 7) // 8 * 8, dtype=dtype, device=device)
+        self.w_in[:s.offsets[4], :width] = torch.cat(mats, 0)
+        self.b_in = None
+        if s.bias:
+            self.b_in = torch.zeros(s.in_cols, dtype=torch.float32, device=device)
+            self.b_in[:s.offsets[1] + s.kv_heads * s.dim] = torch.cat([get("q.b"), get("k.b")]).float()
+        vec = lambda n: get(n).float().contiguous() if s.norm else None
+        self.q_gain, self.k_gain = vec("q.norm"), vec("k.norm")
+        self.slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / s.heads) for h in range(s.heads)], dtype=torch.float32, device=device) if s.biased else None
+
+    def make_pages(self, pages: int, page_tokens: int, device, dtype: torch.dtype) -> tuple:
+        s = self.shape
+        z = lambda n: torch.zeros(pages, page_tokens, s.kv_heads, n, dtype=dtype, device=device)
+        return z(s.dim), z(s.vdim)
+
+    def project(self, B: GroupedBuffers, xa: torch.Tensor, status_ptr) -> None:
+        N.linear(xa, self.w_in, B.proj[:xa.shape[0], :self.shape.in_cols], bias=self.b_in, status_ptr=status_ptr)
+
+    def attend(self, B: GroupedBuffers, m: int, pages: tuple, rope, pos, slot, plan, table, eps: float, out: torch.Tensor, status_ptr) -> None:
+        """``m`` rows of a packed step (``plan``), or decode rows (None), from ``B.proj`` to ``out`` ``[m, >= heads * vdim]``."""
+        s = self.shape
+        proj, q, bf16 = B.proj[:m], B.q[s.heads, s.q_stride, s.dim][:m], B.proj.dtype == torch.bfloat16
+        qo, ko, vo, go, _ = s.offsets
+        qk_norm_rope_write(proj, (qo, ko, vo), self.q_gain, self.k_gain, eps, heads=s.heads, kv_heads=s.kv_heads, dim=s.dim, vdim=s.vdim, rot=s.rot_dims,
+                           interleaved=True, rope=rope, positions=pos, slots=slot, page_table=table, q_out=q, k_cache=pages[0], v_cache=pages[1], whole=s.norm,
+                           status_ptr=status_ptr)
+        gate = proj[:, go:]
+        how = dict(heads=s.heads, window=s.window, scale=s.scale, gate_act="sigmoid", gate_head=True, chunked=s.chunked, cap=s.cap, slopes=self.slopes,
+                   status_ptr=status_ptr)
+        tiled = plan is not None and bool(plan.runs) and s.tiles and bf16
+        if tiled:
+            k, vt = B.ctx[s.kv_heads, s.q_stride]
+            for r, n, sl, p0 in plan.runs:
+                fa_window(q[r:r + n], *pages, table, slot=sl, pos0=p0, ctx_k=k, ctx_vt=vt, out=out[r:r + n], gate=gate[r:r + n], **how)
+        groups = plan.groups if tiled else [(r, min(m, r + B.group)) for r in range(0, m, B.group)]
+        rest = plan.step_positions if tiled else pos
+        if s.splits and bf16:
+            for lo, hi in groups:
+                gqa_window(q[lo:hi], *pages, rest[lo:hi], slot[lo:hi], table, splits=s.splits, scratch=B.scratch, out=out[lo:hi], gate=gate[lo:hi], **how)
+        elif groups:
+            window_attn(q, *pages, rest, slot, table, out=out, gate=gate, **how)

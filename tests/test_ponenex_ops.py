@@ -75,7 +75,7 @@ def test_router_selection_from_logits(experts, top):
     zd, bd = z.cuda(), b.cuda()
     ids, wts, sw = (torch.zeros(M, top, dtype=t, device="cuda") for t in (torch.int32, F32, F32))
     sw = torch.zeros(M, device="cuda")
-    rc = _lib.load().ifab_moe_route(zd.data_ptr(), experts + 1, bd.data_ptr(), M, experts, top, 2, 1, 1.0, ids.data_ptr(), wts.data_ptr(), sw.data_ptr(), _s())
+    rc = _lib.load().ifab_moe_route(zd.data_ptr(), experts + 1, bd.data_ptr(), M, experts, top, 2, 1, 1.0, 1, 1, ids.data_ptr(), wts.data_ptr(), sw.data_ptr(), _s())
     assert rc == 0
     best, want = (z[:, :experts] + b).sort(dim=-1, descending=True, stable=True)
     assert torch.equal(ids.cpu().long(), want[:, :top])
