@@ -117,10 +117,9 @@ def limited_unit(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, limit: flo
     return (g * torch.sigmoid(1.702 * g) * (u + (0.0 if "up_without_one" in faults else 1.0))) @ w[p + "down"].T
 
 
-def route(h: torch.Tensor, w_router: torch.Tensor, correction: torch.Tensor, top: int, count: int, keep: int, faults=()):
-    """``(ids, weights)`` ``[T, top]``: experts chosen by sigmoid score + correction among the ``keep`` best of ``count`` groups (a group is as
-    good as its two best together), weighted by the score alone."""
-    s = torch.sigmoid(h @ w_router.T)
+def choose(s: torch.Tensor, correction: torch.Tensor, top: int, count: int, keep: int, faults=()):
+    """``(ids, weights)`` ``[T, top]``: experts chosen by score + correction among the ``keep`` best of ``count`` groups (a group is as good as its
+    two best together), weighted by the score alone."""
     c = s if "no_correction" in faults else s + correction
     if "all_groups" not in faults:
         T, E = c.shape
@@ -132,6 +131,10 @@ def route(h: torch.Tensor, w_router: torch.Tensor, correction: torch.Tensor, top
     ids = c.sort(dim=-1, descending=True, stable=True).indices[:, :top]
     wts = (c if "weights_with_correction" in faults else s).gather(1, ids)
     return ids, wts / wts.sum(-1, keepdim=True) if "weights_renormed" in faults else wts
+
+
+def route(h: torch.Tensor, w_router: torch.Tensor, correction: torch.Tensor, top: int, count: int, keep: int, faults=()):
+    return choose(torch.sigmoid(h @ w_router.T), correction, top, count, keep, faults)
 
 
 def experts(h: torch.Tensor, m: dict, w: Dict[str, torch.Tensor], p: str, faults=()) -> torch.Tensor:
