@@ -83,6 +83,9 @@ int ifab_gemm_epilogue_bf16(const void* a, long lda, const void* b, long ldb, vo
                             int act, float cap, int M, int N, int K, uint32_t* status, void* stream);
 int ifab_gemm_epilogue_bf16_2sm(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int out_f32, const void* residual, long ldr,
                                 const float* bias, int act, float cap, int persistent, int M, int N, int K, uint32_t* status, void* stream);
+/* f32 parts of A * B^T + bias along K for M <= 128 rows, part_stride apart; their sum is the product */
+int ifab_gemm_split_bf16(const void* a, long lda, const void* b, long ldb, float* c, long ldc, long part_stride, int parts, const float* bias, int M, int N, int K,
+                         uint32_t* status, void* stream);
 /* first half of a gated feed-forward, any number of rows: b = [gate rows | up rows] ([2F, K]), c[M, F] = unit(a gate^T, a up^T). Units: 0 silu(g) u,
  * 1 relu(g) u, 2 g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = u within [-limit, limit] */
 int ifab_gemm_gated_bf16(const void* a, long lda, const void* b, long ldb, void* c, long ldc, int unit, float limit, float alpha, int M, int F, int K,
@@ -199,11 +202,11 @@ int ifab_moe_down_f32_decode(const void* act, int ldact, const int32_t* ids, con
 /* routed experts of decoders with an f32 residual (moe_rows.cu): logits f32 [M, ld] (column E: the shared expert's gate, used when shared_w is given) ->
  * ids, wts [M, topk]; scoring 0 softmax, 1 sigmoid, 2 logit + bias selected, softmax over the chosen, 3 sigmoid + bias selected, sigmoid (over the sum with
  * renorm); of `groups` groups of neighbours only the `keep` best are open (moe_select.cuh). combine_norm: y = weighted sum of the permuted rows
- * (+ shared_w * shared), x += rms(y) * w (without w: y + base) (+ extra), xa = rms(x) * w2 (x without w2) */
+ * (+ shared_w * shared), x += rms(y) * w (without w: y + base, a sum of parts) (+ extra), xa = rms(x) * w2 (x without w2) */
 int ifab_moe_route(const float* logits, long ld, const float* bias, int M, int E, int topk, int scoring, int renorm, float scale, int groups, int keep, int32_t* ids,
                    float* wts, float* shared_w, void* stream);
 int ifab_moe_combine_norm(const void* y, long ldy, const int32_t* route_row, const float* wts, int topk, const void* shared, long lds, const float* shared_w,
-                          const float* w, const float* w2, float eps, const float* base, long ldb, const float* extra, long lde, float* x, long ldx, void* xa,
+                          const float* w, const float* w2, float eps, const float* base, long ldb, int parts, long part_stride, const float* extra, long lde, float* x, long ldx, void* xa,
                           long lda, int f32, int M, int D, void* stream);
 int ifab_moe_down_allreduce_decode(const void* act, const int32_t* ids, const float* wts, int T, int D, int F, int topk,
                                    int e0, int e_local, const void* w_down, const void* w_shared_down, int Fs,
@@ -303,8 +306,8 @@ int ifab_delta_rule_decode(const void* q, const void* k, const void* v, const fl
 /* x = table[id] * scale (and once more to copy, when given); xa = x, or rms(x) * w when w is given */
 int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, float scale, const float* w, float eps, float* x, long ldx, float* copy, void* xa, long lda,
                     int f32, int T, int D, int vocab, uint32_t* status, void* stream);
-/* x += rms(y) * w (y without w, nothing without y) (+ extra); xa = x, or rms(x) * w2 when w2 is given */
-int ifab_post_norm_add(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, const float* extra, long lde, void* xa, long lda,
+/* x += rms(y) * w (y without w, nothing without y) (+ extra), y the sum of `parts` rows part_stride apart; xa = x, or rms(x) * w2 when w2 is given */
+int ifab_post_norm_add(const float* y, long ldy, int parts, long part_stride, const float* w, const float* w2, float eps, float* x, long ldx, const float* extra, long lde, void* xa, long lda,
                        int f32, int T, int D, void* stream);
 /* y [T, F] = gated unit of gu[:, c] and gu[:, up + c] */
 int ifab_gated_rows(const void* gu, long ld, int up, int unit, float limit, float alpha, void* y, long ldy, int f32, int T, int F, void* stream);

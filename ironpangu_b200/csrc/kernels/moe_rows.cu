@@ -5,7 +5,8 @@
 //                            expert's weight sigmoid(logits[:, E]) when the logits carry that column
 //   moe_combine_norm_kernel  y = sum of the chosen experts' rows by weight + shared weight * shared row (f32, slot order); then the
 //                            residual update x += rms(y) * w and the next operand xa = rms(x) * w2 (or x). Without w, y is added
-//                            as it is, together with f32 rows `base` (what ran beside the experts) and `extra`
+//                            as it is, together with f32 rows `base` (what ran beside the experts, perhaps in parts of a
+//                            sum) and `extra`
 #include "moe_select.cuh"
 #include "rope.cuh"
 #include "ifab_kernels.h"
@@ -54,6 +55,7 @@ struct CombineNormParams {
   const float *w, *w2; float eps;
   float* x; long ldx; void* xa; long lda;
   const float *base, *extra; long ldb, lde;      // rows of the residual update (without w), or null
+  int parts; long part_stride;           // of base
   int D, Dp;                             // Dp: D padded to 4 columns; the padding of every operand is zero
 };
 
@@ -110,10 +112,16 @@ __global__ void __launch_bounds__(256) moe_combine_norm_kernel(CombineNormParams
       float r[4];
       load4(xr + c, r);
       if (p.base) {
-        float f[4];
-        load4(p.base + (long)m * p.ldb + c, f);
+        float b[4];
+        load4(p.base + (long)m * p.ldb + c, b);
+        for (int q = 1; q < p.parts; ++q) {
+          float f[4];
+          load4(p.base + q * p.part_stride + (long)m * p.ldb + c, f);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) v[i][j] += f[j];
+          for (int j = 0; j < 4; ++j) b[j] += f[j];
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[i][j] += b[j];
       }
       if (p.extra) {
         float f[4];
@@ -161,12 +169,12 @@ extern "C" int ifab_moe_route(const float* logits, long ld, const float* bias, i
 }
 
 extern "C" int ifab_moe_combine_norm(const void* y, long ldy, const int32_t* route_row, const float* wts, int topk, const void* shared, long lds,
-                                     const float* shared_w, const float* w, const float* w2, float eps, const float* base, long ldb, const float* extra, long lde,
+                                     const float* shared_w, const float* w, const float* w2, float eps, const float* base, long ldb, int parts, long part_stride, const float* extra, long lde,
                                      float* x, long ldx, void* xa, long lda, int f32, int M, int D, void* stream) {
   const int Dp = (D + 3) / 4 * 4;
   if (M < 1 || D < 1 || topk < 1 || topk > MAX_TOPK || ldy % 4 || ldx % 4 || lda % 4 || (shared && lds % 4) || ldy < Dp || ldx < Dp || lda < Dp || (shared && lds < Dp))
     return -1;
-  if ((w && base) || (base && (ldb % 4 || ldb < Dp)) || (extra && (lde % 4 || lde < Dp))) return -1;
-  CombineNormParams p{y, ldy, route_row, wts, topk, shared, lds, shared_w, w, w2, eps, x, ldx, xa, lda, base, extra, ldb, lde, D, Dp};
+  if ((w && base) || (base && (ldb % 4 || ldb < Dp || parts < 1 || part_stride % 4)) || (extra && (lde % 4 || lde < Dp))) return -1;
+  CombineNormParams p{y, ldy, route_row, wts, topk, shared, lds, shared_w, w, w2, eps, x, ldx, xa, lda, base, extra, ldb, lde, parts, part_stride, D, Dp};
   return f32 ? combine<float>(p, M, (cudaStream_t)stream) : combine<bf16>(p, M, (cudaStream_t)stream);
 }

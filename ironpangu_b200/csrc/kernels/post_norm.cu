@@ -4,7 +4,8 @@
 //                          when a gain is given (the norm ahead of the first sublayer); a second f32 copy on request
 //   post_norm_add_kernel   x += rms(y) * w; copy in the activation type (of rms(x) * w2 when a second gain is given: the norm ahead
 //                          of the output matrix). y is the f32 output of the sublayer's last linear; without w
-//                          it is added as it is, without y nothing is; rows of `extra` join the update
+//                          it is added as it is, without y nothing is; rows of `extra` join the update. y may
+//                          come in parts of a sum
 //   rms_rows_kernel        rms(x[row]) * w of selected rows, in the activation type (the norm ahead of the output matrix)
 //   group_norm_gate_kernel (o / rms of each group of columns [* w]) * act(gate): the normalised, gated heads of a recurrent
 //                          mixer. group = one head without a gain, or all heads together with one
@@ -52,7 +53,7 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(const int32_t* ids, con
 
 // one CTA per row
 template <typename A>
-__global__ void __launch_bounds__(256) post_norm_add_kernel(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx,
+__global__ void __launch_bounds__(256) post_norm_add_kernel(const float* y, long ldy, int parts, long part_stride, const float* w, const float* w2, float eps, float* x, long ldx,
                                                             const float* extra, long lde, A* xa, long lda, int D) {
   __shared__ float red[33];
   grid_dep_launch();
@@ -62,7 +63,7 @@ __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* y, long
   const float* er = extra ? extra + (long)t * lde : nullptr;
   float* xr = x + (long)t * ldx;
   A* ar = xa + (long)t * lda;
-  if (D % 4 == 0 && ldy % 4 == 0 && ldx % 4 == 0 && lda % 4 == 0 && lde % 4 == 0 && D <= 256 * 16) {     // the row stays in registers between the passes
+  if (D % 4 == 0 && ldy % 4 == 0 && ldx % 4 == 0 && lda % 4 == 0 && lde % 4 == 0 && part_stride % 4 == 0 && D <= 256 * 16) {     // the row stays in registers between the passes
     float4 v[4], r[4], g[4];
     float ss = 0.f;
 #pragma unroll
@@ -73,6 +74,13 @@ __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* y, long
       g[i] = make_float4(1.f, 1.f, 1.f, 1.f);
       if (c < D) {
         if (yr) v[i] = *reinterpret_cast<const float4*>(yr + c);
+        for (int q = 1; q < parts; ++q) {
+          const float4 a = *reinterpret_cast<const float4*>(yr + q * part_stride + c);
+          v[i].x += a.x;
+          v[i].y += a.y;
+          v[i].z += a.z;
+          v[i].w += a.w;
+        }
         r[i] = *reinterpret_cast<const float4*>(xr + c);
         if (w) g[i] = *reinterpret_cast<const float4*>(w + c);
         if (er) {
@@ -115,13 +123,21 @@ __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* y, long
     return;
   }
   float ss = 0.f;
+  auto value = [&](int c) {
+    float v = yr[c];
+    for (int q = 1; q < parts; ++q) v += yr[q * part_stride + c];
+    return v;
+  };
   if (yr && w)
-    for (int c = threadIdx.x; c < D; c += blockDim.x) ss += yr[c] * yr[c];
+    for (int c = threadIdx.x; c < D; c += blockDim.x) {
+      const float v = value(c);
+      ss += v * v;
+    }
   const float inv = yr && w ? 1.f / sqrtf(block_sum(ss, red) / (float)D + eps) : 1.f;
   ss = 0.f;
   for (int c = threadIdx.x; c < D; c += blockDim.x) {
     float v = xr[c] + (er ? er[c] : 0.f);
-    if (yr) v += yr[c] * inv * (w ? w[c] : 1.f);
+    if (yr) v += value(c) * inv * (w ? w[c] : 1.f);
     xr[c] = v;
     ss += v * v;
     if (!w2) ar[c] = from_f32<A>(v);
@@ -212,12 +228,14 @@ extern "C" int ifab_embed_rows(const int32_t* ids, const void* table, long ldt, 
              : embed<bf16>(ids, table, ldt, scale, w, eps, x, ldx, copy, xa, lda, T, D, vocab, status, s);
 }
 
-extern "C" int ifab_post_norm_add(const float* y, long ldy, const float* w, const float* w2, float eps, float* x, long ldx, const float* extra, long lde, void* xa,
+// y: the sum of `parts` rows, part_stride elements apart
+extern "C" int ifab_post_norm_add(const float* y, long ldy, int parts, long part_stride, const float* w, const float* w2, float eps, float* x, long ldx, const float* extra, long lde, void* xa,
                                   long lda, int f32, int T, int D, void* stream) {
-  if (T < 1 || D < 1) return -1;
+  if (T < 1 || D < 1 || parts < 1) return -1;
+  if (!y) parts = 1;
   cudaStream_t s = (cudaStream_t)stream;
-  return f32 ? launch_chain(post_norm_add_kernel<float>, dim3(T), dim3(256), 0, s, y, ldy, w, w2, eps, x, ldx, extra, lde, (float*)xa, lda, D)
-             : launch_chain(post_norm_add_kernel<bf16>, dim3(T), dim3(256), 0, s, y, ldy, w, w2, eps, x, ldx, extra, lde, (bf16*)xa, lda, D);
+  return f32 ? launch_chain(post_norm_add_kernel<float>, dim3(T), dim3(256), 0, s, y, ldy, parts, part_stride, w, w2, eps, x, ldx, extra, lde, (float*)xa, lda, D)
+             : launch_chain(post_norm_add_kernel<bf16>, dim3(T), dim3(256), 0, s, y, ldy, parts, part_stride, w, w2, eps, x, ldx, extra, lde, (bf16*)xa, lda, D);
 }
 
 // y [T, F] = unit(gu[:, c], gu[:, up + c])

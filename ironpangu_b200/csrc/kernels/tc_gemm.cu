@@ -9,6 +9,7 @@
 //               add the bias / residual, activation or soft limit, store bf16 or f32
 // Gated form: B holds gate rows [0, F) and up rows [F, 2 F); a tile's accumulator takes BN / 2 of each (two boxes per stage) and the
 // epilogue stores the gated unit's value (rope.cuh), so that a feed-forward's first half is one launch for any number of rows.
+// Split form: a product of one tile row with few columns spreads its K over blockIdx.z; its reader adds the parts in their order.
 // A and B are both K-major ("NT"), which is how activations [tokens, K] and weights [out, K] are
 // stored everywhere in this library, so no transposes are needed. M, N and K tails are handled by
 // TMA zero fill plus masked stores. Used for prefill chunks and batched decode (M >= 16); the
@@ -36,6 +37,8 @@ struct GemmParams {
   const float* bias;     // [N] or null
   float cap;             // > 0: the result is cap tanh(result / cap)
   int F; GatedUnit unit; // gated form: output columns (N = 2 F)
+  int k_blocks;          // > 0: CTAs of blockIdx.z take that many K blocks each and write f32 parts of the sum, part_stride apart
+  long part_stride;
 };
 
 // store 32 consecutive columns of one row (values already final)
@@ -101,11 +104,17 @@ __global__ void __launch_bounds__(192) tc_gemm_kernel(const __grid_constant__ CU
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   constexpr int NOUT = GATED ? BN / 2 : BN;
   const int m0 = blockIdx.y * BM, n0 = blockIdx.x * NOUT;
-  const int num_kb = (p.K + BK - 1) / BK;
+  int num_kb = (p.K + BK - 1) / BK, k_first = 0;
+  if (p.k_blocks > 0) {
+    k_first = blockIdx.z * p.k_blocks;
+    num_kb = min(p.k_blocks, num_kb - k_first);
+    p.c = reinterpret_cast<float*>(p.c) + blockIdx.z * p.part_stride;
+    if (blockIdx.z) p.bias = nullptr;
+  }
   grid_dep_launch();
   grid_dep_wait();
   if (warp == 0 && lane == 0) {
-    pipe.produce(&tmap_a, &tmap_b, num_kb, m0, n0, -1, p.spin_limit, p.status, GATED ? p.F + n0 : -1, p.a_rows);
+    pipe.produce(&tmap_a, &tmap_b, num_kb, m0, n0, -1, p.spin_limit, p.status, GATED ? p.F + n0 : -1, p.a_rows, 0, k_first);
   } else if (warp == 1 && lane == 0) {
     pipe.mma(num_kb, p.spin_limit, p.status);
   } else if (warp >= 2) {
@@ -140,7 +149,8 @@ int launch(const CUtensorMap& ta, const CUtensorMap& tb, const GemmParams& p, cu
   constexpr int smem = Cfg<BN, ST>::SMEM;
   if (int rc = opt_in_smem(k, smem)) return rc;
   constexpr int NOUT = GATED ? BN / 2 : BN;
-  dim3 grid(((GATED ? p.F : p.N) + NOUT - 1) / NOUT, (p.M + BM - 1) / BM);
+  const int parts = p.k_blocks > 0 ? ((p.K + BK - 1) / BK + p.k_blocks - 1) / p.k_blocks : 1;
+  dim3 grid(((GATED ? p.F : p.N) + NOUT - 1) / NOUT, (p.M + BM - 1) / BM, parts);
   return launch_chain(k, grid, dim3(192), (size_t)smem, s, ta, tb, p);
 }
 
@@ -234,7 +244,7 @@ extern "C" int ifab_gemm_epilogue_bf16(const void* a, long lda, const void* b, l
   const int a_rows = one_row ? (M + 7) / 8 * 8 : BM;
   if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, (uint32_t)a_rows)) return rc;
   if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)N, (uint64_t)K, (uint64_t)ldb, (uint32_t)BN)) return rc;
-  GemmParams p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, a_rows, act, bias, cap, 0, {}};
+  GemmParams p{c, ldc, out_f32, (const bf16*)residual, ldr, M, N, K, status, 4000000u, a_rows, act, bias, cap, 0, {}, 0, 0};
   cudaStream_t s = (cudaStream_t)stream;
   if (!one_row) return BN == 256 ? launch<256, 4>(ta, tb, p, s) : launch<128, 6>(ta, tb, p, s);
   return BN == 128 ? launch<128, 3>(ta, tb, p, s) : BN == 64 ? launch<64, 4>(ta, tb, p, s) : launch<32, 5>(ta, tb, p, s);
@@ -256,8 +266,25 @@ extern "C" int ifab_gemm_gated_bf16(const void* a, long lda, const void* b, long
   CUtensorMap ta, tb;
   if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, (uint32_t)a_rows)) return rc;
   if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)2 * F, (uint64_t)K, (uint64_t)ldb, (uint32_t)(BN / 2))) return rc;
-  GemmParams p{c, ldc, 0, nullptr, 0, M, 2 * F, K, status, 4000000u, a_rows, 0, nullptr, 0.f, F, gu};
+  GemmParams p{c, ldc, 0, nullptr, 0, M, 2 * F, K, status, 4000000u, a_rows, 0, nullptr, 0.f, F, gu, 0, 0};
   cudaStream_t s = (cudaStream_t)stream;
   if (!one_row) return launch<256, 4, true>(ta, tb, p, s);
   return BN == 128 ? launch<128, 3, true>(ta, tb, p, s) : BN == 64 ? launch<64, 4, true>(ta, tb, p, s) : launch<32, 5, true>(ta, tb, p, s);
+}
+
+// Parts of C[M, N] (f32, M <= 128) = A B^T + bias along K: `parts` of them, part_stride elements apart; C is their sum. Every part gets K blocks of 64
+// columns, all but the last equally many.
+extern "C" int ifab_gemm_split_bf16(const void* a, long lda, const void* b, long ldb, float* c, long ldc, long part_stride, int parts, const float* bias, int M, int N,
+                                    int K, uint32_t* status, void* stream) {
+  const int kb = (K + BK - 1) / BK, per = parts > 0 ? (kb + parts - 1) / parts : 0;
+  if (M < 1 || M > BM || N < 1 || K < 8 || K % 8 || lda % 8 || ldb % 8 || parts < 1 || per * (parts - 1) >= kb || part_stride < (long)(M - 1) * ldc + N) return -1;
+  CUtensorMap ta, tb;
+  int BN = 32;
+  for (; BN < 128 && (N + BN - 1) / BN > 296; BN *= 2) {}
+  const int a_rows = (M + 7) / 8 * 8;
+  if (int rc = make_tmap_bf16_2d(&ta, a, (uint64_t)M, (uint64_t)K, (uint64_t)lda, (uint32_t)a_rows)) return rc;
+  if (int rc = make_tmap_bf16_2d(&tb, b, (uint64_t)N, (uint64_t)K, (uint64_t)ldb, (uint32_t)BN)) return rc;
+  GemmParams p{c, ldc, 1, nullptr, 0, M, N, K, status, 4000000u, a_rows, 0, bias, 0.f, 0, {}, per, part_stride};
+  cudaStream_t s = (cudaStream_t)stream;
+  return BN == 128 ? launch<128, 3>(ta, tb, p, s) : BN == 64 ? launch<64, 4>(ta, tb, p, s) : launch<32, 5>(ta, tb, p, s);
 }

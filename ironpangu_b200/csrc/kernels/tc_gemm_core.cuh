@@ -55,10 +55,11 @@ struct Pipe {
   // a_rows: rows of ta's box when it is shorter than the tile (the rest of the stage's A area then holds anything: rows of the
   // accumulator are independent, and the epilogue stores the live ones only).
   // a_col: first column of A (a multiple of 8), for heads that lie side by side in a row.
+  // k_first: first K block, for products split along K.
   // b_row_hi >= 0: the B tile is two boxes of BN/2 rows (tb's box is BN/2 rows): rows b_row.. fill the first half of
   // the stage's B area and rows b_row_hi.. the second half (paired gate / up projections under one accumulator).
   __device__ __forceinline__ void produce(const CUtensorMap* ta, const CUtensorMap* tb, int num_kb, int a_row, int b_row, int b_batch,
-                                          uint32_t spin_limit, uint32_t* status, int b_row_hi = -1, int a_rows = BM, int a_col = 0) {
+                                          uint32_t spin_limit, uint32_t* status, int b_row_hi = -1, int a_rows = BM, int a_col = 0, int k_first = 0) {
     using C = Cfg<BN, NSTAGES>;
     int issued = 0;
     for (int kb = 0; kb < num_kb; ++kb) {
@@ -68,12 +69,12 @@ struct Pipe {
       if (*abort_flag) break;
       unsigned char* a_dst = smem + s * C::STAGE_BYTES;
       mbar_expect_tx(&full[s], C::B_BYTES + a_rows * (BK * 2));
-      tma_load_2d(a_dst, ta, &full[s], a_col + kb * BK, a_row);
-      if (b_batch >= 0) tma_load_3d(a_dst + C::A_BYTES, tb, &full[s], kb * BK, b_row, b_batch);
-      else tma_load_2d(a_dst + C::A_BYTES, tb, &full[s], kb * BK, b_row);
+      tma_load_2d(a_dst, ta, &full[s], a_col + (k_first + kb) * BK, a_row);
+      if (b_batch >= 0) tma_load_3d(a_dst + C::A_BYTES, tb, &full[s], (k_first + kb) * BK, b_row, b_batch);
+      else tma_load_2d(a_dst + C::A_BYTES, tb, &full[s], (k_first + kb) * BK, b_row);
       if (b_row_hi >= 0) {
-        if (b_batch >= 0) tma_load_3d(a_dst + C::A_BYTES + C::B_BYTES / 2, tb, &full[s], kb * BK, b_row_hi, b_batch);
-        else tma_load_2d(a_dst + C::A_BYTES + C::B_BYTES / 2, tb, &full[s], kb * BK, b_row_hi);
+        if (b_batch >= 0) tma_load_3d(a_dst + C::A_BYTES + C::B_BYTES / 2, tb, &full[s], (k_first + kb) * BK, b_row_hi, b_batch);
+        else tma_load_2d(a_dst + C::A_BYTES + C::B_BYTES / 2, tb, &full[s], (k_first + kb) * BK, b_row_hi);
       }
       issued = kb + 1;
     }

@@ -4,6 +4,7 @@
 //   qk_norm_rope_write_kernel  RMS norm per head of q and k with a shared gain, rotation of the first `rot` columns (either pair
 //                              layout), q to its own rows, k and v into the pages of their sequence
 //   qk_rows_norm_write_kernel  the same with the norm over all heads of q (and all of k) together, a gain per column
+//   qk_chunks_write_kernel     that, or no norm at all, for bf16 heads of whole 16-byte chunks
 //   window_attn_kernel         one CTA per (row, query head): scores, weights and sums in f32; the denominator also holds
 //                              exp(sink_h). Optional output gate, a value per column or per head
 //
@@ -163,6 +164,103 @@ __global__ void __launch_bounds__(256) qk_rows_norm_write_kernel(QkParams p) {
   }
 }
 
+// grid T, 256 threads: a thread keeps up to NV chunks of 8 columns (q, then k, then v) in registers between the row sums and the stores.
+// NORM: gains of all columns of q and k
+template <int NV, bool NORM>
+__global__ void __launch_bounds__(256) qk_chunks_write_kernel(QkParams p) {
+  __shared__ float red[2][8];
+  grid_dep_launch();
+  grid_dep_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = p.positions[t];
+  if (pos < 0) return;
+  const bf16* row = reinterpret_cast<const bf16*>(p.proj) + (long)t * p.ldp;
+  const int lp = pos / p.page_tokens;
+  const int page = lp < p.max_pages ? p.page_table[(long)p.slots[t] * p.max_pages + lp] : -1;
+  if (page < 0 || page >= p.num_pages) {
+    if (threadIdx.x == 0 && p.status) atomicOr(p.status, IFAB_STATUS_BAD_INDEX);
+    return;
+  }
+  const long dst_row = (long)page * p.page_tokens + pos % p.page_tokens;
+  const int nq = p.H * p.d, nk = p.G * p.d, nv = p.G * p.e;
+  const bool same = p.v_off == p.k_off;            // the values are the keys
+  const int total = nq + nk + (same ? 0 : nv);
+  uint4 raw[NV];
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (threadIdx.x + i * 256) * 8;
+    raw[i] = make_uint4(0, 0, 0, 0);
+    if (c < total) raw[i] = *reinterpret_cast<const uint4*>(row + (c < nq ? p.q_off + c : c < nq + nk ? p.k_off + c - nq : p.v_off + c - nq - nk));
+    if (NORM && c < nq + nk) {
+      float f[8], ss = 0.f;
+      unpack8(raw[i], f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss += f[j] * f[j];
+      if (c < nq) sq += ss;
+      else sk += ss;
+    }
+  }
+  float iq = 1.f, ik = 1.f;
+  if (NORM) {
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) {
+      red[0][warp] = sq;
+      red[1][warp] = sk;
+    }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      sq += red[0][i];
+      sk += red[1][i];
+    }
+    iq = 1.f / sqrtf(sq / (float)nq + p.eps);
+    ik = 1.f / sqrtf(sk / (float)nk + p.eps);
+  }
+  const float2* cs = p.rope.cs + (long)t * (p.rope.rot / 2);
+  bf16* vd = reinterpret_cast<bf16*>(p.v_cache) + dst_row * nv;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (threadIdx.x + i * 256) * 8;
+    if (c >= total) break;
+    if (c >= nq + nk) {
+      *reinterpret_cast<uint4*>(vd + c - nq - nk) = raw[i];
+      continue;
+    }
+    const bool is_q = c < nq;
+    const int k = is_q ? c : c - nq, h = k / p.d, col = k - h * p.d;
+    if (!is_q && same) *reinterpret_cast<uint4*>(vd + k) = raw[i];
+    float f[8];
+    unpack8(raw[i], f);
+    if (NORM) {
+      const float4 g0 = *reinterpret_cast<const float4*>((is_q ? p.q_gain : p.k_gain) + k), g1 = *reinterpret_cast<const float4*>((is_q ? p.q_gain : p.k_gain) + k + 4);
+      const float g[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w}, inv = is_q ? iq : ik;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] = f[j] * inv * g[j];
+    }
+    if (col < p.rope.rot) {                          // whole chunks: rot is a multiple of 8
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 r = cs[col / 2 + j];
+        const float a = f[2 * j], b = f[2 * j + 1];
+        f[2 * j] = a * r.x - b * r.y;
+        f[2 * j + 1] = b * r.x + a * r.y;
+      }
+    }
+    bf16* dst = is_q ? reinterpret_cast<bf16*>(p.q_out) + (long)t * p.ldq + (long)h * p.q_stride + col : reinterpret_cast<bf16*>(p.k_cache) + dst_row * nk + k;
+    *reinterpret_cast<uint4*>(dst) = pack8(f);
+  }
+}
+
+template <bool NORM>
+int write_chunks(const QkParams& p, cudaStream_t s) {
+  const int chunks = (p.H * p.d + p.G * p.d + (p.v_off == p.k_off ? 0 : p.G * p.e) + 2047) / 2048;
+  if (chunks <= 2) return launch_chain(qk_chunks_write_kernel<2, NORM>, dim3(p.T), dim3(256), 0, s, p);
+  return launch_chain(qk_chunks_write_kernel<4, NORM>, dim3(p.T), dim3(256), 0, s, p);
+}
+
 struct WinParams {
   const void* q; long ldq;
   const void *k_cache, *v_cache;
@@ -201,6 +299,34 @@ __global__ void __launch_bounds__(256) ctx_gather_pad_kernel(const bf16* k_cache
     src_row[t] = row;
   }
   __syncthreads();
+  if ((d | e) % 8 == 0) {
+    // 16-byte chunks: keys straight through, values by columns of 8 keys
+    for (int i = t; i < 32 * (dp / 8); i += 256) {
+      const int kk = i / (dp / 8), c = (i - kk * (dp / 8)) * 8;
+      const long row = src_row[kk];
+      *reinterpret_cast<uint4*>(k + (long)(j0 + kk) * G * dp + (long)g * dp + c) =
+          (row >= 0 && c < d) ? *reinterpret_cast<const uint4*>(k_cache + (row * G + g) * d + c) : make_uint4(0, 0, 0, 0);
+    }
+    for (int i = t; i < 32 * 16; i += 256) {
+      const int kk = i >> 4, c = (i & 15) * 8;
+      const long row = src_row[kk];
+      const uint4 v = (row >= 0 && c < e) ? *reinterpret_cast<const uint4*>(v_cache + (row * G + g) * e + c) : make_uint4(0, 0, 0, 0);
+      uint32_t* w = reinterpret_cast<uint32_t*>(&tile[kk][c]);
+      w[0] = v.x;
+      w[1] = v.y;
+      w[2] = v.z;
+      w[3] = v.w;
+    }
+    __syncthreads();
+    for (int i = t; i < 128 * 4; i += 256) {
+      const int c = i >> 2, k0 = (i & 3) * 8;
+      union { bf16 h[8]; uint4 u; } o;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) o.h[j] = tile[k0 + j][c];
+      *reinterpret_cast<uint4*>(vt + ((long)g * 128 + c) * ldvt + j0 + k0) = o.u;
+    }
+    return;
+  }
   const bf16 zero = __float2bfloat16_rn(0.f);
   for (int i = t; i < 32 * dp; i += 256) {
     const int kk = i / dp, c = i - kk * dp;
@@ -323,6 +449,10 @@ extern "C" int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int 
   if (T < 1 || T > 65535 || H < 1 || G < 1 || d < 1 || e < 1 || rot < 0 || rot % 2 || rot > d || (rot && !rope) || q_stride < d) return -1;
   QkParams p{proj, ldp, q_off, k_off, v_off, q_gain, k_gain, eps, H, G, d, e, {(const float2*)rope, rot, interleaved}, positions, slots, page_table, max_pages, page_tokens,
              num_pages, q_out, ldq, q_stride, k_cache, v_cache, T, status};
+  const auto odd = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) != 0; };
+  if (!f32 && (whole || (!q_gain && !k_gain)) && !((d | e | rot | q_off | k_off | v_off | q_stride) % 8) && !((ldp | ldq) % 8) && (interleaved || !rot) &&
+      (long)H * d + (long)G * d + (v_off == k_off ? 0 : G * e) <= 8192 && !odd(proj) && !odd(q_out) && !odd(k_cache) && !odd(v_cache) && (!whole || (!odd(q_gain) && !odd(k_gain))))
+    return whole ? write_chunks<true>(p, (cudaStream_t)stream) : write_chunks<false>(p, (cudaStream_t)stream);
   if (whole) {
     if (!q_gain || !k_gain) return -1;
     return f32 ? launch_chain(qk_rows_norm_write_kernel<float>, dim3(T), dim3(256), 0, (cudaStream_t)stream, p)
@@ -348,7 +478,8 @@ extern "C" int ifab_window_attn(const void* q, long ldq, int q_stride, const voi
 extern "C" int ifab_ctx_gather_pad(const void* k_cache, const void* v_cache, const int32_t* page_table, int slot, int max_pages, int page_tokens,
                                    int num_pages, int first, int n, int rows, int G, int d, int dp, int e, void* k, void* vt, long ldvt, uint32_t* status,
                                    void* stream) {
-  if (n < 1 || rows < n || rows % 32 || slot < 0 || first < 0 || G < 1 || d < 1 || dp < d || e < 1 || e > 128 || ldvt < rows) return -1;
+  if (n < 1 || rows < n || rows % 32 || slot < 0 || first < 0 || G < 1 || d < 1 || dp < d || e < 1 || e > 128 || ldvt < rows || dp % 8 || ldvt % 8) return -1;
+  if (((reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(vt)) & 15)) return -1;
   return launch_chain(ctx_gather_pad_kernel, dim3(rows / 32, G), dim3(256), 0, (cudaStream_t)stream, (const bf16*)k_cache, (const bf16*)v_cache, page_table,
                       slot, max_pages, page_tokens, num_pages, first, n, G, d, dp, e, (bf16*)k, (bf16*)vt, ldvt, status);
 }

@@ -311,7 +311,7 @@ class MikutarDecoder(StreamDecoder):
         """All layer runs over ``m`` rows as separate row operators and matrix products; the residual ends in ``B.x``, and with ``final`` the
         normalised rows for the output matrix in ``B.xa``."""
         c, st, W = self.cfg, self.fabric.desc.status, self.cfg.width
-        x, xa, y = B.x[:m, :W], B.xa[:m], B.y[:m, :W]
+        x, xa = B.x[:m, :W], B.xa[:m]
         first = None if B.first is None else B.first[:m, :W]
         N.embed_rows(tok, self.embed, x, xa, gain=self.runs[0]["norm1"], eps=c.eps, copy=first, status_ptr=st)
         B.rotary.fill(pos)
@@ -324,12 +324,12 @@ class MikutarDecoder(StreamDecoder):
             R["mix"].project(B.attn, xa, st)
             R["join"].unit_rows(B.join, xa, st)
             self._attend(B, R, m, pos, slot, plan)
-            R["join"].rows(B.join, m, y, st)
+            y = R["join"].rows(B.join, m, B.y[:m], st)
             then = (None, None) if probe is not None else (gain, extra)
             if R["experts"] is not None:
-                R["experts"].rows(B.experts, m, xa, None, then[0], c.eps, B.x[:m], st, base=B.y[:m], extra=None if then[1] is None else B.first[:m])
+                R["experts"].rows(B.experts, m, xa, None, then[0], c.eps, B.x[:m], st, base=y, extra=None if then[1] is None else B.first[:m])
             else:
-                N.post_norm_add(y, None, c.eps, x, xa, *then)
+                N.post_norm_add(y[..., :W], None, c.eps, x, xa, *then)
             if probe is not None:                  # the residual as the layer leaves it; what comes before the next one follows
                 probe.append(x.clone())
                 N.post_norm_add(None, None, c.eps, x, xa, gain, extra)

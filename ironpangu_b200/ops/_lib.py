@@ -58,10 +58,11 @@ _SIGS = {
     "ifab_gemm_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, _P, _P],
     "ifab_gemm_act_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, c_int, c_int, c_int, c_int, _P, _P],
     "ifab_gemm_epilogue_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, _P, c_int, c_float, c_int, c_int, c_int, _P, _P],
+    "ifab_gemm_split_bf16": [_P, c_long, _P, c_long, _P, c_long, c_long, c_int, _P, c_int, c_int, c_int, _P, _P],
     "ifab_gemm_gated_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, c_float, c_float, c_int, c_int, c_int, _P, _P],
     "ifab_linear_f32": [_P, c_long, _P, c_long, _P, c_long, _P, c_float, c_int, c_int, c_int, c_int, _P],
     "ifab_embed_rows": [_P, _P, c_long, c_float, _P, c_float, _P, c_long, _P, _P, c_long, c_int, c_int, c_int, c_int, _P, _P],
-    "ifab_post_norm_add": [_P, c_long, _P, _P, c_float, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
+    "ifab_post_norm_add": [_P, c_long, c_int, c_long, _P, _P, c_float, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
     "ifab_gated_rows": [_P, c_long, c_int, c_int, c_float, c_float, _P, c_long, c_int, c_int, c_int, _P],
     "ifab_parallel_in_decode": [_P, c_long, _P, c_long, _P, c_float, _P, _P, c_long, _P, c_long, _P, _P, _P, c_long, c_int, _P, c_int, c_int, c_float, c_float, _P, c_long,
                                 _P, _P, c_long, _P, c_int, c_int, c_int, c_int, c_float, c_int, c_int, _P, _P, _P, c_int, c_int, _P],
@@ -88,7 +89,7 @@ _SIGS = {
                          c_long, c_int, c_int, _P, c_long, c_int, _P, _P],
     "ifab_moe_down_f32_decode": [_P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, c_long, _P],
     "ifab_moe_route": [_P, c_long, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, _P, _P, _P, _P],
-    "ifab_moe_combine_norm": [_P, c_long, _P, _P, c_int, _P, c_long, _P, _P, _P, c_float, _P, c_long, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
+    "ifab_moe_combine_norm": [_P, c_long, _P, _P, c_int, _P, c_long, _P, _P, _P, c_float, _P, c_long, c_int, c_long, _P, c_long, _P, c_long, _P, c_long, c_int, c_int, c_int, _P],
     "ifab_linear_f32_batched": [_P, c_long, c_long, _P, c_long, c_long, _P, c_long, c_long, c_int, c_int, c_int, c_int, _P],
     "ifab_grouped_linear_f32": [_P, c_long, _P, c_int, c_int, c_float, c_float, _P, c_int, c_int, _P, _P, c_int, c_int, _P, c_long, _P],
     "ifab_gemm_heads_bf16": [_P, c_long, c_int, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P],

@@ -59,9 +59,16 @@ class Join:
         if self.F:
             N.gated_linear(xa, self.gate_up, self.unit, self.operand(B, m)[:, self.at:], None if B.pair is None else B.pair[:m, :2 * self.F], status_ptr)
 
-    def rows(self, B: "JoinBuffers", m: int, y: torch.Tensor, status_ptr) -> None:
-        """``y`` (f32) = the product and its bias."""
-        N.linear(self.operand(B, m), self.w, y, bias=self.bias, status_ptr=status_ptr)
+    def rows(self, B: "JoinBuffers", m: int, y: torch.Tensor, status_ptr) -> torch.Tensor:
+        """The product and its bias in f32: in ``y``, or for few rows as parts of a sum ``[parts, m, padded width]``; returns which."""
+        width, k = self.w.shape
+        n = 1 if B.parts is None else N.split_count(m, width, k)
+        if n == 1:
+            N.linear(self.operand(B, m), self.w, y[:, :width], bias=self.bias, status_ptr=status_ptr)
+            return y
+        parts = B.parts[:n, :m]
+        N.split_linear(self.operand(B, m), self.w, parts[:, :, :width], self.bias, status_ptr)
+        return parts
 
     def decode(self, B: "JoinBuffers", n: int, y: torch.Tensor, addend: Optional[torch.Tensor]) -> None:
         """The same for decode rows; ``addend`` (f32 rows, may be ``y``) is added."""
@@ -74,6 +81,7 @@ class JoinBuffers:
     def __init__(self, joins, rows: int, dtype: torch.dtype, device):
         self.rows = {j.key: torch.zeros(rows, j.at + j.F, dtype=dtype, device=device) for j in joins}
         widest = max(j.F for j in joins)
+        self.parts = torch.zeros(8, min(rows, 128), _pad(joins[0].w.shape[0]), dtype=F32, device=device) if dtype != F32 else None
         self.pair = torch.zeros(rows, 2 * widest, dtype=dtype, device=device) if widest and dtype == F32 else None
 
 

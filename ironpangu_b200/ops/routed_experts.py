@@ -120,7 +120,7 @@ class RoutedExperts:
 
     def rows(self, B: ExpertBuffers, m: int, xa: torch.Tensor, gain: Optional[torch.Tensor], next_gain: Optional[torch.Tensor], eps: float, x: torch.Tensor,
              status_ptr, base: Optional[torch.Tensor] = None, extra: Optional[torch.Tensor] = None) -> None:
-        """``x += rms(experts(xa)) * gain``, or without a gain ``x += experts(xa) + base`` (f32 rows); ``extra`` (f32 rows) joins either. ``xa`` =
+        """``x += rms(experts(xa)) * gain``, or without a gain ``x += experts(xa) + base`` (f32 rows, or parts of their sum); ``extra`` (f32 rows) joins either. ``xa`` =
         ``rms(x) * next_gain`` (x without one). ``xa``: ``[m, padded width]``."""
         s, lib = self.shape, _lib.load()
         D = self.gate_up.shape[2]
@@ -150,7 +150,7 @@ class RoutedExperts:
                     P.grouped_gemm(xa, self.shared_gate_up[None], B.row_tiles, B.row_ntiles, sact, unit=s.unit, status_ptr=status_ptr)
                 N.linear(sact[:m], self.shared_down, sh[:m], status_ptr=status_ptr)
         check(lib.ifab_moe_combine_norm(y.data_ptr(), y.stride(0), route.route_row.data_ptr(), wts.data_ptr(), s.top, _p(sh), 0 if sh is None else sh.stride(0),
-                                        B.shared_w.data_ptr() if s.shared_ff else None, _p(gain), _p(next_gain), eps, _p(base), 0 if base is None else base.stride(0),
+                                        B.shared_w.data_ptr() if s.shared_ff else None, _p(gain), _p(next_gain), eps, _p(base), *N._parts(base),
                                         _p(extra), 0 if extra is None else extra.stride(0), x.data_ptr(), x.stride(0), xa.data_ptr(), xa.stride(0), _f32(xa), m, s.width, _s()), "moe_combine_norm")
 
     def _grouped_f32(self, xa, index, gate_up, down, tiles, ntiles, act, y, rows: int) -> None:

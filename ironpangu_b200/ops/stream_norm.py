@@ -63,13 +63,20 @@ def embed_rows(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, xa: torc
                                       xa.stride(0), _f32(xa), T, D, table.shape[0], status_ptr, _s()), "embed_rows")
 
 
+def _parts(y: Optional[torch.Tensor]) -> tuple:
+    """Row stride, parts and their distance of rows ``[T, D]`` or of parts of a sum ``[parts, T, D]``."""
+    if y is None:
+        return 0, 1, 0
+    return (y.stride(1), y.shape[0], y.stride(0)) if y.dim() == 3 else (y.stride(0), 1, 0)
+
+
 def post_norm_add(y: Optional[torch.Tensor], w: Optional[torch.Tensor], eps: float, x: torch.Tensor, xa: torch.Tensor, final: Optional[torch.Tensor] = None,
                   extra: Optional[torch.Tensor] = None) -> None:
     """``x += rms(y) * w [+ extra]`` in f32 (``y`` as it is without ``w``, nothing without ``y``); ``xa`` = x, or ``rms(x) * final`` (the norm
-    ahead of the next linears)."""
+    ahead of the next linears). ``y`` may be the parts of a sum, ``[parts, T, D]``."""
     T, D = x.shape
     assert all(t is None or t.dtype == torch.float32 for t in (y, w, x, extra))
-    check(_lib.load().ifab_post_norm_add(_p(y), 0 if y is None else y.stride(0), _p(w), _p(final), eps, x.data_ptr(), x.stride(0), _p(extra),
+    check(_lib.load().ifab_post_norm_add(_p(y), *_parts(y), _p(w), _p(final), eps, x.data_ptr(), x.stride(0), _p(extra),
                                          0 if extra is None else extra.stride(0), xa.data_ptr(), xa.stride(0), _f32(xa), T, D, _s()), "post_norm_add")
 
 
@@ -146,6 +153,25 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: Optional[st
     else:
         check(_lib.load().ifab_gemm_epilogue_bf16(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), _f32(out), None, 0,
                                                   _p(bias), ACTIVATIONS[act], cap, T, N, K, status_ptr, _s()), "gemm_epilogue")
+
+
+def split_count(rows: int, n: int, k: int) -> int:
+    """Parts along K that give a product of one tile row (128) about two CTAs an SM; 1 when it has enough columns or is too short."""
+    if rows > 128:
+        return 1
+    blocks = (k + 63) // 64
+    want = max(1, min(8, 296 // ((n + 31) // 32), blocks // 4))
+    per = (blocks + want - 1) // want
+    return (blocks + per - 1) // per
+
+
+def split_linear(x: torch.Tensor, w: torch.Tensor, parts: torch.Tensor, bias: Optional[torch.Tensor] = None, status_ptr: Optional[int] = None) -> None:
+    """``parts`` (f32 ``[parts, T, N]``, T <= 128): their sum is ``x @ w.T + bias``."""
+    T, K = x.shape
+    S, _, N = parts.shape
+    assert parts.shape[1] == T and w.shape == (N, K) and x.dtype == w.dtype == BF16 and parts.stride(2) == 1
+    check(_lib.load().ifab_gemm_split_bf16(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), parts.data_ptr(), parts.stride(1), parts.stride(0), S, _p(bias), T, N, K,
+                                           status_ptr, _s()), "gemm_split")
 
 
 def gated_linear(x: torch.Tensor, w: torch.Tensor, unit: GatedUnit, out: torch.Tensor, pair: Optional[torch.Tensor] = None, status_ptr: Optional[int] = None) -> None:

@@ -126,13 +126,14 @@ def mikutar_arm(size, prompt: int, chunk_rows: int, batches: List[int], t: Timer
         pos = torch.arange(prompt - n, prompt, dtype=torch.int32, device=dev)
         setup(B, n, pos)
         x, xa, y = B.x[:n], B.xa[:n], B.y[:n]
+        own = dense[0]["join"].rows(B.join, n, y, st)
         group(f"input projection, {n} rows", dec.runs, lambda R: R["mix"].project(B.attn, xa, st), w_in, n * w_in)
         group(f"gated unit of dense layers, {n} rows", dense, lambda R: R["join"].unit_rows(B.join, xa, st), gu_d, n * gu_d)
         group(f"gated unit of routed layers, {n} rows", routed, lambda R: R["join"].unit_rows(B.join, xa, st), gu_m, n * gu_m)
         group(f"output product of dense layers, {n} rows", dense, lambda R: R["join"].rows(B.join, n, y, st), join_d, n * join_d)
         group(f"output product of routed layers, {n} rows", routed, lambda R: R["join"].rows(B.join, n, y, st), join_m, n * join_m)
-        group(f"residual and next norm, {n} rows", dense, lambda R: N.post_norm_add(y, None, eps, x, xa, R["norm1"]), n * cfg.width * 14.0)
-        group(f"router, routed experts, residual and next norm, {n} rows", routed, lambda R: R["experts"].rows(B.experts, n, xa, None, R["norm1"], eps, x, st, base=y),
+        group(f"residual and next norm, {n} rows", dense, lambda R: N.post_norm_add(own, None, eps, x, xa, R["norm1"]), n * cfg.width * 14.0)
+        group(f"router, routed experts, residual and next norm, {n} rows", routed, lambda R: R["experts"].rows(B.experts, n, xa, None, R["norm1"], eps, x, st, base=own),
               hit * unit + w_router, n * c["top"] * unit)
     m = chunk_rows
     pos, sl = torch.arange(prompt - m, prompt, dtype=torch.int32, device=dev), torch.zeros(m, dtype=torch.int32, device=dev)

@@ -50,6 +50,24 @@ def test_linear_with_bias_and_soft_limit(dtype, rows, cols, width):
         assert _rel(out, z - b.double() + add.double()) < 1e-5
 
 
+@pytest.mark.parametrize("rows,cols,width,parts", [(1, 40, 64, 1), (3, 33, 512, 8), (8, 131, 1000, 3), (64, 1024, 5120, 8), (128, 96, 328, 6), (70, 10000, 256, 2)])
+def test_product_in_parts(rows, cols, width, parts):
+    """Parts along K, the ragged last one included; the row operators add them up."""
+    from ironpangu_b200.ops import stream_norm as N
+
+    g = torch.Generator().manual_seed(cols)
+    x, w, b = torch.randn(rows, width, generator=g).to(BF16), (torch.randn(cols, width, generator=g) * width ** -0.5).to(BF16), torch.randn(cols, generator=g)
+    out = torch.full((parts, rows, _pad(cols)), 5.0, device="cuda")
+    N.split_linear(x.cuda(), w.cuda(), out[:, :, :cols], b.cuda())
+    want = x.double() @ w.double().T + b.double()
+    assert _rel(out.sum(0)[:, :cols], want) < 2e-5 and (out[:, :, cols:] == 5).all()
+    r = torch.randn(rows, _pad(cols), generator=g)
+    xd, xa = r.cuda(), torch.zeros(rows, _pad(cols), device="cuda")
+    N.post_norm_add(out[:, :, :cols], None, 1e-3, xd[:, :cols], xa)
+    assert _rel(xd[:, :cols], r[:, :cols].double() + want) < 2e-5
+    assert N.split_count(rows, cols, width) >= 1 and N.split_count(200, cols, width) == 1
+
+
 UNITS = [("relu", 0.0, 1.0), ("limited", 0.7, 1.702), ("limited", 7.0, 0.9), ("silu", 0.0, 1.0)]
 
 
@@ -289,7 +307,8 @@ def test_routed_experts_beside_another_sublayer(dtype, width, experts, top, grou
     gain = 1 + 0.2 * torch.randn(width, generator=g)
     xd, xa = pad(x, F32), pad(h, dtype)
     B.start(rows)
-    ex.rows(B, rows, xa, None, gain.cuda(), 1e-4, xd, None, base=pad(base, F32), extra=pad(extra, F32))
+    part = pad(0.25 * base, F32), pad(0.75 * base, F32)                   # what ran beside the experts, as one piece and as parts of a sum
+    ex.rows(B, rows, xa, None, gain.cuda(), 1e-4, xd, None, base=pad(base, F32) if rows == 9 else torch.stack(part), extra=pad(extra, F32))
     want = x.double() + base.double() + extra.double() + y
     assert _rel(xd[:, :width], want) < _lim(dtype, 3e-6, 8e-3)
     assert _rel(xa[:, :width], O.rms(want, 1e-4, gain.double())) < _lim(dtype, 3e-6, 1.2e-2) and not xd[:, width:].any() and not xa[:, width:].any()
@@ -354,5 +373,6 @@ def test_front_and_end_of_a_parallel_layer(rows, width, heads, ff, experts):
         want = mixed.double() @ d("o").T + d("o.b") + (act @ d("down").T if ff else 0)
         got, got2 = out.cuda(), torch.zeros(rows, width, device="cuda")
         join.decode(JB, rows, got, got)
-        join.rows(JB, rows, got2, None)
+        got2 = join.rows(JB, rows, got2, None)
+        got2 = got2.sum(0) if got2.dim() == 3 else got2
         assert _rel(got, want + out.double()) < 1e-5 and _rel(got2, want) < 4e-5
