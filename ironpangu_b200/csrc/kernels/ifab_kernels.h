@@ -356,8 +356,31 @@ int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int 
                             void* v_cache, int whole, int T, uint32_t* status, void* stream);
 int ifab_window_attn(const void* q, long ldq, int q_stride, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,
                      const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int H, int G, int d, int e, int window, float scale, float cap,
-                     const float* slopes, int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, void* out, long ldo, int T,
-                     uint32_t* status, void* stream);
+                     const float* slopes, int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, int keep, int pool,
+                     const void* pool_k, const void* pool_v, float factor, void* out, long ldo, int T, uint32_t* status, void* stream);
+/* means of the blocks of `pool` positions that end with a row of the step, into pool_k / pool_v [pages, ceil(page_tokens / pool), G, .] */
+int ifab_pool_write(const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots, const int32_t* page_table, int max_pages,
+                    int page_tokens, int num_pages, int G, int d, int e, int pool, void* pool_k, void* pool_v, int T, uint32_t* status, void* stream);
+/* residual streams side by side with a convolution ahead of every sublayer (hyper_streams.cu) */
+int ifab_embed_norm(const int32_t* ids, const void* table, long ldt, const float* gain, float eps, float* x, long ldx, int f32, int T, int D, int vocab,
+                    uint32_t* status, void* stream);
+int ifab_step_epoch(const int32_t* slots, int32_t* epoch, int T, void* stream);
+int ifab_streams_rows(const float* x_in, long ldr_in, long lds_in, float* x_out, long ldr_out, long lds_out, const float* y, long ldy, int parts,
+                      long part_stride, const float* mix, const float* out, const float* in, const float* gain, float eps, const float* taps_w, int taps,
+                      float* history, const int32_t* epoch, const int32_t* positions, const int32_t* slots, float* sum, long ldsum, void* xa, long lda, int f32,
+                      int T, int S, int D, int block, void* stream);
+/* recurrences with a decay per token (gated_recurrence.cu, gated_delta.cu). kind: 0 state-space duality, 1 delta rule, 2 matrix memory */
+int ifab_gr_prepare(const void* proj, long ldp, int f32, const int32_t* sections, const float* scales, float* q, float* k, float* v, const float* taps_w,
+                    const float* bias, int taps, int C, void* history, const int32_t* epoch, int kind, int H, int decay_col, int weight_col, const float* a_log,
+                    const float* decay_bias, const float* weight_bias, float cap, float* log_decay, float* weight, const int32_t* positions,
+                    const int32_t* slots, int T, void* stream);
+int ifab_gr_step(const float* q, const float* k, const float* v, const float* log_decay, const float* weight, int kind, int H, int G, int d, int E, float* state,
+                 float* m_state, const int32_t* epoch, float* m_rows, const int32_t* positions, const int32_t* slots, float* o, long ldo, int T, void* stream);
+int ifab_gr_chunks(const float* q, const float* k, const float* v, const float* log_decay, const float* weight, int kind, int H, int G, int d, int E,
+                   const int32_t* chunks, int n, const int32_t* positions, float* cstate, uint64_t cstate_bytes, float* cdecay, float* w_rows, float* u_rows,
+                   float* state, float* m_state, const int32_t* epoch, float* m_rows, float* o, long ldo, void* stream);
+int ifab_gr_finish(const float* o, long ldo, int H, int e, int E, const float* m, const float* v, const float* skip, const void* gate, long ldg, int act,
+                   int gate_first, int groups, float eps, const float* gain, void* y, long ldy, int f32, int T, void* stream);
 /* operands of the tensor-core windowed attention: keys / values first .. first + n - 1 of a sequence, heads zero-padded to dp / 128 columns */
 int ifab_ctx_gather_pad(const void* k_cache, const void* v_cache, const int32_t* page_table, int slot, int max_pages, int page_tokens, int num_pages,
                         int first, int n, int rows, int G, int d, int dp, int e, void* k, void* vt, long ldvt, uint32_t* status, void* stream);

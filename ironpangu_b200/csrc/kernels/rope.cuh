@@ -52,13 +52,17 @@ __device__ __forceinline__ float sigmoid_f32(float x) {
 template <bool FAST = false>
 __device__ __forceinline__ float gelu_tanh_f32(float z) { return z * sigmoid_f32<FAST>(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
 
-// elementwise activations by number: 0 none, 1 SiLU, 2 sigmoid, 3 GELU (tanh form)
+// 0.5 z (1 + erf(z / sqrt 2)), without cancellation for negative z
+__device__ __forceinline__ float gelu_erf_f32(float z) { return 0.5f * z * erfcf(-0.70710678118654752f * z); }
+
+// elementwise activations by number: 0 none, 1 SiLU, 2 sigmoid, 3 GELU (tanh form), 4 GELU (erf form)
 template <bool FAST = false>
 __device__ __forceinline__ float activate(float z, int act) {
   switch (act) {
     case 1: return z * sigmoid_f32<FAST>(z);
     case 2: return sigmoid_f32<FAST>(z);
     case 3: return gelu_tanh_f32<FAST>(z);
+    case 4: return gelu_erf_f32(z);
     default: return z;
   }
 }

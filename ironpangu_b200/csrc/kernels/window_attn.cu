@@ -6,7 +6,9 @@
 //   qk_rows_norm_write_kernel  the same with the norm over all heads of q (and all of k) together, a gain per column
 //   qk_chunks_write_kernel     that, or no norm at all, for bf16 heads of whole 16-byte chunks
 //   window_attn_kernel         one CTA per (row, query head): scores, weights and sums in f32; the denominator also holds
-//                              exp(sink_h). Optional output gate, a value per column or per head
+//                              exp(sink_h). Optional output gate, a value per column or per head, and a factor on the result
+//   pool_write_kernel          means of the keys and values of the blocks that end with a row of the step, out of the pages into the
+//                              entries of AheadRule
 //
 // v may be the columns of k (v_off == k_off): the values are then the keys as projected.
 //
@@ -275,6 +277,8 @@ struct WinParams {
   uint32_t* status;
   ScoreRule rule;
   int gate_head;                 // the gate has one value per head: [T, H]
+  AheadRule ahead;
+  float factor;                  // of the result
 };
 
 // Keys and values first .. first + n - 1 of one sequence out of its pages: k [rows, G * dp] (columns d .. dp - 1 of a head zero) and
@@ -364,22 +368,26 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
     acc[u] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  for (int k0 = first + warp; k0 <= pos; k0 += WARPS * KB) {
+  const int ahead = p.ahead.count(first), n = ahead + pos + 1 - first;      // what the query sees: entries ahead of the window, then its positions
+  for (int k0 = warp; k0 < n; k0 += WARPS * KB) {
     float s[KB];
     long r[KB];
+    const A* vr[KB];
 #pragma unroll
     for (int b = 0; b < KB; ++b) {
-      const int key = k0 + b * WARPS;
+      const int i = k0 + b * WARPS;
       r[b] = -1;
       s[b] = 0.f;
-      if (key <= pos) {
-        const int lp = key / p.page_tokens;
+      if (i < n) {
+        const bool pooled = i < ahead && p.ahead.pool > 0;
+        const int key = i < ahead ? p.ahead.position(i) : first + i - ahead, lp = key / p.page_tokens;
         const int page = lp < p.max_pages ? table[lp] : -1;
         if (page < 0 || page >= p.num_pages) {
           if (lane == 0 && p.status) atomicOr(p.status, IFAB_STATUS_BAD_INDEX);
         } else {
-          r[b] = ((long)page * p.page_tokens + key % p.page_tokens) * p.G + g;
-          const A* kr = reinterpret_cast<const A*>(p.k_cache) + r[b] * p.d;
+          r[b] = ((pooled ? (long)page * p.ahead.per_page + p.ahead.row(i, p.page_tokens) : (long)page * p.page_tokens + key % p.page_tokens)) * p.G + g;
+          const A* kr = reinterpret_cast<const A*>(pooled ? p.ahead.k : p.k_cache) + r[b] * p.d;
+          vr[b] = reinterpret_cast<const A*>(pooled ? p.ahead.v : p.v_cache) + r[b] * p.e;
 #pragma unroll
           for (int u = 0; u < EPL; ++u)
             if (32 * u < p.d && lane + 32 * u < p.d) s[b] = fmaf(q[u], to_f32(kr[lane + 32 * u]), s[b]);
@@ -391,7 +399,7 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
     if (!p.rule.plain()) {
 #pragma unroll
       for (int b = 0; b < KB; ++b)
-        if (r[b] >= 0) s[b] = ruled_score<sizeof(A) == 2>(s[b], p.rule, slope, pos - k0 - b * WARPS);
+        if (r[b] >= 0) s[b] = ruled_score<sizeof(A) == 2>(s[b], p.rule, slope, n - 1 - k0 - b * WARPS);
     }
     float mn = m;
 #pragma unroll
@@ -406,10 +414,9 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
       if (r[b] < 0) continue;
       const float w = expf(s[b] - mn);
       l += w;
-      const A* vr = reinterpret_cast<const A*>(p.v_cache) + r[b] * p.e;
 #pragma unroll
       for (int u = 0; u < EPL; ++u)
-        if (32 * u < p.e && lane + 32 * u < p.e) acc[u] = fmaf(w, to_f32(vr[lane + 32 * u]), acc[u]);
+        if (32 * u < p.e && lane + 32 * u < p.e) acc[u] = fmaf(w, to_f32(vr[b][lane + 32 * u]), acc[u]);
     }
     m = mn;
   }
@@ -429,7 +436,7 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
     wgt[w] = sm_m[w] == -INFINITY ? 0.f : expf(sm_m[w] - M);
     den += wgt[w] * sm_l[w];
   }
-  const float inv = den > 0.f ? 1.f / den : 0.f;
+  const float inv = den > 0.f ? p.factor / den : 0.f;
   for (int c = threadIdx.x; c < p.e; c += blockDim.x) {
     float v = 0.f;
 #pragma unroll
@@ -440,7 +447,57 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
   }
 }
 
+// grid (T, G), 128 threads: the block that ends at a row's position, if one does
+template <typename A>
+__global__ void __launch_bounds__(128) pool_write_kernel(const A* k_cache, const A* v_cache, const int32_t* positions, const int32_t* slots, const int32_t* page_table,
+                                                         int max_pages, int page_tokens, int num_pages, int G, int d, int e, AheadRule rule, uint32_t* status) {
+  grid_dep_launch();
+  grid_dep_wait();
+  const int t = blockIdx.x, g = blockIdx.y, pos = positions[t], P = rule.pool;
+  if (pos < 0 || (pos + 1) % P) return;
+  const int32_t* table = page_table + (long)slots[t] * max_pages;
+  const int last = pos / page_tokens < max_pages ? table[pos / page_tokens] : -1;
+  bool ok = last >= 0 && last < num_pages;
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};      // d + e <= 512 columns
+  for (int j = pos - P + 1; j <= pos && ok; ++j) {
+    const int page = j / page_tokens < max_pages ? table[j / page_tokens] : -1;
+    if (page < 0 || page >= num_pages) {
+      ok = false;
+      break;
+    }
+    const long row = ((long)page * page_tokens + j % page_tokens) * G + g;
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int c = threadIdx.x + 128 * u;
+      if (c < d + e) acc[u] += to_f32(c < d ? k_cache[row * d + c] : v_cache[row * e + c - d]);
+    }
+  }
+  if (!ok) {
+    if (threadIdx.x == 0 && status) atomicOr(status, IFAB_STATUS_BAD_INDEX);
+    return;
+  }
+  const long row = ((long)last * rule.per_page + rule.row(pos / P, page_tokens)) * G + g;
+#pragma unroll
+  for (int u = 0; u < 4; ++u) {
+    const int c = threadIdx.x + 128 * u;
+    if (c >= d + e) break;
+    A* dst = c < d ? reinterpret_cast<A*>(const_cast<void*>(rule.k)) + row * d + c : reinterpret_cast<A*>(const_cast<void*>(rule.v)) + row * e + c - d;
+    *dst = from_f32<A>(acc[u] / (float)P);
+  }
+}
+
 }  // namespace
+
+extern "C" int ifab_pool_write(const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots, const int32_t* page_table, int max_pages,
+                               int page_tokens, int num_pages, int G, int d, int e, int pool, void* pool_k, void* pool_v, int T, uint32_t* status, void* stream) {
+  if (T < 1 || G < 1 || G > 65535 || d < 1 || d > 256 || e < 1 || e > 256 || pool < 1 || !pool_k || !pool_v) return -1;
+  const AheadRule rule = ahead_rule(0, pool, pool_k, pool_v, page_tokens);
+  const dim3 grid(T, G);
+  return f32 ? launch_chain(pool_write_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, (const float*)k_cache, (const float*)v_cache, positions, slots, page_table,
+                            max_pages, page_tokens, num_pages, G, d, e, rule, status)
+             : launch_chain(pool_write_kernel<bf16>, grid, dim3(128), 0, (cudaStream_t)stream, (const bf16*)k_cache, (const bf16*)v_cache, positions, slots, page_table,
+                            max_pages, page_tokens, num_pages, G, d, e, rule, status);
+}
 
 extern "C" int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, const float* q_gain, const float* k_gain,
                                        float eps, int H, int G, int d, int e, int rot, int interleaved, const void* rope, const int32_t* positions,
@@ -466,10 +523,13 @@ extern "C" int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int 
 extern "C" int ifab_window_attn(const void* q, long ldq, int q_stride, const void* k_cache, const void* v_cache, int f32, const int32_t* positions, const int32_t* slots,
                                 const int32_t* page_table, int max_pages, int page_tokens, int num_pages, int H, int G, int d, int e, int window,
                                 float scale, float cap, const float* slopes, int chunked, const float* sink, const void* gate, long ldg, int gate_act,
-                                int gate_per_head, void* out, long ldo, int T, uint32_t* status, void* stream) {
+                                int gate_per_head, int keep, int pool, const void* pool_k, const void* pool_v, float factor, void* out, long ldo, int T,
+                                uint32_t* status, void* stream) {
+  const AheadRule ahead = ahead_rule(keep, pool, pool_k, pool_v, page_tokens);
+  if (!ahead_ok(ahead, window, chunked) || (ahead.any() && (cap > 0.f || slopes))) return -1;
   if (cap < 0.f || T < 1 || T > 65535 || H < 1 || G < 1 || H % G || d < 1 || d > 256 || e < 1 || e > 256 || window < 0) return -1;
   WinParams p{q, ldq, k_cache, v_cache, positions, slots, page_table, max_pages, page_tokens, num_pages, H, G, d, e, window, scale, sink, gate, ldg, gate_act,
-              out, ldo, q_stride, status, {cap, slopes, chunked}, gate_per_head};
+              out, ldo, q_stride, status, {cap, slopes, chunked}, gate_per_head, ahead, factor};
   const dim3 grid(H, T);
   return f32 ? launch_chain(window_attn_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, p)
              : launch_chain(window_attn_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)stream, p);

@@ -46,7 +46,7 @@ def load(path, config_of: Callable[[dict], object], shapes_of: Callable[[object]
         _, _, _, dt, have = src.tensors[name]
         if tuple(have) != tuple(shape) or dt not in DTYPES:
             raise ValueError(f"{name}: {dt} {list(have)} in the checkpoint, {list(shape)} expected")
-        out[name] = torch.from_numpy(src.bytes_of(name).copy()).view(DTYPES[dt]).view(*shape)
+        out[name] = torch.from_numpy(src.bytes_of(name).copy()).view(DTYPES[dt]).view(tuple(shape))
     return c, out
 
 

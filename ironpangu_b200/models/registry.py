@@ -25,7 +25,8 @@ class Family:
 
 FAMILIES: Tuple[Family, ...] = (Family("Falinex", "falinex", "FalinexDecoder", "FalinexRows", True, ("falinex-tiny", "falinex2b")),
                                 Family("Ponenex", "ponenex", "PonenexDecoder", "PonenexRows", True, ("ponenex-tiny", "ponenex-text")),
-                                Family("Mikutar", "mikutar", "MikutarDecoder", "MikutarRows", True, ("mikutar-tiny", "mikutar-text")))
+                                Family("Mikutar", "mikutar", "MikutarDecoder", "MikutarRows", True, ("mikutar-tiny", "mikutar-text")),
+                                Family("Fubelorn", "fubelorn", "FubelornDecoder", "FubelornRows", True, ("fubelorn-tiny", "fubelorn-text")))
 
 
 def family_of(checkpoint_dir) -> Family:

@@ -2,6 +2,8 @@
 per-sequence f32 states, for any head sizes."""
 from __future__ import annotations
 
+import math
+from dataclasses import dataclass
 from typing import Optional, Sequence
 
 import torch
@@ -14,25 +16,50 @@ CHUNK = 64            # rows of a chunk of the f32 form
 TILE = 128            # rows of a chunk of the tensor-core form
 
 
-def rotary_frequencies(dims: int, base: float, device) -> torch.Tensor:
-    """``base^(-2 i / dims)`` for i < dims / 2, in double."""
-    return torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64, device=device)
+@dataclass(frozen=True)
+class RotaryScaling:
+    """Stretching of long wavelengths: a frequency whose wavelength is above ``original / low`` is divided by ``factor``, one below ``original /
+    high`` stays, between them the two are mixed in proportion to ``original / wavelength``."""
+
+    factor: float
+    low: float
+    high: float
+    original: float
+
+    def check(self) -> None:
+        if self.factor <= 0 or self.original <= 0 or not 0 < self.low < self.high:
+            raise ValueError(f"rotation scaling {self} is not supported")
+
+    def apply(self, f: float) -> float:
+        turns = self.original * f / (2.0 * math.pi)          # of the pair over the original context
+        if turns > self.high:
+            return f
+        if turns < self.low:
+            return f / self.factor
+        s = (turns - self.low) / (self.high - self.low)
+        return (1.0 - s) * f / self.factor + s * f
+
+
+def rotary_frequencies(dims: int, base: float, device, scaling: Optional[RotaryScaling] = None) -> torch.Tensor:
+    """``base^(-2 i / dims)`` for i < dims / 2, scaled, in double."""
+    f = [float(base) ** (-2.0 * i / dims) for i in range(dims // 2)]
+    return torch.tensor([scaling.apply(v) for v in f] if scaling else f, dtype=torch.float64, device=device)
 
 
 class RotaryTables:
-    """(cos, sin) of every rotation a model uses, for the rows of a step: one table f32 ``[rows, dims / 2, 2]`` per (dims, base), filled by
+    """(cos, sin) of every rotation a model uses, for the rows of a step: one table f32 ``[rows, dims / 2, 2]`` per (dims, base[, scaling]), filled by
     one launch each per step and read by all layers."""
 
     def __init__(self, rotations, rows: int, device):
-        self.freq = {r: rotary_frequencies(r[0], r[1], device) for r in sorted(set(rotations)) if r[0]}
+        self.freq = {r: rotary_frequencies(r[0], r[1], device, r[2]) for r in {(*r, None)[:3] for r in rotations} if r[0]}
         self.table = {r: torch.zeros(rows, r[0] // 2, 2, dtype=torch.float32, device=device) for r in self.freq}
 
     def fill(self, positions: torch.Tensor) -> None:
         for r, f in self.freq.items():
             check(_lib.load().ifab_rope_table(positions.data_ptr(), f.data_ptr(), self.table[r].data_ptr(), positions.numel(), f.numel(), _s()), "rope_table")
 
-    def get(self, dims: int, base: float) -> Optional[torch.Tensor]:
-        return self.table[(dims, base)] if dims else None
+    def get(self, dims: int, base: float, scaling: Optional[RotaryScaling] = None) -> Optional[torch.Tensor]:
+        return self.table[(dims, base, scaling)] if dims else None
 
 
 def decay_powers(decay: Sequence[float], device) -> torch.Tensor:

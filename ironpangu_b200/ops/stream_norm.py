@@ -12,7 +12,7 @@ from . import _lib
 from ._lib import check
 
 BF16 = torch.bfloat16
-ACTIVATIONS = {None: 0, "silu": 1, "sigmoid": 2, "gelu_tanh": 3}
+ACTIVATIONS = {None: 0, "silu": 1, "sigmoid": 2, "gelu_tanh": 3, "gelu_erf": 4}
 
 
 UNITS = {"silu": 0, "relu": 1, "limited": 2}

@@ -3,7 +3,10 @@
 
 The mask: the last ``window`` positions (0: all), or with ``chunked`` the positions of the query's own stretch of ``window``, counted from
 position 0 of the sequence. A score is ``q k scale``, with ``cap`` > 0 ``cap * tanh(score / cap)``, and with ``slopes`` (f32 ``[heads]``) less
-``slope * (distance of the key)``. A gate has a value per column of the result, or one per head (``gate_head``)."""
+``slope * (distance of the key)``. A gate has a value per column of the result, or one per head (``gate_head``).
+
+Beside its window a query may see entries ahead of it, in the same softmax (:class:`Ahead`): the first ``keep`` positions, or one mean key and
+value per block of ``pool`` positions that lies wholly before the window."""
 from __future__ import annotations
 
 from dataclasses import dataclass
@@ -14,7 +17,33 @@ import torch
 from . import _lib
 from . import stream_norm as N
 from ._lib import check
+from .linear_attn import RotaryScaling
 from .stream_norm import ACTIVATIONS, _f32, _p, _s
+
+
+@dataclass(frozen=True)
+class Ahead:
+    """``pages``: the blocks' keys and values ``[pages, entries, kv_heads, .]`` (an entry lives in the page of its block's last position)."""
+
+    keep: int = 0
+    pool: int = 0
+    pages: Optional[tuple] = None
+
+    @property
+    def args(self) -> tuple:
+        k, v = self.pages or (None, None)
+        return self.keep, self.pool, _p(k), _p(v)
+
+
+NOTHING_AHEAD = Ahead()
+
+
+def pool_write(k_cache: torch.Tensor, v_cache: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, page_table: torch.Tensor, ahead: Ahead, status_ptr=None) -> None:
+    """The means of the blocks that end with a row of the step, out of the pages into ``ahead.pages``."""
+    pages, pt, G, d = k_cache.shape
+    check(_lib.load().ifab_pool_write(k_cache.data_ptr(), v_cache.data_ptr(), _f32(k_cache), positions.data_ptr(), slots.data_ptr(), page_table.data_ptr(),
+                                      page_table.shape[1], pt, pages, G, d, v_cache.shape[3], ahead.pool, ahead.pages[0].data_ptr(), ahead.pages[1].data_ptr(),
+                                      positions.numel(), status_ptr, _s()), "pool_write")
 
 
 def qk_norm_rope_write(proj: torch.Tensor, offsets, q_gain: Optional[torch.Tensor], k_gain: Optional[torch.Tensor], eps: float, *, heads: int, kv_heads: int,
@@ -34,13 +63,13 @@ def qk_norm_rope_write(proj: torch.Tensor, offsets, q_gain: Optional[torch.Tenso
 def window_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, page_table: torch.Tensor, *,
                 heads: int, window: int, scale: float, out: torch.Tensor, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                 gate_act: Optional[str] = None, gate_head: bool = False, chunked: bool = False, cap: float = 0.0, slopes: Optional[torch.Tensor] = None,
-                status_ptr=None) -> None:
-    """Rows of any sequences, any head sizes: exp(sink) joins the denominator, the result is multiplied by ``gate_act(gate)``."""
+                ahead: Ahead = NOTHING_AHEAD, factor: float = 1.0, status_ptr=None) -> None:
+    """Rows of any sequences, any head sizes: exp(sink) joins the denominator, the result is multiplied by ``gate_act(gate)`` and ``factor``."""
     pages, pt, G, d = k_cache.shape
     check(_lib.load().ifab_window_attn(q.data_ptr(), q.stride(0), q.shape[1] // heads, k_cache.data_ptr(), v_cache.data_ptr(), _f32(q), positions.data_ptr(), slots.data_ptr(),
                                        page_table.data_ptr(), page_table.shape[1], pt, pages, heads, G, d, v_cache.shape[3], window, scale, cap, _p(slopes), int(chunked), _p(sink), _p(gate),
-                                       0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], int(gate_head), out.data_ptr(), out.stride(0), q.shape[0], status_ptr,
-                                       _s()), "window_attn")
+                                       0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], int(gate_head), *ahead.args, factor, out.data_ptr(), out.stride(0), q.shape[0],
+                                       status_ptr, _s()), "window_attn")
 
 
 SPLIT_KEYS = 64            # fewest keys per split of the split-KV decode form
@@ -115,11 +144,18 @@ class GroupedShape:
     chunked: bool = False
     cap: float = 0.0               # soft limit of the scores
     biased: bool = False           # distance bias with slope 2^(-8 (h + 1) / heads)
-    rot_dims: int = 0              # rotated columns of a head, interleaved pairs
+    rot_dims: int = 0              # rotated columns of a head
     rot_base: float = 10000.0
+    rot_scaling: Optional[RotaryScaling] = None
+    rot_halves: bool = False       # pairs (i, i + rot_dims / 2) instead of neighbours
     norm: bool = False             # rms of all of q and of all of k before the rotation
+    head_norm: bool = False        # rms of every head of q and k instead, without a gain
     keys_are_values: bool = False  # values = keys as projected
     bias: bool = False             # of the q, k and output projections
+    gated: bool = True             # a gate per head
+    keep: int = 0                  # first positions seen beside the window
+    pool: int = 0                  # positions of a block seen beside the window
+    factor: float = 1.0            # of the result
 
     def check(self) -> None:
         if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
@@ -130,13 +166,19 @@ class GroupedShape:
             raise ValueError(f"attention: rotation of {self.rot_dims} columns in heads of {self.dim}")
         if self.window < 0 or self.cap < 0:
             raise ValueError("attention: window and cap must not be negative")
+        if min(self.keep, self.pool) < 0 or (self.keep and self.pool) or ((self.keep or self.pool) and (self.chunked or self.cap or self.biased or not self.window)):
+            raise ValueError(f"attention: {self.keep} kept positions, blocks of {self.pool} beside a window of {self.window} are not supported")
+        if self.rot_scaling:
+            self.rot_scaling.check()
+        if self.norm and self.head_norm:
+            raise ValueError("attention: one norm of q and k at most")
 
     @property
     def offsets(self) -> tuple:
         """Where q, k, v and the head gates start in a projection row, and where it ends."""
         q, k = self.heads * self.dim, self.kv_heads * self.dim
         v = 0 if self.keys_are_values else self.kv_heads * self.vdim
-        return 0, q, q if self.keys_are_values else q + k, q + k + v, q + k + v + self.heads
+        return 0, q, q if self.keys_are_values else q + k, q + k + v, q + k + v + self.heads * self.gated
 
     @property
     def in_cols(self) -> int:
@@ -160,14 +202,26 @@ class GroupedShape:
         """Elements a token holds in the pages."""
         return self.kv_heads * (self.dim + self.vdim)
 
+    def page(self, page_tokens: int) -> int:
+        """Elements of a page, with the entries of the blocks that may end in it."""
+        return self.row * (page_tokens + self.entries(page_tokens))
+
+    def entries(self, page_tokens: int) -> int:
+        return (page_tokens + self.pool - 1) // self.pool if self.pool else 0
+
+    @property
+    def rotation(self) -> tuple:
+        return self.rot_dims, self.rot_base, self.rot_scaling
+
 
 class GroupedBuffers:
     """Work buffers of the grouped attention layers of a model for up to ``rows`` rows; ``chunked``: for packed steps."""
 
-    def __init__(self, shapes, rows: int, dtype: torch.dtype, device, *, chunked: bool, max_context: int, group: int):
+    def __init__(self, shapes, rows: int, dtype: torch.dtype, device, *, chunked: bool, max_context: int, group: int, in_cols: int = 0):
+        """``in_cols``: columns of the projection rows when others share them."""
         self.group = group
         z = lambda *s: torch.zeros(*s, dtype=dtype, device=device)
-        self.proj = z(rows, max(s.in_cols for s in shapes))
+        self.proj = z(rows, max([s.in_cols for s in shapes] + [in_cols]))
         # queries at the stride of the tensor-core tiles where they have one (padding columns stay zero: one buffer per shape)
         self.q = {(s.heads, s.q_stride, s.dim): z(rows, s.heads * s.q_stride) for s in shapes}
         need = [s.heads * s.splits * (s.vdim + 2) for s in shapes if s.splits]
@@ -192,7 +246,7 @@ class GroupedAttention:
         s = shape
         self.shape = s
         get = lambda n: W[p + n].to(device)
-        mats = [get(n).to(dtype) for n in ("q", "k") + (() if s.keys_are_values else ("v",)) + ("g",)]
+        mats = [get(n).to(dtype) for n in ("q", "k") + (() if s.keys_are_values else ("v",)) + (("g",) if s.gated else ())]
         width = mats[0].shape[1]
         self.w_in = torch.zeros(s.in_cols, (width + 7) // 8 * 8, dtype=dtype, device=device)
         self.w_in[:s.offsets[4], :width] = torch.cat(mats, 0)
@@ -202,12 +256,16 @@ class GroupedAttention:
             self.b_in[:s.offsets[1] + s.kv_heads * s.dim] = torch.cat([get("q.b"), get("k.b")]).float()
         vec = lambda n: get(n).float().contiguous() if s.norm else None
         self.q_gain, self.k_gain = vec("q.norm"), vec("k.norm")
+        if s.head_norm:
+            self.q_gain = self.k_gain = torch.ones(s.dim, dtype=torch.float32, device=device)
         self.slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / s.heads) for h in range(s.heads)], dtype=torch.float32, device=device) if s.biased else None
 
     def make_pages(self, pages: int, page_tokens: int, device, dtype: torch.dtype) -> tuple:
+        """Keys and values of the tokens, then - with blocks - of the blocks."""
         s = self.shape
-        z = lambda n: torch.zeros(pages, page_tokens, s.kv_heads, n, dtype=dtype, device=device)
-        return z(s.dim), z(s.vdim)
+        z = lambda m, n: torch.zeros(pages, m, s.kv_heads, n, dtype=dtype, device=device)
+        m = s.entries(page_tokens)
+        return (z(page_tokens, s.dim), z(page_tokens, s.vdim)) + ((z(m, s.dim), z(m, s.vdim)) if m else ())
 
     def project(self, B: GroupedBuffers, xa: torch.Tensor, status_ptr) -> None:
         N.linear(xa, self.w_in, B.proj[:xa.shape[0], :self.shape.in_cols], bias=self.b_in, status_ptr=status_ptr)
@@ -218,20 +276,24 @@ class GroupedAttention:
         proj, q, bf16 = B.proj[:m], B.q[s.heads, s.q_stride, s.dim][:m], B.proj.dtype == torch.bfloat16
         qo, ko, vo, go, _ = s.offsets
         qk_norm_rope_write(proj, (qo, ko, vo), self.q_gain, self.k_gain, eps, heads=s.heads, kv_heads=s.kv_heads, dim=s.dim, vdim=s.vdim, rot=s.rot_dims,
-                           interleaved=True, rope=rope, positions=pos, slots=slot, page_table=table, q_out=q, k_cache=pages[0], v_cache=pages[1], whole=s.norm,
-                           status_ptr=status_ptr)
-        gate = proj[:, go:]
-        how = dict(heads=s.heads, window=s.window, scale=s.scale, gate_act="sigmoid", gate_head=True, chunked=s.chunked, cap=s.cap, slopes=self.slopes,
-                   status_ptr=status_ptr)
-        tiled = plan is not None and bool(plan.runs) and s.tiles and bf16
+                           interleaved=not s.rot_halves, rope=rope, positions=pos, slots=slot, page_table=table, q_out=q, k_cache=pages[0], v_cache=pages[1],
+                           whole=s.norm, status_ptr=status_ptr)
+        ahead, pages = Ahead(s.keep, s.pool, pages[2:] or None), pages[:2]
+        if s.pool:
+            pool_write(*pages, pos, slot, table, ahead, status_ptr)
+        gate = proj[:, go:] if s.gated else None
+        how = dict(heads=s.heads, window=s.window, scale=s.scale, gate_act="sigmoid" if s.gated else None, gate_head=s.gated, chunked=s.chunked, cap=s.cap, slopes=self.slopes,
+                   ahead=ahead, factor=s.factor, status_ptr=status_ptr)
+        plain = not s.keep and not s.pool and s.factor == 1.0
+        tiled = plan is not None and bool(plan.runs) and s.tiles and bf16 and plain
         if tiled:
             k, vt = B.ctx[s.kv_heads, s.q_stride]
             for r, n, sl, p0 in plan.runs:
-                fa_window(q[r:r + n], *pages, table, slot=sl, pos0=p0, ctx_k=k, ctx_vt=vt, out=out[r:r + n], gate=gate[r:r + n], **how)
+                fa_window(q[r:r + n], *pages, table, slot=sl, pos0=p0, ctx_k=k, ctx_vt=vt, out=out[r:r + n], gate=None if gate is None else gate[r:r + n], **how)
         groups = plan.groups if tiled else [(r, min(m, r + B.group)) for r in range(0, m, B.group)]
         rest = plan.step_positions if tiled else pos
-        if s.splits and bf16:
+        if s.splits and bf16 and plain:
             for lo, hi in groups:
-                gqa_window(q[lo:hi], *pages, rest[lo:hi], slot[lo:hi], table, splits=s.splits, scratch=B.scratch, out=out[lo:hi], gate=gate[lo:hi], **how)
+                gqa_window(q[lo:hi], *pages, rest[lo:hi], slot[lo:hi], table, splits=s.splits, scratch=B.scratch, out=out[lo:hi], gate=None if gate is None else gate[lo:hi], **how)
         elif groups:
             window_attn(q, *pages, rest, slot, table, out=out, gate=gate, **how)
