@@ -85,7 +85,25 @@ struct GqaParams {
   const bf16* gate; long ldg; int gate_act;       // the result is multiplied by act(gate [T, Hq * HD]); or null
   int gate_head;                                  // the gate has one value per head instead: [T, Hq]
   ScoreRule rule;
+  AheadRule ahead;                                // entries that count as the first keys of a row
+  float factor;                                   // of the result
 };
+
+// what a row sees: entries ahead of its window, then the positions first .. pos
+struct Seen {
+  int first, ahead, n;
+  __device__ __forceinline__ Seen(const GqaParams& p, int pos) : first(first_key(pos, p.window, p.rule.chunked)) {
+    ahead = p.ahead.count(first);
+    n = ahead + pos + 1 - first;
+  }
+};
+// row of key k of what a row sees; `pooled`: in the caches of the blocks
+__device__ __forceinline__ long key_row(const GqaParams& p, const Seen& seen, int k, int slot, bool* pooled) {
+  *pooled = k < seen.ahead && p.ahead.pool > 0;
+  const int pos = k < seen.ahead ? p.ahead.position(k) : seen.first + k - seen.ahead;
+  const long r = row_of(pos, slot, p.page_table, p.max_pages, p.page_tokens, p.num_pages);
+  return *pooled && r >= 0 ? r / p.page_tokens * p.ahead.per_page + p.ahead.row(k, p.page_tokens) : r;
+}
 
 // HD = head_dim (EPL = HD/32 elements per lane), G = query heads per kv head
 template <int HD, int G>
@@ -100,7 +118,8 @@ __global__ void __launch_bounds__(256) gqa_split_kernel(GqaParams p) {
   const int split = blockIdx.x, kvh = blockIdx.y, t = blockIdx.z;
   const int pos = p.positions[t];
   if (pos < 0) return;
-  const int first = first_key(pos, p.window, p.rule.chunked), n = pos + 1 - first;
+  const Seen seen(p, pos);
+  const int n = seen.n;
   const int k_begin = split * p.kps;
   if (k_begin >= n) return;
   // the last split also takes every key beyond max_splits * keys_per_split, so a long context is slower, never clipped
@@ -132,13 +151,14 @@ __global__ void __launch_bounds__(256) gqa_split_kernel(GqaParams p) {
       const int k = kb + 8 * j;
       ok[j] = k < k_end;
       if (ok[j]) {
-        const long r = row_of(first + k, slot, p.page_table, p.max_pages, p.page_tokens, p.num_pages);
+        bool pooled;
+        const long r = key_row(p, seen, k, slot, &pooled);
         if (r < 0) {
           if (lane == 0 && p.status) atomicOr(p.status, IFAB_STATUS_BAD_INDEX);
           ok[j] = false;
         } else {
-          const bf16* kr = p.k_cache + r * kv_elems + (long)kvh * HD + lane * EPL;
-          const bf16* vr = p.v_cache + r * kv_elems + (long)kvh * HD + lane * EPL;
+          const bf16* kr = (pooled ? (const bf16*)p.ahead.k : p.k_cache) + r * kv_elems + (long)kvh * HD + lane * EPL;
+          const bf16* vr = (pooled ? (const bf16*)p.ahead.v : p.v_cache) + r * kv_elems + (long)kvh * HD + lane * EPL;
 #pragma unroll
           for (int i = 0; i < EPL; i += 2) {
             const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(kr + i));
@@ -215,7 +235,8 @@ __global__ void __launch_bounds__(256, 2) gqa_split_shared_kernel(GqaParams p) {
   const int split = blockIdx.x, kvh = blockIdx.y, t = blockIdx.z;
   const int pos = p.positions[t];
   if (pos < 0) return;
-  const int first = first_key(pos, p.window, p.rule.chunked), n = pos + 1 - first;
+  const Seen seen(p, pos);
+  const int n = seen.n;
   const int k_begin = split * p.kps;
   if (k_begin >= n) return;
   const int k_end = (split == p.max_splits - 1) ? n : min(n, k_begin + p.kps);
@@ -246,13 +267,14 @@ __global__ void __launch_bounds__(256, 2) gqa_split_shared_kernel(GqaParams p) {
       ok[b] = k < k_end;
       kr[b] = vr[b] = make_uint4(0, 0, 0, 0);
       if (ok[b]) {
-        const long r = row_of(first + k, slot, p.page_table, p.max_pages, p.page_tokens, p.num_pages);
+        bool pooled;
+        const long r = key_row(p, seen, k, slot, &pooled);
         if (r < 0) {
           if (sub == 0 && p.status) atomicOr(p.status, IFAB_STATUS_BAD_INDEX);
           ok[b] = false;
         } else {
-          kr[b] = *reinterpret_cast<const uint4*>(p.k_cache + r * kv_elems + head);
-          vr[b] = *reinterpret_cast<const uint4*>(p.v_cache + r * kv_elems + head);
+          kr[b] = *reinterpret_cast<const uint4*>((pooled ? (const bf16*)p.ahead.k : p.k_cache) + r * kv_elems + head);
+          vr[b] = *reinterpret_cast<const uint4*>((pooled ? (const bf16*)p.ahead.v : p.v_cache) + r * kv_elems + head);
         }
       }
     }
@@ -352,7 +374,7 @@ __global__ void gqa_merge_kernel(GqaParams p, bf16* out, long ldo) {
   const int h = blockIdx.x, t = blockIdx.y;
   const int pos = p.positions[t];
   if (pos < 0) return;
-  const int n = pos + 1 - first_key(pos, p.window, p.rule.chunked);
+  const int n = Seen(p, pos).n;
   int ns = (n + p.kps - 1) / p.kps;
   if (ns > p.max_splits) ns = p.max_splits;
   const float* base = p.scratch + ((long)t * p.Hq + h) * p.max_splits * (HD + 2);
@@ -369,7 +391,7 @@ __global__ void gqa_merge_kernel(GqaParams p, bf16* out, long ldo) {
     if (threadIdx.x == 0) Ls = L;
   }
   __syncthreads();
-  const float invL = Ls > 0.f ? 1.f / Ls : 0.f;
+  const float invL = Ls > 0.f ? p.factor / Ls : 0.f;
   for (int c = threadIdx.x; c < HD; c += blockDim.x) {
     float v = 0.f;
     for (int s = 0; s < ns; ++s) v += wgt[s] * base[(long)s * (HD + 2) + c];
@@ -419,21 +441,25 @@ extern "C" int ifab_gqa_decode_attention(const void* q, long ldq, const void* k_
                                          int head_dim, int keys_per_split, int max_splits, float* scratch,
                                          uint64_t scratch_bytes, void* out, long ldo, uint32_t* status, void* stream) {
   return ifab_gqa_window_attention(q, ldq, k_cache, v_cache, positions, slots, page_table, max_pages, page_tokens, num_pages, scale, 0, 0.f, nullptr, 0, nullptr, nullptr,
-                                   0, 0, 0, T, Hq, Hkv, head_dim, keys_per_split, max_splits, scratch, scratch_bytes, out, ldo, status, stream);
+                                   0, 0, 0, 0, 0, nullptr, nullptr, 1.f, T, Hq, Hkv, head_dim, keys_per_split, max_splits, scratch, scratch_bytes, out, ldo, status, stream);
 }
 
 // The same over the last `window` positions (0: all) or, `chunked`, the query's own stretch of as many; with a cap of the scores (0: none), slopes [Hq]
-// of the distance bias, a sink logit per query head in the denominator and an output gate, [T, Hq * HD] or [T, Hq].
+// of the distance bias, a sink logit per query head in the denominator and an output gate, [T, Hq * HD] or [T, Hq]; entries ahead of the window
+// (attn_rule.cuh); a factor on the result.
 extern "C" int ifab_gqa_window_attention(const void* q, long ldq, const void* k_cache, const void* v_cache, const int32_t* positions, const int32_t* slots,
                                          const int32_t* page_table, int max_pages, int page_tokens, int num_pages, float scale, int window, float cap,
-                                         const float* slopes, int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, int T, int Hq, int Hkv, int head_dim,
+                                         const float* slopes, int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, int keep, int pool, const void* pool_k,
+                                         const void* pool_v, float factor, int T, int Hq, int Hkv, int head_dim,
                                          int keys_per_split, int max_splits, float* scratch, uint64_t scratch_bytes, void* out, long ldo,
                                          uint32_t* status, void* stream) {
   if (Hkv < 1 || Hq % Hkv || max_splits < 1 || max_splits > 64 || keys_per_split < 8 || window < 0 || cap < 0.f) return -1;
+  const AheadRule ahead = ahead_rule(keep, pool, pool_k, pool_v, page_tokens);
+  if (!ahead_ok(ahead, window, chunked) || (ahead.any() && (cap > 0.f || slopes))) return -1;
   if ((uint64_t)T * Hq * max_splits * (head_dim + 2) * sizeof(float) > scratch_bytes) return -5;
   GqaParams p{(const bf16*)q, ldq, (const bf16*)k_cache, (const bf16*)v_cache, positions, slots, page_table,
               max_pages, page_tokens, num_pages, scale, window, T, Hq, Hkv, keys_per_split, max_splits, scratch, status, sink, (const bf16*)gate, ldg,
-              gate_act, gate_per_head, {cap, slopes, chunked}};
+              gate_act, gate_per_head, {cap, slopes, chunked}, ahead, factor};
   cudaStream_t s = (cudaStream_t)stream;
   switch (head_dim) {
     case 64: return dispatch_g<64>(p, (bf16*)out, ldo, s);

@@ -54,6 +54,9 @@ struct FaParams {
   int chunked;                               // `window` is the size of the stretches that queries stay in (attn_rule.cuh)
   float cap_log2, cap_exp;                   // RULED: cap * log2(e) (0: no cap) and 2 * scale * log2(e) / cap
   const float* slopes;                       // RULED: distance bias [H], or null
+  AheadRule ahead;                           // entries ahead of the windows: rows 0 .. of the context operands, filled up to `ahead_rows` (whole key tiles)
+  int ahead_rows, base;                      // base: position of the row behind them
+  float factor;                              // of the result
   int ordered;                               // blockIdx.y counts places in `order`: query tiles with most key tiles first (else query tiles)
   uint8_t order[64];
 };
@@ -100,7 +103,8 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
   const int last_row = min(q0 + BQ, p.m) - 1;
   const int t_end = min((p.ctx + BKEY - 1) / BKEY, (p.pos0 + last_row) / BKEY + 1);
   const int t_begin = first_key(p.pos0 + q0, p.window, p.chunked) / BKEY;
-  const int n_tiles = t_end - t_begin;
+  const int t_ahead = p.ahead_rows ? (p.ahead.count(p.base + first_key(p.pos0 + last_row, p.window, p.chunked)) + BKEY - 1) / BKEY : 0;
+  const int n_tiles = t_ahead + t_end - t_begin;
 
   if (threadIdx.x == 0) {
     mbar_init(&B->q_full, 1);
@@ -140,7 +144,7 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
     for (int pp = 0; pp < NQ; ++pp) tma_load_2d(Qs + pp * PANEL_BYTES, &tmap_q, &B->q_full, h * p.q_head_stride + pp * 64, q0);
     int armed_k = 0, armed_v = 0;
     for (int j = 0; j < n_tiles && !*abort_flag; ++j) {
-      const int key0 = (t_begin + j) * BKEY, s = j % KST, round = j / KST;
+      const int key0 = j < t_ahead ? j * BKEY : p.ahead_rows + (t_begin + j - t_ahead) * BKEY, s = j % KST, round = j / KST;
       if (round > 0 && !mbar_wait(&B->k_empty[s], (round - 1) & 1, p.spin_limit)) { fail(); break; }
       unsigned char* kd = Ks + s * NQ * PANEL_BYTES;
       mbar_expect_tx(&B->k_full[s], NQ * PANEL_BYTES);
@@ -206,6 +210,7 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
     const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
     const int q_pos = p.pos0 + q0 + r;
     const int lo = first_key(q_pos, p.window, p.chunked);       // first visible key
+    const int last_ahead = p.ahead_rows ? p.ahead.count(p.base + lo) - 1 : -1;
     const float slope = RULED && p.slopes ? p.slopes[h] * 1.4426950408889634f : 0.f;
     constexpr int HK = BKEY / PARTS, HV = DV / PARTS;
     float m_ref = -INFINITY, l_run = 0.f;     // reference maximum (base-2 domain, may lag the true maximum by up to 8); sum over this thread's columns
@@ -243,7 +248,9 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
       return true;
     };
     for (int j = 0; j < n_tiles && ok; ++j) {
-      const int key0 = (t_begin + j) * BKEY + half * HK, s = j & 1;
+      const bool front = j < t_ahead;                            // a tile of entries ahead of the windows
+      const int key0 = (front ? j : t_begin + j - t_ahead) * BKEY + half * HK, s = j & 1;
+      const int first_seen = front ? 0 : lo, last_seen = front ? last_ahead : q_pos;
       // the warp leaves the loop together: the TMEM accesses and the votes below are warp-wide
       if (!__all_sync(0xffffffffu, mbar_wait(&B->s_full[s], (j >> 1) & 1, p.spin_limit) && !*abort_flag)) { ok = false; break; }
       tc_fence_after();
@@ -279,7 +286,7 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
         const int key = key0 + i;
         float z = sv[i];
         if (RULED) z -= slope * (float)(q_pos - key);
-        sv[i] = (key <= q_pos && key >= lo) ? z : -INFINITY;
+        sv[i] = (key <= last_seen && key >= first_seen) ? z : -INFINITY;
         mx[i & 3] = fmaxf(mx[i & 3], sv[i]);
       }
       const float my_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
@@ -361,7 +368,7 @@ __global__ void __launch_bounds__(THREADS, 1) fa_prefill_kernel(const __grid_con
       if (lane == 0) fail();
     } else if (q0 + r < p.m) {
       if (p.sink) l_run += exp2f(p.sink[h] * 1.4426950408889634f - m_ref);
-      float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv = l_run > 0.f ? p.factor / l_run : 0.f;
       if (p.gate && p.gate_head) inv *= activate<true>(__bfloat162float(p.gate[(long)(q0 + r) * p.ldg + h]), p.gate_act);
       const int c0 = half * HV;
       bf16* dst = p.out + (long)(q0 + r) * p.ldo + (long)h * p.e + c0;
@@ -409,6 +416,7 @@ int launch_fa(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& t
     for (int i = 0; i < tiles; ++i) {
       const int last = std::min((i + 1) * BQ, p.m) - 1;
       cost[i] = (p.pos0 + last) / BKEY - first_key(p.pos0 + i * BQ, p.window, p.chunked) / BKEY;
+      if (p.ahead_rows) cost[i] += (p.ahead.count(p.base + first_key(p.pos0 + last, p.window, p.chunked)) + BKEY - 1) / BKEY;
       p.order[i] = (uint8_t)i;
     }
     std::stable_sort(p.order, p.order + tiles, [&](uint8_t a, uint8_t b) { return cost[a] > cost[b]; });
@@ -442,7 +450,7 @@ extern "C" int ifab_fa_prefill_bf16(const void* q, long ldq, int q_head_stride, 
   }
   if (int rc = make_tmap_bf16_2d(&tv, vt, (uint64_t)vt_rows, (uint64_t)ctx, (uint64_t)ldvt, DV)) return rc;
   FaParams p{(bf16*)out, ldo, m, ctx, kv_group, pos0, window, q_head_stride, k_head_stride, vt_head_stride, vt_row0,
-             scale * 1.4426950408889634f, DV, nullptr, nullptr, 0, 0, 0, status, 4000000u, 0, 0.f, 0.f, nullptr, 0, {}};
+             scale * 1.4426950408889634f, DV, nullptr, nullptr, 0, 0, 0, status, 4000000u, 0, 0.f, 0.f, nullptr, {}, 0, 0, 1.f, 0, {}};
   cudaStream_t s = (cudaStream_t)stream;
   if (d1 == 128 && d2 == 64) return launch_fa<2, 1>(tq, tk, tk2, tv, p, H, s);
   if (d1 == 128 && d2 == 0) return launch_fa<2, 0>(tq, tk, tk2, tv, p, H, s);
@@ -454,22 +462,27 @@ extern "C" int ifab_fa_prefill_bf16(const void* q, long ldq, int q_head_stride, 
 // of any width: q [m, H * (d + d2)] and k [ctx, G * d] with d in {64, 128} columns per head (narrower heads are zero-padded by the caller),
 // k2 [ctx, d2] key columns shared by all heads (d2 0 or 64), vt [G * 128, ldvt >= ctx] (rows past a narrower value head are zero), out
 // [m, H * e], e <= 128; gate [m, H * e], or [m, H] with gate_per_head. `chunked`: `window` is the size of the stretches queries stay in (position 0 of
-// the operands starts one); cap (0: none) and slopes [H] (or null) act on the scores (attn_rule.cuh), without k2.
+// the operands starts one); cap (0: none) and slopes [H] (or null) act on the scores (attn_rule.cuh), without k2. keep / pool: entries ahead of the
+// windows (attn_rule.cuh) lie in rows / columns 0 .. of k and vt, zero-filled up to ahead_rows (a multiple of 128); the ctx positions, of which the
+// first is position `base` of the sequence, follow them. factor: of the result.
 extern "C" int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const void* k2, long ldk2, int d2, const void* vt, long ldvt, void* out, long ldo,
                                    int m, int ctx, int H, int kv_group, int d, int e, int pos0, int window, float scale, float cap, const float* slopes,
-                                   int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, uint32_t* status, void* stream) {
+                                   int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, int keep, int pool,
+                                   int ahead_rows, int base, float factor, uint32_t* status, void* stream) {
   if (m < 1 || ctx < 1 || H < 1 || kv_group < 1 || H % kv_group || pos0 < 0 || pos0 + m > ctx || window < 0) return -1;
-  if ((d != 64 && d != 128) || (d2 != 0 && d2 != 64) || (d2 && (!k2 || ldk2 % 8)) || e < 1 || e > DV || ldq % 8 || ldk % 8 || ldvt % 8 || ldvt < ctx) return -1;
+  if (ahead_rows < 0 || ahead_rows % BKEY || base < 0 || (ahead_rows && ((keep > 0) == (pool > 0) || !window || chunked || cap > 0.f || slopes || d2))) return -1;
+  if ((d != 64 && d != 128) || (d2 != 0 && d2 != 64) || (d2 && (!k2 || ldk2 % 8)) || e < 1 || e > DV || ldq % 8 || ldk % 8 || ldvt % 8 || ldvt < ctx + ahead_rows) return -1;
   const int G = H / kv_group;
   CUtensorMap tq, tk, tk2, tv;
   if (int rc = make_tmap_bf16_2d(&tq, q, (uint64_t)m, (uint64_t)H * (d + d2), (uint64_t)ldq, BQ)) return rc;
-  if (int rc = make_tmap_bf16_2d(&tk, k, (uint64_t)ctx, (uint64_t)G * d, (uint64_t)ldk, BKEY)) return rc;
+  if (int rc = make_tmap_bf16_2d(&tk, k, (uint64_t)(ahead_rows + ctx), (uint64_t)G * d, (uint64_t)ldk, BKEY)) return rc;
   tk2 = tk;
   if (d2)
     if (int rc = make_tmap_bf16_2d(&tk2, k2, (uint64_t)ctx, (uint64_t)d2, (uint64_t)ldk2, BKEY)) return rc;
-  if (int rc = make_tmap_bf16_2d(&tv, vt, (uint64_t)G * DV, (uint64_t)ctx, (uint64_t)ldvt, DV)) return rc;
+  if (int rc = make_tmap_bf16_2d(&tv, vt, (uint64_t)G * DV, (uint64_t)(ahead_rows + ctx), (uint64_t)ldvt, DV)) return rc;
   FaParams p{(bf16*)out, ldo, m, ctx, kv_group, pos0, window, d + d2, d, DV, 0, scale * 1.4426950408889634f, e, sink, (const bf16*)gate, ldg, gate_act,
-             gate_per_head, status, 4000000u, chunked, cap * 1.4426950408889634f, cap > 0.f ? 2.f * scale * 1.4426950408889634f / cap : 0.f, slopes, 0, {}};
+             gate_per_head, status, 4000000u, chunked, cap * 1.4426950408889634f, cap > 0.f ? 2.f * scale * 1.4426950408889634f / cap : 0.f, slopes, ahead_rule(keep, pool, nullptr, nullptr, 1), ahead_rows, base,
+             factor, 0, {}};
   cudaStream_t s = (cudaStream_t)stream;
   if (cap > 0.f || slopes)
     return d2 ? -1 : d == 128 ? launch_fa<2, 0, true, true>(tq, tk, tk2, tv, p, H, s) : launch_fa<1, 0, true, true>(tq, tk, tk2, tv, p, H, s);

@@ -383,10 +383,12 @@ int ifab_gr_finish(const float* o, long ldo, int H, int e, int E, const float* m
                    int gate_first, int groups, float eps, const float* gain, void* y, long ldy, int f32, int T, void* stream);
 /* operands of the tensor-core windowed attention: keys / values first .. first + n - 1 of a sequence, heads zero-padded to dp / 128 columns */
 int ifab_ctx_gather_pad(const void* k_cache, const void* v_cache, const int32_t* page_table, int slot, int max_pages, int page_tokens, int num_pages,
-                        int first, int n, int rows, int G, int d, int dp, int e, void* k, void* vt, long ldvt, uint32_t* status, void* stream);
+                        int first, int n, int rows, int keep, int pool, const void* pool_k, const void* pool_v, int n_ahead, int ahead_rows, int G, int d, int dp, int e, void* k,
+                        void* vt, long ldvt, uint32_t* status, void* stream);
 int ifab_fa_window_bf16(const void* q, long ldq, const void* k, long ldk, const void* k2, long ldk2, int d2, const void* vt, long ldvt, void* out, long ldo,
                         int m, int ctx, int H, int kv_group, int d, int e, int pos0, int window, float scale, float cap, const float* slopes, int chunked,
-                        const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, uint32_t* status, void* stream);
+                        const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, int keep, int pool, int ahead_rows, int base, float factor,
+                        uint32_t* status, void* stream);
 /* latent attention over paged rows [latent padded to Lp | rotated key part padded to Rp], any sizes, bf16 or f32 (latent_attn.cu). splits <= 64, the last
  * takes what is left of the keys a row sees; scratch f32 [T, H, splits, Lp + 2] */
 int ifab_latent_prepare(const void* proj, long ldp, int f32, int q_off, int q_rank, int kv_off, int kv_rank, int rot_dim, const float* q_gain,
@@ -414,8 +416,8 @@ int ifab_latent_gather(const void* cache, const int32_t* page_table, int slot, i
                        int Rp, int tile, void* lat, void* rot, uint32_t* status, void* stream);
 int ifab_gqa_window_attention(const void* q, long ldq, const void* k_cache, const void* v_cache, const int32_t* positions, const int32_t* slots,
                               const int32_t* page_table, int max_pages, int page_tokens, int num_pages, float scale, int window, float cap, const float* slopes,
-                              int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, int T, int Hq, int Hkv, int head_dim, int keys_per_split, int max_splits,
-                              float* scratch, uint64_t scratch_bytes, void* out, long ldo, uint32_t* status, void* stream);
+                              int chunked, const float* sink, const void* gate, long ldg, int gate_act, int gate_per_head, int keep, int pool, const void* pool_k, const void* pool_v,
+                              float factor, int T, int Hq, int Hkv, int head_dim, int keys_per_split, int max_splits, float* scratch, uint64_t scratch_bytes, void* out, long ldo, uint32_t* status, void* stream);
 /* indexer: q bf16 [T, heads, dim], w f32 [T, heads], keys paged bf16 [pages, page_tokens, dim]; scores = scratch f32 [T, ctx];
  * out int32 [T, topk]: the top-k key positions (<= the query position) in ascending order, -1 padded */
 int ifab_sparse_index(const void* q, const float* w, const void* keys, const int32_t* positions, const int32_t* slots,

@@ -281,23 +281,29 @@ struct WinParams {
   float factor;                  // of the result
 };
 
-// Keys and values first .. first + n - 1 of one sequence out of its pages: k [rows, G * dp] (columns d .. dp - 1 of a head zero) and
+// The first n_ahead entries ahead of a window (rows 0 .. ahead_rows - 1, zero-filled), then keys and values first .. first + n - 1 of one sequence out of its pages: k [rows, G * dp] (columns d .. dp - 1 of a head zero) and
 // transposed values vt [G * 128, ld] (rows e .. 127 of a head zero), rows / columns from n on zero - the operands of the tensor-core
 // attention. grid (ceil(rows / 32), G): one CTA per 32 keys of a head, values turned through shared memory.
 __global__ void __launch_bounds__(256) ctx_gather_pad_kernel(const bf16* k_cache, const bf16* v_cache, const int32_t* page_table, int slot, int max_pages,
-                                                             int page_tokens, int num_pages, int first, int n, int G, int d, int dp, int e, bf16* k,
-                                                             bf16* vt, long ldvt, uint32_t* status) {
+                                                             int page_tokens, int num_pages, int first, int n, AheadRule ahead, int n_ahead, int ahead_rows,
+                                                             int G, int d, int dp, int e, bf16* k, bf16* vt, long ldvt, uint32_t* status) {
   __shared__ bf16 tile[32][128 + 2];
   __shared__ long src_row[32];
   grid_dep_launch();
   grid_dep_wait();
   const int j0 = blockIdx.x * 32, g = blockIdx.y, t = threadIdx.x;
+  const bool front = j0 < ahead_rows, pooled = front && ahead.pool > 0;
+  if (pooled) {
+    k_cache = reinterpret_cast<const bf16*>(ahead.k);
+    v_cache = reinterpret_cast<const bf16*>(ahead.v);
+  }
   if (t < 32) {
     long row = -1;
-    if (j0 + t < n) {
-      const int pos = first + j0 + t, lp = pos / page_tokens;
+    const int i = front ? j0 + t : j0 + t - ahead_rows;
+    if (i < (front ? n_ahead : n)) {
+      const int pos = front ? ahead.position(i) : first + i, lp = pos / page_tokens;
       const int page = lp < max_pages ? page_table[(long)slot * max_pages + lp] : -1;
-      if (page >= 0 && page < num_pages) row = (long)page * page_tokens + pos % page_tokens;
+      if (page >= 0 && page < num_pages) row = pooled ? (long)page * ahead.per_page + ahead.row(i, page_tokens) : (long)page * page_tokens + pos % page_tokens;
       else if (status) atomicOr(status, IFAB_STATUS_BAD_INDEX);
     }
     src_row[t] = row;
@@ -536,12 +542,14 @@ extern "C" int ifab_window_attn(const void* q, long ldq, int q_stride, const voi
 }
 
 extern "C" int ifab_ctx_gather_pad(const void* k_cache, const void* v_cache, const int32_t* page_table, int slot, int max_pages, int page_tokens,
-                                   int num_pages, int first, int n, int rows, int G, int d, int dp, int e, void* k, void* vt, long ldvt, uint32_t* status,
-                                   void* stream) {
-  if (n < 1 || rows < n || rows % 32 || slot < 0 || first < 0 || G < 1 || d < 1 || dp < d || e < 1 || e > 128 || ldvt < rows || dp % 8 || ldvt % 8) return -1;
+                                   int num_pages, int first, int n, int rows, int keep, int pool, const void* pool_k, const void* pool_v, int n_ahead, int ahead_rows,
+                                   int G, int d, int dp, int e, void* k, void* vt, long ldvt, uint32_t* status, void* stream) {
+  const AheadRule ahead = ahead_rule(keep, pool, pool_k, pool_v, page_tokens);
+  if (!ahead_ok(ahead, 1, 0) || n_ahead < 0 || ahead_rows < n_ahead || ahead_rows % 32 || (n_ahead && !ahead.any())) return -1;
+  if (n < 1 || rows < n || rows % 32 || slot < 0 || first < 0 || G < 1 || d < 1 || dp < d || e < 1 || e > 128 || ldvt < rows + ahead_rows || dp % 8 || ldvt % 8) return -1;
   if (((reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(vt)) & 15)) return -1;
-  return launch_chain(ctx_gather_pad_kernel, dim3(rows / 32, G), dim3(256), 0, (cudaStream_t)stream, (const bf16*)k_cache, (const bf16*)v_cache, page_table,
-                      slot, max_pages, page_tokens, num_pages, first, n, G, d, dp, e, (bf16*)k, (bf16*)vt, ldvt, status);
+  return launch_chain(ctx_gather_pad_kernel, dim3((rows + ahead_rows) / 32, G), dim3(256), 0, (cudaStream_t)stream, (const bf16*)k_cache, (const bf16*)v_cache,
+                      page_table, slot, max_pages, page_tokens, num_pages, first, n, ahead, n_ahead, ahead_rows, G, d, dp, e, (bf16*)k, (bf16*)vt, ldvt, status);
 }
 
 extern "C" int ifab_rope_table(const int32_t* positions, const double* freq, void* cs, int T, int pairs, void* stream) {

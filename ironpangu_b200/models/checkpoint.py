@@ -24,7 +24,7 @@ def save(path, cfg, weights: Dict[str, torch.Tensor]) -> None:
     (d / "config.json").write_text(json.dumps(cfg.to_dict(), indent=1))
     hdr, blobs, at = {}, [], 0
     for n, t in weights.items():
-        raw = t.detach().to(torch.bfloat16).cpu().contiguous().view(torch.uint8).numpy().tobytes()
+        raw = t.detach().to(torch.bfloat16).cpu().contiguous().reshape(-1).view(torch.uint8).numpy().tobytes()
         hdr[n] = {"dtype": "BF16", "shape": list(t.shape), "data_offsets": [at, at + len(raw)]}
         blobs.append(raw)
         at += len(raw)

@@ -80,11 +80,12 @@ _SIGS = {
     "ifab_la_chunks": [_P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, _P, _P, c_u64, _P, _P, c_long, _P],
     "ifab_qk_norm_rope_write": [_P, c_long, c_int, c_int, c_int, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_int, c_int,
                                 c_int, _P, c_long, c_int, _P, _P, c_int, c_int, _P, _P],
-    "ifab_ctx_gather_pad": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_long, _P, _P],
+    "ifab_ctx_gather_pad": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_long,
+                            _P, _P],
     "ifab_fa_window_bf16": [_P, c_long, _P, c_long, _P, c_long, c_int, _P, c_long, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                            c_float, c_float, _P, c_int, _P, _P, c_long, c_int, c_int, _P, _P],
+                            c_float, c_float, _P, c_int, _P, _P, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P],
     "ifab_gqa_window_attention": [_P, c_long, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, c_float, _P, c_int, _P, _P, c_long, c_int, c_int, c_int, c_int,
-                                  c_int, c_int, c_int, c_int, _P, c_u64, _P, c_long, _P, _P],
+                                  _P, _P, c_float, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_u64, _P, c_long, _P, _P],
     "ifab_window_attn": [_P, c_long, c_int, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, _P, c_int, _P, _P,
                          c_long, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, c_long, c_int, _P, _P],
     "ifab_pool_write": [_P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, _P],

@@ -261,7 +261,7 @@ class LatentMixer:
         q, out, gate = self._q(B)[lo:lo + n], B.mixed[H * s.vdim][lo:lo + n], B.proj[lo:lo + n, s.gate_off:]
         check(lib.ifab_fa_window_bf16(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), rot.data_ptr(), rot.stride(0), 64, vt.data_ptr(), vt.stride(0),
                                       out.data_ptr(), out.stride(0), n, ctx, H, 1, n1, s.vdim, pos0 - first, s.window, s.scale, 0.0, None, 0, None, gate.data_ptr(),
-                                      gate.stride(0), ACTIVATIONS["sigmoid"], 1, status_ptr, _s()), "fa_window")
+                                      gate.stride(0), ACTIVATIONS["sigmoid"], 1, 0, 0, 0, 0, 1.0, status_ptr, _s()), "fa_window")
 
     def mix(self, B: LatentBuffers, m: int, rope, pos, slot, plan, table, eps: float, status_ptr) -> None:
         """``m`` rows of a packed step (``plan``), or decode rows (None), from ``B.proj`` to ``B.mixed`` as matrix products and row kernels."""

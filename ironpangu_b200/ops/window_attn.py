@@ -34,6 +34,10 @@ class Ahead:
         k, v = self.pages or (None, None)
         return self.keep, self.pool, _p(k), _p(v)
 
+    def count(self, first: int) -> int:
+        """Entries that a query sees whose window starts at position ``first`` (at most)."""
+        return min(self.keep, first) if self.keep else first // self.pool if self.pool else 0
+
 
 NOTHING_AHEAD = Ahead()
 
@@ -76,25 +80,26 @@ SPLIT_KEYS = 64            # fewest keys per split of the split-KV decode form
 SPLIT_CTAS = 600           # CTAs the splits of a launch aim at: more rows, longer splits
 
 
-def split_form(heads: int, kv_heads: int, dim: int, vdim: int, window: int) -> int:
-    """Most splits the split-KV decode kernels take for this shape, 0 when it needs the general kernel."""
+def split_form(heads: int, kv_heads: int, dim: int, vdim: int, window: int, ahead: int = 0) -> int:
+    """Most splits the split-KV decode kernels take for this shape (``ahead``: most entries ahead of a window), 0 when it needs the general kernel."""
     if dim != vdim or dim not in (64, 128, 256) or heads // kv_heads not in (1, 2, 4, 8) or (dim == 256 and heads // kv_heads == 8) or not window:
         return 0
-    return max(1, min(64, (window + SPLIT_KEYS - 1) // SPLIT_KEYS))
+    return max(1, min(64, (window + ahead + SPLIT_KEYS - 1) // SPLIT_KEYS))
 
 
 def gqa_window(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, page_table: torch.Tensor, *,
                heads: int, window: int, scale: float, splits: int, scratch: torch.Tensor, out: torch.Tensor, sink: Optional[torch.Tensor] = None,
                gate: Optional[torch.Tensor] = None, gate_act: Optional[str] = None, gate_head: bool = False, chunked: bool = False, cap: float = 0.0,
-               slopes: Optional[torch.Tensor] = None, status_ptr=None) -> None:
-    """:func:`window_attn` by splits of the window (query heads of a group share the key loads), bf16, shapes of :func:`split_form`.
-    ``splits``: the most to use; launches of many rows use fewer, longer ones."""
+               slopes: Optional[torch.Tensor] = None, ahead: Ahead = NOTHING_AHEAD, most_ahead: int = 0, factor: float = 1.0, status_ptr=None) -> None:
+    """:func:`window_attn` by splits of what a row sees (query heads of a group share the key loads), bf16, shapes of :func:`split_form`.
+    ``splits``: the most to use; launches of many rows use fewer, longer ones. ``most_ahead``: how many entries ahead of its window a row may see."""
     pages, pt, G, d = k_cache.shape
     splits = max(1, min(splits, SPLIT_CTAS // (q.shape[0] * G)))
-    kps = ((window + splits - 1) // splits + 31) // 32 * 32
+    kps = ((window + most_ahead + splits - 1) // splits + 31) // 32 * 32
     check(_lib.load().ifab_gqa_window_attention(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), positions.data_ptr(), slots.data_ptr(),
                                                 page_table.data_ptr(), page_table.shape[1], pt, pages, scale, window, cap, _p(slopes), int(chunked), _p(sink), _p(gate),
-                                                0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], int(gate_head), q.shape[0], heads, G, d, kps, splits,
+                                                0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], int(gate_head), *ahead.args, factor, q.shape[0], heads, G, d,
+                                                kps, splits,
                                                 scratch.data_ptr(), scratch.numel() * 4, out.data_ptr(), out.stride(0), status_ptr, _s()), "gqa_window")
 
 
@@ -108,26 +113,34 @@ def context_rows(count: int, window: int) -> int:
     return (count + window - 1 + 31) // 32 * 32
 
 
+def ahead_rows(count: int) -> int:
+    """Context rows that ``count`` entries ahead of the windows take: whole key tiles."""
+    return (count + 127) // 128 * 128
+
+
 def fa_window(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor, *, slot: int, pos0: int, heads: int, window: int,
               scale: float, ctx_k: torch.Tensor, ctx_vt: torch.Tensor, out: torch.Tensor, sink: Optional[torch.Tensor] = None,
               gate: Optional[torch.Tensor] = None, gate_act: Optional[str] = None, gate_head: bool = False, chunked: bool = False, cap: float = 0.0,
-              slopes: Optional[torch.Tensor] = None, status_ptr=None) -> None:
+              slopes: Optional[torch.Tensor] = None, ahead: Ahead = NOTHING_AHEAD, factor: float = 1.0, status_ptr=None) -> None:
     """Prompt attention of consecutive positions ``pos0 ..`` of one sequence (keys already in its pages) on the tensor cores: the keys
     and values the rows can see are gathered out of the pages into ``ctx_k`` ``[rows, kv_heads * tile]`` / ``ctx_vt`` ``[kv_heads * 128,
-    rows]``. ``q``: ``[m, heads * tile]``, columns past the head width zero; ``window`` 0: the whole context."""
+    rows]``, entries ahead of the windows first. ``q``: ``[m, heads * tile]``, columns past the head width zero; ``window`` 0: the whole context."""
     pages, pt, G, d = k_cache.shape
     m, e = q.shape[0], v_cache.shape[3]
     dp = q.shape[1] // heads
     first = 0 if not window else pos0 // window * window if chunked else max(0, pos0 - window + 1)
     n = pos0 + m - first
     rows = (n + 31) // 32 * 32
-    assert dp == tile_width(d) and e <= 128 and ctx_k.shape[0] >= rows and ctx_vt.shape[1] >= rows and ctx_k.shape[1] == G * dp
+    seen = ahead.count(max(0, pos0 + m - window)) if window else 0         # by the last row
+    front = ahead_rows(seen)
+    assert dp == tile_width(d) and e <= 128 and ctx_k.shape[0] >= front + rows and ctx_vt.shape[1] >= front + rows and ctx_k.shape[1] == G * dp
     lib = _lib.load()
-    check(lib.ifab_ctx_gather_pad(k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr(), slot, page_table.shape[1], pt, pages, first, n, rows, G, d,
-                                  dp, e, ctx_k.data_ptr(), ctx_vt.data_ptr(), ctx_vt.stride(0), status_ptr, _s()), "ctx_gather_pad")
+    check(lib.ifab_ctx_gather_pad(k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr(), slot, page_table.shape[1], pt, pages, first, n, rows, *ahead.args,
+                                  seen, front, G, d, dp, e, ctx_k.data_ptr(), ctx_vt.data_ptr(), ctx_vt.stride(0), status_ptr, _s()), "ctx_gather_pad")
     check(lib.ifab_fa_window_bf16(q.data_ptr(), q.stride(0), ctx_k.data_ptr(), ctx_k.stride(0), None, 0, 0, ctx_vt.data_ptr(), ctx_vt.stride(0), out.data_ptr(),
                                   out.stride(0), m, n, heads, heads // G, dp, e, pos0 - first, window, scale, cap, _p(slopes), int(chunked), _p(sink), _p(gate),
-                                  0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], int(gate_head), status_ptr, _s()), "fa_window")
+                                  0 if gate is None else gate.stride(0), ACTIVATIONS[gate_act], int(gate_head), ahead.keep, ahead.pool, front, first, factor, status_ptr, _s()),
+          "fa_window")
 
 
 # ---------------------------------------------------------------------------------------------------------------------------
@@ -193,9 +206,12 @@ class GroupedShape:
     def q_stride(self) -> int:
         return tile_width(self.dim) if self.tiles else self.dim
 
-    @property
-    def splits(self) -> int:
-        return split_form(self.heads, self.kv_heads, self.dim, self.vdim, self.window) if self.q_stride == self.dim else 0
+    def most_ahead(self, context: int) -> int:
+        """Most entries a row sees ahead of its window in sequences of ``context`` positions."""
+        return Ahead(self.keep, self.pool).count(max(0, context - self.window)) if self.window else 0
+
+    def splits(self, context: int) -> int:
+        return split_form(self.heads, self.kv_heads, self.dim, self.vdim, self.window, self.most_ahead(context)) if self.q_stride == self.dim else 0
 
     @property
     def row(self) -> int:
@@ -224,14 +240,15 @@ class GroupedBuffers:
         self.proj = z(rows, max([s.in_cols for s in shapes] + [in_cols]))
         # queries at the stride of the tensor-core tiles where they have one (padding columns stay zero: one buffer per shape)
         self.q = {(s.heads, s.q_stride, s.dim): z(rows, s.heads * s.q_stride) for s in shapes}
-        need = [s.heads * s.splits * (s.vdim + 2) for s in shapes if s.splits]
-        self.scratch = torch.empty(min(rows, group) * max(need), dtype=torch.float32, device=device) if need and dtype == torch.bfloat16 else None
+        self.context = max_context
+        need = [s.heads * s.splits(max_context) * (s.vdim + 2) for s in shapes]
+        self.scratch = torch.empty(min(rows, group) * max(need), dtype=torch.float32, device=device) if any(need) and dtype == torch.bfloat16 else None
         self.ctx = {}
         if chunked and dtype == torch.bfloat16:
             for s in shapes:
                 cap = (max_context + 31) // 32 * 32
                 if s.window:
-                    cap = min(cap, context_rows(rows, s.window))
+                    cap = min(cap, context_rows(rows, s.window)) + ahead_rows(s.most_ahead(max_context))
                 key = (s.kv_heads, s.q_stride)
                 if s.tiles and (key not in self.ctx or self.ctx[key][0].shape[0] < cap):
                     self.ctx[key] = z(cap, s.kv_heads * s.q_stride), z(s.kv_heads * 128, cap)
@@ -284,16 +301,17 @@ class GroupedAttention:
         gate = proj[:, go:] if s.gated else None
         how = dict(heads=s.heads, window=s.window, scale=s.scale, gate_act="sigmoid" if s.gated else None, gate_head=s.gated, chunked=s.chunked, cap=s.cap, slopes=self.slopes,
                    ahead=ahead, factor=s.factor, status_ptr=status_ptr)
-        plain = not s.keep and not s.pool and s.factor == 1.0
-        tiled = plan is not None and bool(plan.runs) and s.tiles and bf16 and plain
+        tiled = plan is not None and bool(plan.runs) and s.tiles and bf16
         if tiled:
             k, vt = B.ctx[s.kv_heads, s.q_stride]
             for r, n, sl, p0 in plan.runs:
                 fa_window(q[r:r + n], *pages, table, slot=sl, pos0=p0, ctx_k=k, ctx_vt=vt, out=out[r:r + n], gate=None if gate is None else gate[r:r + n], **how)
         groups = plan.groups if tiled else [(r, min(m, r + B.group)) for r in range(0, m, B.group)]
         rest = plan.step_positions if tiled else pos
-        if s.splits and bf16 and plain:
+        splits = s.splits(B.context) if bf16 else 0
+        if splits:
             for lo, hi in groups:
-                gqa_window(q[lo:hi], *pages, rest[lo:hi], slot[lo:hi], table, splits=s.splits, scratch=B.scratch, out=out[lo:hi], gate=None if gate is None else gate[lo:hi], **how)
+                gqa_window(q[lo:hi], *pages, rest[lo:hi], slot[lo:hi], table, splits=splits, most_ahead=s.most_ahead(B.context), scratch=B.scratch,
+                           out=out[lo:hi], gate=None if gate is None else gate[lo:hi], **how)
         elif groups:
             window_attn(q, *pages, rest, slot, table, out=out, gate=gate, **how)
