@@ -34,7 +34,7 @@ def parse():
     ap.add_argument("--impl", default="native", choices=["native", "reference", "nccl_cublas"])
     ap.add_argument("--model", default="flagship", choices=["flagship", "tiny", "dense2b"],
                     help="flagship: the 92B-class MLA+MoE model of the headline metric; dense2b: the Qwen-style 2B dense GQA decoder")
-    ap.add_argument("--design", default="", choices=["", "falinex", "ponenex", "mikutar"],
+    ap.add_argument("--design", default="", choices=["", "falinex", "ponenex", "mikutar", "fubelorn"],
                     help="instead of the headline run, prefill and decode throughput of a design beside its closest other model at equal size, one JSON "
                          "line per size (one GPU): falinex beside the dense model (ironpangu_b200/utils/bench_falinex.py), ponenex beside the MLA + MoE "
                          "model (bench_ponenex.py), mikutar beside ponenex and the dense model (bench_mikutar.py)")

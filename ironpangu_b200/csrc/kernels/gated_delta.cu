@@ -19,10 +19,11 @@ constexpr int C = GR_CHUNK, EB = 16;
 struct LocalSmem {
   float a[C][C + 1], t[C][C + 1], tmp[C / 2][C / 2 + 1];
   float x[C][68];
-  GrFactors f;
+  GrFactors<GR_CHUNK> f;
 };
 
 // grid (n, H), 256 threads
+template <typename A>
 __global__ void __launch_bounds__(256) gr_delta_local_kernel(GrChunks p, GrState st, float* w_rows, float* u_rows) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   LocalSmem& S = *reinterpret_cast<LocalSmem*>(smem_raw);
@@ -37,7 +38,7 @@ __global__ void __launch_bounds__(256) gr_delta_local_kernel(GrChunks p, GrState
     __syncthreads();
     for (int i = tid; i < C * 64; i += 256) {
       const int j = i >> 6, x = i & 63;
-      S.x[x][j] = (j < L && d0 + x < r.d) ? r.k[((long)(row0 + j) * r.G + g) * r.d + d0 + x] : 0.f;
+      S.x[x][j] = (j < L && d0 + x < r.d) ? gr_k<A>(r, row0 + j, g, d0 + x) : 0.f;
     }
     __syncthreads();
     const int n = min(64, r.d - d0);
@@ -99,7 +100,7 @@ __global__ void __launch_bounds__(256) gr_delta_local_kernel(GrChunks p, GrState
       const int j = i >> 6, x = i & 63;
       float v = 0.f;
       if (j < L && c0 + x < n) {
-        v = val ? r.v[((long)(row0 + j) * r.H + h) * n + c0 + x] : r.k[((long)(row0 + j) * r.G + g) * n + c0 + x];
+        v = val ? gr_v<A>(r, row0 + j, h, c0 + x) : gr_k<A>(r, row0 + j, g, c0 + x);
         v *= val ? S.f.w[j] : S.f.w[j] * expf((float)S.f.total[j]);
       }
       S.x[j][x] = v;
@@ -128,10 +129,11 @@ __global__ void __launch_bounds__(256) gr_delta_local_kernel(GrChunks p, GrState
 struct ScanSmem {
   float x[C][68];            // 64 columns of T (b g k), or of the decayed keys, [row][column]
   float u[C][EB + 4];
-  GrFactors f;
+  GrFactors<GR_CHUNK> f;
 };
 
 // grid (ceil(E / EB), H, n): CTAs of a run's first chunk walk its chunks. Dynamic shared memory: ScanSmem, then the state slice [d][EB]
+template <typename A>
 __global__ void __launch_bounds__(256) gr_delta_scan_kernel(GrChunks p, GrState st, const float* w_rows, float* u_rows) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   ScanSmem& S = *reinterpret_cast<ScanSmem*>(smem_raw);
@@ -197,7 +199,7 @@ __global__ void __launch_bounds__(256) gr_delta_scan_kernel(GrChunks p, GrState 
       __syncthreads();
       for (int i = tid; i < C * 64; i += 256) {
         const int j = i >> 6, x = i & 63;
-        S.x[j][x] = (j < L && x < n) ? r.k[((long)(row0 + j) * r.G + g) * r.d + d0 + x] : 0.f;
+        S.x[j][x] = (j < L && x < n) ? gr_k<A>(r, row0 + j, g, d0 + x) : 0.f;
       }
       __syncthreads();
       if (sx < n) {
@@ -226,10 +228,15 @@ __global__ void __launch_bounds__(256) gr_delta_scan_kernel(GrChunks p, GrState 
 
 }  // namespace
 
-int ifab::gr_delta_chunks(const GrChunks& p, const GrState& st, float* w_rows, float* u_rows, cudaStream_t s) {
-  if (int rc = opt_in_smem(gr_delta_local_kernel, sizeof(LocalSmem))) return rc;
-  if (int rc = launch_chain(gr_delta_local_kernel, dim3(p.n, p.r.H), dim3(256), sizeof(LocalSmem), s, p, st, w_rows, u_rows)) return rc;
+template <typename A>
+static int chunks(const GrChunks& p, const GrState& st, float* w_rows, float* u_rows, cudaStream_t s) {
+  if (int rc = opt_in_smem(gr_delta_local_kernel<A>, sizeof(LocalSmem))) return rc;
+  if (int rc = launch_chain(gr_delta_local_kernel<A>, dim3(p.n, p.r.H), dim3(256), sizeof(LocalSmem), s, p, st, w_rows, u_rows)) return rc;
   const size_t smem = (sizeof(ScanSmem) + 15) / 16 * 16 + (size_t)p.r.d * EB * sizeof(float);
-  if (int rc = opt_in_smem(gr_delta_scan_kernel, smem)) return rc;
-  return launch_chain(gr_delta_scan_kernel, dim3((p.r.E + EB - 1) / EB, p.r.H, p.n), dim3(256), smem, s, p, st, (const float*)w_rows, u_rows);
+  if (int rc = opt_in_smem(gr_delta_scan_kernel<A>, smem)) return rc;
+  return launch_chain(gr_delta_scan_kernel<A>, dim3((p.r.E + EB - 1) / EB, p.r.H, p.n), dim3(256), smem, s, p, st, (const float*)w_rows, u_rows);
+}
+
+int ifab::gr_delta_chunks(const GrChunks& p, const GrState& st, int f32, float* w_rows, float* u_rows, cudaStream_t s) {
+  return f32 ? chunks<float>(p, st, w_rows, u_rows, s) : chunks<bf16>(p, st, w_rows, u_rows, s);
 }

@@ -1,17 +1,17 @@
-// Recurrences over a matrix state per head with a decay per token, for any head sizes; everything in f32:
+// Recurrences over a matrix state per head with a decay per token, for any head sizes; states, gates and products in f32:
 //
 //   SSD      S = a S + w k v^T                                   o = S^T q      (state-space duality: a = exp(-exp(A) dt), w = dt)
 //   DELTA    S = a S,  u = w (v - S^T k),  S += k u^T            o = S^T q      (gated delta rule: w = beta)
 //   MEMORY   m' = max(f + m, i),  S = exp(f + m - m') S + exp(i - m') k v^T     (exponential gates; one more value column of ones keeps
 //            the sum of the keys, so that S^T q ends with n q)
 //
-//   gr_prepare_kernel  packed projection rows -> q, k, v in f32 (short causal convolution + SiLU, unit vectors or a factor) and the
-//                      gates (softplus, exponentials, soft limits), one CTA per row. The convolution reads rows of the step and the
+//   gr_prepare_kernel  packed projection rows -> q, k, v (short causal convolution + SiLU) in the activation type, the factors that make q and k
+//                      unit vectors, and the gates (softplus, exponentials, soft limits). The convolution reads rows of the step and the
 //                      sequence's last taps - 1 rows before it (history [slots, 2, taps - 1, C] in the activation type, two sides by epoch as in
 //                      hyper_streams.cu)
 //   gr_step_kernel     decode: one CTA per (head, run of rows of one slot, 32 value columns); a run walks its rows through the state.
 //                      The grid depends on the row count only (graph capture)
-//   prompts, by chunks of 64 consecutive rows of one sequence:
+//   prompts, by chunks of 64 consecutive rows of one sequence with f32 products (the tensor-core form: gated_tiles.cu):
 //     gr_maximum_kernel  MEMORY: the running maximum of every row
 //     gr_state_kernel    what a chunk adds to the state; gr_scan_kernel: the states ahead of every chunk (DELTA: gated_delta.cu)
 //     gr_out_kernel      the outputs of a chunk from the state ahead of it and from its rows
@@ -29,8 +29,8 @@ namespace {
 struct Section {
   int col, heads, n;          // where it starts in a projection row, heads and columns of a head
   int channel;                // of the convolution, -1: none
-  float scale; int unit;      // a factor; unit: divided by sqrt(sum of squares + 1e-6) first
-  float* dst; int stride;     // f32 [T, heads * stride]; columns past n get 1
+  void* dst;                  // [T, heads * n]
+  float* factors; float factor;      // [T, heads]: factor / sqrt(sum of squares + 1e-6); or null
 };
 
 struct PrepareParams {
@@ -42,75 +42,114 @@ struct PrepareParams {
   const float *a_log, *decay_bias, *weight_bias; float cap;
   float *log_decay, *weight;
   const int32_t *positions, *slots;
-  int T;
+  int T, rows;                // rows of a CTA
 };
 
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
-// grid T, 256 threads: a warp per head
-template <typename A>
+template <typename A, int V>
+__device__ __forceinline__ void load_v(const A* p, float* f) {
+  if constexpr (V == 4 && sizeof(A) == 2) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else if constexpr (V == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  } else {
+    f[0] = to_f32(*p);
+  }
+}
+template <typename A, int V>
+__device__ __forceinline__ void store_v(A* p, const float* f) {
+  if constexpr (V == 4 && sizeof(A) == 2) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+  } else if constexpr (V == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  } else {
+    *p = from_f32<A>(f[0]);
+  }
+}
+
+// grid (ceil(heads of all sections / 8) + 1, ceil(T / rows)), 256 threads: a warp per head, V columns per lane at a time; the last CTAs make the gates
+template <typename A, int V>
 __global__ void __launch_bounds__(256) gr_prepare_kernel(PrepareParams p) {
   grid_dep_launch();
   grid_dep_wait();
-  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const A* row = reinterpret_cast<const A*>(p.proj) + (long)t * p.ldp;
-  const int pos = p.positions[t], slot = p.slots[t], back = p.taps - 1;
-  if (pos < 0) return;
-  int run = 0;                // rows of the sequence ahead of this one in the step
-  while (run < back && t - run - 1 >= 0 && p.slots[t - run - 1] == slot) ++run;
-  const int side = p.taps > 1 ? p.epoch[slot] & 1 : 0;
-  const A* old = reinterpret_cast<const A*>(p.history) + ((long)slot * 2 + side) * back * p.C;
-  A* fresh = reinterpret_cast<A*>(p.history) + ((long)slot * 2 + (side ^ 1)) * back * p.C;
-  const bool last = p.taps > 1 && (t + 1 == p.T || p.slots[t + 1] != slot);
-  const int total = p.sec[0].heads + p.sec[1].heads + p.sec[2].heads;
-  for (int i = warp; i < total; i += 8) {
-    const int which = i < p.sec[0].heads ? 0 : i < p.sec[0].heads + p.sec[1].heads ? 1 : 2;
-    const Section& s = p.sec[which];
-    const int h = i - (which > 0 ? p.sec[0].heads : 0) - (which > 1 ? p.sec[1].heads : 0);
-    float* dst = s.dst + ((long)t * s.heads + h) * s.stride;
-    float ss = 0.f;
-    for (int c = lane; c < s.n; c += 32) {
-      const int col = h * s.n + c;
-      float v = to_f32(row[s.col + col]);
-      if (s.channel >= 0) {
-        const int ch = s.channel + col;
-        if (last) fresh[ch] = row[s.col + col];
-        v *= p.taps_w[(long)back * p.C + ch];
-        for (int j = 1; j < p.taps; ++j) {
-          A b = from_f32<A>(0.f);
-          if (j <= pos) b = j <= run ? row[s.col + col - (long)j * p.ldp] : old[(long)(j - run - 1) * p.C + ch];
-          v = fmaf(p.taps_w[(long)(back - j) * p.C + ch], to_f32(b), v);
-          if (last && j < back) fresh[(long)j * p.C + ch] = b;
-        }
-        if (p.bias) v += p.bias[ch];
-        v *= sigmoid_f32(v);
-      }
-      if (s.unit) {
-        dst[c] = v;
-        ss = fmaf(v, v, ss);
+  const int t0 = blockIdx.y * p.rows, t1 = min(p.T, t0 + p.rows), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (blockIdx.x == gridDim.x - 1) {
+    for (int i = threadIdx.x; i < (t1 - t0) * p.H; i += 256) {
+      const int t = t0 + i / p.H, h = i % p.H;
+      const A* row = reinterpret_cast<const A*>(p.proj) + (long)t * p.ldp;
+      const float a = to_f32(row[p.decay_col + h]) + (p.decay_bias ? p.decay_bias[h] : 0.f), b = to_f32(row[p.weight_col + h]) + (p.weight_bias ? p.weight_bias[h] : 0.f);
+      float g, w;
+      if (p.kind == GR_MEMORY) {
+        g = -softplus(-p.cap * tanhf(a / p.cap));
+        w = p.cap * tanhf(b / p.cap);
       } else {
-        dst[c] = v * s.scale;
+        const float sp = softplus(a);
+        g = -expf(p.a_log[h]) * sp;
+        w = p.kind == GR_SSD ? sp : sigmoid_f32(b);
       }
+      p.log_decay[(long)t * p.H + h] = g;
+      p.weight[(long)t * p.H + h] = w;
     }
-    if (s.unit) {
-      const float f = s.scale / sqrtf(warp_sum(ss) + 1e-6f);
-      for (int c = lane; c < s.n; c += 32) dst[c] *= f;
-    }
-    for (int c = s.n + lane; c < s.stride; c += 32) dst[c] = 1.f;
+    return;
   }
-  for (int h = threadIdx.x; h < p.H; h += 256) {
-    const float a = to_f32(row[p.decay_col + h]) + (p.decay_bias ? p.decay_bias[h] : 0.f), b = to_f32(row[p.weight_col + h]) + (p.weight_bias ? p.weight_bias[h] : 0.f);
-    float g, w;
-    if (p.kind == GR_MEMORY) {
-      g = -softplus(-p.cap * tanhf(a / p.cap));
-      w = p.cap * tanhf(b / p.cap);
-    } else {
-      const float sp = softplus(a);
-      g = -expf(p.a_log[h]) * sp;
-      w = p.kind == GR_SSD ? sp : sigmoid_f32(b);
+  const int i = blockIdx.x * 8 + warp, h0 = p.sec[0].heads, h1 = h0 + p.sec[1].heads;
+  if (i >= h1 + p.sec[2].heads) return;
+  const Section& s = p.sec[i < h0 ? 0 : i < h1 ? 1 : 2];
+  const int h = i - (i < h0 ? 0 : i < h1 ? h0 : h1), back = p.taps - 1;
+  for (int t = t0; t < t1; ++t) {
+    const int pos = p.positions[t], slot = p.slots[t];
+    if (pos < 0) continue;
+    const A* row = reinterpret_cast<const A*>(p.proj) + (long)t * p.ldp + s.col + h * s.n;
+    A* dst = reinterpret_cast<A*>(s.dst) + ((long)t * s.heads + h) * s.n;
+    int run = 0;                // rows of the sequence ahead of this one in the step
+    while (run < back && t - run - 1 >= 0 && p.slots[t - run - 1] == slot) ++run;
+    const int side = p.taps > 1 ? p.epoch[slot] & 1 : 0, ch0 = s.channel + h * s.n;
+    const A* old = reinterpret_cast<const A*>(p.history) + ((long)slot * 2 + side) * back * p.C + ch0;
+    A* fresh = reinterpret_cast<A*>(p.history) + ((long)slot * 2 + (side ^ 1)) * back * p.C + ch0;
+    const bool last = p.taps > 1 && (t + 1 == p.T || p.slots[t + 1] != slot);
+    float ss = 0.f;
+    for (int c = lane * V; c < s.n; c += 32 * V) {
+      float v[V];
+      load_v<A, V>(row + c, v);
+      if (s.channel >= 0) {
+        float w[V], x[V], acc[V];
+        load_v<float, V>(p.taps_w + (long)back * p.C + ch0 + c, w);
+#pragma unroll
+        for (int u = 0; u < V; ++u) acc[u] = v[u] * w[u];
+        if (last) store_v<A, V>(fresh + c, v);
+        for (int j = 1; j < p.taps; ++j) {
+          if (j <= pos) {
+            load_v<A, V>(j <= run ? row + c - (long)j * p.ldp : old + (long)(j - run - 1) * p.C + c, x);
+            load_v<float, V>(p.taps_w + (long)(back - j) * p.C + ch0 + c, w);
+#pragma unroll
+            for (int u = 0; u < V; ++u) acc[u] = fmaf(w[u], x[u], acc[u]);
+          } else {
+#pragma unroll
+            for (int u = 0; u < V; ++u) x[u] = 0.f;
+          }
+          if (last && j < back) store_v<A, V>(fresh + (long)j * p.C + c, x);
+        }
+        if (p.bias) {
+          load_v<float, V>(p.bias + ch0 + c, w);
+#pragma unroll
+          for (int u = 0; u < V; ++u) acc[u] += w[u];
+        }
+#pragma unroll
+        for (int u = 0; u < V; ++u) v[u] = to_f32(from_f32<A>(acc[u] * sigmoid_f32<sizeof(A) == 2>(acc[u])));
+      }
+      store_v<A, V>(dst + c, v);
+#pragma unroll
+      for (int u = 0; u < V; ++u) ss = fmaf(v[u], v[u], ss);
     }
-    p.log_decay[(long)t * p.H + h] = g;
-    p.weight[(long)t * p.H + h] = w;
+    if (s.factors) {
+      ss = warp_sum(ss);
+      if (lane == 0) s.factors[(long)t * s.heads + h] = s.factor / sqrtf(ss + 1e-6f);
+    }
   }
 }
 
@@ -124,7 +163,7 @@ struct StepParams {
 };
 
 // a warp owns 4 value columns = rows of the state, lanes their d columns (float4s: REG of them per lane; 0: any d, one column at a time)
-template <int REG>
+template <typename A, int REG>
 __global__ void __launch_bounds__(256) gr_step_kernel(StepParams p) {
   grid_dep_launch();
   grid_dep_wait();
@@ -151,8 +190,8 @@ __global__ void __launch_bounds__(256) gr_step_kernel(StepParams p) {
   }
   bool first = empty;
   for (int t = t0; t < p.T && p.slots[t] == slot && p.positions[t] >= 0; ++t) {
-    const float *q = r.q + ((long)t * r.G + g) * d, *k = r.k + ((long)t * r.G + g) * d;
-    const float* vr = r.v + ((long)t * r.H + h) * r.E + col0;
+    const A *q = reinterpret_cast<const A*>(r.q) + ((long)t * r.G + g) * d, *k = reinterpret_cast<const A*>(r.k) + ((long)t * r.G + g) * d;
+    const float fq = r.qs ? r.qs[(long)t * r.G + g] : r.q_factor, fk = r.ks ? r.ks[(long)t * r.G + g] : 1.f;
     const float ld = r.log_decay[(long)t * r.H + h];
     float w = r.weight[(long)t * r.H + h], a;
     if (r.kind == GR_MEMORY) {
@@ -166,14 +205,19 @@ __global__ void __launch_bounds__(256) gr_step_kernel(StepParams p) {
     }
     float v[4], acc[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-    for (int u = 0; u < 4; ++u) v[u] = u < nc ? vr[u] : 0.f;
+    for (int u = 0; u < 4; ++u) v[u] = u < nc ? gr_v<A>(r, t, h, col0 + u) : 0.f;
     if (REG) {
       float4 kr[R], qr[R];
 #pragma unroll
       for (int x = 0; x < R; ++x) {
         const int c = (lane + 32 * x) * 4;
-        kr[x] = c < d ? *reinterpret_cast<const float4*>(k + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-        qr[x] = c < d ? *reinterpret_cast<const float4*>(q + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        float a4[4] = {0.f, 0.f, 0.f, 0.f}, b4[4] = {0.f, 0.f, 0.f, 0.f};
+        if (c < d) {
+          load_v<A, 4>(k + c, a4);
+          load_v<A, 4>(q + c, b4);
+        }
+        kr[x] = make_float4(a4[0] * fk, a4[1] * fk, a4[2] * fk, a4[3] * fk);
+        qr[x] = make_float4(b4[0] * fq, b4[1] * fq, b4[2] * fq, b4[3] * fq);
       }
       float kk[4];
 #pragma unroll
@@ -206,7 +250,7 @@ __global__ void __launch_bounds__(256) gr_step_kernel(StepParams p) {
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
           float kk = 0.f;
-          for (int c = lane; c < d && u < nc; c += 32) kk = fmaf(k[c], S[(long)u * d + c], kk);
+          for (int c = lane; c < d && u < nc; c += 32) kk = fmaf(to_f32(k[c]) * fk, S[(long)u * d + c], kk);
           v[u] = fmaf(-a, warp_sum(kk), v[u]);
         }
       }
@@ -214,9 +258,9 @@ __global__ void __launch_bounds__(256) gr_step_kernel(StepParams p) {
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
           if (u >= nc) break;
-          const float x = fmaf(k[c], w * v[u], first ? 0.f : a * S[(long)u * d + c]);
+          const float x = fmaf(to_f32(k[c]) * fk, w * v[u], first ? 0.f : a * S[(long)u * d + c]);
           S[(long)u * d + c] = x;
-          acc[u] = fmaf(q[c], x, acc[u]);
+          acc[u] = fmaf(to_f32(q[c]) * fq, x, acc[u]);
         }
     }
     first = false;
@@ -238,46 +282,78 @@ __global__ void __launch_bounds__(256) gr_step_kernel(StepParams p) {
   if (r.kind == GR_MEMORY && blockIdx.z == 0 && threadIdx.x == 0) p.st.m[((long)slot * 2 + (side ^ 1)) * r.H + h] = m;
 }
 
-// grid (H, chunks), 32 threads: CTAs of a run's first chunk walk its rows, 32 at a time. m_t = G_t + max(m_0, max over j <= t of (i_j - G_j)), G the sums of f
-__global__ void __launch_bounds__(32) gr_maximum_kernel(GrChunks p, GrState st) {
+// grid (H, chunks), 256 threads: CTAs of a run's first chunk walk its rows, 2048 at a time. m_t = G_t + max(m_0, max over j <= t of (i_j - G_j)), G the sums of f
+__global__ void __launch_bounds__(256) gr_maximum_kernel(GrChunks p, GrState st) {
+  constexpr int R = 8;
+  __shared__ double sums[8], tops[8];
   grid_dep_launch();
   grid_dep_wait();
-  const int h = blockIdx.x, c = blockIdx.y, lane = threadIdx.x, meta = p.chunks[c * 4 + 3];
+  const int h = blockIdx.x, c = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, meta = p.chunks[c * 4 + 3];
   if (!(meta & 1)) return;
   const int row0 = p.chunks[c * 4], slot = p.chunks[c * 4 + 2], count = meta >> 1, lc = c + count - 1;
   const int n = p.chunks[lc * 4] + p.chunks[lc * 4 + 1] - row0, side = st.epoch[slot] & 1;
   const GrRows& r = p.r;
   double sum = 0.0, best = p.positions[row0] == 0 ? 0.0 : (double)st.m[((long)slot * 2 + side) * r.H + h];
-  for (int t0 = 0; t0 < n; t0 += 32) {
-    const int t = t0 + lane;
-    const bool live = t < n;
-    const long at = (long)(row0 + (live ? t : 0)) * r.H + h;
-    double G = live ? (double)r.log_decay[at] : 0.0;
-    const double i = live ? (double)r.weight[at] : -INFINITY;
+  for (int t0 = 0; t0 < n; t0 += 256 * R) {
+    const int t = t0 + threadIdx.x * R;
+    float f[R], in[R];
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const long at = (long)(row0 + min(t + i, n - 1)) * r.H + h;
+      f[i] = t + i < n ? r.log_decay[at] : 0.f;
+      in[i] = t + i < n ? r.weight[at] : -INFINITY;
+    }
+    double G = 0.0, b = -INFINITY;      // of this thread's rows, from their start
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      G += (double)f[i];
+      b = fmax(b, (double)in[i] - G);
+    }
+    // of everything up to and with this thread's rows: sums add, a later maximum is moved back by the sums ahead of it
+    double GS = G, bS = b;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const double x = __shfl_up_sync(0xffffffffu, G, o);
-      if (lane >= o) G += x;
+      const double g = __shfl_up_sync(0xffffffffu, GS, o), x = __shfl_up_sync(0xffffffffu, bS, o);
+      if (lane >= o) {
+        bS = fmax(x, bS - g);
+        GS += g;
+      }
     }
-    G += sum;
-    double b = i - G;
+    __syncthreads();
+    if (lane == 31) {
+      sums[warp] = GS;
+      tops[warp] = bS;
+    }
+    __syncthreads();
+    double ahead = sum, top = best;     // up to this thread's rows
+    for (int w = 0; w < warp; ++w) {
+      top = fmax(top, tops[w] - ahead);
+      ahead += sums[w];
+    }
+    const double gl = __shfl_up_sync(0xffffffffu, GS, 1), bl = __shfl_up_sync(0xffffffffu, bS, 1);
+    if (lane > 0) {
+      top = fmax(top, bl - ahead);
+      ahead += gl;
+    }
 #pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const double x = __shfl_up_sync(0xffffffffu, b, o);
-      if (lane >= o) b = fmax(b, x);
+    for (int i = 0; i < R; ++i) {
+      ahead += (double)f[i];
+      top = fmax(top, (double)in[i] - ahead);
+      if (t + i < n) r.m[(long)(row0 + t + i) * r.H + h] = (float)(ahead + top);
+      if (t + i == n - 1) st.m[((long)slot * 2 + (side ^ 1)) * r.H + h] = (float)(ahead + top);
     }
-    b = fmax(b, best);
-    if (live) r.m[at] = (float)(G + b);
-    if (live && t == n - 1) st.m[((long)slot * 2 + (side ^ 1)) * r.H + h] = (float)(G + b);
-    sum = __shfl_sync(0xffffffffu, G, 31);
-    best = __shfl_sync(0xffffffffu, b, 31);
+    for (int w = 0; w < 8; ++w) {
+      best = fmax(best, tops[w] - sum);
+      sum += sums[w];
+    }
   }
 }
 
 // grid (n, H, tiles of 64 x 64 of the state): sum over the chunk's rows of (weight at the chunk's end) k_j v_j^T
+template <typename A>
 __global__ void __launch_bounds__(256) gr_state_kernel(GrChunks p, GrState st) {
   __shared__ float ks[GR_CHUNK][68], vs[GR_CHUNK][68];
-  __shared__ GrFactors f;
+  __shared__ GrFactors<GR_CHUNK> f;
   grid_dep_launch();
   grid_dep_wait();
   const GrRows& r = p.r;
@@ -286,14 +362,14 @@ __global__ void __launch_bounds__(256) gr_state_kernel(GrChunks p, GrState st) {
   gr_load_factors(p, c, h, st, f);
   if (threadIdx.x < GR_CHUNK) {
     const int j = threadIdx.x;
-    vs[j][64] = j < L ? gr_add(f, L, j) : 0.f;
+    vs[j][64] = j < L ? gr_pair(f, L - 1, j) : 0.f;
     if (j == 0 && blockIdx.z == 0) p.cdecay[(long)c * r.H + h] = gr_carry(f, L - 1);
   }
   __syncthreads();
   for (int i = threadIdx.x; i < GR_CHUNK * 64; i += 256) {
     const int j = i >> 6, x = i & 63;
-    ks[j][x] = (j < L && d0 + x < r.d) ? r.k[((long)(row0 + j) * r.G + g) * r.d + d0 + x] * vs[j][64] : 0.f;
-    vs[j][x] = (j < L && e0 + x < r.E) ? r.v[((long)(row0 + j) * r.H + h) * r.E + e0 + x] : 0.f;
+    ks[j][x] = (j < L && d0 + x < r.d) ? gr_k<A>(r, row0 + j, g, d0 + x) * vs[j][64] : 0.f;
+    vs[j][x] = (j < L && e0 + x < r.E) ? gr_v<A>(r, row0 + j, h, e0 + x) : 0.f;
   }
   __syncthreads();
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -363,9 +439,10 @@ __global__ void __launch_bounds__(256) gr_scan_kernel(GrChunks p, float* state) 
 }
 
 // grid (n, H, ceil(E / 64)): o_i = carry_i S^T q_i + sum over j <= i of pair(i, j) (q_i . k_j) v_j
+template <typename A, typename AV>
 __global__ void __launch_bounds__(256) gr_out_kernel(GrChunks p, GrState st) {
   extern __shared__ float sm[];
-  __shared__ GrFactors f;
+  __shared__ GrFactors<GR_CHUNK> f;
   float(*qs)[68] = reinterpret_cast<float(*)[68]>(sm);                 // [column of q][row], one 64-column slice
   float(*ks)[68] = reinterpret_cast<float(*)[68]>(sm + 64 * 68);       // [column of k][row]; then v rows
   float(*ss)[68] = reinterpret_cast<float(*)[68]>(sm + 2 * 64 * 68);   // a slice of the state; then the weights [j][i]
@@ -383,9 +460,8 @@ __global__ void __launch_bounds__(256) gr_out_kernel(GrChunks p, GrState st) {
     for (int i = threadIdx.x; i < GR_CHUNK * 64; i += 256) {
       const int j = i >> 6, x = i & 63;
       const bool ok = j < L && d0 + x < r.d;
-      const long at = ((long)(row0 + j) * r.G + g) * r.d + d0 + x;
-      qs[x][j] = ok ? r.q[at] : 0.f;
-      ks[x][j] = ok ? r.k[at] : 0.f;
+      qs[x][j] = ok ? gr_q<A>(r, row0 + j, g, d0 + x) : 0.f;
+      ks[x][j] = ok ? gr_k<A>(r, row0 + j, g, d0 + x) : 0.f;
       ss[x][j] = (d0 + x < r.d && e0 + j < r.E) ? S[(long)(e0 + j) * r.d + d0 + x] : 0.f;
     }
     __syncthreads();
@@ -417,7 +493,7 @@ __global__ void __launch_bounds__(256) gr_out_kernel(GrChunks p, GrState st) {
   }
   for (int i = threadIdx.x; i < GR_CHUNK * 64; i += 256) {
     const int j = i >> 6, x = i & 63;
-    ks[j][x] = (j < L && e0 + x < r.E) ? r.v[((long)(row0 + j) * r.H + h) * r.E + e0 + x] : 0.f;
+    ks[j][x] = (j < L && e0 + x < r.E) ? gr_v<AV>(r, row0 + j, h, e0 + x) : 0.f;
   }
   __syncthreads();
   for (int j = 0; j < L; ++j) {
@@ -438,20 +514,20 @@ __global__ void __launch_bounds__(256) gr_out_kernel(GrChunks p, GrState st) {
 struct FinishParams {
   const float* o; long ldo; int H, e, E;       // heads of e columns at stride E in a row
   const float *m;                              // MEMORY: [T, H]
-  const float *v, *skip;                       // SSD: [T, H * E] and D [H], or null
+  const void* v; const float* skip;            // SSD: [T, H * e] and D [H], or null
   const void* gate; long ldg; int act, gate_first;
   int groups; float eps; const float* gain;    // [H * e]
   void* y; long ldy;
 };
 
-// grid T, 256 threads; WPG warps per group
+// grid (CTAs of a row's groups, T), 256 threads; WPG warps per group
 template <typename A, int WPG>
 __global__ void __launch_bounds__(256) gr_finish_kernel(FinishParams p) {
   __shared__ float red[33];
   extern __shared__ float den[];               // MEMORY: 1 / the denominator of every head
   grid_dep_launch();
   grid_dep_wait();
-  const int t = blockIdx.x, n = p.H * p.e / p.groups;
+  const int t = blockIdx.y, n = p.H * p.e / p.groups;
   const float* o = p.o + (long)t * p.ldo;
   const A* gate = reinterpret_cast<const A*>(p.gate) + (long)t * p.ldg;
   if (p.m) {
@@ -462,12 +538,12 @@ __global__ void __launch_bounds__(256) gr_finish_kernel(FinishParams p) {
     const int h = c / p.e, j = c - h * p.e;
     float x = o[(long)h * p.E + j];
     if (p.m) x *= den[h];
-    if (p.skip) x = fmaf(p.skip[h], p.v[((long)t * p.H + h) * p.E + j], x);
+    if (p.skip) x = fmaf(p.skip[h], to_f32(reinterpret_cast<const A*>(p.v)[((long)t * p.H + h) * p.e + j]), x);
     *g = activate<sizeof(A) == 2>(to_f32(gate[c]), p.act);
     return p.gate_first ? x * *g : x;
   };
   constexpr int TPG = 32 * WPG, GPB = 8 / WPG;
-  for (int g0 = 0; g0 < p.groups; g0 += GPB) {
+  for (int g0 = blockIdx.x * GPB; g0 < p.groups; g0 += gridDim.x * GPB) {
     const int g = g0 + threadIdx.x / TPG, i0 = threadIdx.x % TPG;
     if (WPG == 1 && g >= p.groups) break;
     float ss = 0.f, z;
@@ -485,81 +561,108 @@ __global__ void __launch_bounds__(256) gr_finish_kernel(FinishParams p) {
 }
 
 bool rows_ok(const GrRows& r) {
-  return r.kind >= GR_SSD && r.kind <= GR_MEMORY && r.H >= 1 && r.G >= 1 && r.H % r.G == 0 && r.d >= 1 && r.E >= 1 && r.d <= 1024 && r.E <= 1024 && r.H <= 65535;
+  return r.kind >= GR_SSD && r.kind <= GR_MEMORY && r.H >= 1 && r.G >= 1 && r.H % r.G == 0 && r.d >= 1 && r.e >= 1 && r.E == r.e + (r.kind == GR_MEMORY) && r.d <= 1024 &&
+         r.E <= 1024 && r.H <= 65535;
 }
 
 }  // namespace
 
-// Sections q, k, v: {column, heads, columns of a head, convolution channel or -1, unit, stride}, scales apart. History in the type of proj.
-extern "C" int ifab_gr_prepare(const void* proj, long ldp, int f32, const int32_t* sections, const float* scales, float* q, float* k, float* v, const float* taps_w,
-                               const float* bias, int taps, int C, void* history, const int32_t* epoch, int kind, int H, int decay_col, int weight_col,
-                               const float* a_log, const float* decay_bias, const float* weight_bias, float cap, float* log_decay, float* weight,
+int ifab::gr_maximum(const GrChunks& p, const GrState& st, cudaStream_t s) { return launch_chain(gr_maximum_kernel, dim3(p.r.H, p.n), dim3(256), 0, s, p, st); }
+
+int ifab::gr_scan(const GrChunks& p, const GrState& st, cudaStream_t s) {
+  const long total = (long)p.r.H * p.r.d * p.r.E;
+  if ((long)p.r.d * p.r.E % 4 == 0) return launch_chain(gr_scan_kernel<4>, dim3((unsigned)((total + 1023) / 1024), p.n), dim3(256), 0, s, p, st.s);
+  return launch_chain(gr_scan_kernel<1>, dim3((unsigned)((total + 255) / 256), p.n), dim3(256), 0, s, p, st.s);
+}
+
+// Sections q, k, v: {column, heads, columns of a head, convolution channel or -1}. factors: of q and k [T, heads] (DELTA), or null. History in the type of proj.
+extern "C" int ifab_gr_prepare(const void* proj, long ldp, int f32, const int32_t* sections, void* q, void* k, void* v, float* q_factors, float* k_factors, float q_factor,
+                               const float* taps_w, const float* bias, int taps, int C, void* history, const int32_t* epoch, int kind, int H, int decay_col,
+                               int weight_col, const float* a_log, const float* decay_bias, const float* weight_bias, float cap, float* log_decay, float* weight,
                                const int32_t* positions, const int32_t* slots, int T, void* stream) {
   if (T < 1 || H < 1 || taps < 0 || taps > 64 || (taps && !taps_w) || (taps > 1 && (!history || !epoch)) || kind < GR_SSD || kind > GR_MEMORY || (kind == GR_MEMORY ? cap <= 0.f : !a_log))
     return -1;
   PrepareParams p{proj, ldp, {}, taps_w, bias, taps, C, history, epoch, kind, H, decay_col, weight_col, a_log, decay_bias, weight_bias, cap, log_decay, weight,
-                  positions, slots, T};
-  float* dst[3] = {q, k, v};
+                  positions, slots, T, T <= 256 ? 1 : 8};
+  void* dst[3] = {q, k, v};
+  float* factors[3] = {q_factors, k_factors, nullptr};
+  const auto odd = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) != 0; };
+  bool four = !((ldp | C) % 4) && !odd(proj) && !odd(history) && !odd(taps_w) && !odd(bias);
+  int heads = 0;
   for (int i = 0; i < 3; ++i) {
-    const int32_t* s = sections + 6 * i;
-    if (s[0] < 0 || s[1] < 1 || s[2] < 1 || s[5] < s[2] || (s[3] >= 0 && (!taps || s[3] + s[1] * s[2] > C))) return -1;
-    p.sec[i] = Section{s[0], s[1], s[2], s[3], scales[i], s[4], dst[i], s[5]};
+    const int32_t* s = sections + 4 * i;
+    if (s[0] < 0 || s[1] < 1 || s[2] < 1 || (s[3] >= 0 && (!taps || s[3] + s[1] * s[2] > C))) return -1;
+    p.sec[i] = Section{s[0], s[1], s[2], s[3], dst[i], factors[i], i == 0 ? q_factor : 1.f};
+    four = four && !((s[0] | s[2] | (s[3] < 0 ? 0 : s[3])) % 4) && !odd(dst[i]);
+    heads += s[1];
   }
-  return f32 ? launch_chain(gr_prepare_kernel<float>, dim3(T), dim3(256), 0, (cudaStream_t)stream, p)
-             : launch_chain(gr_prepare_kernel<bf16>, dim3(T), dim3(256), 0, (cudaStream_t)stream, p);
+  const dim3 grid((heads + 7) / 8 + 1, (T + p.rows - 1) / p.rows);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (grid.y > 65535) return -1;
+  if (four) return f32 ? launch_chain(gr_prepare_kernel<float, 4>, grid, dim3(256), 0, s, p) : launch_chain(gr_prepare_kernel<bf16, 4>, grid, dim3(256), 0, s, p);
+  return f32 ? launch_chain(gr_prepare_kernel<float, 1>, grid, dim3(256), 0, s, p) : launch_chain(gr_prepare_kernel<bf16, 1>, grid, dim3(256), 0, s, p);
 }
 
 // rows at negative positions are skipped
-extern "C" int ifab_gr_step(const float* q, const float* k, const float* v, const float* log_decay, const float* weight, int kind, int H, int G, int d, int E,
-                            float* state, float* m_state, const int32_t* epoch, float* m_rows, const int32_t* positions, const int32_t* slots, float* o, long ldo,
-                            int T, void* stream) {
-  StepParams p{{q, k, v, log_decay, weight, m_rows, kind, H, G, d, E}, {state, m_state, epoch}, positions, slots, o, ldo, m_rows, T};
+extern "C" int ifab_gr_step(const void* q, const void* k, const void* v, int f32, const float* qs, const float* ks, float q_factor, const float* log_decay,
+                            const float* weight, int kind, int H, int G, int d, int e, float* state, float* m_state, const int32_t* epoch, float* m_rows,
+                            const int32_t* positions, const int32_t* slots, float* o, long ldo, int T, void* stream) {
+  const int E = e + (kind == GR_MEMORY);
+  StepParams p{{q, k, v, qs, ks, q_factor, log_decay, weight, m_rows, kind, H, G, d, e, E}, {state, m_state, epoch}, positions, slots, o, ldo, m_rows, T};
   if (T < 1 || T > 65535 || !rows_ok(p.r) || (kind == GR_MEMORY && (!m_state || !epoch || !m_rows))) return -1;
   const dim3 grid(H, T, (E + 31) / 32);
   cudaStream_t s = (cudaStream_t)stream;
-  if (d % 4 || d > 256) return launch_chain(gr_step_kernel<0>, grid, dim3(256), 0, s, p);
-  return d <= 128 ? launch_chain(gr_step_kernel<1>, grid, dim3(256), 0, s, p) : launch_chain(gr_step_kernel<2>, grid, dim3(256), 0, s, p);
+  const int reg = d % 4 || d > 256 ? 0 : d <= 128 ? 1 : 2;
+  if (f32)
+    return reg == 0 ? launch_chain(gr_step_kernel<float, 0>, grid, dim3(256), 0, s, p)
+                    : reg == 1 ? launch_chain(gr_step_kernel<float, 1>, grid, dim3(256), 0, s, p) : launch_chain(gr_step_kernel<float, 2>, grid, dim3(256), 0, s, p);
+  return reg == 0 ? launch_chain(gr_step_kernel<bf16, 0>, grid, dim3(256), 0, s, p)
+                  : reg == 1 ? launch_chain(gr_step_kernel<bf16, 1>, grid, dim3(256), 0, s, p) : launch_chain(gr_step_kernel<bf16, 2>, grid, dim3(256), 0, s, p);
 }
 
-// Chunks of at most 64 rows. scratch: cstate f32 [n, H, E, d], cdecay [n, H]; DELTA: w_rows [T, H, d] and u_rows [T, H, E] (the corrected values)
-extern "C" int ifab_gr_chunks(const float* q, const float* k, const float* v, const float* log_decay, const float* weight, int kind, int H, int G, int d, int E,
-                              const int32_t* chunks, int n, const int32_t* positions, float* cstate, uint64_t cstate_bytes, float* cdecay, float* w_rows,
-                              float* u_rows, float* state, float* m_state, const int32_t* epoch, float* m_rows, float* o, long ldo, void* stream) {
-  GrChunks p{{q, k, v, log_decay, weight, m_rows, kind, H, G, d, E}, chunks, n, positions, cstate, cdecay, o, ldo};
+// Chunks of at most 64 rows. scratch: cstate f32 [n, H, E, d], cdecay [n, H]; DELTA: w_rows [T, H, d] and u_rows [T, H, e] (the corrected values)
+extern "C" int ifab_gr_chunks(const void* q, const void* k, const void* v, int f32, const float* qs, const float* ks, float q_factor, const float* log_decay,
+                              const float* weight, int kind, int H, int G, int d, int e, const int32_t* chunks, int n, const int32_t* positions, float* cstate,
+                              uint64_t cstate_bytes, float* cdecay, float* w_rows, float* u_rows, float* state, float* m_state, const int32_t* epoch, float* m_rows,
+                              float* o, long ldo, void* stream) {
+  const int E = e + (kind == GR_MEMORY);
+  GrChunks p{{q, k, v, qs, ks, q_factor, log_decay, weight, m_rows, kind, H, G, d, e, E}, chunks, n, positions, cstate, cdecay, o, ldo};
   const GrState st{state, m_state, epoch};
   if (n < 1 || n > 65535 || !rows_ok(p.r) || (kind == GR_MEMORY && (!m_state || !epoch || !m_rows)) || (kind == GR_DELTA && (!w_rows || !u_rows))) return -1;
   if ((uint64_t)n * H * d * E * sizeof(float) > cstate_bytes) return -5;
   cudaStream_t s = (cudaStream_t)stream;
   const int td = (d + 63) / 64, te = (E + 63) / 64;
   if (kind == GR_DELTA) {
-    if (int rc = gr_delta_chunks(p, st, w_rows, u_rows, s)) return rc;
+    if (int rc = gr_delta_chunks(p, st, f32, w_rows, u_rows, s)) return rc;
     p.r.v = u_rows;
     p.r.kind = GR_SSD;             // the outputs: corrected values that count once
     p.r.weight = nullptr;
   } else {
     if (kind == GR_MEMORY)
-      if (int rc = launch_chain(gr_maximum_kernel, dim3(H, n), dim3(32), 0, s, p, st)) return rc;
-    if (int rc = launch_chain(gr_state_kernel, dim3(n, H, td * te), dim3(256), 0, s, p, st)) return rc;
-    const long total = (long)H * d * E;
-    if ((long)d * E % 4 == 0) {
-      if (int rc = launch_chain(gr_scan_kernel<4>, dim3((unsigned)((total + 1023) / 1024), n), dim3(256), 0, s, p, state)) return rc;
-    } else {
-      if (int rc = launch_chain(gr_scan_kernel<1>, dim3((unsigned)((total + 255) / 256), n), dim3(256), 0, s, p, state)) return rc;
-    }
+      if (int rc = gr_maximum(p, st, s)) return rc;
+    const dim3 grid(n, H, td * te);
+    if (int rc = f32 ? launch_chain(gr_state_kernel<float>, grid, dim3(256), 0, s, p, st) : launch_chain(gr_state_kernel<bf16>, grid, dim3(256), 0, s, p, st)) return rc;
+    if (int rc = gr_scan(p, st, s)) return rc;
   }
   const size_t smem = 3 * 64 * 68 * sizeof(float);
-  if (int rc = opt_in_smem(gr_out_kernel, smem)) return rc;
-  return launch_chain(gr_out_kernel, dim3(n, H, te), dim3(256), smem, s, p, st);
+  const auto out = [&](auto kernel) {
+    if (int rc = opt_in_smem(kernel, smem)) return rc;
+    return launch_chain(kernel, dim3(n, H, te), dim3(256), smem, s, p, st);
+  };
+  return f32 ? out(gr_out_kernel<float, float>) : kind == GR_DELTA ? out(gr_out_kernel<bf16, float>) : out(gr_out_kernel<bf16, bf16>);
 }
 
 // y [T, H * e]: see the top of the file. m: MEMORY (heads of o end with n q); v, skip: a skip
-extern "C" int ifab_gr_finish(const float* o, long ldo, int H, int e, int E, const float* m, const float* v, const float* skip, const void* gate, long ldg, int act,
+extern "C" int ifab_gr_finish(const float* o, long ldo, int H, int e, int E, const float* m, const void* v, const float* skip, const void* gate, long ldg, int act,
                               int gate_first, int groups, float eps, const float* gain, void* y, long ldy, int f32, int T, void* stream) {
-  if (T < 1 || H < 1 || H > 2048 || e < 1 || E < e || (m && E <= e) || groups < 1 || (H * e) % groups || !gate || !gain || (skip && !v)) return -1;
+  if (T < 1 || T > 65535 || H < 1 || H > 2048 || e < 1 || E < e || (m && E <= e) || groups < 1 || (H * e) % groups || !gate || !gain || (skip && !v)) return -1;
   FinishParams p{o, ldo, H, e, E, m, v, skip, gate, ldg, act, gate_first, groups, eps, gain, y, ldy};
   const size_t smem = m ? (size_t)H * sizeof(float) : 0;
   cudaStream_t s = (cudaStream_t)stream;
-  if (H * e / groups > 256)
-    return f32 ? launch_chain(gr_finish_kernel<float, 8>, dim3(T), dim3(256), smem, s, p) : launch_chain(gr_finish_kernel<bf16, 8>, dim3(T), dim3(256), smem, s, p);
-  return f32 ? launch_chain(gr_finish_kernel<float, 1>, dim3(T), dim3(256), smem, s, p) : launch_chain(gr_finish_kernel<bf16, 1>, dim3(T), dim3(256), smem, s, p);
+  if (H * e / groups > 256) {
+    const dim3 grid(groups < 8 ? groups : 8, T);
+    return f32 ? launch_chain(gr_finish_kernel<float, 8>, grid, dim3(256), smem, s, p) : launch_chain(gr_finish_kernel<bf16, 8>, grid, dim3(256), smem, s, p);
+  }
+  const dim3 grid(T <= 256 ? (groups + 7) / 8 : 1, T);
+  return f32 ? launch_chain(gr_finish_kernel<float, 1>, grid, dim3(256), smem, s, p) : launch_chain(gr_finish_kernel<bf16, 1>, grid, dim3(256), smem, s, p);
 }

@@ -7,6 +7,7 @@
 //                        norm, the convolution and the operand of the next linears. A CTA takes `block` consecutive rows and recomputes h
 //                        of the few rows ahead of them that the convolution reaches (x_out must not be x_in); the last taps - 1
 //                        values of h before a step come from the sequence's history
+//   streams_tile_kernel  the same for steps of many rows: a warp per row up to the norm, then a thread per column group down the rows
 //
 // History [slots, 2, taps - 1, width] f32, newest first, two sides per slot: a step reads the side `epoch[slot]` names and writes the other
 // (ifab_step_epoch turns the epochs over once per step), so rows of a step may be worked on in any order.
@@ -190,6 +191,140 @@ __global__ void __launch_bounds__(THREADS) streams_rows_kernel(StreamsParams p) 
   }
 }
 
+// Shared memory: h of the CTA's rows and of those recomputed ahead of them, then 1 / rms times the gain of each
+template <typename A, int SMAX>
+__global__ void __launch_bounds__(1024) streams_tile_kernel(StreamsParams p) {
+  extern __shared__ __align__(16) float hs[];
+  __shared__ float mix[SMAX * SMAX], in[SMAX], out[SMAX];
+  grid_dep_launch();
+  for (int i = threadIdx.x; i < p.S * p.S; i += blockDim.x) mix[i] = p.mix ? p.mix[i] : 0.f;
+  if ((int)threadIdx.x < p.S) {
+    in[threadIdx.x] = p.in ? p.in[threadIdx.x] : 1.f;
+    out[threadIdx.x] = p.out ? p.out[threadIdx.x] : 0.f;
+  }
+  const float gain = p.gain ? p.gain[0] : 1.f;
+  __syncthreads();
+  grid_dep_wait();
+  const int r0 = blockIdx.x * p.block, r1 = min(p.T, r0 + p.block), back = max(p.taps - 1, 0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int o = 0;                                   // rows of the same run ahead of this CTA's (as many as matter)
+  while (o < back && r0 - o - 1 >= 0 && p.slots[r0 - o - 1] == p.slots[r0]) ++o;
+  const int rows = o + r1 - r0;
+  float* inv = hs + (long)(p.block + back) * p.D;
+  for (int i = warp; i < rows; i += blockDim.x >> 5) {
+    const int r = r0 - o + i;
+    const bool mine = i >= o;
+    const float* xr = p.x_in + (long)r * p.ldr_in;
+    float* h = hs + (long)i * p.D;
+    float ss = 0.f;
+#pragma unroll 2
+    for (int c = lane * 4; c < p.D; c += 128) {
+      Vec<4> x[SMAX], u;
+#pragma unroll
+      for (int s = 0; s < SMAX; ++s)
+        if (s < p.S) x[s] = ld<4>(xr + s * p.lds_in + c);
+      if (p.y) {
+        Vec<4> y = ld<4>(p.y + (long)r * p.ldy + c), n[SMAX];
+        for (int q = 1; q < p.parts; ++q) {
+          const Vec<4> a = ld<4>(p.y + q * p.part_stride + (long)r * p.ldy + c);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) y.f[k] += a.f[k];
+        }
+#pragma unroll
+        for (int t = 0; t < SMAX; ++t) {
+          if (t >= p.S) break;
+#pragma unroll
+          for (int k = 0; k < 4; ++k) n[t].f[k] = out[t] * y.f[k];
+#pragma unroll
+          for (int s = 0; s < SMAX; ++s) {
+            if (s >= p.S) break;
+#pragma unroll
+            for (int k = 0; k < 4; ++k) n[t].f[k] = fmaf(mix[s * p.S + t], x[s].f[k], n[t].f[k]);
+          }
+          if (mine && p.x_out) st<4>(p.x_out + (long)r * p.ldr_out + t * p.lds_out + c, n[t]);
+        }
+#pragma unroll
+        for (int t = 0; t < SMAX; ++t) x[t] = n[t];
+      }
+#pragma unroll
+      for (int k = 0; k < 4; ++k) u.f[k] = 0.f;
+#pragma unroll
+      for (int s = 0; s < SMAX; ++s) {
+        if (s >= p.S) break;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) u.f[k] = fmaf(in[s], x[s].f[k], u.f[k]);
+      }
+#pragma unroll
+      for (int k = 0; k < 4; ++k) ss = fmaf(u.f[k], u.f[k], ss);
+      st<4>(h + c, u);
+      if (mine && p.sum) st<4>(p.sum + (long)r * p.ldsum + c, u);
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) inv[i] = gain / sqrtf(ss / (float)p.D + p.eps);
+  }
+  __syncthreads();
+  if (!p.xa) return;
+  for (int c = threadIdx.x * 4; c < p.D; c += blockDim.x * 4) {
+    int run = o;                               // rows of the run ahead of row r in the step (as many as matter)
+    for (int i = o; i < rows; ++i) {
+      const int r = r0 - o + i, slot = p.slots[r];
+      if (i > o) run = p.slots[r - 1] == slot ? run + 1 : 0;
+      Vec<4> v = ld<4>(hs + (long)i * p.D + c);
+      const float f = inv[i];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v.f[k] *= f;
+      Vec<4> a = v;
+      if (p.taps) {
+        const int pos = p.positions[r], side = p.taps > 1 ? p.epoch[slot] & 1 : 0;
+        const float* old = p.history + ((long)slot * 2 + side) * back * p.D;
+        const bool last = p.taps > 1 && (r + 1 == p.T || p.slots[r + 1] != slot);
+        float* fresh = p.history + ((long)slot * 2 + (side ^ 1)) * back * p.D;
+        const Vec<4> w = ld<4>(p.taps_w + (long)back * p.D + c);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) a.f[k] = fmaf(w.f[k], v.f[k], a.f[k]);
+        if (last) st<4>(fresh + c, v);
+        for (int j = 1; j < p.taps; ++j) {
+          Vec<4> b;
+          float g = 1.f;
+          if (j > pos) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k) b.f[k] = 0.f;
+          } else if (j <= run) {
+            b = ld<4>(hs + (long)(i - j) * p.D + c);
+            g = inv[i - j];
+          } else {
+            b = ld<4>(old + (long)(j - run - 1) * p.D + c);
+          }
+          const Vec<4> wj = ld<4>(p.taps_w + (long)(back - j) * p.D + c);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            b.f[k] *= g;
+            a.f[k] = fmaf(wj.f[k], b.f[k], a.f[k]);
+          }
+          if (last && j < back) st<4>(fresh + (long)j * p.D + c, b);
+        }
+      }
+      st<4>(reinterpret_cast<A*>(p.xa) + (long)r * p.lda + c, a);
+    }
+  }
+}
+
+// rows of a CTA so that one wave of CTAs takes all of them, as far as shared memory allows; 0: the other kernel
+int tile_rows(const StreamsParams& p) {
+  const int back = p.taps > 1 ? p.taps - 1 : 0, room = (int)(200 * 1024 / (p.D * sizeof(float) + sizeof(float))) - back;
+  if (p.T <= 256 || room < 4) return 0;
+  const int want = (p.T + 147) / 148;
+  return want < 4 ? 4 : want < room ? want : room;
+}
+template <typename A, int SMAX>
+int launch_tile(StreamsParams p, cudaStream_t s) {
+  p.block = tile_rows(p);
+  const int rows = p.block + (p.taps > 1 ? p.taps - 1 : 0);
+  const size_t smem = (size_t)rows * (p.D + 1) * sizeof(float);
+  auto k = streams_tile_kernel<A, SMAX>;
+  if (int rc = opt_in_smem(k, smem)) return rc;
+  return launch_chain(k, dim3((p.T + p.block - 1) / p.block), dim3(32 * (rows < 32 ? (rows < 8 ? 8 : rows) : 32)), smem, s, p);
+}
+
 template <typename A, int SMAX, int V>
 int launch_rows(const StreamsParams& p, cudaStream_t s) {
   const size_t smem = (size_t)(p.taps > 1 ? p.taps : 1) * p.D * sizeof(float);
@@ -204,6 +339,7 @@ int by_streams(const StreamsParams& p, cudaStream_t s) {
   const bool four = !((p.D | p.ldr_in | p.lds_in | p.ldr_out | p.lds_out | p.ldy | p.part_stride | p.ldsum | p.lda) % 4) && !odd(p.x_in) && !odd(p.x_out) && !odd(p.y) &&
                     !odd(p.taps_w) && !odd(p.history) && !odd(p.sum) && !odd(p.xa);
   if (!four) return launch_rows<A, MAX_S, 1>(p, s);
+  if (p.S <= 4 && tile_rows(p)) return p.S <= 1 ? launch_tile<A, 1>(p, s) : p.S == 2 ? launch_tile<A, 2>(p, s) : launch_tile<A, 4>(p, s);
   if (p.S == 1) return launch_rows<A, 1, 4>(p, s);
   if (p.S == 2) return launch_rows<A, 2, 4>(p, s);
   if (p.S <= 4) return launch_rows<A, 4, 4>(p, s);

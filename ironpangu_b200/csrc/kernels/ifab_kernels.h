@@ -369,17 +369,24 @@ int ifab_streams_rows(const float* x_in, long ldr_in, long lds_in, float* x_out,
                       long part_stride, const float* mix, const float* out, const float* in, const float* gain, float eps, const float* taps_w, int taps,
                       float* history, const int32_t* epoch, const int32_t* positions, const int32_t* slots, float* sum, long ldsum, void* xa, long lda, int f32,
                       int T, int S, int D, int block, void* stream);
-/* recurrences with a decay per token (gated_recurrence.cu, gated_delta.cu). kind: 0 state-space duality, 1 delta rule, 2 matrix memory */
-int ifab_gr_prepare(const void* proj, long ldp, int f32, const int32_t* sections, const float* scales, float* q, float* k, float* v, const float* taps_w,
-                    const float* bias, int taps, int C, void* history, const int32_t* epoch, int kind, int H, int decay_col, int weight_col, const float* a_log,
-                    const float* decay_bias, const float* weight_bias, float cap, float* log_decay, float* weight, const int32_t* positions,
-                    const int32_t* slots, int T, void* stream);
-int ifab_gr_step(const float* q, const float* k, const float* v, const float* log_decay, const float* weight, int kind, int H, int G, int d, int E, float* state,
-                 float* m_state, const int32_t* epoch, float* m_rows, const int32_t* positions, const int32_t* slots, float* o, long ldo, int T, void* stream);
-int ifab_gr_chunks(const float* q, const float* k, const float* v, const float* log_decay, const float* weight, int kind, int H, int G, int d, int E,
-                   const int32_t* chunks, int n, const int32_t* positions, float* cstate, uint64_t cstate_bytes, float* cdecay, float* w_rows, float* u_rows,
-                   float* state, float* m_state, const int32_t* epoch, float* m_rows, float* o, long ldo, void* stream);
-int ifab_gr_finish(const float* o, long ldo, int H, int e, int E, const float* m, const float* v, const float* skip, const void* gate, long ldg, int act,
+/* recurrences with a decay per token (gated_recurrence.cu, gated_delta.cu). kind: 0 state-space duality, 1 delta rule, 2 matrix memory. q, k [T, G, d] and
+ * v [T, H, e] in the activation type, qs / ks [T, G]: factors of their rows or null; the state [slots, H, e (+ 1 for kind 2), d] */
+int ifab_gr_prepare(const void* proj, long ldp, int f32, const int32_t* sections, void* q, void* k, void* v, float* q_factors, float* k_factors, float q_factor,
+                    const float* taps_w, const float* bias, int taps, int C, void* history, const int32_t* epoch, int kind, int H, int decay_col,
+                    int weight_col, const float* a_log, const float* decay_bias, const float* weight_bias, float cap, float* log_decay, float* weight,
+                    const int32_t* positions, const int32_t* slots, int T, void* stream);
+int ifab_gr_step(const void* q, const void* k, const void* v, int f32, const float* qs, const float* ks, float q_factor, const float* log_decay,
+                 const float* weight, int kind, int H, int G, int d, int e, float* state, float* m_state, const int32_t* epoch, float* m_rows,
+                 const int32_t* positions, const int32_t* slots, float* o, long ldo, int T, void* stream);
+int ifab_gr_chunks(const void* q, const void* k, const void* v, int f32, const float* qs, const float* ks, float q_factor, const float* log_decay,
+                   const float* weight, int kind, int H, int G, int d, int e, const int32_t* chunks, int n, const int32_t* positions, float* cstate,
+                   uint64_t cstate_bytes, float* cdecay, float* w_rows, float* u_rows, float* state, float* m_state, const int32_t* epoch, float* m_rows,
+                   float* o, long ldo, void* stream);
+int ifab_gr_tiles(const void* q, const void* k, const void* v, const float* qs, const float* ks, float q_factor, const float* log_decay, const float* weight, int kind,
+                  int H, int G, int d, int e, const int32_t* chunks, int n, const int32_t* positions, float* cstate, uint64_t cstate_bytes, float* cdecay, float* u,
+                  void* images, uint64_t image_bytes_given, float* state, float* m_state, const int32_t* epoch, float* m_rows, float* o, long ldo,
+                  const void* gate, long ldg, int gate_act, const float* gain, float eps, void* y, long ldy, uint32_t* status, void* stream);
+int ifab_gr_finish(const float* o, long ldo, int H, int e, int E, const float* m, const void* v, const float* skip, const void* gate, long ldg, int act,
                    int gate_first, int groups, float eps, const float* gain, void* y, long ldy, int f32, int T, void* stream);
 /* operands of the tensor-core windowed attention: keys / values first .. first + n - 1 of a sequence, heads zero-padded to dp / 128 columns */
 int ifab_ctx_gather_pad(const void* k_cache, const void* v_cache, const int32_t* page_table, int slot, int max_pages, int page_tokens, int num_pages,

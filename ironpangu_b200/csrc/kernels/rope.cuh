@@ -52,8 +52,15 @@ __device__ __forceinline__ float sigmoid_f32(float x) {
 template <bool FAST = false>
 __device__ __forceinline__ float gelu_tanh_f32(float z) { return z * sigmoid_f32<FAST>(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
 
-// 0.5 z (1 + erf(z / sqrt 2)), without cancellation for negative z
-__device__ __forceinline__ float gelu_erf_f32(float z) { return 0.5f * z * erfcf(-0.70710678118654752f * z); }
+// 0.5 z (1 + erf(z / sqrt 2)) = z - 0.5 z erfc(z / sqrt 2). FAST: erfc by formula 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical Functions
+// (absolute error below 1.5e-7)
+template <bool FAST = false>
+__device__ __forceinline__ float gelu_erf_f32(float z) {
+  if (!FAST) return 0.5f * z * erfcf(-0.70710678118654752f * z);
+  const float x = 0.70710678118654752f * fabsf(z), t = __fdividef(1.f, fmaf(0.3275911f, x, 1.f));
+  const float c = t * (0.254829592f + t * (-0.284496736f + t * (1.421413741f + t * (-1.453152027f + t * 1.061405429f)))) * __expf(-x * x);
+  return fmaxf(z, 0.f) - 0.5f * fabsf(z) * c;
+}
 
 // elementwise activations by number: 0 none, 1 SiLU, 2 sigmoid, 3 GELU (tanh form), 4 GELU (erf form)
 template <bool FAST = false>
@@ -62,7 +69,7 @@ __device__ __forceinline__ float activate(float z, int act) {
     case 1: return z * sigmoid_f32<FAST>(z);
     case 2: return sigmoid_f32<FAST>(z);
     case 3: return gelu_tanh_f32<FAST>(z);
-    case 4: return gelu_erf_f32(z);
+    case 4: return gelu_erf_f32<FAST>(z);
     default: return z;
   }
 }

@@ -22,7 +22,7 @@ import torch
 
 from ..ops import hyper_streams as HS
 from ..ops import stream_norm as N
-from ..ops.gated_recurrence import CHUNK, GatedRecurrence, RecurrenceBuffers, RecurrenceShape
+from ..ops.gated_recurrence import CHUNK, TILE, GatedRecurrence, RecurrenceBuffers, RecurrenceShape
 from ..ops.linear_attn import DevicePlan, RotaryScaling, RotaryTables
 from ..ops.window_attn import GroupedAttention, GroupedBuffers, GroupedShape
 from ..parallel.fabric import Fabric
@@ -30,7 +30,7 @@ from . import checkpoint
 from .checkpoint import pad8
 from .stream_decoder import ATTN_ROWS, BF16, F32, StreamDecoder, StreamRows
 
-KERNEL_UNITS = ("misc", "post_norm", "hyper_streams", "gated_recurrence", "gated_delta", "linear_f32", "window_attn", "decode_gqa", "fa_prefill", "decode_post_norm",
+KERNEL_UNITS = ("misc", "post_norm", "hyper_streams", "gated_recurrence", "gated_delta", "gated_tiles", "linear_f32", "window_attn", "decode_gqa", "fa_prefill", "decode_post_norm",
                 "decode_moe", "sampling", "tc_gemm", "tc_gemm_2sm")
 MIXERS = ("parallel", "mamba2", "parallel_2")
 
@@ -265,7 +265,7 @@ class _Rows:
         self.streams = [torch.zeros(rows, max(c.streams, 1), pad8(c.width), dtype=F32, device=dev) for _ in range(2)]
         left = [l.left for l in c.layers if l.left]
         self.attn = GroupedBuffers(left, rows, A, dev, chunked=chunked, max_context=dec.max_context, group=ATTN_ROWS, in_cols=max(l.in_cols for l in c.layers))
-        self.rec = RecurrenceBuffers([l.right for l in c.layers], rows, dev, chunked=chunked, slots=dec.num_slots)
+        self.rec = RecurrenceBuffers([l.right for l in c.layers], rows, A, dev, chunk=dec.chunk if chunked else 0, slots=dec.num_slots)
         self.mixed = {l.mixed: z(sum(l.mixed)) for l in c.layers}                        # one per pair of widths: the padding columns must stay zero
         self.act = {l.ff: z(l.ff) for l in c.layers if l.ff}
         self.parts = torch.zeros(8, min(rows, 128), pad8(c.width), dtype=F32, device=dev) if A == BF16 else None
@@ -276,7 +276,6 @@ class FubelornDecoder(StreamDecoder):
     """Decode executor: see :class:`StreamDecoder`."""
 
     name = "fubelorn"
-    chunk = CHUNK
 
     def make_rows(self, rows: int, chunked: bool) -> _Rows:
         return _Rows(self, rows, chunked)
@@ -307,6 +306,8 @@ class FubelornDecoder(StreamDecoder):
             sub = [HS.Sublayer(W, p, q, c.streams, c.mult, c.taps, c.width, dev) for q in ((1, 2) if l.ff else (1,))]
             self.layers.append({"c": l, "left": left, "right": right, "in": w_in, "out": w_out, "sub": sub,
                                 "up": self._mat(W, p + "mlp.up") if l.ff else None, "down": self._mat(W, p + "mlp.down") if l.ff else None})
+        # prompts: recurrences on the tensor cores in bf16 when every head fits a tile, f32 products otherwise
+        self.chunk = TILE if self.dtype == BF16 and all(l.right.tiles for l in c.layers) else CHUNK
         self.fused = False
 
     def _state_bytes(self) -> tuple:
@@ -336,7 +337,7 @@ class FubelornDecoder(StreamDecoder):
         out = B.mixed[l.mixed][:m]
         if l.left:
             L["left"].attend(B.attn, m, L["pages"], B.rotary.get(*l.left.rotation), pos, slot, plan, self.page_table, self.cfg.eps, out, st)
-        L["right"].mix(B.rec, L["state"], B.attn.proj[:m], pos, slot, plan, self.epoch, self.cfg.eps, out[:, l.mixed[0]:])
+        L["right"].mix(B.rec, L["state"], B.attn.proj[:m], pos, slot, plan, self.epoch, self.cfg.eps, out[:, l.mixed[0]:], st)
         return out
 
     def _product(self, B: _Rows, x: torch.Tensor, w: torch.Tensor, m: int) -> torch.Tensor:

@@ -1,5 +1,5 @@
 """Recurrences over a matrix state per head with a decay per token - state-space duality, gated delta rule, matrix memory with exponential
-gates - between a packed input projection and the operand of the output projection (``csrc/kernels/gated_recurrence.cu``, ``gated_delta.cu``)."""
+gates - between a packed input projection and the operand of the output projection (``csrc/kernels/gated_recurrence.cu``, ``gated_delta.cu``, ``gated_tiles.cu``)."""
 from __future__ import annotations
 
 import ctypes
@@ -14,7 +14,8 @@ from .linear_attn import DevicePlan
 from .stream_norm import ACTIVATIONS, _f32, _p, _s
 
 F32 = torch.float32
-CHUNK = 64               # rows of a chunk
+CHUNK = 64               # rows of a chunk of the f32 form
+TILE = 128               # of the tensor-core form (bf16, heads up to 128 columns)
 KINDS = {"ssd": 0, "delta": 1, "memory": 2}
 
 
@@ -75,27 +76,45 @@ class RecurrenceShape:
         return 2 * self.kv_heads * self.dim + self.inner if self.taps else 0
 
     @property
+    def tiles(self) -> bool:
+        """Fits the tensor-core form."""
+        return max(self.dim, self.vdim) <= 128
+
+    @property
+    def image_bytes(self) -> int:
+        """Of the delta rule's operands of a chunk and head."""
+        return (4 if self.dim <= 64 else 6) * 16384
+
+    @property
     def slot_floats(self) -> int:
         """32-bit words a sequence holds besides the convolution's history."""
         return self.heads * self.E * self.dim + (2 * self.heads if self.kind == "memory" else 0)
 
 
 class RecurrenceBuffers:
-    """Work buffers of the recurrences of a model for up to ``rows`` rows; ``chunked``: for packed steps over ``slots`` sequences."""
+    """Work buffers of the recurrences of a model for up to ``rows`` rows; ``chunk`` > 0: for packed steps over ``slots`` sequences with chunks of so many
+    rows (TILE: all recurrences take the tensor-core form)."""
 
-    def __init__(self, shapes, rows: int, device, *, chunked: bool, slots: int):
-        f = lambda n: torch.empty(max(n, 1), dtype=F32, device=device)
+    def __init__(self, shapes, rows: int, dtype: torch.dtype, device, *, chunk: int, slots: int):
+        f = lambda n, dt=F32: torch.empty(max(n, 1), dtype=dt, device=device)
         most = lambda fn: max([fn(s) for s in shapes] or [1])
-        self.q, self.k = f(rows * most(lambda s: s.kv_heads * s.dim)), f(rows * most(lambda s: s.kv_heads * s.dim))
-        self.v, self.o = f(rows * most(lambda s: s.heads * s.E)), f(rows * most(lambda s: s.heads * s.E))
+        self.q, self.k = f(rows * most(lambda s: s.kv_heads * s.dim), dtype), f(rows * most(lambda s: s.kv_heads * s.dim), dtype)
+        self.v, self.o = f(rows * most(lambda s: s.inner), dtype), f(rows * most(lambda s: s.heads * s.E))
+        self.qs, self.ks = f(rows * most(lambda s: s.kv_heads)), f(rows * most(lambda s: s.kv_heads))
         self.log_decay, self.weight, self.m = (f(rows * most(lambda s: s.heads)) for _ in range(3))
-        self.cstate = self.cdecay = self.w_rows = self.u_rows = None
-        if chunked and shapes:
-            n = rows // CHUNK + slots + 1                    # chunks of a step: whole ones and one ragged end per sequence
+        self.chunk = chunk
+        self.cstate = self.cdecay = self.w_rows = self.u_rows = self.images = None
+        if chunk and shapes:
+            assert chunk == CHUNK or (chunk == TILE and dtype == torch.bfloat16 and all(s.tiles for s in shapes))
+            n = rows // chunk + slots + 1                    # chunks of a step: whole ones and one ragged end per sequence
             self.cstate, self.cdecay = f(n * most(lambda s: s.heads * s.dim * s.E)), f(n * most(lambda s: s.heads))
             delta = [s for s in shapes if s.kind == "delta"]
             if delta:
-                self.w_rows, self.u_rows = f(rows * max(s.heads * s.dim for s in delta)), f(rows * max(s.heads * s.E for s in delta))
+                self.u_rows = f(rows * max(s.inner for s in delta))
+                if chunk == TILE:
+                    self.images = f(n * max(s.heads * s.image_bytes for s in delta), torch.uint8)
+                else:
+                    self.w_rows = f(rows * max(s.heads * s.dim for s in delta))
 
 
 class GatedRecurrence:
@@ -114,15 +133,15 @@ class GatedRecurrence:
         for n, w in s.columns.items():
             self.col[n] = c
             c += w
-        qk, E = s.kv_heads * s.dim, s.E
+        qk = s.kv_heads * s.dim
         channel = {"v": 0, "k": s.inner, "q": s.inner + qk} if s.kind == "ssd" else {"q": 0, "k": qk, "v": 2 * qk}
         if not s.taps:
             channel = dict.fromkeys("qkv", -1)
         sec = []
-        for n, heads, w, stride in (("q", s.kv_heads, s.dim, s.dim), ("k", s.kv_heads, s.dim, s.dim), ("v", s.heads, s.vdim, E)):
-            sec += [self.col[n], heads, w, channel[n], int(s.kind == "delta" and n != "v"), stride]
-        self.sections = (ctypes.c_int32 * 18)(*sec)
-        self.scales = (ctypes.c_float * 3)(s.dim ** -0.5 if s.kind != "ssd" else 1.0, 1.0, 1.0)
+        for n, heads, w in (("q", s.kv_heads, s.dim), ("k", s.kv_heads, s.dim), ("v", s.heads, s.vdim)):
+            sec += [self.col[n], heads, w, channel[n]]
+        self.sections = (ctypes.c_int32 * 12)(*sec)
+        self.q_factor = s.dim ** -0.5 if s.kind != "ssd" else 1.0
         self.taps_w = self.bias = self.a_log = self.decay_bias = self.weight_bias = self.skip = None
         if s.taps:
             conv = [get("conv")] if s.kind == "ssd" else [get(n + ".conv") for n in "qkv"]
@@ -141,31 +160,46 @@ class GatedRecurrence:
         return RecurrenceState(self.shape, slots, device, dtype)
 
     def mix(self, B: RecurrenceBuffers, state: "RecurrenceState", proj: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, plan: Optional[DevicePlan], epoch: torch.Tensor,
-            eps: float, out: torch.Tensor) -> None:
+            eps: float, out: torch.Tensor, status_ptr=None) -> None:
         """Rows of a packed step (``plan``), or decode rows (None), from ``proj`` to ``out`` ``[m, >= heads * vdim]``."""
         self.prepare(B, state, proj, pos, slot, epoch)
-        self.run(B, state, pos, slot, plan, epoch)
-        self.finish(B, proj, eps, out)
+        # norm and gate belong to the tensor-core form when every row is one of its and the norm is per head
+        whole = plan is not None and plan.table is not None and not plan.groups and B.chunk == TILE and self.shape.kind != "ssd"
+        self.run(B, state, pos, slot, plan, epoch, (proj[:, self.col[self.gate]:], out, eps) if whole else None, status_ptr)
+        if not whole:
+            self.finish(B, proj, eps, out)
 
     def prepare(self, B, state, proj, pos, slot, epoch) -> None:
         s = self.shape
-        check(_lib.load().ifab_gr_prepare(proj.data_ptr(), proj.stride(0), _f32(proj), self.sections, self.scales, B.q.data_ptr(), B.k.data_ptr(), B.v.data_ptr(),
-                                          _p(self.taps_w), _p(self.bias), s.taps, s.channels, _p(state.history), epoch.data_ptr(), self.kind, s.heads, self.decay_col,
-                                          self.weight_col, _p(self.a_log), _p(self.decay_bias), _p(self.weight_bias), s.gate_cap, B.log_decay.data_ptr(),
-                                          B.weight.data_ptr(), pos.data_ptr(), slot.data_ptr(), proj.shape[0], _s()), "gr_prepare")
+        unit = s.kind == "delta"
+        check(_lib.load().ifab_gr_prepare(proj.data_ptr(), proj.stride(0), _f32(proj), self.sections, B.q.data_ptr(), B.k.data_ptr(), B.v.data_ptr(),
+                                          B.qs.data_ptr() if unit else None, B.ks.data_ptr() if unit else None, self.q_factor, _p(self.taps_w), _p(self.bias), s.taps,
+                                          s.channels, _p(state.history), epoch.data_ptr(), self.kind, s.heads, self.decay_col, self.weight_col, _p(self.a_log),
+                                          _p(self.decay_bias), _p(self.weight_bias), s.gate_cap, B.log_decay.data_ptr(), B.weight.data_ptr(), pos.data_ptr(),
+                                          slot.data_ptr(), proj.shape[0], _s()), "gr_prepare")
 
-    def run(self, B, state, pos, slot, plan: Optional[DevicePlan], epoch) -> None:
+    def run(self, B, state, pos, slot, plan: Optional[DevicePlan], epoch, finish=None, status_ptr=None) -> None:
+        """The prepared rows through the states, into ``B.o`` - or with ``finish`` (gate rows, result, eps) through norm and gate too."""
         s, m = self.shape, pos.numel()
-        rows = (B.q.data_ptr(), B.k.data_ptr(), B.v.data_ptr(), B.log_decay.data_ptr(), B.weight.data_ptr(), self.kind, s.heads, s.kv_heads, s.dim, s.E)
+        unit = s.kind == "delta"
+        qkv = B.q.data_ptr(), B.k.data_ptr(), B.v.data_ptr()
+        rows = (B.qs.data_ptr() if unit else None, B.ks.data_ptr() if unit else None, self.q_factor, B.log_decay.data_ptr(), B.weight.data_ptr(), self.kind, s.heads, s.kv_heads,
+                s.dim, s.vdim)
         ldo = s.heads * s.E
         long = plan is not None and plan.table is not None
         if long:
-            check(_lib.load().ifab_gr_chunks(*rows, plan.table.data_ptr(), plan.table.shape[0], pos.data_ptr(), B.cstate.data_ptr(), B.cstate.numel() * 4, B.cdecay.data_ptr(),
-                                             _p(B.w_rows), _p(B.u_rows), state.s.data_ptr(), _p(state.m), epoch.data_ptr(), B.m.data_ptr(), B.o.data_ptr(), ldo, _s()),
-                  "gr_chunks")
+            chunks = plan.table.data_ptr(), plan.table.shape[0], pos.data_ptr(), B.cstate.data_ptr(), B.cstate.numel() * 4, B.cdecay.data_ptr()
+            states = state.s.data_ptr(), _p(state.m), epoch.data_ptr(), B.m.data_ptr()
+            if B.chunk == TILE:
+                gate, out, eps = finish or (None, None, 0.0)
+                check(_lib.load().ifab_gr_tiles(*qkv, *rows, *chunks, _p(B.u_rows), _p(B.images), 0 if B.images is None else B.images.numel(), *states, B.o.data_ptr(), ldo,
+                                                _p(gate), 0 if gate is None else gate.stride(0), self.gate_act, self.gain.data_ptr(), eps, _p(out),
+                                                0 if out is None else out.stride(0), status_ptr, _s()), "gr_tiles")
+            else:
+                check(_lib.load().ifab_gr_chunks(*qkv, _f32(B.q), *rows, *chunks, _p(B.w_rows), _p(B.u_rows), *states, B.o.data_ptr(), ldo, _s()), "gr_chunks")
         if not long or plan.groups:
-            check(_lib.load().ifab_gr_step(*rows, state.s.data_ptr(), _p(state.m), epoch.data_ptr(), B.m.data_ptr(), (pos if plan is None else plan.step_positions).data_ptr(),
-                                           slot.data_ptr(), B.o.data_ptr(), ldo, m, _s()), "gr_step")
+            check(_lib.load().ifab_gr_step(*qkv, _f32(B.q), *rows, state.s.data_ptr(), _p(state.m), epoch.data_ptr(), B.m.data_ptr(),
+                                           (pos if plan is None else plan.step_positions).data_ptr(), slot.data_ptr(), B.o.data_ptr(), ldo, m, _s()), "gr_step")
 
     def finish(self, B, proj, eps: float, out: torch.Tensor) -> None:
         s = self.shape

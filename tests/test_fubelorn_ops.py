@@ -237,13 +237,16 @@ class Recurrence:
         n, v = sum(c for *_, c in step), self.shape.inner
         pos = [p for _, _, lo, c in step for p in range(lo, lo + c)]
         slots = [s for _, s, _, c in step for _ in range(c)]
-        plan = StepPlan(slots, pos, short=short, chunk=self.GR.CHUNK)
+        chunk = self.GR.TILE if self.dtype == BF16 and self.shape.tiles else self.GR.CHUNK
+        plan = StepPlan(slots, pos, short=short, chunk=chunk)
         dp, ds = torch.tensor(pos, dtype=torch.int32, device="cuda"), torch.tensor(slots, dtype=torch.int32, device="cuda")
-        B = self.GR.RecurrenceBuffers([self.shape], n, "cuda", chunked=True, slots=4)
+        B = self.GR.RecurrenceBuffers([self.shape], n, self.dtype, "cuda", chunk=chunk, slots=4)
         out = torch.full((n, _pad(v) + 8), 5.0, dtype=self.dtype, device="cuda")
         HS.step_epoch(ds, self.epoch)
         proj = torch.cat([self.proj[k][lo:lo + c] for k, _, lo, c in step]).cuda()
-        self.mixer.mix(B, self.state, proj, dp, ds, plan.bind(plan.control.cuda(), dp), self.epoch, self.eps, out[:, 4:])
+        st = torch.zeros(1, dtype=torch.int32, device="cuda")
+        self.mixer.mix(B, self.state, proj, dp, ds, plan.bind(plan.control.cuda(), dp), self.epoch, self.eps, out[:, 4:], st.data_ptr())
+        assert int(st) == 0
         assert (out[:, :4] == 5).all() and (out[:, 4 + v:] == 5).all()
         return torch.split(out[:, 4:4 + v].cpu(), [c for *_, c in step])
 
@@ -266,20 +269,22 @@ def test_recurrence_in_portions(shape, dtype):
     """Whole, in portions around the chunk size, in pairs, and token by token; then several sequences over slots that are used again."""
     lens = {"a": 200, "b": 3, "c": 70, "d": 129, "e": 1, "f": 64, "g": 21}
     r = Recurrence(shape, dtype, lens)
-    lim = _lim(dtype, 2e-5, 1e-2)
-    for cuts in (_cuts(200, 200), _cuts(200, 64), _cuts(200, 65), _cuts(200, 63), _cuts(200, 7), _cuts(60, 2), _cuts(60, 1), [[("a", 1, 0, 130)]] + [[("a", 1, i, 1)] for i in range(130, 160)]):
+    lim = _lim(dtype, 2e-5, 8e-2)          # in 16 bits the convolved rows are rounded
+    for cuts in (_cuts(200, 200), _cuts(200, 128), _cuts(200, 129), _cuts(200, 64), _cuts(200, 65), _cuts(200, 63), _cuts(200, 7), _cuts(60, 2), _cuts(60, 1), [[("a", 1, 0, 130)]] + [[("a", 1, i, 1)] for i in range(130, 160)]):
         assert r.error(cuts) < lim, cuts[0]
     assert r.error(batches(random.Random(3), lens, [1, 1, 2, 4, 5, 17, 64, 66, 130])) < lim
 
 
 @gpu
-@pytest.mark.parametrize("shape", [SHAPES["delta"][1], SHAPES["ssd"][0], SHAPES["memory"][1]], ids=str)
-def test_recurrence_of_long_and_short_memory(shape):
+@pytest.mark.parametrize("shape,dtype", [(SHAPES["delta"][1], F32), (SHAPES["ssd"][0], F32), (SHAPES["memory"][1], F32), (("delta", 2, 1, 128, 128, 4), BF16), (("delta", 1, 1, 40, 72, 2), BF16),
+                                         (("ssd", 2, 1, 128, 64, 4, 1), BF16), (("memory", 2, 2, 64, 128), BF16), (("memory", 1, 1, 128, 96), BF16)], ids=str)
+def test_recurrence_of_long_and_short_memory(shape, dtype):
     """Decays so strong that a chunk's logs sum to hundreds, and gates so large that the running maximum jumps; a state that hardly decays
     over a thousand rows."""
     for strong, n in ((30.0, 300), (0.002, 1000)):
-        r = Recurrence(shape, F32, {"a": n}, strong=strong, seed=4)
-        assert r.error(_cuts(n, n)) < 5e-5 and r.error(_cuts(n, 100)) < 5e-5
+        r = Recurrence(shape, dtype, {"a": n}, strong=strong, seed=4)
+        lim = 5e-5 if dtype == F32 else 2e-2
+        assert r.error(_cuts(n, n)) < lim and r.error(_cuts(n, 100)) < lim
 
 
 def test_restated_recurrences_by_hand():
