@@ -97,58 +97,80 @@ __global__ void __launch_bounds__(256) gr_prepare_kernel(PrepareParams p) {
     }
     return;
   }
+  // what the rows need to know: rows of their sequence ahead of them in the step, position, slot, whether they are its last
+  __shared__ int run_of[8], pos_of[8], slot_of[8], last_of[8], side_of[8];
+  const int back = p.taps - 1;
+  if ((int)threadIdx.x < t1 - t0) {
+    const int t = t0 + threadIdx.x, slot = p.slots[t];
+    int run = 0;
+    while (run < back && t - run - 1 >= 0 && p.slots[t - run - 1] == slot) ++run;
+    run_of[threadIdx.x] = run;
+    pos_of[threadIdx.x] = p.positions[t];
+    slot_of[threadIdx.x] = slot;
+    last_of[threadIdx.x] = p.taps > 1 && (t + 1 == p.T || p.slots[t + 1] != slot);
+    side_of[threadIdx.x] = p.taps > 1 ? p.epoch[slot] & 1 : 0;
+  }
+  __syncthreads();
   const int i = blockIdx.x * 8 + warp, h0 = p.sec[0].heads, h1 = h0 + p.sec[1].heads;
   if (i >= h1 + p.sec[2].heads) return;
   const Section& s = p.sec[i < h0 ? 0 : i < h1 ? 1 : 2];
-  const int h = i - (i < h0 ? 0 : i < h1 ? h0 : h1), back = p.taps - 1;
-  for (int t = t0; t < t1; ++t) {
-    const int pos = p.positions[t], slot = p.slots[t];
-    if (pos < 0) continue;
-    const A* row = reinterpret_cast<const A*>(p.proj) + (long)t * p.ldp + s.col + h * s.n;
-    A* dst = reinterpret_cast<A*>(s.dst) + ((long)t * s.heads + h) * s.n;
-    int run = 0;                // rows of the sequence ahead of this one in the step
-    while (run < back && t - run - 1 >= 0 && p.slots[t - run - 1] == slot) ++run;
-    const int side = p.taps > 1 ? p.epoch[slot] & 1 : 0, ch0 = s.channel + h * s.n;
-    const A* old = reinterpret_cast<const A*>(p.history) + ((long)slot * 2 + side) * back * p.C + ch0;
-    A* fresh = reinterpret_cast<A*>(p.history) + ((long)slot * 2 + (side ^ 1)) * back * p.C + ch0;
-    const bool last = p.taps > 1 && (t + 1 == p.T || p.slots[t + 1] != slot);
-    float ss = 0.f;
-    for (int c = lane * V; c < s.n; c += 32 * V) {
+  const int h = i - (i < h0 ? 0 : i < h1 ? h0 : h1);
+  float sum[8];
+#pragma unroll
+  for (int z = 0; z < 8; ++z) sum[z] = 0.f;
+  for (int c = lane * V; c < s.n; c += 32 * V) {
+    float w0[V], bias[V];
+    if (s.channel >= 0) {
+      load_v<float, V>(p.taps_w + (long)back * p.C + s.channel + h * s.n + c, w0);
+      if (p.bias) load_v<float, V>(p.bias + s.channel + h * s.n + c, bias);
+    }
+#pragma unroll
+    for (int z = 0; z < 8; ++z) {
+      const int t = t0 + z, pos = t < t1 ? pos_of[z] : -1;
+      if (pos < 0) continue;
+      const A* row = reinterpret_cast<const A*>(p.proj) + (long)t * p.ldp + s.col + h * s.n;
+      A* dst = reinterpret_cast<A*>(s.dst) + ((long)t * s.heads + h) * s.n;
       float v[V];
       load_v<A, V>(row + c, v);
       if (s.channel >= 0) {
+        const int run = run_of[z], ch = s.channel + h * s.n + c;
+        const bool last = last_of[z];
+        A* fresh = reinterpret_cast<A*>(p.history) + ((long)slot_of[z] * 2 + (side_of[z] ^ 1)) * back * p.C + ch;
+        const A* old = reinterpret_cast<const A*>(p.history) + ((long)slot_of[z] * 2 + side_of[z]) * back * p.C + ch;
         float w[V], x[V], acc[V];
-        load_v<float, V>(p.taps_w + (long)back * p.C + ch0 + c, w);
 #pragma unroll
-        for (int u = 0; u < V; ++u) acc[u] = v[u] * w[u];
-        if (last) store_v<A, V>(fresh + c, v);
+        for (int u = 0; u < V; ++u) acc[u] = v[u] * w0[u];
+        if (last) store_v<A, V>(fresh, v);
         for (int j = 1; j < p.taps; ++j) {
           if (j <= pos) {
-            load_v<A, V>(j <= run ? row + c - (long)j * p.ldp : old + (long)(j - run - 1) * p.C + c, x);
-            load_v<float, V>(p.taps_w + (long)(back - j) * p.C + ch0 + c, w);
+            load_v<A, V>(j <= run ? row + c - (long)j * p.ldp : old + (long)(j - run - 1) * p.C, x);
+            load_v<float, V>(p.taps_w + (long)(back - j) * p.C + ch, w);
 #pragma unroll
             for (int u = 0; u < V; ++u) acc[u] = fmaf(w[u], x[u], acc[u]);
           } else {
 #pragma unroll
             for (int u = 0; u < V; ++u) x[u] = 0.f;
           }
-          if (last && j < back) store_v<A, V>(fresh + (long)j * p.C + c, x);
+          if (last && j < back) store_v<A, V>(fresh + (long)j * p.C, x);
         }
         if (p.bias) {
-          load_v<float, V>(p.bias + ch0 + c, w);
 #pragma unroll
-          for (int u = 0; u < V; ++u) acc[u] += w[u];
+          for (int u = 0; u < V; ++u) acc[u] += bias[u];
         }
 #pragma unroll
         for (int u = 0; u < V; ++u) v[u] = to_f32(from_f32<A>(acc[u] * sigmoid_f32<sizeof(A) == 2>(acc[u])));
       }
       store_v<A, V>(dst + c, v);
 #pragma unroll
-      for (int u = 0; u < V; ++u) ss = fmaf(v[u], v[u], ss);
+      for (int u = 0; u < V; ++u) sum[z] = fmaf(v[u], v[u], sum[z]);
     }
-    if (s.factors) {
-      ss = warp_sum(ss);
-      if (lane == 0) s.factors[(long)t * s.heads + h] = s.factor / sqrtf(ss + 1e-6f);
+  }
+  if (s.factors) {
+#pragma unroll
+    for (int z = 0; z < 8; ++z) {
+      if (t0 + z >= t1 || pos_of[z] < 0) continue;
+      const float ss = warp_sum(sum[z]);
+      if (lane == 0) s.factors[(long)(t0 + z) * s.heads + h] = s.factor / sqrtf(ss + 1e-6f);
     }
   }
 }
@@ -560,6 +582,49 @@ __global__ void __launch_bounds__(256) gr_finish_kernel(FinishParams p) {
   }
 }
 
+// One CTA per row and group, the values in registers between the sum and the stores; whole chunks of 4 columns. ITER: chunks of a thread
+template <typename A, int ITER>
+__global__ void __launch_bounds__(256) gr_finish_wide_kernel(FinishParams p) {
+  __shared__ float red[33];
+  grid_dep_launch();
+  grid_dep_wait();
+  const int t = blockIdx.y, n = p.H * p.e / p.groups, base = blockIdx.x * n;
+  const float* o = p.o + (long)t * p.ldo;
+  const A* gate = reinterpret_cast<const A*>(p.gate) + (long)t * p.ldg;
+  float x[ITER][4], z[ITER][4], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < ITER; ++i) {
+    const int k = (threadIdx.x + i * 256) * 4, c = base + k;
+    if (k >= n) break;
+    const int h = c / p.e, j = c - h * p.e;
+    load_v<float, 4>(o + (long)h * p.E + j, x[i]);
+    load_v<A, 4>(gate + c, z[i]);
+    if (p.skip) {
+      float v[4];
+      load_v<A, 4>(reinterpret_cast<const A*>(p.v) + (long)t * p.H * p.e + c, v);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) x[i][u] = fmaf(p.skip[h], v[u], x[i][u]);
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      z[i][u] = activate<sizeof(A) == 2>(z[i][u], p.act);
+      if (p.gate_first) x[i][u] *= z[i][u];
+      ss = fmaf(x[i][u], x[i][u], ss);
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)n + p.eps);
+#pragma unroll
+  for (int i = 0; i < ITER; ++i) {
+    const int k = (threadIdx.x + i * 256) * 4, c = base + k;
+    if (k >= n) break;
+    float g[4];
+    load_v<float, 4>(p.gain + c, g);
+#pragma unroll
+    for (int u = 0; u < 4; ++u) g[u] *= x[i][u] * inv * (p.gate_first ? 1.f : z[i][u]);
+    store_v<A, 4>(reinterpret_cast<A*>(p.y) + (long)t * p.ldy + c, g);
+  }
+}
+
 bool rows_ok(const GrRows& r) {
   return r.kind >= GR_SSD && r.kind <= GR_MEMORY && r.H >= 1 && r.G >= 1 && r.H % r.G == 0 && r.d >= 1 && r.e >= 1 && r.E == r.e + (r.kind == GR_MEMORY) && r.d <= 1024 &&
          r.E <= 1024 && r.H <= 65535;
@@ -659,7 +724,15 @@ extern "C" int ifab_gr_finish(const float* o, long ldo, int H, int e, int E, con
   FinishParams p{o, ldo, H, e, E, m, v, skip, gate, ldg, act, gate_first, groups, eps, gain, y, ldy};
   const size_t smem = m ? (size_t)H * sizeof(float) : 0;
   cudaStream_t s = (cudaStream_t)stream;
-  if (H * e / groups > 256) {
+  const int n = H * e / groups;
+  const auto odd = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) != 0; };
+  const auto off = [&](const void* a) { return (reinterpret_cast<uintptr_t>(a) & (f32 ? 15 : 7)) != 0; };
+  if (n > 256 && n <= 8192 && !m && !((n | e | E | ldo | ldg | ldy) % 4) && !odd(o) && !odd(gain) && !off(gate) && !off(y) && !off(v)) {
+    const dim3 grid(groups, T);
+    if (f32) return n <= 4096 ? launch_chain(gr_finish_wide_kernel<float, 4>, grid, dim3(256), 0, s, p) : launch_chain(gr_finish_wide_kernel<float, 8>, grid, dim3(256), 0, s, p);
+    return n <= 4096 ? launch_chain(gr_finish_wide_kernel<bf16, 4>, grid, dim3(256), 0, s, p) : launch_chain(gr_finish_wide_kernel<bf16, 8>, grid, dim3(256), 0, s, p);
+  }
+  if (n > 256) {
     const dim3 grid(groups < 8 ? groups : 8, T);
     return f32 ? launch_chain(gr_finish_kernel<float, 8>, grid, dim3(256), smem, s, p) : launch_chain(gr_finish_kernel<bf16, 8>, grid, dim3(256), smem, s, p);
   }

@@ -660,11 +660,11 @@ __global__ void __launch_bounds__(THREADS, 1) gr_tile_delta_kernel(TileParams p)
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
-// DELTA: over the chunks of a sequence. 128 threads: a TMEM lane each (a row of the chunk, then a key column of the state)
+// DELTA: over the chunks of a sequence. 256 threads: two per TMEM lane (a row of the chunk, then a key column of the state), half of the value columns each
 // ---------------------------------------------------------------------------------------------------------------------------
-constexpr int EN = 32;                           // value columns of a CTA
+constexpr int EN = 32, EH = EN / 2;              // value columns of a CTA, of a thread
 struct ScanSmall {
-  double last[CT];                               // scratch of the running sums
+  double last[8];                                // scratch of the running sums
   uint64_t full[2], done[2];
   uint32_t tmem_slot;
 };
@@ -679,10 +679,25 @@ __device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t b
   asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar))
                : "memory");
 }
+// 16 consecutive f32 columns of a thread's TMEM lane (tc_common.cuh has the form of 32)
+__device__ __forceinline__ void tmem_ld_32x16(uint32_t taddr, float* v) {
+  uint32_t* r = reinterpret_cast<uint32_t*>(v);
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]),
+                 "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+               : "r"(taddr)
+               : "memory");
+}
+__device__ __forceinline__ void tmem_st_32x16(uint32_t taddr, const float* v) {
+  const uint32_t* r = reinterpret_cast<const uint32_t*>(v);
+  asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};" ::"r"(taddr), "r"(r[0]), "r"(r[1]),
+               "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
+               : "memory");
+}
 
 // grid (ceil(e / EN), H, n): CTAs of a run's first chunk walk its chunks
 template <int NP>
-__global__ void __launch_bounds__(128, 1) gr_tile_scan_kernel(TileParams p) {
+__global__ void __launch_bounds__(256, 1) gr_tile_scan_kernel(TileParams p) {
   using Y = ScanLayout<NP>;
   constexpr uint32_t U_COL = 0, S_COL = 32;
   constexpr int IMAGE = image_bytes(NP);
@@ -691,7 +706,8 @@ __global__ void __launch_bounds__(128, 1) gr_tile_scan_kernel(TileParams p) {
   unsigned char *Ss = smem + Y::S, *Us = smem + Y::U;
   ScanSmall& X = *reinterpret_cast<ScanSmall*>(smem + Y::SMALL);
   const GrRows& r = p.c.r;
-  const int first = blockIdx.z, h = blockIdx.y, e0 = blockIdx.x * EN, g = h / (r.H / r.G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, ne = min(EN, r.e - e0);
+  const int first = blockIdx.z, h = blockIdx.y, g = h / (r.H / r.G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int quarter = warp & 3, half = warp >> 2, row = quarter * 32 + lane, e0 = blockIdx.x * EN + half * EH, ne = min(EH, max(r.e - e0, 0));
   grid_dep_wait();
   const int meta = p.c.chunks[first * 4 + 3], count = meta >> 1, slot = p.c.chunks[first * 4 + 2];
   if (!(meta & 1)) return;
@@ -705,7 +721,7 @@ __global__ void __launch_bounds__(128, 1) gr_tile_scan_kernel(TileParams p) {
   if (warp == 0) tmem_alloc(&X.tmem_slot, 64);
   __syncthreads();               // tensor memory is taken before a dependent kernel may start beside this one
   grid_dep_launch();
-  const uint32_t tmem = X.tmem_slot, mine = tmem + ((uint32_t)(warp * 32) << 16);
+  const uint32_t tmem = X.tmem_slot, mine = tmem + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(half * EH);
   const bool fresh = p.c.positions[p.c.chunks[first * 4]] == 0;
   float* state = p.st.s + (((long)slot * r.H + h) * r.E + e0) * r.d;
   auto load = [&](int c) {
@@ -713,97 +729,97 @@ __global__ void __launch_bounds__(128, 1) gr_tile_scan_kernel(TileParams p) {
     mbar_expect_tx(&X.full[b], IMAGE);
     bulk_load(smem + Y::IMG + b * IMAGE, p.images + ((long)c * r.H + h) * IMAGE, IMAGE, &X.full[b]);
   };
-  float s[EN];
   int issued = min(count, 2);
   bool ok = true;
   if (tid == 0) {
     load(first);
     if (count > 1) load(first + 1);
   }
+  // what this thread's row of a chunk brings: its part of T (b v), its log decay, the factor of its key
+  struct Row {
+    float u[EH], log_decay, kn;
+    float* at;
+    bool live;
+  };
+  auto fetch = [&](int c, Row& x) {
+    const int row0 = p.c.chunks[c * 4], L = p.c.chunks[c * 4 + 1];
+    x.live = row < L;
+    const long t = row0 + (x.live ? row : 0);
+    x.at = p.u + (t * r.H + h) * r.e + e0;
+    x.log_decay = x.live ? r.log_decay[t * r.H + h] : 0.f;
+    x.kn = x.live && r.ks ? r.ks[t * r.G + g] : 1.f;
+    if (r.e % 4 == 0) {
 #pragma unroll
-  for (int i = 0; i < EN; ++i) s[i] = (i < ne && tid < r.d && !fresh) ? state[(long)i * r.d + tid] : 0.f;
-  constexpr uint32_t idesc = umma_idesc_bf16(128, EN);
-  int n = 0;
-  for (; n < count && ok; ++n) {
-    const int c = first + n, row0 = p.c.chunks[c * 4], L = p.c.chunks[c * 4 + 1], b = n & 1;
-    // this thread's key column of the state ahead of the chunk: into the chunk's place and, in two terms, into the operand
-    float* ahead = p.c.cstate + (((long)c * r.H + h) * r.E + e0) * r.d;
-    if (tid < 64 * NP) {
-#pragma unroll
-      for (int i = 0; i < EN; ++i) {
-        if (i < ne && tid < r.d) ahead[(long)i * r.d + tid] = s[i];
-        put2(Ss, Ss + NP * EN * 128, at(i, tid, EN), s[i]);
-      }
-    }
-    // running sums of the log decays; this thread's row
-    double total = tid < L ? (double)r.log_decay[(long)(row0 + tid) * r.H + h] : 0.0;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const double x = __shfl_up_sync(0xffffffffu, total, o);
-      if (lane >= o) total += x;
-    }
-    if (lane == 31) X.last[warp] = total;
-    float u[EN];
-    const bool live = tid < L;
-    float* ur = p.u + ((long)(row0 + tid) * r.H + h) * r.e + e0;
-    if (live && r.e % 4 == 0) {
-#pragma unroll
-      for (int i = 0; i < EN; i += 4) {
-        const float4 x = i < ne ? *reinterpret_cast<const float4*>(ur + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-        u[i] = x.x; u[i + 1] = x.y; u[i + 2] = x.z; u[i + 3] = x.w;
+      for (int i = 0; i < EH; i += 4) {
+        const float4 v = x.live && i < ne ? *reinterpret_cast<const float4*>(x.at + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        x.u[i] = v.x; x.u[i + 1] = v.y; x.u[i + 2] = v.z; x.u[i + 3] = v.w;
       }
     } else {
 #pragma unroll
-      for (int i = 0; i < EN; ++i) u[i] = live && i < ne ? ur[i] : 0.f;
+      for (int i = 0; i < EH; ++i) x.u[i] = x.live && i < ne ? x.at[i] : 0.f;
     }
-    const float kn = live && r.ks ? r.ks[(long)(row0 + tid) * r.G + g] : 1.f;
+  };
+  float s[EH];
+#pragma unroll
+  for (int i = 0; i < EH; ++i) s[i] = (i < ne && row < r.d && !fresh) ? state[(long)i * r.d + row] : 0.f;
+  Row next;
+  fetch(first, next);
+  constexpr uint32_t idesc = umma_idesc_bf16(128, EN);
+  for (int n = 0; n < count && ok; ++n) {
+    const int c = first + n, b = n & 1;
+    Row x = next;
+    // running sums of the log decays
+    double total = (double)x.log_decay;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const double y = __shfl_up_sync(0xffffffffu, total, o);
+      if (lane >= o) total += y;
+    }
+    if (lane == 31) X.last[warp] = total;
+    // this thread's key column of the state ahead of the chunk, in two terms
+    if (row < 64 * NP) {
+#pragma unroll
+      for (int i = 0; i < EH; ++i) put2(Ss, Ss + NP * EN * 128, at(half * EH + i, row, EN), s[i]);
+    }
     operands_ready();
+    unsigned char* img = smem + Y::IMG + b * IMAGE;
+    if (tid == 0 && mbar_wait(&X.full[b], (n >> 1) & 1, p.spin_limit)) {
+      tc_fence_after();
+      const uint32_t w = smem_u32(img), sb = smem_u32(Ss);
+      bool acc = false;
+      mma_panels(tmem + U_COL, w, sb, PANEL, EN * 128, NP, idesc, &acc);
+      mma_panels(tmem + U_COL, w, sb + NP * EN * 128, PANEL, EN * 128, NP, idesc, &acc);
+      mma_panels(tmem + U_COL, w + NP * PANEL, sb, PANEL, EN * 128, NP, idesc, &acc);
+      umma_commit(&X.done[0]);
+    }
+    __syncwarp();
+    if (n + 1 < count) fetch(c + 1, next);
+    // the state ahead of the chunk for the outputs; as it enters the sum: decayed
+    float* ahead = p.c.cstate + (((long)c * r.H + h) * r.E + e0) * r.d;
     double all = 0.0;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
-      if (w < warp) total += X.last[w];
-      all += X.last[w];
+      const double y = X.last[half * 4 + w];
+      if (w < quarter) total += y;
+      all += y;
     }
-    const float carry = expf((float)all);
-    unsigned char* img = smem + Y::IMG + b * IMAGE;
-    if (tid == 0) {
-      if (mbar_wait(&X.full[b], (n >> 1) & 1, p.spin_limit)) {
-        tc_fence_after();
-        const uint32_t w = smem_u32(img), sb = smem_u32(Ss);
-        bool acc = false;
-        mma_panels(tmem + U_COL, w, sb, PANEL, EN * 128, NP, idesc, &acc);
-        mma_panels(tmem + U_COL, w, sb + NP * EN * 128, PANEL, EN * 128, NP, idesc, &acc);
-        mma_panels(tmem + U_COL, w + NP * PANEL, sb, PANEL, EN * 128, NP, idesc, &acc);
-        umma_commit(&X.done[0]);
-      }
-    }
-    __syncwarp();
-    // the state as it enters the sum: decayed
+    const float carry = expf((float)all), tail = x.live ? expf((float)(all - total)) * x.kn : 0.f;
 #pragma unroll
-    for (int i = 0; i < EN; ++i) s[i] *= carry;
-    tmem_st_32x32(mine + S_COL, s);
+    for (int i = 0; i < EH; ++i) {
+      if (i < ne && row < r.d) ahead[(long)i * r.d + row] = s[i];
+      s[i] *= carry;
+    }
+    tmem_st_32x16(mine + S_COL, s);
     tmem_st_wait();
     ok = __all_sync(0xffffffffu, mbar_wait(&X.done[0], n & 1, p.spin_limit));
     tc_fence_after();
-    float wv[EN];
-    tmem_ld_32x32(mine + U_COL, wv);
+    float wv[EH];
+    tmem_ld_32x16(mine + U_COL, wv);
     tmem_ld_wait();
-    const float tail = live ? expf((float)(all - total)) * kn : 0.f;
 #pragma unroll
-    for (int i = 0; i < EN; ++i) {
-      u[i] -= wv[i];
-      put2(Us, Us + 2 * EN * 128, at(i, tid, EN), u[i] * tail);
-    }
-    if (live && ok) {
-      if (r.e % 4 == 0) {
-#pragma unroll
-        for (int i = 0; i < EN; i += 4)
-          if (i < ne) *reinterpret_cast<float4*>(ur + i) = make_float4(u[i], u[i + 1], u[i + 2], u[i + 3]);
-      } else {
-#pragma unroll
-        for (int i = 0; i < EN; ++i)
-          if (i < ne) ur[i] = u[i];
-      }
+    for (int i = 0; i < EH; ++i) {
+      x.u[i] -= wv[i];
+      put2(Us, Us + 2 * EN * 128, at(half * EH + i, row, EN), x.u[i] * tail);
     }
     ok = __syncthreads_and(ok);      // all warps leave the loop together
     if (!ok) break;
@@ -816,9 +832,20 @@ __global__ void __launch_bounds__(128, 1) gr_tile_scan_kernel(TileParams p) {
       umma_commit(&X.done[1]);
     }
     __syncwarp();
+    if (x.live) {
+      if (r.e % 4 == 0) {
+#pragma unroll
+        for (int i = 0; i < EH; i += 4)
+          if (i < ne) *reinterpret_cast<float4*>(x.at + i) = make_float4(x.u[i], x.u[i + 1], x.u[i + 2], x.u[i + 3]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < EH; ++i)
+          if (i < ne) x.at[i] = x.u[i];
+      }
+    }
     ok = __all_sync(0xffffffffu, mbar_wait(&X.done[1], n & 1, p.spin_limit));
     tc_fence_after();
-    tmem_ld_32x32(mine + S_COL, s);
+    tmem_ld_32x16(mine + S_COL, s);
     tmem_ld_wait();
     ok = __syncthreads_and(ok);      // the products have read this chunk's image
     if (ok && n + 2 < count) {
@@ -833,8 +860,8 @@ __global__ void __launch_bounds__(128, 1) gr_tile_scan_kernel(TileParams p) {
     }
   } else {
 #pragma unroll
-    for (int i = 0; i < EN; ++i)
-      if (i < ne && tid < r.d) state[(long)i * r.d + tid] = s[i];
+    for (int i = 0; i < EH; ++i)
+      if (i < ne && row < r.d) state[(long)i * r.d + row] = s[i];
   }
   tc_fence_before();
   __syncthreads();
@@ -856,7 +883,7 @@ int tiles(const TileParams& p, cudaStream_t s) {
   const int n = p.c.n;
   if (r.kind == GR_DELTA) {
     if (int rc = run(gr_tile_delta_kernel<NP>, dim3(n, r.H), THREADS, DeltaLayout::SMEM, s, p)) return rc;
-    if (int rc = run(gr_tile_scan_kernel<NP>, dim3((r.e + EN - 1) / EN, r.H, n), 128, ScanLayout<NP>::SMEM, s, p)) return rc;
+    if (int rc = run(gr_tile_scan_kernel<NP>, dim3((r.e + EN - 1) / EN, r.H, n), 256, ScanLayout<NP>::SMEM, s, p)) return rc;
     TileParams o = p;
     o.c.r.weight = nullptr;      // corrected values count once
     return run(gr_tile_out_kernel<NP, true>, dim3(n, r.H), THREADS, out_smem<true>(), s, o);

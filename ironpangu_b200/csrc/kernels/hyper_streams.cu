@@ -90,11 +90,12 @@ __device__ __forceinline__ void st(bf16* p, const Vec<V>& v) {
 
 // SMAX: most streams; V: columns of a thread at a time. Shared memory: the last `taps` (at least 1) rows of h, columns private to their threads
 template <typename A, int SMAX, int V>
-__global__ void __launch_bounds__(THREADS) streams_rows_kernel(StreamsParams p) {
+__global__ void __launch_bounds__(SMAX <= 2 ? 1024 : SMAX <= 4 ? 512 : THREADS) streams_rows_kernel(StreamsParams p) {
   extern __shared__ __align__(16) float ring[];
   __shared__ float red[33], mix[SMAX * SMAX], in[SMAX], out[SMAX];
   grid_dep_launch();
-  for (int i = threadIdx.x; i < p.S * p.S; i += THREADS) mix[i] = p.mix ? p.mix[i] : 0.f;
+  const int nthr = blockDim.x;
+  for (int i = threadIdx.x; i < p.S * p.S; i += nthr) mix[i] = p.mix ? p.mix[i] : 0.f;
   if ((int)threadIdx.x < p.S) {
     in[threadIdx.x] = p.in ? p.in[threadIdx.x] : 1.f;
     out[threadIdx.x] = p.out ? p.out[threadIdx.x] : 0.f;
@@ -112,7 +113,7 @@ __global__ void __launch_bounds__(THREADS) streams_rows_kernel(StreamsParams p) 
     float* h = ring + (long)(r % deep) * p.D;
     const float* xr = p.x_in + (long)r * p.ldr_in;
     float ss = 0.f;
-    for (int c = threadIdx.x * V; c < p.D; c += THREADS * V) {
+    for (int c = threadIdx.x * V; c < p.D; c += nthr * V) {
       Vec<V> x[SMAX], u;
 #pragma unroll
       for (int s = 0; s < SMAX; ++s)
@@ -160,7 +161,7 @@ __global__ void __launch_bounds__(THREADS) streams_rows_kernel(StreamsParams p) 
     const float* old = p.history + ((long)slot * 2 + side) * back * p.D;
     const bool last = p.taps > 1 && mine && (r + 1 == p.T || p.slots[r + 1] != slot);
     float* fresh = p.history + ((long)slot * 2 + (side ^ 1)) * back * p.D;
-    for (int c = threadIdx.x * V; c < p.D; c += THREADS * V) {
+    for (int c = threadIdx.x * V; c < p.D; c += nthr * V) {
       Vec<V> v = ld<V>(h + c);
 #pragma unroll
       for (int i = 0; i < V; ++i) v.f[i] *= f;
@@ -192,8 +193,9 @@ __global__ void __launch_bounds__(THREADS) streams_rows_kernel(StreamsParams p) 
 }
 
 // Shared memory: h of the CTA's rows and of those recomputed ahead of them, then 1 / rms times the gain of each
+constexpr int tile_threads(int smax) { return smax <= 2 ? 768 : 512; }
 template <typename A, int SMAX>
-__global__ void __launch_bounds__(1024) streams_tile_kernel(StreamsParams p) {
+__global__ void __launch_bounds__(tile_threads(SMAX)) streams_tile_kernel(StreamsParams p) {
   extern __shared__ __align__(16) float hs[];
   __shared__ float mix[SMAX * SMAX], in[SMAX], out[SMAX];
   grid_dep_launch();
@@ -308,12 +310,12 @@ __global__ void __launch_bounds__(1024) streams_tile_kernel(StreamsParams p) {
   }
 }
 
-// rows of a CTA so that one wave of CTAs takes all of them, as far as shared memory allows; 0: the other kernel
+// rows of a CTA: even waves of CTAs, as many as shared memory asks for; 0: the other kernel
 int tile_rows(const StreamsParams& p) {
   const int back = p.taps > 1 ? p.taps - 1 : 0, room = (int)(200 * 1024 / (p.D * sizeof(float) + sizeof(float))) - back;
   if (p.T <= 256 || room < 4) return 0;
-  const int want = (p.T + 147) / 148;
-  return want < 4 ? 4 : want < room ? want : room;
+  const int want = (p.T + 147) / 148, waves = (want + room - 1) / room, rows = (want + waves - 1) / waves;
+  return rows < 4 ? 4 : rows;
 }
 template <typename A, int SMAX>
 int launch_tile(StreamsParams p, cudaStream_t s) {
@@ -322,7 +324,7 @@ int launch_tile(StreamsParams p, cudaStream_t s) {
   const size_t smem = (size_t)rows * (p.D + 1) * sizeof(float);
   auto k = streams_tile_kernel<A, SMAX>;
   if (int rc = opt_in_smem(k, smem)) return rc;
-  return launch_chain(k, dim3((p.T + p.block - 1) / p.block), dim3(32 * (rows < 32 ? (rows < 8 ? 8 : rows) : 32)), smem, s, p);
+  return launch_chain(k, dim3((p.T + p.block - 1) / p.block), dim3(rows < 8 ? 256 : 32 * rows < tile_threads(SMAX) ? 32 * rows : tile_threads(SMAX)), smem, s, p);
 }
 
 template <typename A, int SMAX, int V>
@@ -331,7 +333,8 @@ int launch_rows(const StreamsParams& p, cudaStream_t s) {
   auto k = streams_rows_kernel<A, SMAX, V>;
   if (smem > 200 * 1024) return -1;
   if (int rc = opt_in_smem(k, smem)) return rc;
-  return launch_chain(k, dim3((p.T + p.block - 1) / p.block), dim3(THREADS), smem, s, p);
+  const int most = SMAX <= 2 ? 1024 : SMAX <= 4 ? 512 : THREADS, want = (p.D + 32 * V - 1) / (32 * V) * 32;
+  return launch_chain(k, dim3((p.T + p.block - 1) / p.block), dim3(want < 64 ? 64 : want < most ? want : most), smem, s, p);
 }
 template <typename A>
 int by_streams(const StreamsParams& p, cudaStream_t s) {

@@ -465,17 +465,25 @@ __global__ void __launch_bounds__(128) pool_write_kernel(const A* k_cache, const
   const int last = pos / page_tokens < max_pages ? table[pos / page_tokens] : -1;
   bool ok = last >= 0 && last < num_pages;
   float acc[4] = {0.f, 0.f, 0.f, 0.f};      // d + e <= 512 columns
-  for (int j = pos - P + 1; j <= pos && ok; ++j) {
-    const int page = j / page_tokens < max_pages ? table[j / page_tokens] : -1;
-    if (page < 0 || page >= num_pages) {
-      ok = false;
-      break;
+  constexpr int B = 8;                      // positions in flight
+  for (int j0 = pos - P + 1; j0 <= pos && ok; j0 += B) {
+    long row[B];
+#pragma unroll
+    for (int b = 0; b < B; ++b) {
+      const int j = min(j0 + b, pos), page = j / page_tokens < max_pages ? table[j / page_tokens] : -1;
+      ok = ok && page >= 0 && page < num_pages;
+      row[b] = ((long)max(page, 0) * page_tokens + j % page_tokens) * G + g;
     }
-    const long row = ((long)page * page_tokens + j % page_tokens) * G + g;
+    if (!ok) break;
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
       const int c = threadIdx.x + 128 * u;
-      if (c < d + e) acc[u] += to_f32(c < d ? k_cache[row * d + c] : v_cache[row * e + c - d]);
+      if (c >= d + e) break;
+      float v[B];
+#pragma unroll
+      for (int b = 0; b < B; ++b) v[b] = j0 + b <= pos ? to_f32(c < d ? k_cache[row[b] * d + c] : v_cache[row[b] * e + c - d]) : 0.f;
+#pragma unroll
+      for (int b = 0; b < B; ++b) acc[u] += v[b];
     }
   }
   if (!ok) {
