@@ -118,6 +118,42 @@ __global__ void __launch_bounds__(256) gr_prepare_kernel(PrepareParams p) {
   float sum[8];
 #pragma unroll
   for (int z = 0; z < 8; ++z) sum[z] = 0.f;
+  // eight rows in the middle of a run: every input is loaded once
+  if (t1 - t0 == 8 && run_of[0] == back && run_of[7] == back && slot_of[0] == slot_of[7] && pos_of[0] >= 0 && p.taps <= 4 && s.channel >= 0) {
+    const A* row = reinterpret_cast<const A*>(p.proj) + (long)t0 * p.ldp + s.col + h * s.n;
+    A* dst = reinterpret_cast<A*>(s.dst) + ((long)t0 * s.heads + h) * s.n;
+    A* fresh = reinterpret_cast<A*>(p.history) + ((long)slot_of[0] * 2 + (side_of[0] ^ 1)) * back * p.C + s.channel + h * s.n;
+    for (int c = lane * V; c < s.n; c += 32 * V) {
+      float x[11][V], w[4][V], bias[V];        // x[3 + z]: of row z
+#pragma unroll
+      for (int z = 0; z < 11; ++z)
+        if (z >= 3 - back) load_v<A, V>(row + (long)(z - 3) * p.ldp + c, x[z]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (j < p.taps) load_v<float, V>(p.taps_w + (long)(back - j) * p.C + s.channel + h * s.n + c, w[j]);
+#pragma unroll
+      for (int u = 0; u < V; ++u) bias[u] = 0.f;
+      if (p.bias) load_v<float, V>(p.bias + s.channel + h * s.n + c, bias);
+#pragma unroll
+      for (int z = 0; z < 8; ++z) {
+        float v[V];
+#pragma unroll
+        for (int u = 0; u < V; ++u) {
+          float acc = bias[u];
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (j < p.taps) acc = fmaf(w[j][u], x[3 + z - j][u], acc);
+          v[u] = to_f32(from_f32<A>(acc * sigmoid_f32<sizeof(A) == 2>(acc)));
+          sum[z] = fmaf(v[u], v[u], sum[z]);
+        }
+        store_v<A, V>(dst + (long)z * s.heads * s.n + c, v);
+      }
+      if (last_of[7])
+#pragma unroll
+        for (int j = 0; j < 3; ++j)
+          if (j < back) store_v<A, V>(fresh + (long)j * p.C + c, x[10 - j]);
+    }
+  } else
   for (int c = lane * V; c < s.n; c += 32 * V) {
     float w0[V], bias[V];
     if (s.channel >= 0) {

@@ -218,47 +218,62 @@ __global__ void __launch_bounds__(tile_threads(SMAX)) streams_tile_kernel(Stream
     const float* xr = p.x_in + (long)r * p.ldr_in;
     float* h = hs + (long)i * p.D;
     float ss = 0.f;
-#pragma unroll 2
-    for (int c = lane * 4; c < p.D; c += 128) {
-      Vec<4> x[SMAX], u;
+    constexpr int U = SMAX <= 1 ? 4 : 2;        // column groups whose loads are in flight together
+    for (int c0 = lane * 4; c0 < p.D; c0 += 128 * U) {
+      Vec<4> x[U][SMAX], y[U];
 #pragma unroll
-      for (int s = 0; s < SMAX; ++s)
-        if (s < p.S) x[s] = ld<4>(xr + s * p.lds_in + c);
-      if (p.y) {
-        Vec<4> y = ld<4>(p.y + (long)r * p.ldy + c), n[SMAX];
-        for (int q = 1; q < p.parts; ++q) {
-          const Vec<4> a = ld<4>(p.y + q * p.part_stride + (long)r * p.ldy + c);
+      for (int z = 0; z < U; ++z) {
+        const int c = c0 + 128 * z;
+        if (c >= p.D) break;
 #pragma unroll
-          for (int k = 0; k < 4; ++k) y.f[k] += a.f[k];
+        for (int s = 0; s < SMAX; ++s)
+          if (s < p.S) x[z][s] = ld<4>(xr + s * p.lds_in + c);
+        if (p.y) {
+          y[z] = ld<4>(p.y + (long)r * p.ldy + c);
+          for (int q = 1; q < p.parts; ++q) {
+            const Vec<4> a = ld<4>(p.y + q * p.part_stride + (long)r * p.ldy + c);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) y[z].f[k] += a.f[k];
+          }
         }
+      }
 #pragma unroll
-        for (int t = 0; t < SMAX; ++t) {
-          if (t >= p.S) break;
+      for (int z = 0; z < U; ++z) {
+        const int c = c0 + 128 * z;
+        if (c >= p.D) break;
+        Vec<4> u;
 #pragma unroll
-          for (int k = 0; k < 4; ++k) n[t].f[k] = out[t] * y.f[k];
+        for (int k = 0; k < 4; ++k) u.f[k] = 0.f;
+        if (p.y) {
+#pragma unroll
+          for (int t = 0; t < SMAX; ++t) {
+            if (t >= p.S) break;
+            Vec<4> n;
+#pragma unroll
+            for (int k = 0; k < 4; ++k) n.f[k] = out[t] * y[z].f[k];
+#pragma unroll
+            for (int s = 0; s < SMAX; ++s) {
+              if (s >= p.S) break;
+#pragma unroll
+              for (int k = 0; k < 4; ++k) n.f[k] = fmaf(mix[s * p.S + t], x[z][s].f[k], n.f[k]);
+            }
+            if (mine && p.x_out) st<4>(p.x_out + (long)r * p.ldr_out + t * p.lds_out + c, n);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) u.f[k] = fmaf(in[t], n.f[k], u.f[k]);
+          }
+        } else {
 #pragma unroll
           for (int s = 0; s < SMAX; ++s) {
             if (s >= p.S) break;
 #pragma unroll
-            for (int k = 0; k < 4; ++k) n[t].f[k] = fmaf(mix[s * p.S + t], x[s].f[k], n[t].f[k]);
+            for (int k = 0; k < 4; ++k) u.f[k] = fmaf(in[s], x[z][s].f[k], u.f[k]);
           }
-          if (mine && p.x_out) st<4>(p.x_out + (long)r * p.ldr_out + t * p.lds_out + c, n[t]);
         }
 #pragma unroll
-        for (int t = 0; t < SMAX; ++t) x[t] = n[t];
+        for (int k = 0; k < 4; ++k) ss = fmaf(u.f[k], u.f[k], ss);
+        st<4>(h + c, u);
+        if (mine && p.sum) st<4>(p.sum + (long)r * p.ldsum + c, u);
       }
-#pragma unroll
-      for (int k = 0; k < 4; ++k) u.f[k] = 0.f;
-#pragma unroll
-      for (int s = 0; s < SMAX; ++s) {
-        if (s >= p.S) break;
-#pragma unroll
-        for (int k = 0; k < 4; ++k) u.f[k] = fmaf(in[s], x[s].f[k], u.f[k]);
-      }
-#pragma unroll
-      for (int k = 0; k < 4; ++k) ss = fmaf(u.f[k], u.f[k], ss);
-      st<4>(h + c, u);
-      if (mine && p.sum) st<4>(p.sum + (long)r * p.ldsum + c, u);
     }
     ss = warp_sum(ss);
     if (lane == 0) inv[i] = gain / sqrtf(ss / (float)p.D + p.eps);

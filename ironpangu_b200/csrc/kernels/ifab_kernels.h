@@ -386,6 +386,18 @@ int ifab_gr_tiles(const void* q, const void* k, const void* v, const float* qs, 
                   int H, int G, int d, int e, const int32_t* chunks, int n, const int32_t* positions, float* cstate, uint64_t cstate_bytes, float* cdecay, float* u,
                   void* images, uint64_t image_bytes_given, float* state, float* m_state, const int32_t* epoch, float* m_rows, float* o, long ldo,
                   const void* gate, long ldg, int gate_act, const float* gain, float eps, void* y, long ldy, uint32_t* status, void* stream);
+/* one or two decode rows (decode_hyper.cu): a linear behind the streams, a linear behind a recurrence, convolution + gates + step in one */
+int ifab_gemv_streams(const float* x_in, long ldr_in, long lds_in, float* x_out, long ldr_out, long lds_out, const float* y, long ldy, const float* mix,
+                      const float* out, const float* in, const float* gain, float eps, const float* taps_w, int taps, float* history, const int32_t* epoch,
+                      const int32_t* positions, const int32_t* slots, int S, const void* w, void* z, long ldz, int out_f32, int act, int T, int N, int K,
+                      void* stream);
+int ifab_gemv_mixed(const void* x, long ldx, int K1, const float* o, long ldo, int H, int e, int E, const float* m, const void* v, const float* skip,
+                    const void* gate, long ldg, int gate_act, int gate_first, int groups, float eps, const float* gain, const void* w, float* z, long ldz, int T,
+                    int N, int K, void* stream);
+int ifab_gr_decode(const void* proj, long ldp, const int32_t* cols, const int32_t* channels, int unit, float q_factor, const float* taps_w, const float* bias, int taps,
+                   int C, void* history, int kind, int H, int G, int d, int e, int decay_col, int weight_col, const float* a_log, const float* decay_bias,
+                   const float* weight_bias, float cap, float* state, float* m_state, const int32_t* epoch, void* v, float* m_rows, const int32_t* positions,
+                   const int32_t* slots, float* o, long ldo, int T, void* stream);
 int ifab_gr_finish(const float* o, long ldo, int H, int e, int E, const float* m, const void* v, const float* skip, const void* gate, long ldg, int act,
                    int gate_first, int groups, float eps, const float* gain, void* y, long ldy, int f32, int T, void* stream);
 /* operands of the tensor-core windowed attention: keys / values first .. first + n - 1 of a sequence, heads zero-padded to dp / 128 columns */

@@ -31,7 +31,7 @@ from .checkpoint import pad8
 from .stream_decoder import ATTN_ROWS, BF16, F32, StreamDecoder, StreamRows
 
 KERNEL_UNITS = ("misc", "post_norm", "hyper_streams", "gated_recurrence", "gated_delta", "gated_tiles", "linear_f32", "window_attn", "decode_gqa", "fa_prefill", "decode_post_norm",
-                "decode_moe", "sampling", "tc_gemm", "tc_gemm_2sm")
+                "decode_hyper", "decode_moe", "sampling", "tc_gemm", "tc_gemm_2sm")
 MIXERS = ("parallel", "mamba2", "parallel_2")
 
 
@@ -308,7 +308,9 @@ class FubelornDecoder(StreamDecoder):
                                 "up": self._mat(W, p + "mlp.up") if l.ff else None, "down": self._mat(W, p + "mlp.down") if l.ff else None})
         # prompts: recurrences on the tensor cores in bf16 when every head fits a tile, f32 products otherwise
         self.chunk = TILE if self.dtype == BF16 and all(l.right.tiles for l in c.layers) else CHUNK
-        self.fused = False
+        # the fused decode chain needs operand widths that are whole 16-byte chunks
+        self.fused = self.dtype == BF16 and c.streams <= HS.FUSED_STREAMS and c.width % 8 == 0 and c.width <= 8192 and all(l.ff % 8 == 0 for l in c.layers) and \
+            all(L["right"].fusable for L in self.layers)
 
     def _state_bytes(self) -> tuple:
         c, es = self.cfg, torch.empty((), dtype=self.dtype).element_size()
@@ -331,13 +333,18 @@ class FubelornDecoder(StreamDecoder):
         return cls(c, w, fabric, **kw)
 
     # -- layers ------------------------------------------------------------------------------------------------------------
-    def _mix(self, B: _Rows, L: dict, m: int, pos, slot, plan: Optional[DevicePlan]) -> torch.Tensor:
-        """The mixer of one layer between its input projection (``B.attn.proj``) and the operand of its output projection, which it returns."""
-        l, st = L["c"], self.fabric.desc.status
+    def _attend(self, B: _Rows, L: dict, m: int, pos, slot, plan: Optional[DevicePlan]) -> torch.Tensor:
+        """The attention of a layer that has one; returns the operand of the output projection, whose first part it leaves there."""
+        l = L["c"]
         out = B.mixed[l.mixed][:m]
         if l.left:
-            L["left"].attend(B.attn, m, L["pages"], B.rotary.get(*l.left.rotation), pos, slot, plan, self.page_table, self.cfg.eps, out, st)
-        L["right"].mix(B.rec, L["state"], B.attn.proj[:m], pos, slot, plan, self.epoch, self.cfg.eps, out[:, l.mixed[0]:], st)
+            L["left"].attend(B.attn, m, L["pages"], B.rotary.get(*l.left.rotation), pos, slot, plan, self.page_table, self.cfg.eps, out, self.fabric.desc.status)
+        return out
+
+    def _mix(self, B: _Rows, L: dict, m: int, pos, slot, plan: Optional[DevicePlan]) -> torch.Tensor:
+        """The mixer of one layer between its input projection (``B.attn.proj``) and the operand of its output projection, which it returns."""
+        out = self._attend(B, L, m, pos, slot, plan)
+        L["right"].mix(B.rec, L["state"], B.attn.proj[:m], pos, slot, plan, self.epoch, self.cfg.eps, out[:, L["c"].mixed[0]:], self.fabric.desc.status)
         return out
 
     def _product(self, B: _Rows, x: torch.Tensor, w: torch.Tensor, m: int) -> torch.Tensor:
@@ -386,6 +393,33 @@ class FubelornDecoder(StreamDecoder):
                 front(None, operand=None, total=t)
                 probe.append(t)
         front(None, operand=xa if final else None, total=x)
+
+
+    def _layers_fused(self, B: _Rows, n: int, tok, pos, slot) -> None:
+        """One or two decode rows: streams, norm and convolution at the front of the linear that reads them, convolution, gates and step of a recurrence in one
+        launch, its norm and gate at the front of the output projection. Ends like :meth:`_layers` with ``final``."""
+        c, W = self.cfg, self.cfg.width
+        x, y = B.x[:n, :W], B.y[:n]
+        HS.step_epoch(slot, self.epoch)
+        HS.embed_norm(tok, self.embed, self.embed_gain, c.eps, x, self.fabric.desc.status)
+        B.rotary.fill(pos)
+        now, spare = x[:, None].expand(-1, max(c.streams, 1), -1), [t[:n, :, :W] for t in B.streams]
+        before = None
+        for L in self.layers:
+            l, proj = L["c"], B.attn.proj[:n]
+            for sub, w, out, act in ((L["sub"][0], L["in"], proj, None),) + (((L["sub"][1], L["up"], B.act[l.ff][:n], "gelu_erf"),) if l.ff else ()):
+                HS.gemv_streams(now, None if before is None else spare[0], None if before is None else y, before, sub, c.eps, self.epoch, pos, slot, w, out, act)
+                if before is not None:
+                    now = spare[0]
+                    spare.reverse()
+                before = sub
+                if act is None:
+                    mixed = self._attend(B, L, n, pos, slot, None)
+                    L["right"].decode(B.rec, L["state"], proj, pos, slot, self.epoch)
+                    L["right"].gemv_mixed(B.rec, proj, c.eps, mixed, l.mixed[0], L["out"], y)
+                else:
+                    N.gemv_act(out, L["down"], y)
+        HS.streams_rows(now, None, y, before, None, self.final_gain, c.eps, self.epoch, pos, slot, B.xa[:n], x)
 
 
 class FubelornRows(StreamRows):

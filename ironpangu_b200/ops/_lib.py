@@ -99,6 +99,11 @@ _SIGS = {
     "ifab_gr_chunks": [_P, _P, _P, c_int, _P, _P, c_float, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, c_u64, _P, _P, _P, _P, _P, _P, _P, _P, c_long, _P],
     "ifab_gr_tiles": [_P, _P, _P, _P, _P, c_float, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, c_u64, _P, _P, _P, c_u64, _P, _P, _P, _P, _P, c_long,
                       _P, c_long, c_int, _P, c_float, _P, c_long, _P, _P],
+    "ifab_gemv_streams": [_P, c_long, c_long, _P, c_long, c_long, _P, c_long, _P, _P, _P, _P, c_float, _P, c_int, _P, _P, _P, _P, c_int, _P, _P, c_long, c_int, c_int, c_int,
+                          c_int, c_int, _P],
+    "ifab_gemv_mixed": [_P, c_long, c_int, _P, c_long, c_int, c_int, c_int, _P, _P, _P, _P, c_long, c_int, c_int, c_int, c_float, _P, _P, _P, c_long, c_int, c_int, c_int, _P],
+    "ifab_gr_decode": [_P, c_long, C.POINTER(C.c_int32), C.POINTER(C.c_int32), c_int, c_float, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P,
+                       _P, _P, c_float, _P, _P, _P, _P, _P, _P, _P, _P, c_long, c_int, _P],
     "ifab_gr_finish": [_P, c_long, c_int, c_int, c_int, _P, _P, _P, _P, c_long, c_int, c_int, c_int, c_float, _P, _P, c_long, c_int, c_int, _P],
     "ifab_moe_down_f32_decode": [_P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, c_long, _P],
     "ifab_moe_route": [_P, c_long, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, _P, _P, _P, _P],

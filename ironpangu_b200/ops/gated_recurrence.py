@@ -1,5 +1,6 @@
 """Recurrences over a matrix state per head with a decay per token - state-space duality, gated delta rule, matrix memory with exponential
-gates - between a packed input projection and the operand of the output projection (``csrc/kernels/gated_recurrence.cu``, ``gated_delta.cu``, ``gated_tiles.cu``)."""
+gates - between a packed input projection and the operand of the output projection (``csrc/kernels/gated_recurrence.cu``, ``gated_delta.cu``, ``gated_tiles.cu``, for
+decode rows ``decode_hyper.cu``)."""
 from __future__ import annotations
 
 import ctypes
@@ -141,6 +142,7 @@ class GatedRecurrence:
         for n, heads, w in (("q", s.kv_heads, s.dim), ("k", s.kv_heads, s.dim), ("v", s.heads, s.vdim)):
             sec += [self.col[n], heads, w, channel[n]]
         self.sections = (ctypes.c_int32 * 12)(*sec)
+        self.cols, self.channels = (ctypes.c_int32 * 3)(*(self.col[n] for n in "qkv")), (ctypes.c_int32 * 3)(*(channel[n] for n in "qkv"))
         self.q_factor = s.dim ** -0.5 if s.kind != "ssd" else 1.0
         self.taps_w = self.bias = self.a_log = self.decay_bias = self.weight_bias = self.skip = None
         if s.taps:
@@ -200,6 +202,30 @@ class GatedRecurrence:
         if not long or plan.groups:
             check(_lib.load().ifab_gr_step(*qkv, _f32(B.q), *rows, state.s.data_ptr(), _p(state.m), epoch.data_ptr(), B.m.data_ptr(),
                                            (pos if plan is None else plan.step_positions).data_ptr(), slot.data_ptr(), B.o.data_ptr(), ldo, m, _s()), "gr_step")
+
+    @property
+    def fusable(self) -> bool:
+        """The fused decode form takes this shape (bf16)."""
+        s = self.shape
+        return s.dim % 4 == 0 and s.dim <= 256 and s.vdim % 4 == 0 and s.inner // s.groups % 4 == 0 and self.col[self.gate] % 4 == 0
+
+    def decode(self, B, state, proj, pos, slot, epoch) -> None:
+        """:meth:`prepare` and :meth:`run` of decode rows in one launch."""
+        s = self.shape
+        check(_lib.load().ifab_gr_decode(proj.data_ptr(), proj.stride(0), self.cols, self.channels, int(s.kind == "delta"), self.q_factor, _p(self.taps_w), _p(self.bias), s.taps,
+                                         s.channels, _p(state.history), self.kind, s.heads, s.kv_heads, s.dim, s.vdim, self.decay_col, self.weight_col, _p(self.a_log),
+                                         _p(self.decay_bias), _p(self.weight_bias), s.gate_cap, state.s.data_ptr(), _p(state.m), epoch.data_ptr(),
+                                         B.v.data_ptr() if s.kind == "ssd" else None, B.m.data_ptr(), pos.data_ptr(), slot.data_ptr(), B.o.data_ptr(), s.heads * s.E,
+                                         proj.shape[0], _s()), "gr_decode")
+
+    def gemv_mixed(self, B, proj, eps: float, x: torch.Tensor, K1: int, w: torch.Tensor, out: torch.Tensor) -> None:
+        """``out`` (f32) = ``[first K1 columns of x | finished recurrence] @ w.T`` for one or two rows (:meth:`finish` and the output projection in one launch)."""
+        s = self.shape
+        gate = proj[:, self.col[self.gate]:]
+        assert w.is_contiguous() and x.dtype == torch.bfloat16
+        check(_lib.load().ifab_gemv_mixed(x.data_ptr(), x.stride(0), K1, B.o.data_ptr(), s.heads * s.E, s.heads, s.vdim, s.E, B.m.data_ptr() if s.kind == "memory" else None,
+                                          B.v.data_ptr(), _p(self.skip), gate.data_ptr(), proj.stride(0), self.gate_act, int(s.kind == "ssd"), s.groups, eps,
+                                          self.gain.data_ptr(), w.data_ptr(), out.data_ptr(), out.stride(0), proj.shape[0], w.shape[0], w.shape[1], _s()), "gemv_mixed")
 
     def finish(self, B, proj, eps: float, out: torch.Tensor) -> None:
         s = self.shape

@@ -1,5 +1,5 @@
 """Residual streams side by side with fixed mixing weights and a short causal convolution ahead of every sublayer
-(``csrc/kernels/hyper_streams.cu``)."""
+(``csrc/kernels/hyper_streams.cu``, for decode rows ``decode_hyper.cu``)."""
 from __future__ import annotations
 
 from typing import Dict, Optional
@@ -8,10 +8,11 @@ import torch
 
 from . import _lib
 from ._lib import check
-from .stream_norm import _f32, _p, _parts, _s
+from .stream_norm import ACTIVATIONS, _f32, _p, _parts, _s
 
 F32 = torch.float32
 MOST_STREAMS, MOST_TAPS = 16, 16
+FUSED_STREAMS = 4        # most streams of the fused decode form
 BLOCK = 8                # rows of a CTA in steps of many rows
 
 
@@ -64,3 +65,17 @@ def streams_rows(x_in: torch.Tensor, x_out: Optional[torch.Tensor], y: Optional[
         (a.gain if a else gain).data_ptr(), eps, _p(a.taps_w) if a else None, a.taps if a else 0, _p(a.history) if a else None, epoch.data_ptr(), positions.data_ptr(),
         slots.data_ptr(), _p(total), 0 if total is None else total.stride(0), _p(xa), 0 if xa is None else xa.stride(0), _f32(some), T, S, D,
         1 if T <= 256 else BLOCK, _s()), "streams_rows")
+
+
+def gemv_streams(x_in: torch.Tensor, x_out: Optional[torch.Tensor], y: Optional[torch.Tensor], before: Optional[Sublayer], after: Sublayer, eps: float, epoch: torch.Tensor,
+                 positions: torch.Tensor, slots: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: Optional[str] = None) -> None:
+    """:func:`streams_rows` and a linear over its operand (bf16 ``w`` ``[N, D]``, ``out = act(operand @ w.T)``) in one launch, for one or two rows of up to
+    four streams."""
+    T, S, D = x_in.shape
+    N, a = w.shape[0], after
+    assert w.shape[1] == D and w.is_contiguous() and (y is None or y.dim() == 2)
+    check(_lib.load().ifab_gemv_streams(
+        x_in.data_ptr(), x_in.stride(0), x_in.stride(1), _p(x_out), 0 if x_out is None else x_out.stride(0), 0 if x_out is None else x_out.stride(1), _p(y),
+        0 if y is None else y.stride(0), None if y is None else before.mix.data_ptr(), None if y is None else before.out.data_ptr(), a.inp.data_ptr(), a.gain.data_ptr(), eps,
+        _p(a.taps_w), a.taps, _p(a.history), epoch.data_ptr(), positions.data_ptr(), slots.data_ptr(), S, w.data_ptr(), out.data_ptr(), out.stride(0), _f32(out),
+        ACTIVATIONS[act], T, N, D, _s()), "gemv_streams")

@@ -88,12 +88,26 @@ def fubelorn_arm(size, prompt: int, chunk_rows: int, batches: List[int], t: Time
             keys = min(l.window, prompt + 1) + l.most_ahead(prompt + 1)
             group(f"window attention, {what} (norm, rotation, pages, attention, gate), {n} sequences", kinds[k], attend,
                   n * keys * l.row * 2 + n * (l.heads + 2 * l.kv_heads) * l.dim * 4)
-        for k, what in (("parallel", "delta rule"), ("mamba2", "state-space"), ("parallel_2", "matrix memory")):
+        for k, what in (("parallel", "delta rule"), ("mamba2", "state-space"), ("parallel_2", "matrix memory")) if n > 1 else ():
             r = shape(k)
             group(f"recurrence step, {what} (convolution, gates, step, norm), {n} sequences", kinds[k],
                   lambda L: L["right"].mix(B.rec, L["state"], B.attn.proj[:n], pos, sl, None, dec.epoch, cfg.eps, B.mixed[L["c"].mixed][:n, L["c"].mixed[0]:]),
                   n * (8.0 * r.heads * r.E * r.dim + 2 * r.in_cols + 2 * r.inner))
-    for n in (1, 64, chunk_rows):
+    # the fused launches of one decode row
+    B, pos, sl = dec.rows, torch.full((1,), prompt, dtype=torch.int32, device=dev), torch.zeros(1, dtype=torch.int32, device=dev)
+    xs, proj = [t[:1, :, :W] for t in B.streams], B.attn.proj[:1]
+    front = lambda L, q, w, out, act=None: HS.gemv_streams(xs[0], xs[1], B.y[:1], L["sub"][0], L["sub"][q], cfg.eps, dec.epoch, pos, sl, w, out, act)
+    for k, name in (("parallel", "parallel"), ("mamba2", "state-space")):
+        group(f"input projection behind streams, norm and convolution, {name} layer, 1 row", kinds[k], lambda L: front(L, 0, L["in"], proj), projection(kinds[k][0]))
+    for k, what in (("parallel", "delta rule"), ("mamba2", "state-space"), ("parallel_2", "matrix memory")):
+        r = shape(k)
+        group(f"recurrence step, {what} (convolution, gates, step), 1 row", kinds[k], lambda L: L["right"].decode(B.rec, L["state"], proj, pos, sl, dec.epoch),
+              8.0 * r.heads * r.E * r.dim + 2 * r.in_cols)
+        group(f"output projection behind norm and gate, {what}, 1 row", kinds[k],
+              lambda L: L["right"].gemv_mixed(B.rec, proj, cfg.eps, B.mixed[L["c"].mixed][:1], L["c"].mixed[0], L["out"], B.y[:1]), 2.0 * W * sum(kinds[k][0]["c"].mixed))
+    group("up projection behind streams, norm and convolution + GELU, 1 row", dec.layers, lambda L: front(L, 1, L["up"], B.act[ff][:1], "gelu_erf"), 2.0 * W * ff)
+    group("down projection, 1 row", dec.layers, lambda L: N.gemv_act(B.act[ff][:1], L["down"], B.y[:1]), 2.0 * W * ff)
+    for n in (64, chunk_rows):
         B = dec.rows if n <= 8 else rows.B
         pos = torch.arange(prompt - n, prompt, dtype=torch.int32, device=dev) if n == chunk_rows else torch.full((n,), prompt, dtype=torch.int32, device=dev)
         sl = torch.zeros(n, dtype=torch.int32, device=dev) if n == chunk_rows else torch.arange(n, dtype=torch.int32, device=dev)

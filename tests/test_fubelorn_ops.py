@@ -132,6 +132,50 @@ def test_streams_and_convolution(dtype, S, taps, width):
 
 
 @gpu
+@pytest.mark.parametrize("S,taps,width,N", [(1, 4, 64, 40), (2, 4, 264, 2400), (3, 2, 136, 9), (4, 7, 1032, 5000), (2, 0, 40, 33), (1, 1, 24, 100), (4, 3, 2048, 300)])
+def test_linear_behind_the_streams(S, taps, width, N):
+    """Decode rows: the fused launch against streams, norm, convolution and a linear of the restatement, over sequences from their first token on, alone, two sequences
+    together, and two rows of one sequence."""
+    from ironpangu_b200.ops import hyper_streams as HS
+
+    g = torch.Generator().manual_seed(width + S)
+    rn = lambda *s: torch.randn(s, generator=g)
+    W = {"hc1.mix": rn(S, S), "hc1.in": rn(S), "hc1.out": rn(S), "norm1": rn(), "canon1": rn(width, taps)}
+    a = HS.Sublayer(W, "", 1, S, 0.7, taps, width, "cuda")
+    a.make_history(3, width, "cuda")
+    if taps > 1:
+        a.history.fill_(float("nan"))
+    eps, n = 1e-2, 24
+    w = (rn(N, width) * width ** -0.5).to(BF16)
+    X, Y = {k: rn(n, S, width) for k in "ab"}, {k: rn(n, width) for k in "ab"}
+    new = {k: torch.einsum("st,nsw->ntw", W["hc1.mix"].double(), X[k].double()) + 0.7 * W["hc1.out"].double()[:, None] * Y[k].double()[:, None] for k in "ab"}
+    h = {k: O.unit_rms(torch.einsum("s,nsw->nw", W["hc1.in"].double(), new[k]), eps) * W["norm1"].double() for k in "ab"}
+    z = {k: torch.nn.functional.gelu((h[k] + O.short_conv(h[k], W["canon1"].double())) @ w.double().T) for k in "ab"}
+    epoch = torch.zeros(3, dtype=torch.int32, device="cuda")
+    at, slot = {"a": 0, "b": 0}, {"a": 2, "b": 0}
+    for step in ("a", "a", "b", "ab", "aa", "ba", "bb", "a", "aa", "aa", "ab", "b", "bb", "ab"):
+        rows = []
+        for k in step:
+            rows.append((k, at[k]))
+            at[k] += 1
+        cat = lambda src: torch.stack([src[k][i] for k, i in rows])
+        m = len(rows)
+        pos, slots = torch.tensor([i for _, i in rows], dtype=torch.int32, device="cuda"), torch.tensor([slot[k] for k, _ in rows], dtype=torch.int32, device="cuda")
+        x_out, out = torch.zeros(m, S, width, device="cuda"), torch.full((m, N + 3), 5.0, device="cuda")
+        HS.step_epoch(slots, epoch)
+        HS.gemv_streams(cat(X).cuda(), x_out, cat(Y).cuda(), a, a, eps, epoch, pos, slots, w.cuda(), out[:, :N], "gelu_erf")
+        assert _rel(x_out, cat(new)) < 2e-6 and (out[:, N:] == 5).all()
+        assert _rel(out[:, :N], cat(z)) < 8e-3, step
+    first = torch.zeros(1, N, device="cuda")                # a sequence's first token ahead of the first layer: one row for every stream, nothing to add
+    HS.step_epoch(torch.tensor([1], dtype=torch.int32, device="cuda"), epoch)
+    x = rn(1, 1, width)
+    HS.gemv_streams(x.cuda().expand(1, S, width), None, None, None, a, eps, epoch, torch.zeros(1, dtype=torch.int32, device="cuda"), torch.ones(1, dtype=torch.int32, device="cuda"),
+                    w.cuda(), first)
+    h = O.unit_rms(x[0].double() * W["hc1.in"].double().sum(), eps) * W["norm1"].double()
+    assert _rel(first, (h + O.short_conv(h, W["canon1"].double())) @ w.double().T) < 8e-3
+
+
+@gpu
 @DTYPES
 def test_embedding_norm_and_plain_residual(dtype):
     from ironpangu_b200.ops import hyper_streams as HS
@@ -285,6 +329,44 @@ def test_recurrence_of_long_and_short_memory(shape, dtype):
         r = Recurrence(shape, dtype, {"a": n}, strong=strong, seed=4)
         lim = 5e-5 if dtype == F32 else 2e-2
         assert r.error(_cuts(n, n)) < lim and r.error(_cuts(n, 100)) < lim
+
+
+@gpu
+@pytest.mark.parametrize("shape", [("delta", 6, 2, 32, 24, 3), ("delta", 2, 1, 136, 72, 2), ("delta", 4, 4, 64, 128, 4), ("delta", 1, 1, 4, 4, 1), ("ssd", 4, 2, 16, 24, 4, 2),
+                                   ("ssd", 6, 1, 32, 16, 2, 1), ("ssd", 2, 1, 128, 64, 4, 2), ("ssd", 2, 2, 200, 136, 4, 1), ("memory", 3, 3, 32, 24), ("memory", 2, 2, 136, 72),
+                                   ("memory", 2, 2, 64, 128)], ids=str)
+@pytest.mark.parametrize("K1", [0, 24])
+def test_fused_decode_of_recurrences(shape, K1):
+    """Step and output projection in two launches: one or two rows, of one sequence or two, behind a prompt and from the first token on."""
+    from ironpangu_b200.ops import hyper_streams as HS
+
+    r = Recurrence(shape, BF16, {"a": 40, "b": 40}, seed=2)
+    g = torch.Generator().manual_seed(9)
+    v, N = r.shape.inner, 72
+    w = torch.zeros(N, K1 + _pad(v))
+    w[:, :K1 + v] = torch.randn(N, K1 + v, generator=g) * (K1 + v) ** -0.5
+    w = w.to(BF16)
+    r.error([[("a", 1, 0, 20)]])
+    at, slot = {"a": 20, "b": 0}, {"a": 1, "b": 3}
+    proj0 = {k: torch.nn.functional.pad(x, (1, 0)) for k, x in r.proj.items()}          # columns from 4 on: whole loads
+    mixer = r.GR.GatedRecurrence(r.shape, r.w, "", "cuda", BF16, at=4, factor=0.75)
+    assert mixer.fusable
+    for step in ("a", "b", "ab", "aa", "bb", "ba", "b", "a", "bb", "aa"):
+        rows = []
+        for k in step:
+            rows.append((k, at[k]))
+            at[k] += 1
+        m = len(rows)
+        pos, slots = torch.tensor([i for _, i in rows], dtype=torch.int32, device="cuda"), torch.tensor([slot[k] for k, _ in rows], dtype=torch.int32, device="cuda")
+        proj = torch.stack([proj0[k][i] for k, i in rows])
+        proj = torch.nn.functional.pad(proj, (0, -proj.shape[1] % 8)).cuda()
+        B = r.GR.RecurrenceBuffers([r.shape], m, BF16, "cuda", chunk=0, slots=4)
+        x, y = torch.randn(m, K1 + 8, generator=g).to(BF16), torch.full((m, N), 5.0, device="cuda")
+        HS.step_epoch(slots, r.epoch)
+        mixer.decode(B, r.state, proj, pos, slots, r.epoch)
+        mixer.gemv_mixed(B, proj, r.eps, x.cuda(), K1, w.cuda(), y)
+        want = torch.cat([x[:, :K1].double(), torch.stack([r.want[k][i] for k, i in rows])], 1) @ w[:, :K1 + v].double().T
+        assert _rel(y, want) < 5e-2, step
 
 
 def test_restated_recurrences_by_hand():
