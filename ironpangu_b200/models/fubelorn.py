@@ -309,6 +309,7 @@ class FubelornDecoder(StreamDecoder):
         # prompts: recurrences on the tensor cores in bf16 when every head fits a tile, f32 products otherwise
         self.chunk = TILE if self.dtype == BF16 and all(l.right.tiles for l in c.layers) else CHUNK
         # the fused decode chain needs operand widths that are whole 16-byte chunks
+        self.side = torch.cuda.Stream()
         self.fused = self.dtype == BF16 and c.streams <= HS.FUSED_STREAMS and c.width % 8 == 0 and c.width <= 8192 and all(l.ff % 8 == 0 for l in c.layers) and \
             all(L["right"].fusable for L in self.layers)
 
@@ -333,19 +334,26 @@ class FubelornDecoder(StreamDecoder):
         return cls(c, w, fabric, **kw)
 
     # -- layers ------------------------------------------------------------------------------------------------------------
-    def _attend(self, B: _Rows, L: dict, m: int, pos, slot, plan: Optional[DevicePlan]) -> torch.Tensor:
-        """The attention of a layer that has one; returns the operand of the output projection, whose first part it leaves there."""
+    def _side_by_side(self, B: _Rows, L: dict, m: int, pos, slot, plan: Optional[DevicePlan], recurrence) -> torch.Tensor:
+        """The mixer of one layer between its input projection (``B.attn.proj``) and the operand of its output projection, which it returns. A layer with an
+        attention runs it beside ``recurrence(operand's second part)``, on a stream of its own between two events."""
         l = L["c"]
         out = B.mixed[l.mixed][:m]
-        if l.left:
-            L["left"].attend(B.attn, m, L["pages"], B.rotary.get(*l.left.rotation), pos, slot, plan, self.page_table, self.cfg.eps, out, self.fabric.desc.status)
+        right = out[:, l.mixed[0]:]
+        if l.left is None:
+            recurrence(right)
+            return out
+        main = torch.cuda.current_stream()
+        self.side.wait_stream(main)
+        with torch.cuda.stream(self.side):
+            recurrence(right)
+        L["left"].attend(B.attn, m, L["pages"], B.rotary.get(*l.left.rotation), pos, slot, plan, self.page_table, self.cfg.eps, out, self.fabric.desc.status)
+        main.wait_stream(self.side)
         return out
 
     def _mix(self, B: _Rows, L: dict, m: int, pos, slot, plan: Optional[DevicePlan]) -> torch.Tensor:
-        """The mixer of one layer between its input projection (``B.attn.proj``) and the operand of its output projection, which it returns."""
-        out = self._attend(B, L, m, pos, slot, plan)
-        L["right"].mix(B.rec, L["state"], B.attn.proj[:m], pos, slot, plan, self.epoch, self.cfg.eps, out[:, L["c"].mixed[0]:], self.fabric.desc.status)
-        return out
+        run = lambda out: L["right"].mix(B.rec, L["state"], B.attn.proj[:m], pos, slot, plan, self.epoch, self.cfg.eps, out, self.fabric.desc.status)
+        return self._side_by_side(B, L, m, pos, slot, plan, run)
 
     def _product(self, B: _Rows, x: torch.Tensor, w: torch.Tensor, m: int) -> torch.Tensor:
         """f32 rows ``x w^T``: in ``B.y``, or for few rows as parts of a sum ``[parts, m, width]``."""
@@ -414,8 +422,7 @@ class FubelornDecoder(StreamDecoder):
                     spare.reverse()
                 before = sub
                 if act is None:
-                    mixed = self._attend(B, L, n, pos, slot, None)
-                    L["right"].decode(B.rec, L["state"], proj, pos, slot, self.epoch)
+                    mixed = self._side_by_side(B, L, n, pos, slot, None, lambda _: L["right"].decode(B.rec, L["state"], proj, pos, slot, self.epoch))
                     L["right"].gemv_mixed(B.rec, proj, c.eps, mixed, l.mixed[0], L["out"], y)
                 else:
                     N.gemv_act(out, L["down"], y)
