@@ -453,51 +453,63 @@ __global__ void __launch_bounds__(256) window_attn_kernel(WinParams p) {
   }
 }
 
-// grid (T, G), 128 threads: the block that ends at a row's position, if one does
-template <typename A>
+// grid T, 128 threads: the block that ends at a row's position, if one does. All heads of a position are one row, keys and values; V columns per thread at a time
+template <typename A, int V>
 __global__ void __launch_bounds__(128) pool_write_kernel(const A* k_cache, const A* v_cache, const int32_t* positions, const int32_t* slots, const int32_t* page_table,
-                                                         int max_pages, int page_tokens, int num_pages, int G, int d, int e, AheadRule rule, uint32_t* status) {
+                                                         int max_pages, int page_tokens, int num_pages, int nk, int nv, AheadRule rule, uint32_t* status) {
+  constexpr int B = 32;                     // positions looked up together
+  __shared__ long rows[B];
+  __shared__ int bad;
   grid_dep_launch();
   grid_dep_wait();
-  const int t = blockIdx.x, g = blockIdx.y, pos = positions[t], P = rule.pool;
+  const int t = blockIdx.x, pos = positions[t], P = rule.pool;
   if (pos < 0 || (pos + 1) % P) return;
   const int32_t* table = page_table + (long)slots[t] * max_pages;
-  const int last = pos / page_tokens < max_pages ? table[pos / page_tokens] : -1;
-  bool ok = last >= 0 && last < num_pages;
-  float acc[4] = {0.f, 0.f, 0.f, 0.f};      // d + e <= 512 columns
-  constexpr int B = 8;                      // positions in flight
-  for (int j0 = pos - P + 1; j0 <= pos && ok; j0 += B) {
-    long row[B];
+  const auto find = [&](int j) {
+    const int lp = j / page_tokens, page = lp < max_pages ? table[lp] : -1;
+    return page >= 0 && page < num_pages ? page : -1;
+  };
+  const int last = find(pos);
+  if (threadIdx.x == 0) bad = last < 0;
+  const long entry = (long)last * rule.per_page + rule.row(pos / P, page_tokens);
+  for (int c0 = 0; c0 < nk + nv; c0 += 128 * V) {             // every thread takes every round: the barriers are the CTA's
+    const int c = c0 + threadIdx.x * V;
+    float acc[V];
 #pragma unroll
-    for (int b = 0; b < B; ++b) {
-      const int j = min(j0 + b, pos), page = j / page_tokens < max_pages ? table[j / page_tokens] : -1;
-      ok = ok && page >= 0 && page < num_pages;
-      row[b] = ((long)max(page, 0) * page_tokens + j % page_tokens) * G + g;
+    for (int u = 0; u < V; ++u) acc[u] = 0.f;
+    for (int j0 = pos - P + 1; j0 <= pos; j0 += B) {
+      __syncthreads();
+      if (threadIdx.x < B) {
+        const int j = min(j0 + (int)threadIdx.x, pos), page = find(j);
+        if (page < 0) bad = 1;
+        rows[threadIdx.x] = (long)max(page, 0) * page_tokens + j % page_tokens;
+      }
+      __syncthreads();
+      if (bad || c >= nk + nv) continue;
+      const int n = min(B, pos - j0 + 1), ld = c < nk ? nk : nv;
+      const A* src = c < nk ? k_cache + c : v_cache + c - nk;
+#pragma unroll 8
+      for (int b = 0; b < n; ++b) {
+        const A* p = src + rows[b] * ld;
+        if constexpr (V == 8) {
+          float f[8];
+          unpack8(*reinterpret_cast<const uint4*>(p), f);
+#pragma unroll
+          for (int u = 0; u < 8; ++u) acc[u] += f[u];
+        } else {
+          acc[0] += to_f32(*p);
+        }
+      }
     }
-    if (!ok) break;
+    if (bad || c >= nk + nv) continue;
+    A* dst = c < nk ? reinterpret_cast<A*>(const_cast<void*>(rule.k)) + entry * nk + c : reinterpret_cast<A*>(const_cast<void*>(rule.v)) + entry * nv + c - nk;
 #pragma unroll
-    for (int u = 0; u < 4; ++u) {
-      const int c = threadIdx.x + 128 * u;
-      if (c >= d + e) break;
-      float v[B];
-#pragma unroll
-      for (int b = 0; b < B; ++b) v[b] = j0 + b <= pos ? to_f32(c < d ? k_cache[row[b] * d + c] : v_cache[row[b] * e + c - d]) : 0.f;
-#pragma unroll
-      for (int b = 0; b < B; ++b) acc[u] += v[b];
-    }
+    for (int u = 0; u < V; ++u) acc[u] /= (float)P;
+    if constexpr (V == 8) *reinterpret_cast<uint4*>(dst) = pack8(acc);
+    else *dst = from_f32<A>(acc[0]);
   }
-  if (!ok) {
-    if (threadIdx.x == 0 && status) atomicOr(status, IFAB_STATUS_BAD_INDEX);
-    return;
-  }
-  const long row = ((long)last * rule.per_page + rule.row(pos / P, page_tokens)) * G + g;
-#pragma unroll
-  for (int u = 0; u < 4; ++u) {
-    const int c = threadIdx.x + 128 * u;
-    if (c >= d + e) break;
-    A* dst = c < d ? reinterpret_cast<A*>(const_cast<void*>(rule.k)) + row * d + c : reinterpret_cast<A*>(const_cast<void*>(rule.v)) + row * e + c - d;
-    *dst = from_f32<A>(acc[u] / (float)P);
-  }
+  __syncthreads();
+  if (bad && threadIdx.x == 0 && status) atomicOr(status, IFAB_STATUS_BAD_INDEX);
 }
 
 }  // namespace
@@ -506,11 +518,17 @@ extern "C" int ifab_pool_write(const void* k_cache, const void* v_cache, int f32
                                int page_tokens, int num_pages, int G, int d, int e, int pool, void* pool_k, void* pool_v, int T, uint32_t* status, void* stream) {
   if (T < 1 || G < 1 || G > 65535 || d < 1 || d > 256 || e < 1 || e > 256 || pool < 1 || !pool_k || !pool_v) return -1;
   const AheadRule rule = ahead_rule(0, pool, pool_k, pool_v, page_tokens);
-  const dim3 grid(T, G);
-  return f32 ? launch_chain(pool_write_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, (const float*)k_cache, (const float*)v_cache, positions, slots, page_table,
-                            max_pages, page_tokens, num_pages, G, d, e, rule, status)
-             : launch_chain(pool_write_kernel<bf16>, grid, dim3(128), 0, (cudaStream_t)stream, (const bf16*)k_cache, (const bf16*)v_cache, positions, slots, page_table,
-                            max_pages, page_tokens, num_pages, G, d, e, rule, status);
+  const int nk = G * d, nv = G * e;
+  const auto odd = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) != 0; };
+  cudaStream_t s = (cudaStream_t)stream;
+  if (f32)
+    return launch_chain(pool_write_kernel<float, 1>, dim3(T), dim3(128), 0, s, (const float*)k_cache, (const float*)v_cache, positions, slots, page_table, max_pages,
+                        page_tokens, num_pages, nk, nv, rule, status);
+  if (!((nk | nv) % 8) && !odd(k_cache) && !odd(v_cache) && !odd(pool_k) && !odd(pool_v))
+    return launch_chain(pool_write_kernel<bf16, 8>, dim3(T), dim3(128), 0, s, (const bf16*)k_cache, (const bf16*)v_cache, positions, slots, page_table, max_pages,
+                        page_tokens, num_pages, nk, nv, rule, status);
+  return launch_chain(pool_write_kernel<bf16, 1>, dim3(T), dim3(128), 0, s, (const bf16*)k_cache, (const bf16*)v_cache, positions, slots, page_table, max_pages,
+                      page_tokens, num_pages, nk, nv, rule, status);
 }
 
 extern "C" int ifab_qk_norm_rope_write(const void* proj, long ldp, int f32, int q_off, int k_off, int v_off, const float* q_gain, const float* k_gain,
