@@ -522,11 +522,11 @@ def test_attention_with_entries_ahead(form, dtype, shape, rule):
 def test_a_single_entry_at_the_edges(form, dtype, shape):
     """A key, or the keys of a block, that take most of a query's weight: the last kept position and the one behind it, the window's oldest and the one
     before it, a block that is just seen and one that is not yet, the first tokens."""
-    size, keep, pool, scale = 96, 6, 12, shape[2] ** -0.5
-    for query in (299, 203, 202, 107, 108, 101):
-        for rule, keys in (((size, keep, 0), ([0], [5], [6], [query - 95], [query - 96], [query])),
-                           ((size, 0, pool), ([query - 95], [query - 96], range(0, 12), range((query - 96 + 1) // 12 * 12 - 12, (query - 96 + 1) // 12 * 12),
-                                              range((query - 96 + 1) // 12 * 12, (query - 96 + 1) // 12 * 12 + 12)))):
+    size, keep, pool, scale = 88, 5, 11, shape[2] ** -0.5
+    for query in (299, 196, 195, 99, 98, 94):
+        old, seen = query - size, (query - size + 1) // pool * pool          # the position just outside the window, the first position of no seen block
+        for rule, keys in (((size, keep, 0), ([0], [keep - 1], [keep], [old + 1], [old], [query])),
+                           ((size, 0, pool), ([old + 1], [old], range(pool), range(seen - pool, seen), range(seen, seen + pool)))):
             for some in keys:
                 some = [k for k in some if k >= 0]
                 K = Keys(*shape, dtype, n=300, seed=query)
